@@ -290,6 +290,13 @@ int32_t vn_model_status(vn_model* m, int32_t* bad_token, int32_t* wait_timeout);
  * GMLA) for a "vda" layer; vn_kv_read's `layer` counts these pairs.  A GMLA module caches the K / V rebuilt from
  * its latents. */
 int32_t vn_kv_create(vn_model* m, int32_t max_batch, int32_t max_seq, vn_kv** out);
+/* The same with the cache of a composed model (a configuration with "family": "composed", see vn_model_create) sized
+ * explicitly.  pool_tokens > 0: latents live in a pool of pages for that many tokens (rounded up to pages of 64) shared
+ * by all sequences; a sequence takes pages as it grows and gives them back when it is reset.  0: every sequence owns
+ * the pages of max_seq positions.  max_pending: rows a sequence may append and cut back with vn_kv_commit; the cache
+ * keeps that many recurrent states besides the committed one.  A longer append (a prompt) can only be kept whole. */
+int32_t vn_kv_create_ex(vn_model* m, int32_t max_batch, int32_t max_seq, int32_t pool_tokens, int32_t max_pending, vn_kv** out);
+int32_t vn_kv_pages(vn_kv* kv, int32_t* total, int32_t* free_pages);
 int32_t vn_kv_destroy(vn_kv* kv);
 /* A second handle on sequences [first, first + count) of a cache: forwards, commits, resets and length calls on it
  * act on those sequences only (a serving loop prefills one free slot while the others keep their state).  The view
@@ -319,6 +326,18 @@ int32_t vn_kv_read(vn_kv* kv, int32_t layer, int32_t seq, int32_t which /*0=k 1=
 int32_t vn_model_forward(vn_model* m, vn_kv* kv, const int64_t* tokens_dev, int32_t B, int32_t T,
                          const int32_t* parents_host, float* out_hidden_dev, float* out_logits_dev,
                          int32_t last_only, int32_t slot_offset);
+
+/* One step over a ragged batch of a composed model: entry e brings counts_host[e] rows for sequence slots_host[e]
+ * (each sequence at most once), its rows standing one after another in tokens_dev [sum of counts] in entry order.
+ * Portions of prompts and single decoded tokens may be mixed.  Everything is appended AND committed.  Final-norm hidden
+ * rows and logits are written for the n_out rows named by out_rows_host (indices into the step's rows), in that order:
+ * out_hidden_dev [n_out, dim], out_logits_dev [n_out, vocab], either may be NULL. */
+int32_t vn_model_forward_ragged(vn_model* m, vn_kv* kv, const int64_t* tokens_dev, int32_t n_entries, const int32_t* slots_host,
+                                const int32_t* counts_host, int32_t n_out, const int32_t* out_rows_host, float* out_hidden_dev,
+                                float* out_logits_dev);
+/* Diagnostic for composed models: while probe_dev is set, every forward of M rows copies the residual stream after layer
+ * run i (a looped layer counts once per pass) to probe_dev + i * M * dim.  NULL switches it off. */
+int32_t vn_model_set_probe(vn_model* m, float* probe_dev);
 
 /* The draft side of one speculative round with a draft MODEL (the north star's replacement for the k linear heads of
  * SpeculativeDecoder.draft, speculative.py:110-162): k proposals per request, token by token, all on the device.

@@ -119,6 +119,8 @@ PROTOTYPES = {
     "vn_model_probe_wait": [_p, C.POINTER(_i64)],
     "vn_model_status": [_p, C.POINTER(_i32), C.POINTER(_i32)],
     "vn_kv_create": [_p, _i32, _i32, C.POINTER(_p)],
+    "vn_kv_create_ex": [_p, _i32, _i32, _i32, _i32, C.POINTER(_p)],
+    "vn_kv_pages": [_p, C.POINTER(_i32), C.POINTER(_i32)],
     "vn_kv_destroy": [_p],
     "vn_kv_view": [_p, _i32, _i32, C.POINTER(_p)],
     "vn_kv_reset_seq": [_p, _i32],
@@ -126,6 +128,8 @@ PROTOTYPES = {
     "vn_kv_set_lengths": [_p, _p],
     "vn_kv_commit": [_p, _i32, _p, _i32, _p, _i32],
     "vn_kv_read": [_p, _i32, _i32, _i32, _p, _i32],
+    "vn_model_forward_ragged": [_p, _p, _p, _i32, _p, _p, _i32, _p, _p, _p],
+    "vn_model_set_probe": [_p, _p],
     "vn_model_forward": [_p, _p, _p, _i32, _i32, _p, _p, _p, _i32, _i32],
 }
 _RESTYPE = {"vn_last_error": C.c_char_p, "vn_topk_row_bytes": C.c_size_t}

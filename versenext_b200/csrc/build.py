@@ -68,10 +68,23 @@ def build(force: bool = False, verbose: bool = False) -> str:
                 if verbose:
                     print("compiled", os.path.basename(done))
     if jobs or not os.path.exists(OUT):
-        r = subprocess.run([NVCC, "-shared", "-o", OUT, *objs, "-lcudart", "-ldl"], capture_output=True, text=True)
+        part = f"{OUT}.{os.getpid()}"
+        r = subprocess.run([NVCC, "-shared", "-o", part, *objs, "-lcudart", "-ldl"], capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+        os.replace(part, OUT)
     return OUT
+
+
+def ensure_built() -> str:
+    """The library, compiled now if this checkout has none yet (one process at a time)."""
+    if os.path.exists(OUT):
+        return OUT
+    import fcntl
+    os.makedirs(OBJ_DIR, exist_ok=True)
+    with open(os.path.join(OBJ_DIR, "lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return OUT if os.path.exists(OUT) else build()
 
 
 if __name__ == "__main__":

@@ -5,7 +5,7 @@
 enum GemmEpilogue {
   EPI_STORE = 0,    // C = acc (+ bias)
   EPI_ADD = 1,      // C += acc              (residual stream, fp32)
-  EPI_SWIGLU = 2    // out[m, n/2] = silu(acc[m, n]) * acc[m, n+1], n even (gate / up rows interleaved in W)
+  EPI_SWIGLU = 2    // out[m, n/2] = act(acc[m, n]) * acc[m, n+1], n even (gate / up rows interleaved in W), act: GemmArgs::act
 };
 
 struct GemmArgs {
@@ -27,6 +27,7 @@ struct GemmArgs {
   int nseg = 1;
   int epi = EPI_STORE;
   int c_bf16 = 0;
+  int act = 0;                    // gate activation of EPI_SWIGLU: 0 silu, 1 gelu (tanh form)
   const char* tag = nullptr;      // name of the call site in the per-kernel timing report (string literal)
   // weight-only quantisation: W points at INT8 / packed INT4 bytes, ldw and w_stride stay in ELEMENTS
   int wq = 0;                     // 0 dense, 1 int8, 2 int4 per output row, 3 int4 with one scale per 128 inputs
@@ -39,6 +40,12 @@ __device__ __forceinline__ float ld_f(const __nv_bfloat16* p) { return __bfloat1
 
 // silu as the reference computes it: x * 0.5 * (1 + tanh(x / 2))   (verse_torch/tensor.py:853-856)
 __device__ __forceinline__ float silu_ref(float x) { return x * (0.5f * (1.0f + tanhf(0.5f * x))); }
+
+// tanh form of gelu: 0.5 x (1 + tanh(sqrt(2 / pi) (x + 0.044715 x^3)))
+__device__ __forceinline__ float gelu_tanh(float x) {
+  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
+__device__ __forceinline__ float glu_act(float x, int act) { return act ? gelu_tanh(x) : silu_ref(x); }
 
 template <typename T>
 __device__ __forceinline__ void store_out(void* C, long long idx, float v, int c_bf16) {
@@ -106,7 +113,7 @@ __global__ void __launch_bounds__(256) gemm_nt_simt_kernel(GemmArgs g) {
       for (int j = 0; j < 4; j += 2) {
         const int n = n0 + tx * 4 + j;
         if (n + 1 < g.N) {
-          const float v = silu_ref(acc[i][j]) * acc[i][j + 1];
+          const float v = glu_act(acc[i][j], g.act) * acc[i][j + 1];
           store_out<float>(g.C, c_base + crow * g.ldc + (n >> 1), v, g.c_bf16);
         }
       }

@@ -43,7 +43,8 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
   if (g.seg_cnt) { row0 = g.seg_off[z]; Mz = g.seg_cnt[z]; }
   const int m0 = blockIdx.x * BM, n0 = blockIdx.y * BN;
   if (m0 >= Mz) return;
-  const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(g.A);
+  const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(g.A) + (g.seg_cnt ? 0 : (long long)z * g.a_stride);
+  const long long c_base = g.seg_cnt ? 0 : (long long)z * g.c_stride;
   const __nv_bfloat16* W = reinterpret_cast<const __nv_bfloat16*>(g.W) + (long long)z * g.w_stride;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int wm = warp / WARPS_N, wn = warp % WARPS_N;
@@ -133,20 +134,20 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
     for (int half = 0; half < 2; ++half) {
       const int m = m0 + wm * 32 + i * 16 + (lane >> 2) + half * 8;
       if (m >= Mz) continue;
-      const long long crow = (long long)(row0 + m);
+      const long long crow = (long long)(row0 + m) * g.ldc + c_base;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int n = n0 + wn * 32 + j * 8 + (lane & 3) * 2;
         const float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
         if (g.epi == EPI_SWIGLU) {
-          if (n + 1 < g.N) store_out<float>(g.C, crow * g.ldc + (n >> 1), silu_ref(v0) * v1, g.c_bf16);
+          if (n + 1 < g.N) store_out<float>(g.C, crow + (n >> 1), glu_act(v0, g.act) * v1, g.c_bf16);
         } else if (g.epi == EPI_ADD) {
-          float* c = reinterpret_cast<float*>(g.C) + crow * g.ldc + n;
+          float* c = reinterpret_cast<float*>(g.C) + crow + n;
           if (n < g.N) c[0] += v0;
           if (n + 1 < g.N) c[1] += v1;
         } else {
-          if (n < g.N) store_out<float>(g.C, crow * g.ldc + n, v0 + (g.bias ? g.bias[n] : 0.f), g.c_bf16);
-          if (n + 1 < g.N) store_out<float>(g.C, crow * g.ldc + n + 1, v1 + (g.bias ? g.bias[n + 1] : 0.f), g.c_bf16);
+          if (n < g.N) store_out<float>(g.C, crow + n, v0 + (g.bias ? g.bias[n] : 0.f), g.c_bf16);
+          if (n + 1 < g.N) store_out<float>(g.C, crow + n + 1, v1 + (g.bias ? g.bias[n + 1] : 0.f), g.c_bf16);
         }
       }
     }
@@ -156,7 +157,7 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
 
 inline bool gemm_mma_supported(const GemmArgs& g) {
   return g.K % 8 == 0 && g.lda % 8 == 0 && g.ldw % 8 == 0 && g.ldw_k == 1 && g.w_stride % 8 == 0 &&
-         ((uintptr_t)g.A & 15) == 0 && ((uintptr_t)g.W & 15) == 0 && (g.seg_cnt != nullptr || g.nseg == 1);
+         ((uintptr_t)g.A & 15) == 0 && ((uintptr_t)g.W & 15) == 0 && (g.seg_cnt != nullptr || g.a_stride % 8 == 0);
 }
 
 inline int32_t launch_gemm_mma(vn_ctx* ctx, const GemmArgs& g) {

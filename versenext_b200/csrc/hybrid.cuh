@@ -1,0 +1,801 @@
+// Composed models: a list of layers of different kinds (latent attention, selective scan, gated delta rule), each with
+// an optional gated feed-forward, and optionally a block of layers that is run several times with the same weights.
+// Weights, the per-sequence cache (paged latents, rings of convolution inputs and of recurrent states), and the forward
+// over new rows of a uniform or a ragged batch.  Included by model.cu: it uses that file's GEMM helpers.
+//
+// One forward serves prompts, portions of prompts, single tokens and mixtures.  Projections of at most 256 rows of a
+// bf16 model are split-K tcgen05 GEMMs whose slices are summed by the kernel that needs them; longer ones go through
+// the tcgen05 segment kernel; an fp32 model uses the fp32 GEMM.  When every entry brings one token, a mixer's
+// recurrence and what surrounds it is one kernel (mamba_step_kernel, delta_step_kernel).
+#pragma once
+#include "json_value.h"
+#include "latent_attn.cuh"
+#include "scan_delta.cuh"
+#include "scan_mamba.cuh"
+#include "seq_ops.cuh"
+
+namespace hybrid {
+
+enum Kind { LATENT = 0, MAMBA1 = 1, DELTA = 2 };
+
+struct HLayer {
+  int kind = 0;
+  // latent: H, d, vd, R (kv_rank), window, scale.  mamba: inner, dt_rank, nstate, taps.  delta: H, KH, d, vd, taps, ra, rg
+  int H = 0, KH = 0, d = 0, vd = 0, R = 0, window = 0, taps = 1, inner = 0, dt_rank = 0, nstate = 0, ra = 0, rg = 0;
+  float scale = 1.f;
+  int ff = 0, act = 0;             // feed-forward width (0: none), activation
+  int dp = 0, Rp = 0, dtp = 0, rap = 0, rgp = 0, n_in = 0, n_x = 0, ffp = 0;    // padded sizes
+  float* norm1 = nullptr; float* norm2 = nullptr;                               // 1 + stored weight
+  void* w_in = nullptr;            // first projection, all its parts stacked [n_in, D]
+  void* w_o = nullptr;
+  void* w_uk = nullptr;            // latent: per head W_uk^T [H][Rp][dp];  delta: a2 [H d, rap];  mamba: dt [inner, dtp]
+  void* w_uv = nullptr;            // latent: [H][vd][Rp];                  delta: g2 [H vd, rgp];  mamba: x [n_x, inner]
+  float* f_a = nullptr;            // latent: norm of the latent;  delta: norm [vd];         mamba: A = -exp(A_log)
+  float* f_b = nullptr;            // latent: sink [H];            delta: exp(A_log) [H];    mamba: D
+  float* f_c = nullptr;            //                              delta: dt_bias [H d];     mamba: dt bias
+  float* conv = nullptr; float* conv_b = nullptr;
+  void* w_gu = nullptr; void* w_down = nullptr;
+  int conv_ch() const { return kind == MAMBA1 ? inner : 2 * KH * d + H * vd; }
+  long long state_elems() const { return kind == MAMBA1 ? (long long)inner * nstate : (long long)H * d * vd; }
+};
+
+struct Run { int layer; int pass; };      // pass: -1 outside the loop
+
+struct Model {
+  int D = 0, vocab = 0, sinusoidal = 0;
+  float eps = 1e-6f;
+  std::vector<HLayer> layers;
+  int loop_start = 0, loop_stop = 0, loop_times = 0;
+  std::vector<Run> runs;
+  void* w_loop = nullptr;          // [D, 2 D]
+  float* loop_step = nullptr;      // [times, D]
+  double* freq = nullptr;          // [ceil(D / 2)]
+  std::set<std::string> want;
+  float* x0 = nullptr; void* cat = nullptr; char* ws = nullptr; size_t ws_bytes = 0;
+  int* meta = nullptr; int meta_cap = 0;
+  float* probe = nullptr;          // residual stream after every layer run, [runs][M][D], or null
+};
+
+// what a cache of such a model keeps besides the lengths; owned by the root cache, shared by its views
+struct Cache {
+  int pending = 1, ring = 2;       // rows that can be appended and cut back; state snapshots per sequence
+  bool pooled = false;
+  int max_pages = 0, n_pages = 0, slots = 0;
+  int* table_dev = nullptr;
+  std::vector<int> table, used;    // [slots][max_pages]; pages held by each slot
+  std::vector<int> free_pages;
+};
+
+inline int up8(int n) { return (n + 7) & ~7; }
+inline int up4(int n) { return (n + 3) & ~3; }
+// latent rows are padded to a multiple of 32 that the tensor-core kernel has an instance for
+inline int latent_pitch(int R) {
+  static const int tiles[] = {1, 2, 3, 4, 6, 8, 12, 16};
+  for (int t : tiles)
+    if (R <= 32 * t) return 32 * t;
+  return (R + 31) & ~31;
+}
+
+struct Arena {
+  char* base = nullptr;
+  size_t off = 0;
+  template <typename P> void take(P** p, size_t bytes) {
+    *p = base ? reinterpret_cast<P*>(base + off) : nullptr;
+    off += (bytes + 255) & ~size_t(255);
+  }
+};
+struct Buffers {
+  float* proj = nullptr;           // [M, n_in] when the projection is not split (also [M, D] of the loop entry)
+  void* mix = nullptr;             // [M, H vd | inner] input of the output projection
+  void* act = nullptr;             // [M, ffp]
+  void *q = nullptr, *qc = nullptr, *oc = nullptr;                    // latent
+  float *gate = nullptr, *part_o = nullptr, *part_ml = nullptr;
+  void *xc = nullptr, *z = nullptr, *dtb = nullptr; float *p = nullptr, *dt = nullptr;       // mamba
+  float *dq = nullptr, *dk = nullptr, *dv = nullptr, *beta = nullptr, *g = nullptr, *gg = nullptr, *o = nullptr;   // delta
+  void *low_a = nullptr, *low_g = nullptr;
+};
+constexpr int SPLIT_ROWS = 64, MAX_SPLITS = 16;   // key splits of the latent attention: forwards of few rows
+
+inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& A, Buffers& b) {
+  A.off = 0;
+  A.take(&b.proj, M * std::max(L.n_in, hm.D) * 4);
+  A.take(&b.mix, M * (size_t)(L.kind == MAMBA1 ? L.inner : L.H * L.vd) * e);
+  if (L.ff) A.take(&b.act, M * L.ffp * e);
+  if (L.kind == LATENT) {
+    A.take(&b.q, M * L.H * L.dp * e);
+    A.take(&b.qc, M * L.H * L.Rp * e);
+    A.take(&b.oc, M * L.H * L.Rp * e);
+    A.take(&b.gate, M * L.H * 4);
+    if (M <= SPLIT_ROWS) {
+      A.take(&b.part_o, (size_t)MAX_SPLITS * M * L.H * L.Rp * 4);
+      A.take(&b.part_ml, (size_t)MAX_SPLITS * M * L.H * 2 * 4);
+    }
+  } else if (L.kind == MAMBA1) {
+    A.take(&b.xc, M * L.inner * e);
+    A.take(&b.z, M * L.inner * e);
+    A.take(&b.dtb, M * L.dtp * e);
+    A.take(&b.p, M * L.n_x * 4);
+    A.take(&b.dt, M * L.inner * 4);
+  } else {
+    A.take(&b.dq, M * L.KH * L.d * 4);
+    A.take(&b.dk, M * L.KH * L.d * 4);
+    A.take(&b.dv, M * L.H * L.vd * 4);
+    A.take(&b.beta, M * L.H * 4);
+    A.take(&b.g, M * L.H * L.d * 4);
+    A.take(&b.gg, M * L.H * L.vd * 4);
+    A.take(&b.o, M * L.H * L.vd * 4);
+    A.take(&b.low_a, M * L.rap * e);
+    A.take(&b.low_g, M * L.rgp * e);
+  }
+}
+
+// ---- configuration ---------------------------------------------------------------------------------------------
+int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
+  c->vocab = (int)j.number("vocab_size", 0);
+  c->dim = (int)j.number("dim", 0);
+  const std::string dt = j.text("dtype");
+  VN_REQUIRE(ctx, dt.empty() || dt == "f32" || dt == "bf16", "dtype must be \"f32\" or \"bf16\", got %s", dt.c_str());
+  c->bf16 = dt == "bf16";
+  c->tie = 0;
+  c->max_seq_len = (int)j.number("max_seq_len", 2048);
+  hm->D = c->dim; hm->vocab = c->vocab;
+  hm->eps = (float)j.number("norm_eps", 1e-6);
+  hm->sinusoidal = j.text("positions") == "sinusoidal";
+  const JsonValue* ls = j.find("layers");
+  VN_REQUIRE(ctx, c->vocab > 0 && c->dim > 0 && ls && ls->kind == JsonValue::ARR && !ls->arr.empty(),
+             "a composed model needs vocab_size, dim and layers");
+  for (size_t i = 0; i < ls->arr.size(); ++i) {
+    const JsonValue& l = ls->arr[i];
+    HLayer L;
+    const std::string t = l.text("mixer");
+    auto I = [&](const char* k, int dflt = 0) { return (int)l.number(k, dflt); };
+    L.kind = t == "latent_attention" ? LATENT : t == "mamba1" ? MAMBA1 : t == "channel_delta" ? DELTA : -1;
+    VN_REQUIRE(ctx, L.kind >= 0, "layer %zu: mixer %s unknown (latent_attention | mamba1 | channel_delta)", i, t.c_str());
+    L.ff = I("mlp_hidden");
+    const std::string act = l.text("mlp_act");
+    VN_REQUIRE(ctx, !L.ff || act == "gelu_tanh" || act == "silu", "layer %zu: activation %s unknown (gelu_tanh | silu)", i, act.c_str());
+    L.act = act == "gelu_tanh";
+    L.ffp = up8(L.ff);
+    L.H = I("heads"); L.d = I("dim"); L.vd = I("vdim"); L.taps = I("conv", 1);
+    if (L.kind == LATENT) {
+      L.R = I("kv_rank"); L.window = I("window"); L.scale = (float)l.number("scale", 0);
+      VN_REQUIRE(ctx, L.H > 0 && L.d > 0 && L.vd > 0 && L.R > 0 && L.R <= 1024 && L.window >= 0, "layer %zu: latent attention sizes", i);
+      L.dp = up8(L.d); L.Rp = latent_pitch(L.R);
+      L.n_in = up8(L.H * L.d + L.R + L.H);
+    } else if (L.kind == MAMBA1) {
+      L.inner = I("inner"); L.dt_rank = I("dt_rank"); L.nstate = I("state");
+      VN_REQUIRE(ctx, L.inner > 0 && L.dt_rank > 0 && L.nstate > 0 && L.nstate <= 128 && L.taps >= 1, "layer %zu: selective scan sizes", i);
+      L.dtp = up8(L.dt_rank);
+      L.n_in = 2 * L.inner;
+      L.n_x = up8(L.dtp + 2 * L.nstate);
+    } else {
+      L.KH = I("kv_heads"); L.ra = I("decay_rank"); L.rg = I("gate_rank");
+      VN_REQUIRE(ctx, L.H > 0 && L.KH > 0 && L.H % L.KH == 0 && L.d > 0 && L.d <= 256 && L.vd > 0 && L.vd <= 512 && L.ra > 0 &&
+                 L.rg > 0 && L.taps >= 1, "layer %zu: delta rule sizes", i);
+      L.rap = up8(L.ra); L.rgp = up8(L.rg);
+      L.n_in = up8(2 * L.KH * L.d + L.H * L.vd + L.H + L.ra + L.rg);
+    }
+    hm->layers.push_back(L);
+  }
+  const int n = (int)hm->layers.size();
+  if (const JsonValue* lp = j.find("loop")) {
+    if (lp->kind == JsonValue::OBJ) {
+      hm->loop_start = (int)lp->number("start", 0);
+      hm->loop_stop = (int)lp->number("stop", 0);
+      hm->loop_times = (int)lp->number("times", 0);
+      VN_REQUIRE(ctx, hm->loop_start >= 0 && hm->loop_start < hm->loop_stop && hm->loop_stop <= n && hm->loop_times >= 1,
+                 "loop over layers %d .. %d, %d times, of %d layers", hm->loop_start, hm->loop_stop, hm->loop_times, n);
+    }
+  }
+  const int a = hm->loop_times ? hm->loop_start : n, b = hm->loop_times ? hm->loop_stop : n;
+  for (int i = 0; i < a; ++i) hm->runs.push_back({i, -1});
+  for (int t = 0; t < hm->loop_times; ++t)
+    for (int i = a; i < b; ++i) hm->runs.push_back({i, t});
+  for (int i = b; i < n; ++i) hm->runs.push_back({i, -1});
+  return VN_OK;
+}
+
+int32_t zalloc(vn_model* m, void** p, size_t bytes) {
+  TRY(dev_alloc(m->ctx, p, bytes));
+  m->param_bytes += bytes;
+  VN_CUDA(m->ctx, cudaMemsetAsync(*p, 0, bytes ? bytes : 16, m->ctx->stream));
+  return VN_OK;
+}
+
+int32_t alloc(vn_model* m) {
+  Model& hm = *m->hyb;
+  const size_t e = m->esz, D = hm.D;
+  auto W = [&](void** p, size_t n) { return zalloc(m, p, n * e); };
+  auto F = [&](float** p, size_t n) { return zalloc(m, (void**)p, n * 4); };
+  TRY(W(&m->emb, hm.vocab * D));
+  TRY(W(&m->head, hm.vocab * D));
+  TRY(F(&m->norm_f, D));
+  TRY(dev_alloc(m->ctx, (void**)&m->status, 4));
+  VN_CUDA(m->ctx, cudaMemsetAsync(m->status, 0, 4, m->ctx->stream));
+  hm.want = {"embed", "head", "final.norm"};
+  if (hm.loop_times) {
+    TRY(W(&hm.w_loop, D * 2 * D));
+    TRY(F(&hm.loop_step, hm.loop_times * D));
+    hm.want.insert("loop.in"); hm.want.insert("loop.step");
+  }
+  if (hm.sinusoidal) {
+    std::vector<double> f((D + 1) / 2);
+    for (size_t i = 0; i < f.size(); ++i) f[i] = pow(10000.0, -2.0 * (double)i / (double)D);
+    TRY(dev_alloc(m->ctx, (void**)&hm.freq, f.size() * 8));
+    VN_CUDA(m->ctx, cudaMemcpyAsync(hm.freq, f.data(), f.size() * 8, cudaMemcpyHostToDevice, m->ctx->stream));
+    VN_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));
+  }
+  for (size_t i = 0; i < hm.layers.size(); ++i) {
+    HLayer& L = hm.layers[i];
+    const std::string p = "l" + std::to_string(i) + ".";
+    auto need = [&](std::initializer_list<const char*> names) { for (const char* s : names) hm.want.insert(p + s); };
+    TRY(F(&L.norm1, D));
+    TRY(W(&L.w_in, (size_t)L.n_in * D));
+    need({"norm1", "mix.o"});
+    if (L.kind == LATENT) {
+      TRY(W(&L.w_uk, (size_t)L.H * L.Rp * L.dp));
+      TRY(W(&L.w_uv, (size_t)L.H * L.vd * L.Rp));
+      TRY(W(&L.w_o, D * L.H * L.vd));
+      TRY(F(&L.f_a, L.R));
+      TRY(F(&L.f_b, L.H));
+      need({"mix.q", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv", "mix.sink", "mix.g"});
+    } else if (L.kind == MAMBA1) {
+      TRY(W(&L.w_uk, (size_t)L.inner * L.dtp));
+      TRY(W(&L.w_uv, (size_t)L.n_x * L.inner));
+      TRY(W(&L.w_o, D * L.inner));
+      TRY(F(&L.f_a, (size_t)L.inner * L.nstate));
+      TRY(F(&L.f_b, L.inner));
+      TRY(F(&L.f_c, L.inner));
+      TRY(F(&L.conv, (size_t)L.inner * L.taps));
+      TRY(F(&L.conv_b, L.inner));
+      need({"mix.in", "mix.conv", "mix.conv.b", "mix.x", "mix.dt", "mix.dt.b", "mix.A_log", "mix.D"});
+    } else {
+      TRY(W(&L.w_uk, (size_t)L.H * L.d * L.rap));
+      TRY(W(&L.w_uv, (size_t)L.H * L.vd * L.rgp));
+      TRY(W(&L.w_o, D * L.H * L.vd));
+      TRY(F(&L.f_a, L.vd));
+      TRY(F(&L.f_b, L.H));
+      TRY(F(&L.f_c, (size_t)L.H * L.d));
+      TRY(F(&L.conv, (size_t)L.conv_ch() * L.taps));
+      need({"mix.q", "mix.q.conv", "mix.k", "mix.k.conv", "mix.v", "mix.v.conv", "mix.b", "mix.A_log", "mix.norm", "mix.a1",
+            "mix.a2", "mix.dt_bias", "mix.g1", "mix.g2"});
+    }
+    if (L.ff) {
+      TRY(F(&L.norm2, D));
+      TRY(W(&L.w_gu, (size_t)2 * L.ffp * D));
+      TRY(W(&L.w_down, D * L.ffp));
+      need({"norm2", "mlp.gate", "mlp.up", "mlp.down"});
+    }
+  }
+  return VN_OK;
+}
+
+void destroy(vn_model* m) {
+  if (!m->hyb) return;
+  auto F = [](void* p) { if (p) cudaFree(p); };
+  Model& hm = *m->hyb;
+  for (auto& L : hm.layers) {
+    F(L.norm1); F(L.norm2); F(L.w_in); F(L.w_o); F(L.w_uk); F(L.w_uv); F(L.f_a); F(L.f_b); F(L.f_c); F(L.conv); F(L.conv_b);
+    F(L.w_gu); F(L.w_down);
+  }
+  F(hm.w_loop); F(hm.loop_step); F(hm.freq); F(hm.x0); F(hm.cat); F(hm.ws); F(hm.meta);
+  delete m->hyb;
+  m->hyb = nullptr;
+}
+
+// ---- weights: checkpoint names to their places in the stacked, padded matrices -----------------------------------
+int32_t load(vn_model* m, const std::string& n, const float* data, long long r, long long cl) {
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  const long long D = hm.D;
+  int32_t st = VN_OK;
+  // expected shape; a vector is (n, 1)
+  auto shape = [&](long long er, long long ec) -> bool {
+    if (r == er && cl == ec) return true;
+    st = vn_fail(ctx, VN_ERR_INVALID, "%s: shape (%lld, %lld) expected (%lld, %lld)", n.c_str(), r, cl, er, ec);
+    return false;
+  };
+  auto rows = [&](void* dst, long long ld, long long row_off = 0, long long row_mul = 1) {
+    return upload(m, data, dst, r, cl, ld, row_mul, row_off);
+  };
+  auto f32 = [&](const float* src, float* dst, long long count) { return upload(m, src, dst, 1, count, count, 1, 0, true); };
+  std::vector<float> tmp;
+  auto mapped = [&](float* dst, long long count, float (*fn)(float)) {
+    tmp.resize(count);
+    for (long long i = 0; i < count; ++i) tmp[i] = fn(data[i]);
+    return f32(tmp.data(), dst, count);
+  };
+  auto one_plus = [](float w) { return 1.0f + w; };
+  auto rate = [](float a) { return expf(a); };
+  auto neg_rate = [](float a) { return -expf(a); };
+  if (!hm.want.count(n)) return vn_fail(ctx, VN_ERR_INVALID, "unexpected tensor %s", n.c_str());
+#define PUT(er, ec, expr) do { if (!shape((er), (ec))) return st; TRY(expr); return VN_OK; } while (0)
+  if (n == "embed") PUT(hm.vocab, D, rows(m->emb, D));
+  if (n == "head") PUT(hm.vocab, D, rows(m->head, D));
+  if (n == "final.norm") PUT(D, 1, mapped(m->norm_f, D, one_plus));
+  if (n == "loop.in") PUT(D, 2 * D, rows(hm.w_loop, 2 * D));
+  if (n == "loop.step") PUT(hm.loop_times, D, f32(data, hm.loop_step, r * cl));
+  const size_t dot = n.find('.');
+  HLayer& L = hm.layers[atoi(n.substr(1, dot - 1).c_str())];      // the name is in `want`: the layer exists
+  const std::string s = n.substr(dot + 1);
+  if (s == "norm1") PUT(D, 1, mapped(L.norm1, D, one_plus));
+  if (s == "norm2") PUT(D, 1, mapped(L.norm2, D, one_plus));
+  if (s == "mlp.gate") PUT(L.ff, D, rows(L.w_gu, D, 0, 2));
+  if (s == "mlp.up") PUT(L.ff, D, rows(L.w_gu, D, 1, 2));
+  if (s == "mlp.down") PUT(D, L.ff, rows(L.w_down, L.ffp));
+  if (L.kind == LATENT) {
+    const long long hd = (long long)L.H * L.d, hv = (long long)L.H * L.vd;
+    if (s == "mix.q") PUT(hd, D, rows(L.w_in, D));
+    if (s == "mix.dkv") PUT(L.R, D, rows(L.w_in, D, hd));
+    if (s == "mix.g") PUT(L.H, D, rows(L.w_in, D, hd + L.R));
+    if (s == "mix.dkv.norm") PUT(L.R, 1, f32(data, L.f_a, L.R));
+    if (s == "mix.sink") PUT(L.H, 1, f32(data, L.f_b, L.H));
+    if (s == "mix.uv") PUT(hv, L.R, rows(L.w_uv, L.Rp));
+    if (s == "mix.o") PUT(D, hv, rows(L.w_o, hv));
+    if (s == "mix.uk") {          // stored per head as [d, R], used as its transpose
+      if (!shape(hd, L.R)) return st;
+      tmp.assign((size_t)L.H * L.Rp * L.dp, 0.f);
+      for (long long h = 0; h < L.H; ++h)
+        for (long long i = 0; i < L.d; ++i)
+          for (long long c = 0; c < L.R; ++c) tmp[(h * L.Rp + c) * L.dp + i] = data[(h * L.d + i) * L.R + c];
+      return upload(m, tmp.data(), L.w_uk, (long long)L.H * L.Rp, L.dp, L.dp);
+    }
+  } else if (L.kind == MAMBA1) {
+    if (s == "mix.in") PUT(2ll * L.inner, D, rows(L.w_in, D));
+    if (s == "mix.conv") PUT(L.inner, L.taps, f32(data, L.conv, r * cl));
+    if (s == "mix.conv.b") PUT(L.inner, 1, f32(data, L.conv_b, r));
+    if (s == "mix.x") {           // dt rows first, B and C behind the padded dt block
+      if (!shape(L.dt_rank + 2ll * L.nstate, L.inner)) return st;
+      TRY(upload(m, data, L.w_uv, L.dt_rank, L.inner, L.inner));
+      return upload(m, data + (long long)L.dt_rank * L.inner, L.w_uv, 2ll * L.nstate, L.inner, L.inner, 1, L.dtp);
+    }
+    if (s == "mix.dt") PUT(L.inner, L.dt_rank, rows(L.w_uk, L.dtp));
+    if (s == "mix.dt.b") PUT(L.inner, 1, f32(data, L.f_c, r));
+    if (s == "mix.A_log") PUT(L.inner, L.nstate, mapped(L.f_a, r * cl, neg_rate));
+    if (s == "mix.D") PUT(L.inner, 1, f32(data, L.f_b, r));
+    if (s == "mix.o") PUT(D, L.inner, rows(L.w_o, L.inner));
+  } else {
+    const long long kd = (long long)L.KH * L.d, hv = (long long)L.H * L.vd, b0 = 2 * kd + hv;
+    if (s == "mix.q") PUT(kd, D, rows(L.w_in, D));
+    if (s == "mix.k") PUT(kd, D, rows(L.w_in, D, kd));
+    if (s == "mix.v") PUT(hv, D, rows(L.w_in, D, 2 * kd));
+    if (s == "mix.b") PUT(L.H, D, rows(L.w_in, D, b0));
+    if (s == "mix.a1") PUT(L.ra, D, rows(L.w_in, D, b0 + L.H));
+    if (s == "mix.g1") PUT(L.rg, D, rows(L.w_in, D, b0 + L.H + L.ra));
+    if (s == "mix.q.conv") PUT(kd, L.taps, f32(data, L.conv, r * cl));
+    if (s == "mix.k.conv") PUT(kd, L.taps, f32(data, L.conv + kd * L.taps, r * cl));
+    if (s == "mix.v.conv") PUT(hv, L.taps, f32(data, L.conv + 2 * kd * L.taps, r * cl));
+    if (s == "mix.a2") PUT((long long)L.H * L.d, L.ra, rows(L.w_uk, L.rap));
+    if (s == "mix.g2") PUT(hv, L.rg, rows(L.w_uv, L.rgp));
+    if (s == "mix.A_log") PUT(L.H, 1, mapped(L.f_b, r, rate));
+    if (s == "mix.dt_bias") PUT((long long)L.H * L.d, 1, f32(data, L.f_c, r));
+    if (s == "mix.norm") PUT(L.vd, 1, f32(data, L.f_a, r));
+    if (s == "mix.o") PUT(D, hv, rows(L.w_o, hv));
+  }
+#undef PUT
+  return vn_fail(ctx, VN_ERR_INVALID, "unexpected tensor %s", n.c_str());
+}
+
+int32_t finalize(vn_model* m) {
+  for (auto& w : m->hyb->want)
+    if (!m->loaded.count(w)) return vn_fail(m->ctx, VN_ERR_INVALID, "missing tensor %s", w.c_str());
+  m->finalized = true;
+  return VN_OK;
+}
+
+// ---- activations ---------------------------------------------------------------------------------------------------
+int32_t ensure(vn_model* m, int M) {
+  if (M <= m->cap_rows) return VN_OK;
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+  m->cap_rows = 0;
+  void** bufs[] = {(void**)&m->x, &m->h, (void**)&m->row_seg, (void**)&hm.x0, &hm.cat, (void**)&hm.ws};
+  for (void** b : bufs) { if (*b) cudaFree(*b); *b = nullptr; }
+  const size_t R = (size_t)M + (M >> 2) + 32, D = hm.D, e = m->esz;
+  TRY(dev_alloc(ctx, (void**)&m->x, R * D * 4));
+  TRY(dev_alloc(ctx, &m->h, R * D * e));
+  m->row_seg_cap = (int)(R / 256 + 2);
+  TRY(dev_alloc(ctx, (void**)&m->row_seg, (size_t)2 * m->row_seg_cap * sizeof(int)));
+  TRY(dev_alloc(ctx, (void**)&hm.x0, R * D * 4));
+  if (hm.loop_times) TRY(dev_alloc(ctx, &hm.cat, R * 2 * D * e));
+  size_t need = 0;
+  for (auto& L : hm.layers)
+    for (size_t rows : {R, std::min(R, (size_t)SPLIT_ROWS)}) {
+      Arena A;
+      Buffers b;
+      layout(hm, L, rows, e, A, b);
+      need = std::max(need, A.off);
+    }
+  TRY(dev_alloc(ctx, (void**)&hm.ws, need));
+  hm.ws_bytes = need;
+  m->cap_rows = (int)R;
+  return VN_OK;
+}
+
+// ---- projections -----------------------------------------------------------------------------------------------------
+bool tc_rows(const vn_model* m, const GemmArgs& g) {
+  return m->cfg.bf16 && m->use_tc && g.M <= 256 && g.N % 4 == 0 && gemm_tc_supported(g);
+}
+GemmArgs gemm_args(const void* A, int lda, const void* W, int N, int K, int M, const char* tag) {
+  GemmArgs g;
+  g.A = A; g.lda = lda; g.W = W; g.ldw = K; g.M = M; g.N = N; g.K = K; g.tag = tag;
+  return g;
+}
+// out = A W^T in fp32: split-K slices in the workspace, or the matrix `direct`
+int32_t project(vn_model* m, GemmArgs g, float* direct, Src* out) {
+  *out = Src();
+  out->ld = g.N;
+  if (tc_rows(m, g)) {
+    int sp = 1;
+    TRY(tc_partial(m, g, g.M, g.M, &sp));
+    out->p = m->partial; out->splits = sp; out->pstride = (long long)g.M * g.N;
+    return VN_OK;
+  }
+  g.C = direct; g.ldc = g.N;
+  out->p = direct;
+  return linear(m, g);
+}
+// x += A W^T; then h = RMSNorm(x) * next_norm when given
+template <typename T>
+int32_t close_block(vn_model* m, GemmArgs g, const float* next_norm) {
+  vn_ctx* ctx = m->ctx;
+  const Model& hm = *m->hyb;
+  const int D = hm.D, M = g.M;
+  if (tc_rows(m, g)) {
+    int sp = 1;
+    TRY(tc_partial(m, g, M, M, &sp));
+    if (D % 4 == 0 && D <= 2048) {
+      VN_LAUNCH_PDL_BIT(ctx, 4, splitk_add_norm_kernel<T>, M, 256, 0, m->partial, sp, (long long)M * D, m->x, next_norm,
+                        (T*)m->h, (float*)nullptr, D, hm.eps);
+    } else {
+      Src s;
+      s.p = m->partial; s.splits = sp; s.pstride = (long long)M * D; s.ld = D;
+      VN_LAUNCH(ctx, rowsum_norm_kernel<T>, M, 256, 0, s, (const float*)nullptr, 1, m->x, next_norm, (T*)m->h, D, hm.eps);
+    }
+    return VN_OK;
+  }
+  g.C = m->x; g.ldc = D; g.epi = EPI_ADD;
+  TRY(linear(m, g));
+  if (next_norm)
+    VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, next_norm, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
+  return VN_OK;
+}
+// nseg products of equal shape, one per head
+int32_t batched(vn_model* m, const GemmArgs& g) {
+  if (m->cfg.bf16 && gemm_mma_supported(g)) return launch_gemm_mma(m->ctx, g);
+  if (m->cfg.bf16) return launch_gemm_simt<__nv_bfloat16, __nv_bfloat16>(m->ctx, g);
+  return launch_gemm_simt<float, float>(m->ctx, g);
+}
+
+// ---- mixers: m->h -> the input of the output projection -----------------------------------------------------------
+template <typename T>
+int32_t latent_attention(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+  vn_ctx* ctx = m->ctx;
+  const int M = rows.M, D = m->hyb->D, H = L.H;
+  Src s;
+  TRY(project(m, gemm_args(m->h, D, L.w_in, L.n_in, D, M, "gemm_latent_in"), b.proj, &s));
+  VN_LAUNCH(ctx, latent_append_kernel<T>, M, 256, (size_t)L.R * 4, s, H, L.d, L.dp, L.R, L.Rp, L.f_a, m->hyb->eps, (T*)b.q,
+            b.gate, (T*)kv->k[run], hc.table_dev, hc.max_pages, rows);
+  GemmArgs g = gemm_args(b.q, H * L.dp, L.w_uk, L.Rp, L.dp, M, "gemm_latent_uk");
+  g.C = b.qc; g.ldc = (long long)H * L.Rp; g.c_bf16 = m->cfg.bf16;
+  g.nseg = H; g.a_stride = L.dp; g.w_stride = (long long)L.Rp * L.dp; g.c_stride = L.Rp;
+  TRY(batched(m, g));
+  LatentArgs a;
+  a.qc = b.qc; a.plane = kv->k[run]; a.table = hc.table_dev; a.max_pages = hc.max_pages; a.Rp = L.Rp; a.H = H;
+  a.window = L.window; a.scale = L.scale; a.sink = L.f_b; a.gate = b.gate; a.out = b.oc; a.rows = rows;
+  const bool mma = m->cfg.bf16 && L.Rp <= 512 && !m->force_simt_attn;
+  if (mma && M <= SPLIT_ROWS) {       // few rows: several CTAs share a tile's key pages
+    const int tile = latent_tile_rows(L.Rp, rows.max_n * H), tiles = rows.n_ent * ceil_div(rows.max_n * H, tile);
+    const int pages = L.window > 0 ? std::min(hc.max_pages, (L.window + rows.max_n) / KV_PAGE + 2) : hc.max_pages;
+    a.splits = std::max(1, std::min(std::min(MAX_SPLITS, pages / 2), 2 * ctx->sm_count / std::max(1, tiles)));
+    a.part_o = b.part_o; a.part_ml = b.part_ml;
+  }
+  TRY(vn_latent_attention(ctx, a, m->cfg.bf16 != 0, mma));
+  g = gemm_args(b.oc, H * L.Rp, L.w_uv, L.vd, L.Rp, M, "gemm_latent_uv");
+  g.C = b.mix; g.ldc = (long long)H * L.vd; g.c_bf16 = m->cfg.bf16;
+  g.nseg = H; g.a_stride = L.Rp; g.w_stride = (long long)L.vd * L.Rp; g.c_stride = L.vd;
+  return batched(m, g);
+}
+
+template <typename T>
+ConvIn<T> conv_in(const HLayer& L, const Cache& hc, const Src& s, void* ring) {
+  ConvIn<T> c;
+  c.src = s; c.ring = (T*)ring; c.RC = L.taps - 1 + hc.pending; c.C = L.conv_ch(); c.taps = L.taps; c.w = L.conv; c.bias = L.conv_b;
+  return c;
+}
+
+template <typename T>
+int32_t mamba1(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+  vn_ctx* ctx = m->ctx;
+  const int M = rows.M, D = m->hyb->D, n = L.inner;
+  Src s;
+  TRY(project(m, gemm_args(m->h, D, L.w_in, L.n_in, D, M, "gemm_mamba_in"), b.proj, &s));
+  const ConvIn<T> cv = conv_in<T>(L, hc, s, kv->k[run]);
+  VN_LAUNCH(ctx, mamba_conv_kernel<T>, dim3(ceil_div(n, 32), ceil_div(M, 8)), dim3(32, 8), 0, cv, rows, (T*)b.xc, (T*)b.z, hc.pending);
+  if (rows.max_n > hc.pending)
+    VN_LAUNCH(ctx, conv_tail_kernel<T>, dim3(ceil_div(n, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
+  MambaArgs a;
+  TRY(project(m, gemm_args(b.xc, n, L.w_uv, L.n_x, n, M, "gemm_mamba_x"), b.p, &a.p));
+  a.xc = b.xc; a.z = b.z; a.dt_cols = L.dtp; a.dt_rank = L.dt_rank; a.w_dt = L.w_uk; a.dt_bias = L.f_c; a.A = L.f_a; a.D = L.f_b;
+  a.state = (float*)kv->v[run]; a.R = hc.ring; a.inner = n; a.nstate = L.nstate; a.out = b.mix; a.rows = rows;
+  if (rows.max_n == 1) {
+    TRY(vn_mamba_step(ctx, a, m->cfg.bf16 != 0));
+    return VN_OK;
+  }
+  VN_LAUNCH(ctx, cast_cols_kernel<T>, M, 64, 0, a.p, 0, L.dt_rank, (T*)b.dtb, L.dtp);
+  GemmArgs g = gemm_args(b.dtb, L.dtp, L.w_uk, n, L.dtp, M, "gemm_mamba_dt");
+  g.C = b.dt; g.ldc = n;
+  TRY(linear(m, g));
+  a.dt = b.dt;
+  return vn_mamba_scan(ctx, a, m->cfg.bf16 != 0);
+}
+
+template <typename T>
+int32_t channel_delta(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+  vn_ctx* ctx = m->ctx;
+  const int M = rows.M, D = m->hyb->D, H = L.H, KH = L.KH, d = L.d, vd = L.vd;
+  Src s;
+  TRY(project(m, gemm_args(m->h, D, L.w_in, L.n_in, D, M, "gemm_delta_in"), b.proj, &s));
+  const ConvIn<T> cv = conv_in<T>(L, hc, s, kv->k[run]);
+  DeltaIn in;
+  in.src = s; in.H = H; in.KH = KH; in.d = d; in.vd = vd; in.ra = L.ra; in.rg = L.rg; in.ra_ld = L.rap; in.rg_ld = L.rgp;
+  in.col_b = 2 * KH * d + H * vd; in.col_a = in.col_b + H; in.col_g = in.col_a + L.ra;
+  in.q = b.dq; in.k = b.dk; in.v = b.dv; in.beta = b.beta; in.low_a = b.low_a; in.low_g = b.low_g;
+  in.rows = rows; in.pending = hc.pending;
+  if (rows.max_n == 1) {
+    DeltaStepArgs<T> a;
+    a.conv = cv; a.in = in; a.w_a = (const T*)L.w_uk; a.w_g = (const T*)L.w_uv; a.decay_rate = L.f_b; a.dt_bias = L.f_c;
+    a.norm_w = L.f_a; a.state = (float*)kv->v[run]; a.R = hc.ring; a.eps = m->hyb->eps; a.out = (T*)b.mix;
+    TRY(vn_delta_step(ctx, a));
+    return VN_OK;
+  }
+  TRY(vn_delta_inputs(ctx, cv, in));
+  if (rows.max_n > hc.pending)
+    VN_LAUNCH(ctx, conv_tail_kernel<T>, dim3(ceil_div(cv.C, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
+  GemmArgs g = gemm_args(b.low_a, L.rap, L.w_uk, H * d, L.rap, M, "gemm_delta_a2");
+  g.C = b.g; g.ldc = H * d;
+  TRY(linear(m, g));
+  const long long ng = (long long)M * H * d;
+  VN_LAUNCH(ctx, delta_decay_kernel, (unsigned)ceil_div(ng, 256ll), 256, 0, b.g, L.f_b, L.f_c, ng, H, d);
+  g = gemm_args(b.low_g, L.rgp, L.w_uv, H * vd, L.rgp, M, "gemm_delta_g2");
+  g.C = b.gg; g.ldc = H * vd;
+  TRY(linear(m, g));
+  DeltaRuleArgs a;
+  a.q = b.dq; a.k = b.dk; a.v = b.dv; a.g = b.g; a.beta = b.beta; a.o = b.o; a.state = (float*)kv->v[run];
+  a.R = hc.ring; a.H = H; a.KH = KH; a.d = d; a.vd = vd; a.rows = rows;
+  TRY(vn_delta_scan(ctx, a));
+  const long long nh = (long long)M * H;
+  VN_LAUNCH(ctx, delta_out_kernel<T>, (unsigned)ceil_div(nh, 8ll), 256, 0, b.o, b.gg, L.f_a, (T*)b.mix, nh, vd, m->hyb->eps);
+  return VN_OK;
+}
+
+// ---- the forward ---------------------------------------------------------------------------------------------------
+// where the output rows come from: all rows, the entries' last rows of a uniform batch, or a list (device)
+struct Pick { const int* list = nullptr; int n = 0, mul = 1, add = 0; };
+
+template <typename T>
+int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows, const Pick& pick, float* out_hidden,
+                float* out_logits) {
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  Cache& hc = *kv->hyb;
+  const int M = rows.M, D = hm.D, n_runs = (int)hm.runs.size();
+  TRY(ensure_partial(m, 1024));
+  VN_LAUNCH(ctx, embed_pos_kernel<T>, M, 256, 0, (const long long*)tokens, (const T*)m->emb, hm.freq, m->x, hm.x0, rows, D,
+            hm.vocab, m->status);
+  auto enters_pass = [&](int i) { return i < n_runs && hm.runs[i].pass >= 0 && hm.runs[i].layer == hm.loop_start; };
+  for (int i = 0; i < n_runs; ++i) {
+    const HLayer& L = hm.layers[hm.runs[i].layer];
+    Arena A;
+    Buffers b;
+    A.base = hm.ws;
+    layout(hm, L, M, m->esz, A, b);
+    if (enters_pass(i)) {
+      // x = W [x | x0] + step vector of the pass, and the first layer's norm
+      VN_LAUNCH(ctx, concat_cast_kernel<T>, M, 256, 0, m->x, hm.x0, (T*)hm.cat, D);
+      Src s;
+      TRY(project(m, gemm_args(hm.cat, 2 * D, hm.w_loop, D, 2 * D, M, "gemm_loop_in"), b.proj, &s));
+      VN_LAUNCH(ctx, rowsum_norm_kernel<T>, M, 256, 0, s, hm.loop_step + (long long)hm.runs[i].pass * D, 0, m->x, L.norm1,
+                (T*)m->h, D, hm.eps);
+    } else if (i == 0) {
+      VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, L.norm1, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
+    }
+    const float* next_norm = i + 1 < n_runs && !enters_pass(i + 1) ? hm.layers[hm.runs[i + 1].layer].norm1 : nullptr;
+    if (L.kind == LATENT) TRY(latent_attention<T>(m, kv, hc, L, i, rows, b));
+    else if (L.kind == MAMBA1) TRY(mamba1<T>(m, kv, hc, L, i, rows, b));
+    else TRY(channel_delta<T>(m, kv, hc, L, i, rows, b));
+    const int width = L.kind == MAMBA1 ? L.inner : L.H * L.vd;
+    TRY(close_block<T>(m, gemm_args(b.mix, width, L.w_o, D, width, M, "gemm_mix_out"), L.ff ? L.norm2 : next_norm));
+    if (L.ff) {
+      GemmArgs g = gemm_args(m->h, D, L.w_gu, 2 * L.ffp, D, M, "gemm_ff_gateup");
+      if (tc_rows(m, g)) {
+        int sp = 1;
+        TRY(tc_partial(m, g, M, M, &sp));
+        const long long pairs = (long long)M * L.ffp;
+        VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp,
+                          (long long)M * 2 * L.ffp, (T*)b.act, 2 * L.ffp, pairs, L.act);
+      } else {
+        g.C = b.act; g.ldc = L.ffp; g.epi = EPI_SWIGLU; g.act = L.act; g.c_bf16 = m->cfg.bf16;
+        TRY(linear(m, g));
+      }
+      TRY(close_block<T>(m, gemm_args(b.act, L.ffp, L.w_down, D, L.ffp, M, "gemm_ff_down"), next_norm));
+    }
+    if (hm.probe)
+      VN_CUDA(ctx, cudaMemcpyAsync(hm.probe + (size_t)i * M * D, m->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, ctx->stream));
+  }
+  if (pick.n == 0) return VN_OK;
+  if (pick.list)
+    VN_LAUNCH(ctx, rmsnorm_pick_kernel<T>, pick.n, 256, 0, m->x, m->norm_f, (T*)m->h, out_hidden, pick.list, 1, 0, D, hm.eps);
+  else
+    VN_LAUNCH(ctx, rmsnorm_kernel<T>, pick.n, 256, 0, m->x, m->norm_f, (T*)m->h, out_hidden, pick.mul, pick.add, D, hm.eps);
+  if (out_logits) {
+    GemmArgs g = gemm_args(m->h, D, m->head, hm.vocab, D, pick.n, "gemm_head");
+    g.C = out_logits; g.ldc = hm.vocab;
+    if (tc_rows(m, g)) {
+      TcPlan direct;
+      direct.error_flag = m->tc_error;
+      return tc_launch(ctx, g, pick.n, direct);
+    }
+    return linear(m, g);
+  }
+  return VN_OK;
+}
+
+// ---- cache -----------------------------------------------------------------------------------------------------------
+int32_t push_table(vn_ctx* ctx, Cache& hc, int slot) {
+  VN_CUDA(ctx, cudaMemcpyAsync(hc.table_dev + (size_t)slot * hc.max_pages, hc.table.data() + (size_t)slot * hc.max_pages,
+                               (size_t)hc.max_pages * 4, cudaMemcpyHostToDevice, ctx->stream));
+  return VN_OK;
+}
+
+int32_t cache_create(vn_model* m, vn_kv* kv, int pool_tokens, int pending) {
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  Cache* hc = kv->hyb = new Cache();
+  hc->pending = pending;
+  hc->ring = pending + 1;
+  hc->slots = kv->max_batch;
+  hc->max_pages = ceil_div(kv->max_seq, KV_PAGE);
+  hc->pooled = pool_tokens > 0;
+  hc->n_pages = hc->pooled ? ceil_div(pool_tokens, KV_PAGE) : hc->slots * hc->max_pages;
+  hc->table.assign((size_t)hc->slots * hc->max_pages, 0);
+  hc->used.assign(hc->slots, 0);
+  if (hc->pooled) {
+    for (int p = hc->n_pages - 1; p >= 0; --p) hc->free_pages.push_back(p);
+  } else {
+    for (size_t i = 0; i < hc->table.size(); ++i) hc->table[i] = (int)i;
+    hc->used.assign(hc->slots, hc->max_pages);
+  }
+  TRY(dev_alloc(ctx, (void**)&hc->table_dev, hc->table.size() * 4));
+  VN_CUDA(ctx, cudaMemcpyAsync(hc->table_dev, hc->table.data(), hc->table.size() * 4, cudaMemcpyHostToDevice, ctx->stream));
+  for (const Run& r : hm.runs) {
+    const HLayer& L = hm.layers[r.layer];
+    void *a = nullptr, *b = nullptr;
+    int32_t st;
+    if (L.kind == LATENT) {
+      st = dev_alloc(ctx, &a, (size_t)hc->n_pages * KV_PAGE * L.Rp * m->esz);
+    } else {
+      st = dev_alloc(ctx, &a, (size_t)hc->slots * (L.taps - 1 + pending) * L.conv_ch() * m->esz);
+      if (st == VN_OK) st = dev_alloc(ctx, &b, (size_t)hc->slots * hc->ring * L.state_elems() * 4);
+    }
+    kv->k.push_back(a); kv->v.push_back(b);
+    TRY(st);
+  }
+  VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+  return VN_OK;
+}
+
+void cache_free(vn_kv* kv) {
+  if (!kv->hyb || kv->parent) return;
+  if (kv->hyb->table_dev) cudaFree(kv->hyb->table_dev);
+  delete kv->hyb;
+  kv->hyb = nullptr;
+}
+
+// pages for `tokens` positions of a slot (pooled caches); *grew tells whether the device table is behind
+int32_t reserve(vn_ctx* ctx, Cache& hc, int slot, int tokens) {
+  const int need = ceil_div(tokens, KV_PAGE);
+  if (!hc.pooled || need <= hc.used[slot]) return VN_OK;
+  if (need - hc.used[slot] > (int)hc.free_pages.size())
+    return vn_fail(ctx, VN_ERR_OVERFLOW, "KV cache overflow: sequence %d needs %d more pages of %d tokens, the pool has %zu free",
+                   slot, need - hc.used[slot], KV_PAGE, hc.free_pages.size());
+  while (hc.used[slot] < need) {
+    hc.table[(size_t)slot * hc.max_pages + hc.used[slot]++] = hc.free_pages.back();
+    hc.free_pages.pop_back();
+  }
+  return push_table(ctx, hc, slot);
+}
+
+// a slot whose sequence is gone gives its pages back (later work of the stream may overwrite them)
+void release(Cache& hc, int slot) {
+  if (!hc.pooled) return;
+  while (hc.used[slot] > 0) hc.free_pages.push_back(hc.table[(size_t)slot * hc.max_pages + --hc.used[slot]]);
+}
+
+int32_t run_forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows, const Pick& pick, float* hidden, float* logits) {
+  TRY(ensure(m, rows.M));
+  if (m->cfg.bf16) return forward<__nv_bfloat16>(m, kv, tokens, rows, pick, hidden, logits);
+  return forward<float>(m, kv, tokens, rows, pick, hidden, logits);
+}
+
+// T new rows for sequences 0 .. B-1 of `kv` (a cache or a view); capacity has been checked
+int32_t forward_uniform(vn_model* m, vn_kv* kv, const int64_t* tokens, int B, int T, int slot_offset, float* hidden,
+                        float* logits, int last_only) {
+  vn_ctx* ctx = m->ctx;
+  Cache& hc = *kv->hyb;
+  VN_REQUIRE(ctx, slot_offset == 0 || slot_offset + T <= hc.pending,
+             "%d uncommitted rows, +%d: this cache keeps %d (max_pending)", slot_offset, T, hc.pending);
+  if (hc.pooled) {
+    // the host's bound on a length may be above it after cut-back appends: exact before a page is taken
+    bool grow = false;
+    for (int b = 0; b < B; ++b) grow |= ceil_div(kv_ub(kv, b) + slot_offset + T, KV_PAGE) > hc.used[kv->parent_first + b];
+    if (grow) { std::vector<int32_t> lens(kv->max_batch); TRY(vn_kv_lengths(kv, lens.data())); }
+    for (int b = 0; b < B; ++b) TRY(reserve(ctx, hc, kv->parent_first + b, kv_ub(kv, b) + slot_offset + T));
+  }
+  Rows r;
+  r.T = T; r.slot0 = kv->parent_first; r.off = slot_offset; r.n_ent = B; r.M = B * T; r.max_n = T;
+  r.lens = kv->lens - kv->parent_first;
+  Pick p;
+  if (last_only) { p.n = B; p.mul = T; p.add = T - 1; } else { p.n = B * T; }
+  return run_forward(m, kv, tokens, r, p, hidden, logits);
+}
+
+// a ragged batch: entry e brings counts[e] rows for sequence slots[e]; everything it appends is committed
+int32_t forward_ragged(vn_model* m, vn_kv* kv, const int64_t* tokens, int n_ent, const int* slots, const int* counts, int n_out,
+                       const int* out_rows, float* hidden, float* logits) {
+  vn_ctx* ctx = m->ctx;
+  Cache& hc = *kv->hyb;
+  Model& hm = *m->hyb;
+  int M = 0, max_n = 0;
+  std::vector<char> seen(kv->max_batch, 0);
+  for (int e = 0; e < n_ent; ++e) {
+    if (slots[e] < 0 || slots[e] >= kv->max_batch) return vn_fail(ctx, VN_ERR_INDEX, "sequence %d out of range (%d)", slots[e], kv->max_batch);
+    VN_REQUIRE(ctx, counts[e] >= 1 && !seen[slots[e]], "entry %d: no rows, or sequence %d named twice", e, slots[e]);
+    seen[slots[e]] = 1;
+    M += counts[e];
+    max_n = std::max(max_n, counts[e]);
+  }
+  bool exact = false;
+  for (int e = 0; e < n_ent; ++e) {
+    if (kv_ub(kv, slots[e]) + counts[e] > kv->max_seq && !exact) {
+      std::vector<int32_t> lens(kv->max_batch);
+      TRY(vn_kv_lengths(kv, lens.data()));
+      exact = true;
+    }
+    if (kv_ub(kv, slots[e]) + counts[e] > kv->max_seq)
+      return vn_fail(ctx, VN_ERR_OVERFLOW, "KV cache overflow: sequence %d holds %d, +%d exceeds the capacity %d", slots[e],
+                     kv_ub(kv, slots[e]), counts[e], kv->max_seq);
+  }
+  for (int i = 0; i < n_out; ++i) VN_REQUIRE(ctx, out_rows[i] >= 0 && out_rows[i] < M, "output row %d of %d", out_rows[i], M);
+  for (int e = 0; e < n_ent; ++e)
+    TRY(reserve(ctx, hc, kv->parent_first + slots[e], kv_ub(kv, slots[e]) + counts[e]));
+  // tables: slot, first row, rows of the entries; entry of each row; wanted rows
+  std::vector<int> t((size_t)3 * n_ent + M + n_out);
+  int *ts = t.data(), *tr = ts + n_ent, *tc = tr + n_ent, *te = tc + n_ent, *to = te + M;
+  for (int e = 0, r = 0; e < n_ent; ++e) {
+    ts[e] = kv->parent_first + slots[e]; tr[e] = r; tc[e] = counts[e];
+    for (int i = 0; i < counts[e]; ++i) te[r++] = e;
+  }
+  std::copy(out_rows, out_rows + n_out, to);
+  if ((int)t.size() > hm.meta_cap) {
+    VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    if (hm.meta) cudaFree(hm.meta);
+    hm.meta = nullptr; hm.meta_cap = 0;
+    TRY(dev_alloc(ctx, (void**)&hm.meta, t.size() * 2 * 4));
+    hm.meta_cap = (int)t.size() * 2;
+  }
+  VN_CUDA(ctx, cudaMemcpyAsync(hm.meta, t.data(), t.size() * 4, cudaMemcpyHostToDevice, ctx->stream));
+  Rows r;
+  r.n_ent = n_ent; r.M = M; r.max_n = max_n;
+  r.slot = hm.meta; r.row0 = r.slot + n_ent; r.cnt = r.row0 + n_ent; r.ent = r.cnt + n_ent;
+  r.lens = kv->lens - kv->parent_first;
+  Pick p;
+  p.list = r.ent + M; p.n = n_out;
+  TRY(run_forward(m, kv, tokens, r, p, hidden, logits));
+  VN_LAUNCH(ctx, rows_advance_kernel, ceil_div(n_ent, 128), 128, 0, r, kv->lens - kv->parent_first);
+  for (int e = 0; e < n_ent; ++e) kv_ub(kv, slots[e]) += counts[e];
+  return VN_OK;
+}
+
+}  // namespace hybrid

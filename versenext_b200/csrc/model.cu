@@ -134,6 +134,8 @@ struct Layer {
 
 }  // namespace
 
+namespace hybrid { struct Model; struct Cache; }   // composed models, hybrid.cuh
+
 struct vn_model {
   vn_ctx* ctx = nullptr;
   Config cfg;
@@ -185,6 +187,7 @@ struct vn_model {
   bool recurrent = false;        // vn_model_set_recurrent: ALiBi path as in the reference's one-token recurrent step
   bool fused_stack = false;      // vn_model_set_fused_stack / VN_DRAFT_STACK=1: the layer stack as one cooperative kernel
   bool use_tc = true;            // VN_GEMM_TC=0 in the environment: keep the mma.sync GEMMs
+  hybrid::Model* hyb = nullptr;  // set for a composed model: its layers live there, `layers` is empty
   bool force_simt_attn = false;  // VN_ATTN_SIMT=1 in the environment: keep the SIMT attention kernel (A/B checks)
 };
 
@@ -199,6 +202,7 @@ struct vn_kv {
   std::vector<int> len_ub;   // host upper bound of every length
   vn_kv* parent = nullptr;   // set for a view (vn_kv_view): planes and lengths belong to the parent
   int parent_first = 0;      // first sequence of the parent this view covers
+  hybrid::Cache* hyb = nullptr;  // composed models: pages, rings (shared with views); k / v hold one pair per layer run
 };
 
 // host upper bound of sequence b's length; a view shares its parent's record
@@ -320,7 +324,10 @@ int32_t alloc_weights(vn_model* m) {
   return VN_OK;
 }
 
+int32_t ensure_hybrid_rows(vn_model* m, int M);
+
 int32_t ensure_rows(vn_model* m, int M) {
+  if (m->hyb) return ensure_hybrid_rows(m, M);
   if (M <= m->cap_rows) return VN_OK;
   vn_ctx* ctx = m->ctx;
   const Config& c = m->cfg;
@@ -991,7 +998,7 @@ int32_t forward_tc(vn_model* m, vn_kv* kv, const int64_t* tokens, int B, int Tn,
         TRY(tc_partial(m, g, cap, M, &sp));
         const long long pairs = (long long)M * c.mlp_hidden;
         VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp,
-                  (long long)M * 2 * c.mlp_hidden, (T*)m->act, 2 * c.mlp_hidden, pairs);
+                  (long long)M * 2 * c.mlp_hidden, (T*)m->act, 2 * c.mlp_hidden, pairs, 0);
       }
       g = GemmArgs();
       g.A = m->act; g.lda = c.mlp_hidden; g.W = L.w_down; g.ldw = c.mlp_hidden; g.M = M; g.N = D; g.K = c.mlp_hidden;
@@ -1240,6 +1247,29 @@ struct NameRoute { int layer; std::string rest; };
 
 }  // namespace
 
+extern "C" int32_t vn_kv_lengths(vn_kv* kv, int32_t* out_host);
+#include "hybrid.cuh"
+
+namespace {
+int32_t ensure_hybrid_rows(vn_model* m, int M) { return hybrid::ensure(m, M); }
+
+int32_t create_hybrid(vn_ctx* ctx, const std::string& config, vn_model** out) {
+  JsonValue j;
+  VN_REQUIRE(ctx, JsonReader::parse(config, &j), "malformed model configuration");
+  vn_model* m = new vn_model();
+  m->ctx = ctx;
+  m->hyb = new hybrid::Model();
+  int32_t st = hybrid::parse(ctx, j, m->hyb, &m->cfg);
+  m->esz = m->cfg.bf16 ? 2 : 4;
+  { const char* e = getenv("VN_ATTN_SIMT"); m->force_simt_attn = e && e[0] == '1'; }
+  { const char* e = getenv("VN_GEMM_TC"); m->use_tc = !(e && e[0] == '0'); }
+  if (st == VN_OK) st = hybrid::alloc(m);
+  if (st != VN_OK) { vn_model_destroy(m); return st; }
+  *out = m;
+  return VN_OK;
+}
+}  // namespace
+
 extern "C" {
 
 int32_t vn_model_create(vn_ctx* ctx, const char* config_json, vn_model** out) {
@@ -1247,6 +1277,8 @@ int32_t vn_model_create(vn_ctx* ctx, const char* config_json, vn_model** out) {
   VN_REQUIRE(ctx, config_json && out, "null argument");
   *out = nullptr;
   const std::string s(config_json);
+  std::string family;
+  if (json_str(s, "family", &family) && family == "composed") return create_hybrid(ctx, s, out);
   Config c;
   double v;
   auto need = [&](const char* key, int* dst) -> bool { if (!json_num(s, key, &v)) return false; *dst = (int)v; return true; };
@@ -1319,6 +1351,7 @@ int32_t vn_model_destroy(vn_model* m) {
     for (auto& S : L.sub) { F(S.wqkv); F(S.w_up); F(S.sink); F(S.sink_k); F(S.sink_v); F(S.head_gate); F(S.head_w); F(S.w_abs); F(S.q[0]); F(S.q[1]); F(S.qs[0]); F(S.qs[1]); }
   for (auto& L : m->layers) F(L.w_vda);
   F(m->lat); F(m->mix);
+  hybrid::destroy(m);
   delete m;
   return VN_OK;
 }
@@ -1331,6 +1364,12 @@ int32_t vn_model_load_tensor(vn_model* m, const char* name, const float* data, i
   VN_REQUIRE(ctx, m->qmode == 0, "the model is quantised: its dense weights are gone, create a new model to reload");
   const Config& c = m->cfg;
   const std::string n(name);
+  if (m->hyb) {
+    TRY(hybrid::load(m, n, data, shape[0], ndim == 2 ? shape[1] : 1));
+    m->loaded.insert(n);
+    m->finalized = false;
+    return VN_OK;
+  }
   if (m->preq_mode) {
     LinearSlot ls;
     VN_REQUIRE(ctx, !locate_linear(m, n, &ls), "%s: this model takes its linears quantised (vn_model_load_quant_tensor)", name);
@@ -1440,6 +1479,7 @@ int32_t vn_model_finalize(vn_model* m) {
   if (!m) return vn_fail(nullptr, VN_ERR_INVALID, "null model");
   vn_ctx* ctx = m->ctx;
   VN_CHECK_CTX(ctx);
+  if (m->hyb) return hybrid::finalize(m);
   if (m->qmode) return VN_OK;   // nothing left to derive once the weights are quantised
   const Config& c = m->cfg;
   // every tensor of the reference's state_dict must have arrived (head.weight may be omitted when tied)
@@ -1847,17 +1887,34 @@ int32_t vn_model_status(vn_model* m, int32_t* bad_token, int32_t* wait_timeout) 
   if (bad_token) *bad_token = tok;
   if (wait_timeout) *wait_timeout = to;
   if (to) return vn_fail(ctx, VN_ERR_TIMEOUT, "a bounded wait inside a GEMM kernel ran out: results of the last forwards are undefined");
+  if (tok == 2) return vn_fail(ctx, VN_ERR_INVALID, "a commit cut back more rows than the cache keeps recurrent states for (max_pending)");
   if (tok) return vn_fail(ctx, VN_ERR_INDEX, "token id outside [0, %d) met by a forward (clamped on the device)", m->cfg.vocab);
   return VN_OK;
 }
 
 int32_t vn_kv_create(vn_model* m, int32_t max_batch, int32_t max_seq, vn_kv** out) {
+  return vn_kv_create_ex(m, max_batch, max_seq, 0, 1, out);
+}
+
+int32_t vn_kv_create_ex(vn_model* m, int32_t max_batch, int32_t max_seq, int32_t pool_tokens, int32_t max_pending, vn_kv** out) {
   if (!m || !out) return vn_fail(nullptr, VN_ERR_INVALID, "null argument");
   vn_ctx* ctx = m->ctx;
   VN_CHECK_CTX(ctx);
   VN_REQUIRE(ctx, max_batch >= 1 && max_seq >= 1, "max_batch and max_seq must be positive");
+  VN_REQUIRE(ctx, pool_tokens >= 0 && max_pending >= 1 && max_pending <= 64, "pool_tokens or max_pending out of range");
+  if (!m->hyb && pool_tokens)
+    return vn_fail(ctx, VN_ERR_UNSUPPORTED, "this model's cache is a fixed slab per sequence: no page pool");
   vn_kv* kv = new vn_kv();
   kv->m = m; kv->ctx = ctx; kv->max_batch = max_batch; kv->max_seq = max_seq;
+  if (m->hyb) {
+    int32_t st = hybrid::cache_create(m, kv, pool_tokens, max_pending);
+    if (st == VN_OK) st = dev_alloc(ctx, (void**)&kv->lens, (size_t)max_batch * 4);
+    if (st != VN_OK) { vn_kv_destroy(kv); return st; }
+    VN_CUDA(ctx, cudaMemsetAsync(kv->lens, 0, (size_t)max_batch * 4, ctx->stream));
+    kv->len_ub.assign(max_batch, 0);
+    *out = kv;
+    return VN_OK;
+  }
   const size_t plane = (size_t)max_batch * max_seq * m->cfg.n_kv * m->cfg.hd * m->esz;
   std::vector<void*> planes;
   for (int i = 0; i < m->n_pairs; ++i) {
@@ -1891,6 +1948,7 @@ int32_t vn_kv_destroy(vn_kv* kv) {
     for (void* p : kv->k) cudaFree(p);
     for (void* p : kv->v) cudaFree(p);
     if (kv->lens) cudaFree(kv->lens);
+    hybrid::cache_free(kv);
   }
   if (kv->planes_dev) cudaFree(kv->planes_dev);
   delete kv;
@@ -1908,6 +1966,12 @@ int32_t vn_kv_view(vn_kv* kv, int32_t first, int32_t count, vn_kv** out) {
   v->m = m; v->ctx = ctx; v->max_batch = count; v->max_seq = kv->max_seq;
   v->parent = kv->parent ? kv->parent : kv;
   v->parent_first = kv->parent_first + first;
+  if (m->hyb) {
+    v->hyb = kv->hyb; v->k = kv->k; v->v = kv->v;
+    v->lens = kv->lens + first;
+    *out = v;
+    return VN_OK;
+  }
   const size_t seq_bytes = (size_t)kv->max_seq * m->cfg.n_kv * m->cfg.hd * m->esz;
   std::vector<void*> planes;
   for (int i = 0; i < m->n_pairs; ++i) {
@@ -1937,6 +2001,18 @@ int32_t vn_kv_set_lengths(vn_kv* kv, const int32_t* lens_host) {
   if (!kv || !lens_host) return vn_fail(nullptr, VN_ERR_INVALID, "null argument");
   vn_ctx* ctx = kv->m->ctx;
   VN_CHECK_CTX(ctx);
+  if (kv->hyb) {
+    // the recurrent state of a sequence exists at its committed length (and at 0): nothing else can be set
+    std::vector<int32_t> now(kv->max_batch);
+    TRY(vn_kv_lengths(kv, now.data()));
+    for (int b = 0; b < kv->max_batch; ++b) {
+      if (lens_host[b] == now[b]) continue;
+      if (lens_host[b] != 0)
+        return vn_fail(ctx, VN_ERR_UNSUPPORTED, "sequence %d cannot be set from length %d to %d: its recurrent state is gone", b, now[b], lens_host[b]);
+      TRY(vn_kv_reset_seq(kv, b));
+    }
+    return VN_OK;
+  }
   for (int b = 0; b < kv->max_batch; ++b)
     if (lens_host[b] < 0 || lens_host[b] > kv->max_seq)
       return vn_fail(ctx, VN_ERR_OVERFLOW, "length %d of sequence %d outside [0, %d]", lens_host[b], b, kv->max_seq);
@@ -1951,6 +2027,8 @@ int32_t vn_kv_reset_seq(vn_kv* kv, int32_t seq) {
   vn_ctx* ctx = kv->m->ctx;
   VN_CHECK_CTX(ctx);
   if (seq >= kv->max_batch) return vn_fail(ctx, VN_ERR_INDEX, "sequence %d out of range (%d)", seq, kv->max_batch);
+  if (kv->hyb)
+    for (int b = seq < 0 ? 0 : seq; b < (seq < 0 ? kv->max_batch : seq + 1); ++b) hybrid::release(*kv->hyb, kv->parent_first + b);
   if (seq < 0) {
     VN_CUDA(ctx, cudaMemsetAsync(kv->lens, 0, (size_t)kv->max_batch * 4, ctx->stream));
     for (int b = 0; b < kv->max_batch; ++b) kv_ub(kv, b) = 0;
@@ -1970,6 +2048,7 @@ int32_t vn_kv_commit(vn_kv* kv, int32_t n_new, const int32_t* keep_idx_dev, int3
   VN_REQUIRE(ctx, n_new >= 0 && n_new <= 4096, "n_new out of range");
   const int B = kv->max_batch;
   if (n_new == 0) return VN_OK;
+  if (keep_idx_dev && m->hyb) return vn_fail(ctx, VN_ERR_UNSUPPORTED, "trees are not available for models with recurrent layers");
   if (keep_idx_dev) {
     VN_REQUIRE(ctx, stride >= 1, "stride must be positive");
     const int row_elems = m->cfg.n_kv * m->cfg.hd;
@@ -1988,7 +2067,8 @@ int32_t vn_kv_commit(vn_kv* kv, int32_t n_new, const int32_t* keep_idx_dev, int3
                 n_keep_dev, keep_add, n_new, kv->max_seq, row_elems);
     }
   }
-  VN_LAUNCH_PDL(ctx, kv_advance_kernel, ceil_div(B, 128), 128, 0, kv->lens, n_keep_dev, keep_add, n_new, kv->max_seq, B);
+  VN_LAUNCH_PDL(ctx, kv_advance_kernel, ceil_div(B, 128), 128, 0, kv->lens, n_keep_dev, keep_add, n_new, kv->max_seq, B,
+                kv->hyb ? kv->hyb->pending : n_new, m->status);
   for (int b = 0; b < B; ++b) kv_ub(kv, b) = std::min(kv_ub(kv, b) + n_new, kv->max_seq);
   return VN_OK;
 }
@@ -1998,6 +2078,7 @@ int32_t vn_kv_read(vn_kv* kv, int32_t layer, int32_t seq, int32_t which, float* 
   vn_model* m = kv->m;
   vn_ctx* ctx = m->ctx;
   VN_CHECK_CTX(ctx);
+  if (m->hyb) return vn_fail(ctx, VN_ERR_UNSUPPORTED, "a composed model's cache holds latents and states, not K / V planes");
   if (layer < 0 || layer >= m->n_pairs) return vn_fail(ctx, VN_ERR_INDEX, "layer %d out of range (%d)", layer, m->n_pairs);
   if (seq < 0 || seq >= kv->max_batch) return vn_fail(ctx, VN_ERR_INDEX, "sequence %d out of range (%d)", seq, kv->max_batch);
   VN_REQUIRE(ctx, n_positions >= 0 && n_positions <= kv->max_seq, "n_positions out of range");
@@ -2040,6 +2121,10 @@ int32_t vn_model_forward(vn_model* m, vn_kv* kv, const int64_t* tokens_dev, int3
                        lens[b] + slot_offset, T, limit);
   }
   const bool tree = parents_host != nullptr;
+  if (m->hyb) {
+    if (tree) return vn_fail(ctx, VN_ERR_UNSUPPORTED, "trees are not available for models with recurrent layers");
+    return hybrid::forward_uniform(m, kv, tokens_dev, B, T, slot_offset, out_hidden_dev, out_logits_dev, last_only);
+  }
   if (tree) {
     VN_REQUIRE(ctx, T <= 64, "a tree may have at most 64 nodes, got %d", T);
     std::vector<int> depth(T);
@@ -2074,6 +2159,34 @@ int32_t vn_model_forward(vn_model* m, vn_kv* kv, const int64_t* tokens_dev, int3
     return forward_tc(m, kv, tokens_dev, B, T, tree, out_hidden_dev, out_logits_dev, last_only, slot_offset);
   if (m->cfg.bf16) return forward_t<__nv_bfloat16>(m, kv, tokens_dev, B, T, tree, out_hidden_dev, out_logits_dev, last_only, slot_offset);
   return forward_t<float>(m, kv, tokens_dev, B, T, tree, out_hidden_dev, out_logits_dev, last_only, slot_offset);
+}
+
+int32_t vn_model_forward_ragged(vn_model* m, vn_kv* kv, const int64_t* tokens_dev, int32_t n_entries, const int32_t* slots_host,
+                                const int32_t* counts_host, int32_t n_out, const int32_t* out_rows_host, float* out_hidden_dev,
+                                float* out_logits_dev) {
+  if (!m || !kv) return vn_fail(nullptr, VN_ERR_INVALID, "null argument");
+  vn_ctx* ctx = m->ctx;
+  VN_CHECK_CTX(ctx);
+  VN_REQUIRE(ctx, m->finalized, "vn_model_finalize has not been called");
+  VN_REQUIRE(ctx, kv->m == m, "KV cache belongs to another model");
+  VN_REQUIRE(ctx, tokens_dev && slots_host && counts_host && n_entries >= 1 && n_out >= 0 && (n_out == 0 || out_rows_host), "bad arguments");
+  if (!m->hyb) return vn_fail(ctx, VN_ERR_UNSUPPORTED, "ragged batches need a composed model: run the entries through views of the cache");
+  return hybrid::forward_ragged(m, kv, tokens_dev, n_entries, slots_host, counts_host, n_out, out_rows_host, out_hidden_dev, out_logits_dev);
+}
+
+int32_t vn_model_set_probe(vn_model* m, float* probe_dev) {
+  if (!m) return vn_fail(nullptr, VN_ERR_INVALID, "null model");
+  if (!m->hyb) return vn_fail(m->ctx, VN_ERR_UNSUPPORTED, "the residual probe is available for composed models");
+  m->hyb->probe = probe_dev;
+  return VN_OK;
+}
+
+int32_t vn_kv_pages(vn_kv* kv, int32_t* total, int32_t* free_pages) {
+  if (!kv) return vn_fail(nullptr, VN_ERR_INVALID, "null argument");
+  if (!kv->hyb) return vn_fail(kv->ctx, VN_ERR_UNSUPPORTED, "this model's cache is a fixed slab per sequence");
+  if (total) *total = kv->hyb->n_pages;
+  if (free_pages) *free_pages = (int32_t)kv->hyb->free_pages.size();
+  return VN_OK;
 }
 
 int32_t vn_draft_propose(vn_model* draft, vn_kv* kv, const int64_t* pair_dev, int32_t B, int32_t k, float temperature,

@@ -4,14 +4,8 @@
 #pragma once
 #include "common.cuh"
 #include "gemm.cuh"
+#include "rows.cuh"
 #include <math_constants.h>
-
-template <typename T> __device__ __forceinline__ float to_f(T v);
-template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename T> __device__ __forceinline__ T from_f(float v);
-template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
 // ---- weight staging: fp32 host rows -> storage dtype, with a row map (dst_row = src_row * mul + off)
 template <typename T>
@@ -556,13 +550,15 @@ __global__ void kv_commit_kernel(T* const* __restrict__ planes, const int* __res
   }
 }
 
-__global__ void kv_advance_kernel(int* __restrict__ lens, const int* __restrict__ n_keep, int keep_add, int n_new, int max_seq, int B) {
+__global__ void kv_advance_kernel(int* __restrict__ lens, const int* __restrict__ n_keep, int keep_add, int n_new, int max_seq, int B,
+                                  int pending, int* __restrict__ status) {
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x * blockDim.x + threadIdx.x;
   if (b >= B) return;
   int nk = n_keep[b] + keep_add;
   nk = nk < 0 ? 0 : (nk > n_new ? n_new : nk);
+  if (n_new > pending && nk != n_new) atomicExch(status, 2);   // a state that cannot be cut back (recurrent layers)
   const int nl = lens[b] + nk;
   lens[b] = nl > max_seq ? max_seq : nl;
 }
@@ -650,10 +646,10 @@ __global__ void splitk_store_kernel(const float* __restrict__ partial, int split
   out[row * ld + n] = acc;
 }
 
-// act[row, j] = silu(sum_s partial[.., 2j]) * sum_s partial[.., 2j+1]
+// act[row, j] = f(sum_s partial[.., 2j]) * sum_s partial[.., 2j+1]
 template <typename T>
 __global__ void splitk_swiglu_kernel(const float* __restrict__ partial, int splits, long long pstride,
-                                     T* __restrict__ act, int N, long long total_pairs) {
+                                     T* __restrict__ act, int N, long long total_pairs, int fn) {
   pdl_trigger();
   pdl_wait();
   const int half = N / 2;
@@ -670,8 +666,8 @@ __global__ void splitk_swiglu_kernel(const float* __restrict__ partial, int spli
       const float4 t = *reinterpret_cast<const float4*>(p + (long long)s * pstride);
       acc.x += t.x; acc.y += t.y; acc.z += t.z; acc.w += t.w;
     }
-    act[row * half + j] = from_f<T>(silu_ref(acc.x) * acc.y);
-    act[row * half + j + 1] = from_f<T>(silu_ref(acc.z) * acc.w);
+    act[row * half + j] = from_f<T>(glu_act(acc.x, fn) * acc.y);
+    act[row * half + j + 1] = from_f<T>(glu_act(acc.z, fn) * acc.w);
     return;
   }
   for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 2, e = 0; e < 2 && i < total_pairs; ++e, ++i) {
@@ -682,7 +678,7 @@ __global__ void splitk_swiglu_kernel(const float* __restrict__ partial, int spli
       const float2 p = *reinterpret_cast<const float2*>(partial + (long long)s * pstride + row * N + 2 * j);
       g += p.x; u += p.y;
     }
-    act[row * half + j] = from_f<T>(silu_ref(g) * u);
+    act[row * half + j] = from_f<T>(glu_act(g, fn) * u);
   }
 }
 

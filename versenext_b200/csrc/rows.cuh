@@ -1,0 +1,99 @@
+// Device-side vocabulary of the row kernels: storage-type conversion, where a row of a (ragged) batch sits in its
+// sequence, sums over split-K slices, and the short causal convolution with its cached inputs.  No kernels here: the file
+// is included by several translation units.
+#pragma once
+#include "common.cuh"
+
+template <typename T> __device__ __forceinline__ float to_f(T v);
+template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// Rows of a forward.  Either a uniform batch (T > 0: entry e = sequence slot0 + e, rows [e*T, e*T + T)) or a ragged
+// one (T == 0: tables).  Row r of an entry that starts at row row0 has position lens[slot] + off + (r - row0).
+struct Rows {
+  int T = 0, slot0 = 0, off = 0, n_ent = 0, M = 0, max_n = 0;
+  const int* ent = nullptr;    // [M] entry of a row
+  const int* slot = nullptr;   // [n_ent]
+  const int* row0 = nullptr;   // [n_ent]
+  const int* cnt = nullptr;    // [n_ent]
+  const int* lens = nullptr;   // [slots] committed tokens
+
+  __device__ __forceinline__ int entry_of(int row) const { return T > 0 ? row / T : ent[row]; }
+  __device__ __forceinline__ void entry(int e, int* s, int* r0, int* n, int* start) const {
+    if (T > 0) { *s = slot0 + e; *r0 = e * T; *n = T; }
+    else { *s = slot[e]; *r0 = row0[e]; *n = cnt[e]; }
+    *start = lens[*s] + off;
+  }
+};
+
+// the fp32 result of a projection: one matrix, or split-K slices that the reader sums in slice order
+struct Src {
+  const float* p = nullptr;
+  int splits = 1;
+  long long pstride = 0;
+  int ld = 0;
+  __device__ __forceinline__ float get(long long row, int col) const {
+    const float* q = p + row * ld + col;
+    float a = *q;
+    for (int s = 1; s < splits; ++s) a += q[(long long)s * pstride];
+    return a;
+  }
+};
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+template <typename T> __device__ __forceinline__ float round_to(float v) { return to_f<T>(from_f<T>(v)); }
+
+// block-wide sum of one value per thread (256 threads), the same total in every thread
+__device__ __forceinline__ float block_sum256(float v, float* sm8) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) sm8[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) tot += sm8[i];
+  return tot;
+}
+
+// ---- short causal convolution over time, one filter per channel ----------------------------------------------
+// The inputs of position p of slot s are kept at ring[(s * RC + p % RC) * C]: the last taps - 1 of them are state, the
+// others are inputs of positions that are appended and not committed yet (a rejected suffix is simply overwritten).
+// An input is rounded to the storage dtype before it is used, so that it does not matter whether it came from this
+// forward or from the ring.
+template <typename T>
+struct ConvIn {
+  Src src;                 // projection rows of this forward
+  int col0 = 0;            // first convolved column
+  T* ring = nullptr;
+  int RC = 1, C = 0, taps = 1;
+  const float* w = nullptr;      // [C, taps]
+  const float* bias = nullptr;   // [C] or null
+
+  __device__ __forceinline__ float input(int row, int r0, int start, int slot, int pos, int c) const {
+    if (pos >= start) return round_to<T>(src.get(r0 + pos - start, col0 + c));
+    if (pos < 0) return 0.f;
+    return to_f<T>(ring[((long long)slot * RC + pos % RC) * C + c]);
+  }
+  // silu(conv) of channel c at `row`; *cur receives the row's own input
+  __device__ __forceinline__ float at(int row, int r0, int start, int slot, int c, float* cur) const {
+    const int pos = start + row - r0;
+    const float* wc = w + (long long)c * taps;
+    float x = input(row, r0, start, slot, pos, c);
+    *cur = x;
+    float acc = x * wc[taps - 1];
+    for (int j = 1; j < taps; ++j) acc = fmaf(input(row, r0, start, slot, pos - j, c), wc[taps - 1 - j], acc);
+    if (bias) acc += bias[c];
+    return acc / (1.0f + expf(-acc));
+  }
+  __device__ __forceinline__ void keep(int slot, int pos, int c, float v) const {
+    ring[((long long)slot * RC + pos % RC) * C + c] = from_f<T>(v);
+  }
+};

@@ -26,13 +26,13 @@ from typing import Optional
 
 import numpy as np
 
-from .model import VerseNexLM, _ptr
+from .model import DeviceLM, _ptr
 
 PURPOSE_DRAFT = 2  # Philox purpose of the draft model's own sampling (0 / 1: accept test / resample)
 
 
 class SpecEngine:
-    def __init__(self, target: VerseNexLM, draft: VerseNexLM, max_batch: int, max_seq: int, k: int = 4,
+    def __init__(self, target: DeviceLM, draft: DeviceLM, max_batch: int, max_seq: int, k: int = 4,
                  temperature: float = 0.0, top_k: int = 0, seed: int = 0, bonus: bool = True,
                  max_new_tokens: int = 4096, graph: bool = True):
         if target.vocab_size != draft.vocab_size:
@@ -46,8 +46,8 @@ class SpecEngine:
         self.temperature, self.top_k, self.seed, self.bonus = float(temperature), int(top_k or 0), int(seed), bool(bonus)
         self.n_verify = self.k + 1 if self.bonus else self.k
         self.max_seq = int(max_seq)
-        self.t_cache = target.new_cache(self.B, max_seq)
-        self.d_cache = draft.new_cache(self.B, max_seq)
+        self.t_cache = target.new_cache(self.B, max_seq, max_pending=self.n_verify)
+        self.d_cache = draft.new_cache(self.B, max_seq, max_pending=self.k + 1)
         ctx, B, k, V = self.ctx, self.B, self.k, self.V
         self.cap = int(max_new_tokens) + k + 1
         self.pair = ctx.zeros((B, 2), np.int64)

@@ -90,15 +90,16 @@ class KVCache:
     (accepted path) and drops the rest (rejected suffix) by compacting in place.
     """
 
-    def __init__(self, model: "VerseNexLM", max_batch: int, max_seq: int, _view_of: Optional["KVCache"] = None,
-                 _first: int = 0):
+    def __init__(self, model: "DeviceLM", max_batch: int, max_seq: int, _view_of: Optional["KVCache"] = None,
+                 _first: int = 0, pool_tokens: int = 0, max_pending: int = 1):
         self.model = model
         self.ctx = model.ctx
         self.max_batch, self.max_seq = int(max_batch), int(max_seq)
         self._parent = _view_of            # keeps the owning cache alive
         h = C.c_void_p()
         if _view_of is None:
-            self.ctx._check(self.ctx.lib.vn_kv_create(model.handle, self.max_batch, self.max_seq, C.byref(h)))
+            self.ctx._check(self.ctx.lib.vn_kv_create_ex(model.handle, self.max_batch, self.max_seq, int(pool_tokens),
+                                                         int(max_pending), C.byref(h)))
         else:
             self.ctx._check(self.ctx.lib.vn_kv_view(_view_of.handle, int(_first), self.max_batch, C.byref(h)))
         self.handle = h
@@ -109,6 +110,13 @@ class KVCache:
         if first < 0 or count < 1 or first + count > self.max_batch:
             raise IndexError(f"sequences [{first}, {first + count}) outside the cache's {self.max_batch}")
         return KVCache(self.model, count, self.max_seq, _view_of=self, _first=first)
+
+    @property
+    def pages(self):
+        """(total, free) pages of the pool a composed model's latents live in."""
+        total, free = C.c_int32(), C.c_int32()
+        self.ctx._check(self.ctx.lib.vn_kv_pages(self.handle, C.byref(total), C.byref(free)))
+        return int(total.value), int(free.value)
 
     @property
     def per_seq_lens(self) -> np.ndarray:
@@ -159,7 +167,143 @@ class KVCache:
             pass
 
 
-class VerseNexLM:
+class DeviceLM:
+    """What every model on the device has, whatever its layers are: a handle, its weights, caches, and the step functions
+    `forward_cached` (a uniform batch, appended but not committed) and `forward_ragged` (entries of any lengths,
+    appended and committed).  Subclasses call `_create` with the configuration the library reads."""
+
+    use_rope = False
+
+    def _create(self, config: dict, device: str):
+        from .backend import _parse_index
+        self.ctx = Context.get(_parse_index(device))
+        h = C.c_void_p()
+        self.handle = None
+        self.ctx._check(self.ctx.lib.vn_model_create(self.ctx.handle, json.dumps(config).encode(), C.byref(h)))
+        self.handle = h
+        self._finalized = False
+        self._scratch_cache: Optional[KVCache] = None
+
+    def eval(self):
+        return self
+
+    def param_bytes(self) -> int:
+        n = C.c_uint64()
+        self.ctx._check(self.ctx.lib.vn_model_param_bytes(self.handle, C.byref(n)))
+        return int(n.value)
+
+    def head_columns(self, hidden, v_lo: int, n_cols: int) -> DeviceArray:
+        """Logits of vocabulary columns [v_lo, v_lo + n_cols) for final-norm hidden rows (R, dim): the LM head of a
+        rank that owns only those columns."""
+        h = as_device(self.ctx, hidden, np.float32)
+        R = h.size // self.dim
+        out = self.ctx.empty((R, n_cols), np.float32)
+        self.ctx._check(self.ctx.lib.vn_model_head(self.handle, _ptr(h), R, int(v_lo), int(n_cols), _ptr(out), n_cols))
+        return out
+
+    def check(self):
+        """Raise what the forwards since the last check ran into on the device: IndexError for a token id outside
+        the vocabulary (as NumPy indexing does in the reference, vnnn.py:453-460), RuntimeError for a kernel
+        wait that ran out.  Synchronises the stream."""
+        self.ctx._check(self.ctx.lib.vn_model_status(self.handle, None, None))
+
+    def load_tensor(self, name: str, array):
+        a = np.ascontiguousarray(np.asarray(array), dtype=np.float32)
+        shape = (C.c_int64 * max(a.ndim, 1))(*(a.shape if a.ndim else (1,)))
+        self.ctx._check(self.ctx.lib.vn_model_load_tensor(self.handle, name.encode(), a.ctypes.data_as(C.c_void_p),
+                                                          max(a.ndim, 1), shape))
+        self._finalized = False
+
+    def finalize(self):
+        self.ctx._check(self.ctx.lib.vn_model_finalize(self.handle))
+        self._finalized = True
+
+    # -- forward -----------------------------------------------------------------
+    def new_cache(self, max_batch: int, max_seq: Optional[int] = None, max_pending: int = 1) -> KVCache:
+        """`max_pending`: rows an engine appends and may cut back again.  Models whose cache is K / V rows only keep
+        any number of them; a model with recurrent layers keeps a state for each."""
+        return KVCache(self, max_batch, max_seq if max_seq is not None else self.max_seq_len, max_pending=max_pending)
+
+    def forward_cached(self, tokens, cache: KVCache, parents=None, last_only: bool = False,
+                       want_logits: bool = True, want_hidden: bool = False, slot_offset: int = 0,
+                       out_logits: Optional[DeviceArray] = None, out_hidden: Optional[DeviceArray] = None):
+        """T new positions per sequence on top of `cache` (appended, not yet committed).
+
+        tokens (B, T) int64 host or device; parents: list of T tree parents (-1 = child of the last
+        committed token) or None for a chain.  Returns logits (B, T | 1, V) and / or hidden."""
+        if not self._finalized:
+            self.finalize()
+        tok = as_device(self.ctx, tokens, np.int64)
+        B, T = tok.shape
+        rows = 1 if last_only else T
+        logits = hidden = None
+        if want_logits:
+            logits = out_logits if out_logits is not None else self.ctx.empty((B, rows, self.vocab_size), np.float32)
+        if want_hidden:
+            hidden = out_hidden if out_hidden is not None else self.ctx.empty((B, rows, self.dim), np.float32)
+        par = None
+        if parents is not None:
+            par = np.ascontiguousarray(parents, dtype=np.int32)
+            if par.shape != (T,):
+                raise ValueError("parents must list one parent per new position")
+        self.ctx._check(self.ctx.lib.vn_model_forward(
+            self.handle, cache.handle, _ptr(tok), B, T,
+            par.ctypes.data_as(C.c_void_p) if par is not None else None, _ptr(hidden), _ptr(logits),
+            int(bool(last_only)), int(slot_offset)))
+        if want_logits and want_hidden:
+            return logits, hidden
+        return logits if want_logits else hidden
+
+    def forward(self, idx):
+        """Whole-sequence forward from position 0, logits (B, T, V) -- CometSparkNexLM.forward."""
+        from .speculative import Tensor, _unwrap
+        ids = _unwrap(idx)
+        ids = ids if isinstance(ids, DeviceArray) else np.asarray(ids, dtype=np.int64)
+        if ids.ndim == 1:
+            ids = ids.reshape(1, -1)
+        B, T = ids.shape
+        c = self._scratch_cache
+        if c is None or c.max_batch < B or c.max_seq < T:
+            self._scratch_cache = c = self.new_cache(max(B, 1), max(T, self.max_seq_len))
+        c.reset()
+        out = Tensor(self.forward_cached(ids, c))
+        self.check()
+        return out
+
+    __call__ = forward
+
+    def forward_ragged(self, cache: KVCache, slots, counts, tokens, out_rows):
+        """One step over a ragged batch: entry e brings `counts[e]` tokens (one after another in `tokens`) for sequence
+        `slots[e]`; all of them are committed.  Returns the logits (len(out_rows), V) at the named rows of `tokens`, or
+        None when no row is named.  Here: entry by entry through views of the cache."""
+        tokens = np.ascontiguousarray(tokens, dtype=np.int64).reshape(-1)
+        out_rows = np.asarray(out_rows, dtype=np.int64).reshape(-1)
+        out = self.ctx.empty((len(out_rows), self.vocab_size), np.float32) if len(out_rows) else None
+        r0 = 0
+        for slot, n in zip(slots, counts):
+            view = cache.view(int(slot), 1)
+            mine = np.flatnonzero((out_rows >= r0) & (out_rows < r0 + n))
+            res = self.forward_cached(tokens[None, r0:r0 + n], view, want_logits=bool(len(mine)),
+                                      want_hidden=not len(mine), last_only=not len(mine))
+            for i in mine:
+                j = int(out_rows[i]) - r0
+                src = res.reshape(n, self.vocab_size)[j:j + 1]
+                self.ctx._check(self.ctx.lib.vn_d2d(self.ctx.handle, _ptr(out[int(i):int(i) + 1]), _ptr(src), src.nbytes))
+            view.commit(n, np.full(1, n, np.int32))
+            r0 += n
+        return out
+
+    def __del__(self):
+        try:
+            self._scratch_cache = None
+            if self.handle:
+                self.ctx.lib.vn_model_destroy(self.handle)
+                self.handle = None
+        except Exception:
+            pass
+
+
+class VerseNexLM(DeviceLM):
     def __init__(self, vocab_size: int, dim: int, n_layer: int, n_head: int, n_kv_head: Optional[int] = None,
                  layer_pattern: Optional[List[str]] = None, window_size: int = 512, num_global_tokens: int = 64,
                  anchor_interval: int = 128, latent_dim=None, use_alibi: bool = True, use_rope: bool = False,
@@ -202,13 +346,7 @@ class VerseNexLM:
                             top_k=int(top_k), expert_hidden=expert_hidden, tie_weights=self.tie_weights,
                             mlp_hidden_multiple=int(mlp_hidden_multiple), embedding_scale=self.embedding_scale,
                             dtype=dtype)
-        from .backend import _parse_index
-        self.ctx = Context.get(_parse_index(device))
-        h = C.c_void_p()
-        self.ctx._check(self.ctx.lib.vn_model_create(self.ctx.handle, json.dumps(self._config).encode(), C.byref(h)))
-        self.handle = h
-        self._finalized = False
-        self._scratch_cache: Optional[KVCache] = None
+        self._create(self._config, device)
 
     @classmethod
     def from_pretrained(cls, path: str, dtype: str = "f32", device: str = "cuda", **overrides) -> "VerseNexLM":
@@ -228,36 +366,6 @@ class VerseNexLM:
     # -- reference-compatible helpers -----------------------------------------
     def get_config(self) -> dict:
         return dict(self._config)
-
-    def eval(self):
-        return self
-
-    def param_bytes(self) -> int:
-        n = C.c_uint64()
-        self.ctx._check(self.ctx.lib.vn_model_param_bytes(self.handle, C.byref(n)))
-        return int(n.value)
-
-    def head_columns(self, hidden, v_lo: int, n_cols: int) -> DeviceArray:
-        """Logits of vocabulary columns [v_lo, v_lo + n_cols) for final-norm hidden rows (R, dim): the LM head of a
-        rank that owns only those columns."""
-        h = as_device(self.ctx, hidden, np.float32)
-        R = h.size // self.dim
-        out = self.ctx.empty((R, n_cols), np.float32)
-        self.ctx._check(self.ctx.lib.vn_model_head(self.handle, _ptr(h), R, int(v_lo), int(n_cols), _ptr(out), n_cols))
-        return out
-
-    def check(self):
-        """Raise what the forwards since the last check ran into on the device: IndexError for a token id outside
-        the vocabulary (as NumPy indexing does in the reference, vnnn.py:453-460), RuntimeError for a kernel
-        wait that ran out.  Synchronises the stream."""
-        self.ctx._check(self.ctx.lib.vn_model_status(self.handle, None, None))
-
-    def load_tensor(self, name: str, array):
-        a = np.ascontiguousarray(np.asarray(array), dtype=np.float32)
-        shape = (C.c_int64 * max(a.ndim, 1))(*(a.shape if a.ndim else (1,)))
-        self.ctx._check(self.ctx.lib.vn_model_load_tensor(self.handle, name.encode(), a.ctypes.data_as(C.c_void_p),
-                                                          max(a.ndim, 1), shape))
-        self._finalized = False
 
     def load_state_dict(self, sd: dict, strict: bool = True):
         """name -> float32 array (vnnn.py:235-285).  A value may also be an already quantised linear: an object
@@ -358,58 +466,6 @@ class VerseNexLM:
         self.ctx._check(self.ctx.lib.vn_model_quantize(self.handle, scheme.encode()))
         self.quantized = scheme
         return self
-
-    def new_cache(self, max_batch: int, max_seq: Optional[int] = None) -> KVCache:
-        return KVCache(self, max_batch, max_seq if max_seq is not None else self.max_seq_len)
-
-    # -- forward -----------------------------------------------------------------
-    def forward_cached(self, tokens, cache: KVCache, parents=None, last_only: bool = False,
-                       want_logits: bool = True, want_hidden: bool = False, slot_offset: int = 0,
-                       out_logits: Optional[DeviceArray] = None, out_hidden: Optional[DeviceArray] = None):
-        """T new positions per sequence on top of `cache` (appended, not yet committed).
-
-        tokens (B, T) int64 host or device; parents: list of T tree parents (-1 = child of the last
-        committed token) or None for a chain.  Returns logits (B, T | 1, V) and / or hidden."""
-        if not self._finalized:
-            self.finalize()
-        tok = as_device(self.ctx, tokens, np.int64)
-        B, T = tok.shape
-        rows = 1 if last_only else T
-        logits = hidden = None
-        if want_logits:
-            logits = out_logits if out_logits is not None else self.ctx.empty((B, rows, self.vocab_size), np.float32)
-        if want_hidden:
-            hidden = out_hidden if out_hidden is not None else self.ctx.empty((B, rows, self.dim), np.float32)
-        par = None
-        if parents is not None:
-            par = np.ascontiguousarray(parents, dtype=np.int32)
-            if par.shape != (T,):
-                raise ValueError("parents must list one parent per new position")
-        self.ctx._check(self.ctx.lib.vn_model_forward(
-            self.handle, cache.handle, _ptr(tok), B, T,
-            par.ctypes.data_as(C.c_void_p) if par is not None else None, _ptr(hidden), _ptr(logits),
-            int(bool(last_only)), int(slot_offset)))
-        if want_logits and want_hidden:
-            return logits, hidden
-        return logits if want_logits else hidden
-
-    def forward(self, idx):
-        """Whole-sequence forward from position 0, logits (B, T, V) -- CometSparkNexLM.forward."""
-        from .speculative import Tensor, _unwrap
-        ids = _unwrap(idx)
-        ids = ids if isinstance(ids, DeviceArray) else np.asarray(ids, dtype=np.int64)
-        if ids.ndim == 1:
-            ids = ids.reshape(1, -1)
-        B, T = ids.shape
-        c = self._scratch_cache
-        if c is None or c.max_batch < B or c.max_seq < T:
-            self._scratch_cache = c = self.new_cache(max(B, 1), max(T, self.max_seq_len))
-        c.reset()
-        out = Tensor(self.forward_cached(ids, c))
-        self.check()
-        return out
-
-    __call__ = forward
 
     def forward_recurrent(self, input_ids, states=None):
         """One decoding step, CometSparkNexLM.forward_recurrent (cometspark.py:737-767): input_ids (B, 1) ->
@@ -546,15 +602,6 @@ class VerseNexLM:
             if res.shape[1] > 0 and not np.all(res[:, -1] == eos_id):
                 res = np.concatenate([res, np.full((B, 1), eos_id, dtype=res.dtype)], axis=1)
         return res
-
-    def __del__(self):
-        try:
-            self._scratch_cache = None
-            if self.handle:
-                self.ctx.lib.vn_model_destroy(self.handle)
-                self.handle = None
-        except Exception:
-            pass
 
 
 CometSparkNexLM = VerseNexLM

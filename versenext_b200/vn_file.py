@@ -13,20 +13,12 @@ from __future__ import annotations
 
 import io
 import json
-import struct
 import zipfile
 from typing import Dict, Iterator, Optional, Tuple
 
 import numpy as np
 
-_ST_DTYPES = {"F64": np.float64, "F32": np.float32, "F16": np.float16, "I64": np.int64, "I32": np.int32,
-              "I16": np.int16, "I8": np.int8, "U8": np.uint8, "BOOL": np.bool_, "U16": np.uint16, "U32": np.uint32,
-              "U64": np.uint64}
-
-
-def _bf16_to_f32(raw: bytes, shape) -> np.ndarray:
-    u = np.frombuffer(raw, dtype=np.uint16).astype(np.uint32) << np.uint32(16)
-    return u.view(np.float32).reshape(shape)
+from .safetensors_file import iter_tensors, read_header
 
 
 class VNFileReader:
@@ -82,33 +74,7 @@ class VNFileReader:
 
     def _iter_safetensors(self):
         with self._zf.open("model.safetensors") as f:
-            (hlen,) = struct.unpack("<Q", f.read(8))
-            if hlen > (100 << 20):
-                raise ValueError("implausible safetensors header length")
-            header = json.loads(f.read(hlen).decode("utf-8"))
-            entries = [(n, e) for n, e in header.items() if n != "__metadata__"]
-            entries.sort(key=lambda ne: ne[1]["data_offsets"][0])
-            pos = 0
-            for name, e in entries:
-                lo, hi = e["data_offsets"]
-                if lo < pos:
-                    raise ValueError(f"{name}: overlapping tensor data")
-                if lo > pos:
-                    f.read(lo - pos)
-                raw = f.read(hi - lo)
-                pos = hi
-                if len(raw) != hi - lo:
-                    raise ValueError(f"{name}: truncated tensor data")
-                shape = tuple(e["shape"])
-                if e["dtype"] == "BF16":
-                    arr = _bf16_to_f32(raw, shape)
-                else:
-                    if e["dtype"] not in _ST_DTYPES:
-                        raise ValueError(f"{name}: unsupported dtype {e['dtype']}")
-                    arr = np.frombuffer(raw, dtype=_ST_DTYPES[e["dtype"]]).reshape(shape)
-                    if arr.dtype in (np.float64, np.float16):
-                        arr = arr.astype(np.float32)
-                yield name, arr
+            yield from iter_tensors(f, read_header(f))
 
     def _iter_npz(self):
         inner = zipfile.ZipFile(io.BytesIO(self._zf.read("model.npz")), "r")
