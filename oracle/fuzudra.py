@@ -23,6 +23,24 @@ def bf16(a):
     return (((u + (((u >> 16) & 1) + 0x7FFF)) >> 16) << 16).astype(np.uint32).view(np.float32)
 
 
+# Applied to the operand of every matrix product and to every value that is kept for later tokens.  `rounded()` makes it
+# a rounding to bfloat16, which shows what storing those in 16 bits costs at every position.
+_store = [lambda a: a]
+
+
+class rounded:
+    def __enter__(self):
+        self.old, _store[0] = _store[0], lambda a: bf16(a).astype(F)
+
+    def __exit__(self, *exc):
+        _store[0] = self.old
+        return False
+
+
+def linear(x, w):
+    return _store[0](x) @ w.T
+
+
 # ---- small pieces -----------------------------------------------------------------------------------------
 def sigmoid(z):
     return 1.0 / (1.0 + np.exp(-z))
@@ -74,11 +92,11 @@ def latent_attention(h, W, cfg, eps):
     H, d, vd, R = cfg["heads"], cfg["dim"], cfg["vdim"], cfg["kv_rank"]
     size = (cfg.get("mask") or {}).get("size")
     T = h.shape[0]
-    q = (h @ W["q"].T).reshape(T, H, d)
-    c = rms(h @ W["dkv"].T, eps) * W["dkv.norm"]
-    k = (c @ W["uk"].T).reshape(T, H, d)
-    v = (c @ W["uv"].T).reshape(T, H, vd)
-    gate = sigmoid(h @ W["g"].T)
+    q = linear(h, W["q"]).reshape(T, H, d)
+    c = _store[0](rms(linear(h, W["dkv"]), eps) * W["dkv.norm"])
+    k = linear(c, W["uk"]).reshape(T, H, d)
+    v = linear(c, W["uv"]).reshape(T, H, vd)
+    gate = sigmoid(linear(h, W["g"]))
     i, j = np.arange(T)[:, None], np.arange(T)[None, :]
     seen = (j <= i) if size is None else ((j <= i) & (i - j < size))
     out = np.zeros((T, H, vd), F)
@@ -87,7 +105,7 @@ def latent_attention(h, W, cfg, eps):
         top = np.maximum(s.max(axis=1), W["sink"][a])
         e = np.exp(s - top[:, None])
         out[:, a] = (e @ v[:, a]) / (e.sum(axis=1) + np.exp(W["sink"][a] - top))[:, None] * gate[:, a:a + 1]
-    return out.reshape(T, H * vd) @ W["o"].T
+    return linear(out.reshape(T, H * vd), W["o"])
 
 
 def selective_scan(x, dt, Bm, Cm, A, D, state=None):
@@ -102,12 +120,12 @@ def selective_scan(x, dt, Bm, Cm, A, D, state=None):
 
 def mamba1(h, W, cfg, eps):
     n, r, N = cfg["inner"], cfg["dt_rank"], cfg["state"]
-    xz = h @ W["in"].T
-    x = silu(causal_conv(xz[:, :n], W["conv"], W["conv.b"]))
-    p = x @ W["x"].T
-    dt = softplus(p[:, :r] @ W["dt"].T + W["dt.b"])
+    xz = linear(h, W["in"])
+    x = _store[0](silu(causal_conv(_store[0](xz[:, :n]), W["conv"], W["conv.b"])))
+    p = linear(x, W["x"])
+    dt = softplus(linear(p[:, :r], W["dt"]) + W["dt.b"])
     y, _ = selective_scan(x, dt, p[:, r:r + N], p[:, r + N:], -np.exp(W["A_log"]), W["D"])
-    return (y * silu(xz[:, n:])) @ W["o"].T
+    return linear(y * silu(_store[0](xz[:, n:])), W["o"])
 
 
 def delta_rule(q, k, v, g, beta, state=None):
@@ -125,28 +143,28 @@ def delta_rule(q, k, v, g, beta, state=None):
 def channel_delta(h, W, cfg, eps):
     H, KH, d, vd = cfg["heads"], cfg["kv_heads"], cfg["dim"], cfg["vdim"]
     T = h.shape[0]
-    q = silu(causal_conv(h @ W["q"].T, W["q.conv"])).reshape(T, KH, d)
-    k = silu(causal_conv(h @ W["k"].T, W["k.conv"])).reshape(T, KH, d)
-    v = silu(causal_conv(h @ W["v"].T, W["v.conv"])).reshape(T, H, vd)
+    q = silu(causal_conv(_store[0](linear(h, W["q"])), W["q.conv"])).reshape(T, KH, d)
+    k = silu(causal_conv(_store[0](linear(h, W["k"])), W["k.conv"])).reshape(T, KH, d)
+    v = silu(causal_conv(_store[0](linear(h, W["v"])), W["v.conv"])).reshape(T, H, vd)
     q = q / np.sqrt((q * q).sum(-1, keepdims=True) + 1e-6) * d ** -0.5
     k = k / np.sqrt((k * k).sum(-1, keepdims=True) + 1e-6)
-    beta = sigmoid(h @ W["b"].T)
-    a = ((h @ W["a1"].T) @ W["a2"].T + W["dt_bias"]).reshape(T, H, d)
+    beta = sigmoid(linear(h, W["b"]))
+    a = (linear(linear(h, W["a1"]), W["a2"]) + W["dt_bias"]).reshape(T, H, d)
     g = np.exp(-np.exp(W["A_log"])[None, :, None] * softplus(a))
-    gate = sigmoid((h @ W["g1"].T) @ W["g2"].T).reshape(T, H, vd)
+    gate = sigmoid(linear(linear(h, W["g1"]), W["g2"])).reshape(T, H, vd)
     out = np.zeros((T, H, vd), F)
     for i in range(H):
         kh = i // (H // KH)
         o, _ = delta_rule(q[:, kh], k[:, kh], v[:, i], g[:, i], beta[:, i])
         out[:, i] = rms(o, eps) * W["norm"] * gate[:, i]
-    return out.reshape(T, H * vd) @ W["o"].T
+    return linear(out.reshape(T, H * vd), W["o"])
 
 
 MIXERS = {"latent_attention": latent_attention, "mamba1": mamba1, "channel_delta": channel_delta}
 
 
 def feed_forward(h, W):
-    return (gelu_tanh(h @ W["gate"].T) * (h @ W["up"].T)) @ W["down"].T
+    return linear(gelu_tanh(linear(h, W["gate"])) * linear(h, W["up"]), W["down"])
 
 
 # ---- the model ----------------------------------------------------------------------------------------------
@@ -180,8 +198,8 @@ def forward(sd, cfg, tokens, collect=None):
     x = x0
     for i, t in layer_runs(cfg):
         if t is not None and i == cfg["loop"]["start"]:
-            x = np.concatenate([x, x0], axis=1) @ np.asarray(sd["loop.in"], F).T + np.asarray(sd["loop.step"], F)[t]
+            x = linear(np.concatenate([x, x0], axis=1), np.asarray(sd["loop.in"], F)) + np.asarray(sd["loop.step"], F)[t]
         x = layer(x, sd, cfg, i)
         if collect is not None:
             collect.append(x)
-    return norm(x, np.asarray(sd["final.norm"], F), cfg["norm"]["eps"]) @ np.asarray(sd["head"], F).T
+    return linear(norm(x, np.asarray(sd["final.norm"], F), cfg["norm"]["eps"]), np.asarray(sd["head"], F))
