@@ -1027,6 +1027,152 @@ def run_layer(args):
         dist.destroy_process_group()
 
 
+FUZUDRA_WIDTHS = (1024, 2048)
+FUZUDRA_CTX, FUZUDRA_DECODE_B, FUZUDRA_PREFILL = 1024, (1, 32, 128), ((1, 4096), (8, 1024))
+
+
+def _decode_ms(m, ctx, B, T0, V, steps, profile=False):
+    """One decoded token for B sequences at context T0: forward, arg-max, commit, replayed from a CUDA graph.  Returns
+    (ms per step, per-kernel times of an eager step or None)."""
+    import ctypes as C
+    from versenext_b200 import sampling
+    from versenext_b200.model import _ptr
+    cache = m.new_cache(B, T0 + 3 * steps + 64)
+    rng = np.random.default_rng(5)
+    part = max(1, 8192 // B)
+    for lo in range(0, T0, part):
+        n = min(part, T0 - lo)
+        m.forward_cached(rng.integers(0, V, (B, n)), cache, want_logits=False, want_hidden=True, last_only=True)
+        cache.commit(n, np.full(B, n, np.int32))
+    tok, one = ctx.from_numpy(rng.integers(0, V, (B, 1))), ctx.from_numpy(np.ones(B, np.int32))
+    logits, length, out = ctx.empty((B, 1, V), np.float32), ctx.empty((B,), np.int32), ctx.empty((B, 1), np.int64)
+    empty = ctx.empty((B, 0), np.int64)
+
+    def step():
+        m.forward_cached(tok, cache, out_logits=logits)
+        sampling.accept(ctx, logits, None, empty, temperature=0.0, shape=(B, 0, V), p_strides=(V, V), q_strides=(0, 0),
+                        out=(length, out))
+        ctx._check(ctx.lib.vn_d2d(ctx.handle, _ptr(tok), _ptr(out), tok.nbytes))
+        cache.commit(1, one)
+    for _ in range(3):
+        step()
+    ctx._check(ctx.lib.vn_graph_begin(ctx.handle))
+    g = C.c_void_p()
+    try:
+        step()
+    finally:
+        ctx._check(ctx.lib.vn_graph_end(ctx.handle, C.byref(g)))
+    flush = ctx.lib.vn_flush_l2
+    times = []
+    for i in range(steps + 3):
+        ctx._check(flush(ctx.handle))
+        e0, e1 = ctx.event(), ctx.event()
+        e0.record()
+        ctx._check(ctx.lib.vn_graph_launch(ctx.handle, g))
+        e1.record()
+        ctx.sync()
+        if i >= 3:
+            times.append(e0.elapsed_ms(e1))
+    ctx._check(ctx.lib.vn_graph_destroy(ctx.handle, g))
+    prof = _profiled(ctx, step) if profile else None
+    m.check()
+    return statistics.median(times), prof
+
+
+def _profiled(ctx, fn, n=4):
+    """Per-kernel times of `fn` (us per call, launches per call), events around every launch, L2 flushed before each call."""
+    ctx.profile(True)
+    try:
+        for _ in range(n):
+            ctx._check(ctx.lib.vn_flush_l2(ctx.handle))
+            fn()
+        rep = ctx.profile_report()
+    finally:
+        ctx.profile(False)
+    out = {}
+    for name, r in rep.items():
+        out[name] = {"us": round(1e3 * r["ms"] / n, 2), "launches": r["launches"] / n}
+    return dict(sorted(out.items(), key=lambda kv: -kv[1]["us"]))
+
+
+def _prefill_ms(m, ctx, B, T, V, steps, profile=False):
+    cache = m.new_cache(B, T + 8)
+    tok = ctx.from_numpy(np.random.default_rng(6).integers(0, V, (B, T)))
+    hidden = ctx.empty((B, 1, m.dim), np.float32)
+
+    def step():
+        cache.reset()
+        m.forward_cached(tok, cache, want_logits=False, want_hidden=True, last_only=True, out_hidden=hidden)
+    for _ in range(3):
+        step()
+    times = []
+    for _ in range(steps):
+        ctx._check(ctx.lib.vn_flush_l2(ctx.handle))
+        e0, e1 = ctx.event(), ctx.event()
+        e0.record()
+        step()
+        e1.record()
+        ctx.sync()
+        times.append(e0.elapsed_ms(e1))
+    prof = _profiled(ctx, step) if profile else None
+    m.check()
+    return statistics.median(times), prof
+
+
+def run_fuzudra(args):
+    """Prefill and decode of the Fuzudra design (random weights, 4 layers) beside VerseNexLM models of the same width,
+    depth, feed-forward, window and vocabulary: all TriSparse, and all GMLA (a latent behind K and V), the closest layers."""
+    import versenext_b200 as vn
+    from versenext_b200 import synthetic as S
+    world, rank, local, dist = dist_setup(args.gpus)
+    ctx = vn.Context.get(local)
+    V = 32000
+    clocks = ClockSampler(local).start() if rank == 0 else None
+    rows, profs, l0 = [], {}, ctx.launch_count()
+    steps = min(max(args.steps, 5), 20)
+    for D in FUZUDRA_WIDTHS:
+        def composed():
+            return S.random_fuzudra(S.fuzudra_config(D, V), dtype="bf16", device=f"cuda:{local}")
+
+        def verse(kind):
+            kw = dict(vocab_size=V, dim=D, n_layer=4, n_head=D // 64, layer_pattern=[kind] * 4, window_size=1024,
+                      num_global_tokens=64, use_alibi=False, use_rope=True, max_seq_len=8192)
+            m = vn.VerseNexLM(dtype="bf16", device=f"cuda:{local}", **kw)
+            S.load_random(m, kw, seed=3)
+            return m
+        for name, make in (("fuzudra", composed), ("trisparse", lambda: verse("trisparse")), ("gmla", lambda: verse("gmla"))):
+            m = make()
+            row = {"model": name, "width": D, "param_mb": round(m.param_bytes() / 1e6, 1)}
+            for B in FUZUDRA_DECODE_B:
+                ms, prof = _decode_ms(m, ctx, B, FUZUDRA_CTX, V, steps, profile=args.kernels)
+                row[f"decode_B{B}_tok_s"] = round(B / ms * 1e3, 1)
+                row[f"decode_B{B}_ms"] = round(ms, 4)
+                if prof:
+                    profs[f"{name}.{D}.decode_B{B}"] = prof
+            for B, T in FUZUDRA_PREFILL:
+                ms, prof = _prefill_ms(m, ctx, B, T, V, steps, profile=args.kernels)
+                row[f"prefill_{B}x{T}_tok_s"] = round(B * T / ms * 1e3, 1)
+                row[f"prefill_{B}x{T}_ms"] = round(ms, 4)
+                if prof:
+                    profs[f"{name}.{D}.prefill_{B}x{T}"] = prof
+            rows.append(row)
+            del m
+    clk = clocks.stop() if clocks else None
+    if rank == 0:
+        head = next(r for r in rows if r["model"] == "fuzudra" and r["width"] == FUZUDRA_WIDTHS[-1])
+        line = {"metric": "composed-model decode throughput", "value": head["decode_B32_tok_s"], "unit": "tokens/s",
+                "n_gpus": world, "steps": steps, "warmup": 3, "ms_per_step": head["decode_B32_ms"], "higher_is_better": True,
+                "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+                "config": {"workload": f"fuzudra: 4 layers, widths {FUZUDRA_WIDTHS}, V={V}, context {FUZUDRA_CTX}, L2 flushed "
+                                       "between steps, decode replayed from a CUDA graph"},
+                "rows": rows, "clocks": clk, "gpu_launches": ctx.launch_count() - l0}
+        if profs:
+            line["kernels"] = profs
+        print(json.dumps(line))
+    if dist is not None:
+        dist.destroy_process_group()
+
+
 def run_small(args):
     import versenext_b200 as vn
     world, rank, local, dist = dist_setup(args.gpus)
@@ -1241,7 +1387,7 @@ def main():
     ap.add_argument("--steps", type=int, default=32)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--workload", default="spec", choices=["spec", "accept", "sharded", "tree", "small", "layer", "delta"])
+    ap.add_argument("--workload", default="spec", choices=["spec", "accept", "sharded", "tree", "small", "layer", "delta", "fuzudra"])
     ap.add_argument("--weak", action="store_true",
                     help="spec workload: 32 requests on every rank (default: the configuration's 32 split over the ranks)")
     ap.add_argument("--no-weak", action="store_true", help="N > 1: skip the extra 32-per-GPU measurement")
@@ -1250,6 +1396,7 @@ def main():
                     help="spec workload: quantise the target's linear weights (not the default benchmark line)")
     ap.add_argument("--pattern", default="mod,trisparse", help="layer workload: comma-separated layer kinds")
     ap.add_argument("--context", type=int, default=1100, help="layer workload: cached positions (a multiple of 220)")
+    ap.add_argument("--kernels", action="store_true", help="fuzudra workload: per-kernel times of every case")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU-baseline leg")
     ap.add_argument("--no-sampler", action="store_true", help="spec workload: skip the sampler GB/s measurement")
     args = ap.parse_args()
@@ -1257,7 +1404,7 @@ def main():
         {"accept": run_reference, "small": run_reference_small}.get(args.workload, run_reference_spec)(args)
     else:
         {"spec": run_spec, "accept": run_accept, "sharded": run_sharded, "tree": run_tree,
-         "small": run_small, "layer": run_layer, "delta": run_delta}[args.workload](args)
+         "small": run_small, "layer": run_layer, "delta": run_delta, "fuzudra": run_fuzudra}[args.workload](args)
 
 
 if __name__ == "__main__":

@@ -115,3 +115,69 @@ def load_random(model, kw: dict, seed: int, init_std: float = 0.02):
 
 def param_count(kw: dict) -> int:
     return int(sum(int(np.prod(s)) for _, s in _shapes(kw)))
+
+
+# ---- composed models (fuzudra.py): layers of the sizes a real model of that width would have ---------------------------
+def fuzudra_config(width: int, vocab: int = 32000, n_layer: int = 4, loop_times: int = 0) -> dict:
+    """config.json contents: latent attention, selective scan and two delta rule layers in turn, a feed-forward behind
+    each (as wide as VerseNexLM's), heads of 128 (64 below width 2048), a window of 1024."""
+    hd = 128 if width >= 2048 else 64
+    heads, ff = width // hd, int((4 * width * 2 / 3 + 63) // 64) * 64
+    mlp = {"kind": "dense", "ff": ff}
+    kinds = [{"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": hd, "vdim": hd, "kv_rank": width // 4,
+              "scale": hd ** -0.5, "mask": {"size": 1024}}},
+             {"type": "mamba1", "mlp": mlp, "mixer": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}},
+             {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": heads, "dim": hd, "vdim": hd, "conv": 4}}]
+    layers = [kinds[(0, 1, 2, 2)[i % 4]] for i in range(n_layer)]
+    return {"architecture": "Fuzudra", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": layers,
+            "loop": {"start": 0, "stop": n_layer, "times": loop_times} if loop_times else None}
+
+
+def fuzudra_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape; the ranks of the two low-rank factors are a head's width."""
+    D, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, D), "head": (V, D), "final.norm": (D,)}
+    if cfg.get("loop"):
+        s["loop.in"], s["loop.step"] = (D, 2 * D), (cfg["loop"]["times"], D)
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        t = {"norm1": (D,)}
+        if L["type"] == "latent_attention":
+            H, d, v, R = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
+            t.update({"mix.q": (H * d, D), "mix.dkv": (R, D), "mix.dkv.norm": (R,), "mix.uk": (H * d, R), "mix.uv": (H * v, R),
+                      "mix.sink": (H,), "mix.g": (H, D), "mix.o": (D, H * v)})
+        elif L["type"] == "mamba1":
+            n, r, N = m["inner"], m["dt_rank"], m["state"]
+            t.update({"mix.in": (2 * n, D), "mix.conv": (n, m["conv"]), "mix.conv.b": (n,), "mix.x": (r + 2 * N, n),
+                      "mix.dt": (n, r), "mix.dt.b": (n,), "mix.A_log": (n, N), "mix.D": (n,), "mix.o": (D, n)})
+        else:
+            H, K, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            t.update({"mix.q": (K * d, D), "mix.q.conv": (K * d, m["conv"]), "mix.k": (K * d, D), "mix.k.conv": (K * d, m["conv"]),
+                      "mix.v": (H * v, D), "mix.v.conv": (H * v, m["conv"]), "mix.b": (H, D), "mix.A_log": (H,),
+                      "mix.norm": (v,), "mix.a1": (d, D), "mix.a2": (H * d, d), "mix.dt_bias": (H * d,), "mix.g1": (v, D),
+                      "mix.g2": (H * v, v), "mix.o": (D, H * v)})
+        if L["mlp"]:
+            t.update({"norm2": (D,), "mlp.gate": (L["mlp"]["ff"], D), "mlp.up": (L["mlp"]["ff"], D), "mlp.down": (D, L["mlp"]["ff"])})
+        s.update({p + n: x for n, x in t.items()})
+    return s
+
+
+def random_fuzudra(cfg: dict, seed: int = 0, **kw):
+    """A FuzudraLM with seeded random weights, tensor by tensor."""
+    from .fuzudra import FuzudraLM
+    shapes = fuzudra_shapes(cfg)
+    model = FuzudraLM(cfg, shapes, **kw)
+    rng = np.random.default_rng(seed)
+    special = {"A_log": (1.0, -1.0), "dt_bias": (1.0, -2.0), "dt.b": (1.0, -3.0), "D": (0.1, 1.0), "sink": (1.0, 0.0)}
+    for name, shape in shapes.items():
+        std, mean = (0.02, 0.0) if len(shape) == 2 else (0.1, 0.0)
+        for end, sm in special.items():
+            if name.endswith("mix." + end):
+                std, mean = sm
+        if name.endswith(".conv"):
+            std = 0.4
+        if name.endswith("mix.norm") or name.endswith("dkv.norm"):
+            mean = 1.0
+        model.load_tensor(name, mean + std * rng.standard_normal(shape, dtype=np.float32))
+    model.finalize()
+    return model
