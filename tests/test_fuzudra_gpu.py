@@ -204,6 +204,34 @@ def test_a_batch_changes_nothing():
     assert err(got[1:], whole(m, np.concatenate([a, b[:5]]))[-1:]) < 1e-5
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_many_sequences_at_once(dtype):
+    """Batches wide enough for the kernels' many-sequence shapes, as a prompt, as short portions that could be cut back,
+    and as single tokens."""
+    cfg = FC.config([FC.delta(heads=8, kv_heads=4, dim=64, vdim=64), FC.mamba(inner=96, state=16, dt_rank=8),
+                     FC.delta(heads=10, kv_heads=10, dim=128, vdim=72, conv=4), FC.latent(heads=8, dim=16, vdim=16, kv_rank=64, window=7)],
+                    width=64)
+    sd = FC.weights(cfg, seed=15)
+    m = build(cfg, sd, dtype)
+    B, T = 40, 29
+    toks = np.stack([prompt(cfg, T, seed=200 + b) for b in range(B)])
+    want = [Expected(sd, cfg, t) for t in toks[::13]]
+    cache = m.new_cache(B, 32, max_pending=3)
+    at, got = 0, []
+    for n in (19, 2, 1, 3, 1, 3):
+        got.append(m.forward_cached(toks[:, at:at + n], cache).numpy())
+        cache.commit(n, np.full(B, n, np.int32))
+        at += n
+    got = np.concatenate(got, axis=1)
+    for i, w in enumerate(want):
+        w.check(got[13 * i], dtype)
+    cache = m.new_cache(B, 32)
+    got = m.forward_ragged(cache, list(range(B)), [T] * B, toks.reshape(-1), range(B * T)).numpy().reshape(B, T, -1)
+    for i, w in enumerate(want):
+        w.check(got[13 * i], dtype)
+    m.check()
+
+
 def greedy(sd, cfg, toks, n):
     toks = list(toks)
     for _ in range(n):

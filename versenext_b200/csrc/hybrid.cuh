@@ -512,7 +512,10 @@ int32_t mamba1(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, cons
   Src s;
   TRY(project(m, gemm_args(m->h, D, L.w_in, L.n_in, D, M, "gemm_mamba_in"), b.proj, &s));
   const ConvIn<T> cv = conv_in<T>(L, hc, s, kv->k[run]);
-  VN_LAUNCH(ctx, mamba_conv_kernel<T>, dim3(ceil_div(n, 32), ceil_div(M, 8)), dim3(32, 8), 0, cv, rows, (T*)b.xc, (T*)b.z, hc.pending);
+  if (rows.max_n == 1)
+    VN_LAUNCH(ctx, (mamba_conv_kernel<T, 1>), dim3(ceil_div(n, 32), ceil_div(M, 8)), dim3(32, 8), 0, cv, rows, (T*)b.xc, (T*)b.z, hc.pending);
+  else
+    VN_LAUNCH(ctx, (mamba_conv_kernel<T, 8>), dim3(ceil_div(n, 32), ceil_div(M, 64)), dim3(32, 8), 0, cv, rows, (T*)b.xc, (T*)b.z, hc.pending);
   if (rows.max_n > hc.pending)
     VN_LAUNCH(ctx, conv_tail_kernel<T>, dim3(ceil_div(n, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
   MambaArgs a;

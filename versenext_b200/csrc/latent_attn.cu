@@ -52,6 +52,6 @@ int32_t vn_latent_attention(vn_ctx* ctx, const LatentArgs& a, bool bf16, bool mm
     default: return vn_fail(ctx, VN_ERR_UNSUPPORTED, "latent pitch %d", a.Rp);
   }
   if (st != VN_OK || a.splits <= 1) return st;
-  VN_LAUNCH(ctx, latent_merge_kernel<__nv_bfloat16>, ceil_div(a.rows.M * a.H, 8), 256, 0, a);
+  VN_LAUNCH(ctx, latent_merge_kernel<__nv_bfloat16>, a.rows.M * a.H, 128, 0, a);
   return VN_OK;
 }

@@ -326,21 +326,33 @@ __global__ void __launch_bounds__(128) latent_attn_mma_kernel(LatentArgs a) {
     }
 }
 
-// merges the key splits: one warp per (row, head).  grid ceil(M H / 8)
+// merges the key splits: one CTA of 128 threads per (row, head).  grid M H
 template <typename T>
-__global__ void __launch_bounds__(256) latent_merge_kernel(LatentArgs a) {
-  const long long n = (long long)a.rows.M * a.H, rf = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentArgs a) {
+  __shared__ float s_w[32];
+  const long long n = (long long)a.rows.M * a.H, rf = blockIdx.x;
   const int lane = threadIdx.x & 31;
-  if (rf >= n) return;
-  float m = a.sink ? a.sink[rf % a.H] : -CUDART_INF_F;
-  for (int s = 0; s < a.splits; ++s) m = fmaxf(m, a.part_ml[2 * (s * n + rf)]);
-  float l = a.sink ? expf(a.sink[rf % a.H] - m) : 0.f;
-  for (int s = 0; s < a.splits; ++s) l += a.part_ml[2 * (s * n + rf) + 1] * expf(a.part_ml[2 * (s * n + rf)] - m);
-  const float w = (a.gate ? a.gate[rf] : 1.f) / l;
-  for (int j = lane; j < a.Rp; j += 32) {
-    float v = 0.f;
-    for (int s = 0; s < a.splits; ++s) v = fmaf(a.part_o[(s * n + rf) * a.Rp + j], expf(a.part_ml[2 * (s * n + rf)] - m), v);
-    reinterpret_cast<T*>(a.out)[rf * a.Rp + j] = from_f<T>(v * w);
+  // every warp: lane s holds split s (at most 32)
+  const float ms = lane < a.splits ? a.part_ml[2 * (lane * n + rf)] : -CUDART_INF_F;
+  const float ls = lane < a.splits ? a.part_ml[2 * (lane * n + rf) + 1] : 0.f;
+  const float sk = a.sink ? a.sink[rf % a.H] : -CUDART_INF_F;
+  float m = fmaxf(ms, sk);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+  const float f = expf(ms - m);
+  const float l = warp_sum(ls * f) + (a.sink ? expf(sk - m) : 0.f);
+  if (threadIdx.x < 32) s_w[lane] = f * ((a.gate ? a.gate[rf] : 1.f) / l);
+  __syncthreads();
+  for (int j = threadIdx.x * 4; j < a.Rp; j += 512) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = 0; s < a.splits; ++s) {
+      const float4 t = *reinterpret_cast<const float4*>(a.part_o + (s * n + rf) * a.Rp + j);
+      const float ws = s_w[s];
+      v.x = fmaf(t.x, ws, v.x); v.y = fmaf(t.y, ws, v.y); v.z = fmaf(t.z, ws, v.z); v.w = fmaf(t.w, ws, v.w);
+    }
+    T* o = reinterpret_cast<T*>(a.out) + rf * a.Rp + j;
+    o[0] = from_f<T>(v.x); o[1] = from_f<T>(v.y); o[2] = from_f<T>(v.z); o[3] = from_f<T>(v.w);
   }
 }
 

@@ -37,8 +37,14 @@ struct Src {
   int ld = 0;
   __device__ __forceinline__ float get(long long row, int col) const {
     const float* q = p + row * ld + col;
-    float a = *q;
-    for (int s = 1; s < splits; ++s) a += q[(long long)s * pstride];
+    if (splits == 1) return *q;
+    float a = 0.f;
+    int s = 0;
+    for (; s + 4 <= splits; s += 4) {          // four slices requested before the first is added; slice order kept
+      const float t0 = q[s * pstride], t1 = q[(s + 1) * pstride], t2 = q[(s + 2) * pstride], t3 = q[(s + 3) * pstride];
+      a += t0; a += t1; a += t2; a += t3;
+    }
+    for (; s < splits; ++s) a += q[s * pstride];
     return a;
   }
 };
@@ -50,6 +56,10 @@ __device__ __forceinline__ float warp_sum(float v) {
 }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// silu of a value that is kept in T: the fast exponential and division where that is 16 bits wide
+template <typename T> __device__ __forceinline__ float silu_as(float z) {
+  return sizeof(T) == 2 ? __fdividef(z, 1.0f + __expf(-z)) : z / (1.0f + expf(-z));
+}
 template <typename T> __device__ __forceinline__ float round_to(float v) { return to_f<T>(from_f<T>(v)); }
 
 // block-wide sum of one value per thread (256 threads), the same total in every thread
@@ -86,12 +96,48 @@ struct ConvIn {
   __device__ __forceinline__ float at(int row, int r0, int start, int slot, int c, float* cur) const {
     const int pos = start + row - r0;
     const float* wc = w + (long long)c * taps;
-    float x = input(row, r0, start, slot, pos, c);
-    *cur = x;
-    float acc = x * wc[taps - 1];
-    for (int j = 1; j < taps; ++j) acc = fmaf(input(row, r0, start, slot, pos - j, c), wc[taps - 1 - j], acc);
+    float acc, x[4], f[4];
+    if (taps <= 4) {                           // the usual lengths: all inputs requested before the first is used
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        f[j] = j < taps ? wc[taps - 1 - j] : 0.f;
+        x[j] = j < taps ? input(row, r0, start, slot, pos - j, c) : 0.f;
+      }
+      acc = x[0] * f[0];
+#pragma unroll
+      for (int j = 1; j < 4; ++j) acc = fmaf(x[j], f[j], acc);
+    } else {
+      x[0] = input(row, r0, start, slot, pos, c);
+      acc = x[0] * wc[taps - 1];
+      for (int j = 1; j < taps; ++j) acc = fmaf(input(row, r0, start, slot, pos - j, c), wc[taps - 1 - j], acc);
+    }
+    *cur = x[0];
+    return activate(acc, c);
+  }
+  __device__ __forceinline__ float activate(float acc, int c) const {
     if (bias) acc += bias[c];
-    return acc / (1.0f + expf(-acc));
+    return silu_as<T>(acc);
+  }
+  // The same for rows row, row + 1, .. row + RB - 1 (those below row_end, all of one entry): every input is read once.
+  // taps <= 4.  Nothing is stored here, so that the loads of several calls can be in flight together.
+  template <int RB>
+  __device__ __forceinline__ void run(int row, int row_end, int r0, int start, int slot, int c, float (&out)[RB]) const {
+    const int pos = start + row - r0;
+    const float* wc = w + (long long)c * taps;
+    float wt[4], x[RB + 3];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) wt[j] = j < taps ? wc[taps - 1 - j] : 0.f;
+#pragma unroll
+    for (int j = 1; j < 4; ++j) x[3 - j] = j < taps ? input(row, r0, start, slot, pos - j, c) : 0.f;
+#pragma unroll
+    for (int i = 0; i < RB; ++i) x[3 + i] = row + i < row_end ? round_to<T>(src.get(row + i, col0 + c)) : 0.f;
+#pragma unroll
+    for (int i = 0; i < RB; ++i) {
+      float acc = x[3 + i] * wt[0];
+#pragma unroll
+      for (int j = 1; j < 4; ++j) acc = fmaf(x[3 + i - j], wt[j], acc);
+      out[i] = activate(acc, c);
+    }
   }
   __device__ __forceinline__ void keep(int slot, int pos, int c, float v) const {
     ring[((long long)slot * RC + pos % RC) * C + c] = from_f<T>(v);

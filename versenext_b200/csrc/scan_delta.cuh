@@ -2,9 +2,9 @@
 //
 //   S <- g * S (row-wise) ; u = beta (v - S^T k) ; S <- S + k u^T ; o = S^T q
 //
-// The columns of S are independent of one another, so a column is the unit of parallelism: eight lanes share one (each
-// holds DK of its rows in registers), a CTA of 128 threads takes 16 columns of one head of one sequence and runs over
-// the sequence's new tokens, with the next CT tokens' q, k, g, v already being copied to shared memory.
+// The columns of S are independent of one another, so a column is the unit of parallelism; a group of lanes holds some
+// columns in registers (rows spread over the lanes) and runs over the sequence's new tokens, while the next tokens'
+// q, k, g, v are already being copied to shared memory.
 // State layout [slot][R][head][vdim][dim] (a column is contiguous); ring of states as in scan_mamba.cuh.
 #pragma once
 #include "gemm_mma.cuh"
@@ -37,50 +37,74 @@ struct DeltaIn {
 constexpr float UNIT_EPS = 1e-6f;   // inside the root of the unit norm of q and k
 
 // Convolution + silu of q, k, v; unit vectors of q and k; beta; the two low-rank factors in the storage dtype.
-// One warp per (row, unit): units 0 .. KH-1 q heads, then KH k heads, H v heads, and one for the rest.
-// grid (2 KH + H + 1, ceil(M / 8)), block (32, 8)
-template <typename T, int NC>      // NC: channels per lane (d, vd <= 32 NC)
+// One warp per (RB rows, unit): units 0 .. KH-1 q heads, then KH k heads, H v heads, and one for the rest.
+// grid (2 KH + H + 1, ceil(M / (8 RB))), block (32, 8)
+template <typename T, int NC, int RB>      // NC: channels per lane (d, vd <= 32 NC)
 __global__ void __launch_bounds__(256) delta_inputs_kernel(ConvIn<T> in, DeltaIn a) {
-  const int row = blockIdx.y * 8 + threadIdx.y, lane = threadIdx.x, unit = blockIdx.x;
-  if (row >= a.rows.M) return;
-  int slot, r0, n, start;
-  a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
-  if (unit == 2 * a.KH + a.H) {
-    for (int h = lane; h < a.H; h += 32) a.beta[(long long)row * a.H + h] = sigmoid_f(a.src.get(row, a.col_b + h));
-    for (int j = lane; j < a.ra_ld; j += 32)
-      reinterpret_cast<T*>(a.low_a)[(long long)row * a.ra_ld + j] = from_f<T>(j < a.ra ? a.src.get(row, a.col_a + j) : 0.f);
-    for (int j = lane; j < a.rg_ld; j += 32)
-      reinterpret_cast<T*>(a.low_g)[(long long)row * a.rg_ld + j] = from_f<T>(j < a.rg ? a.src.get(row, a.col_g + j) : 0.f);
-    return;
-  }
-  const bool is_v = unit >= 2 * a.KH;
+  const int lane = threadIdx.x, unit = blockIdx.x;
+  int row = (blockIdx.y * 8 + threadIdx.y) * RB;
+  const int last = min(row + RB, a.rows.M);
+  const bool is_v = unit >= 2 * a.KH, is_k = !is_v && unit >= a.KH;
   const int w = is_v ? a.vd : a.d;
   const int c0 = is_v ? 2 * a.KH * a.d + (unit - 2 * a.KH) * a.vd : unit * a.d;
-  float val[NC], ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < NC; ++i) {
-    const int j = lane + 32 * i;
-    val[i] = 0.f;
-    if (j < w) {
-      float cur;
-      val[i] = in.at(row, r0, start, slot, c0 + j, &cur);
-      if (n <= a.pending) in.keep(slot, start + row - r0, c0 + j, cur);
-      ss += val[i] * val[i];
+  while (row < last) {                                  // stretches of one entry
+    if (unit == 2 * a.KH + a.H) {
+      for (int h = lane; h < a.H; h += 32) a.beta[(long long)row * a.H + h] = sigmoid_f(a.src.get(row, a.col_b + h));
+      for (int j = lane; j < a.ra_ld; j += 32)
+        reinterpret_cast<T*>(a.low_a)[(long long)row * a.ra_ld + j] = from_f<T>(j < a.ra ? a.src.get(row, a.col_a + j) : 0.f);
+      for (int j = lane; j < a.rg_ld; j += 32)
+        reinterpret_cast<T*>(a.low_g)[(long long)row * a.rg_ld + j] = from_f<T>(j < a.rg ? a.src.get(row, a.col_g + j) : 0.f);
+      ++row;
+      continue;
     }
-  }
-  float* dst;
-  float f = 1.f;
-  if (is_v) {
-    dst = a.v + (long long)row * a.H * a.vd + (unit - 2 * a.KH) * a.vd;
-  } else {
-    const bool is_k = unit >= a.KH;
-    f = 1.f / sqrtf(warp_sum(ss) + UNIT_EPS);
-    if (!is_k) f *= 1.f / sqrtf((float)a.d);
-    dst = (is_k ? a.k : a.q) + (long long)row * a.KH * a.d + (is_k ? unit - a.KH : unit) * a.d;
-  }
+    int slot, r0, n, start;
+    a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
+    const int first = row, end = min(last, r0 + n);
+    float val[RB][NC];
 #pragma unroll
-  for (int i = 0; i < NC; ++i)
-    if (lane + 32 * i < w) dst[lane + 32 * i] = val[i] * f;
+    for (int i = 0; i < NC; ++i) {
+      const int j = lane + 32 * i;
+      float v[RB];
+#pragma unroll
+      for (int r = 0; r < RB; ++r) v[r] = 0.f;
+      if (j < w) {
+        if (RB > 1 && in.taps <= 4) {
+          in.template run<RB>(first, end, r0, start, slot, c0 + j, v);
+        } else {
+#pragma unroll
+          for (int r = 0; r < RB; ++r) {
+            float cur;
+            if (first + r < end) v[r] = in.at(first + r, r0, start, slot, c0 + j, &cur);
+          }
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < RB; ++r) val[r][i] = v[r];
+    }
+    if (n <= a.pending)
+      for (int r = first; r < end; ++r)
+        for (int j = lane; j < w; j += 32) in.keep(slot, start + r - r0, c0 + j, in.src.get(r, in.col0 + c0 + j));
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      if (first + r >= end) break;
+      float* dst;
+      float f = 1.f;
+      if (is_v) {
+        dst = a.v + (long long)(first + r) * a.H * a.vd + (unit - 2 * a.KH) * a.vd;
+      } else {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NC; ++i) ss += val[r][i] * val[r][i];
+        f = 1.f / sqrtf(warp_sum(ss) + UNIT_EPS);
+        if (!is_k) f *= 1.f / sqrtf((float)a.d);
+        dst = (is_k ? a.k : a.q) + (long long)(first + r) * a.KH * a.d + (is_k ? unit - a.KH : unit) * a.d;
+      }
+#pragma unroll
+      for (int i = 0; i < NC; ++i)
+        if (lane + 32 * i < w) dst[lane + 32 * i] = val[r][i] * f;
+    }
+    row = end;
+  }
 }
 
 // g = exp(-exp(A_log_h) softplus(g + dt_bias)), in place over [M, H * d];  decay_rate[h] = exp(A_log_h)
@@ -107,9 +131,8 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const float* __restrict_
   for (int j = lane; j < vd; j += 32) out[i * vd + j] = from_f<T>(oi[j] / r * w[j] * sigmoid_f(gate[i * vd + j]));
 }
 
-// rows of a column held by a lane: register 4 i + e <-> row 32 i + 4 li + e (so that eight lanes read 128 contiguous
+// One-token kernel: eight lanes share a column; rows of it held by a lane: register 4 i + e <-> row 32 i + 4 li + e (so that eight lanes read 128 contiguous
 // bytes of q, k, g, and of a state column)
-constexpr int DR_COLS = 16;
 
 template <int DK>
 __device__ __forceinline__ void delta_col_load(const float* col, int d, int li, bool ok, float (&S)[DK]) {
@@ -139,35 +162,44 @@ __device__ __forceinline__ void delta_col_store(float* col, int d, int li, const
     }
   }
 }
-// one token of one column (the lane's rows): returns the lane's part of o
-template <int DK>
-__device__ __forceinline__ float delta_col_step(float (&S)[DK], const float* q, const float* k, const float* g, int li,
-                                                float v, float beta) {
-  float d0 = 0.f, d1 = 0.f;
+// one token of NP columns (the lane's rows of each); o[p] receives the lane's part of the read-out
+template <int DK, int NP>
+__device__ __forceinline__ void delta_cols_step(float (&S)[NP][DK], const float* q, const float* k, const float* g, int li,
+                                                const float (&v)[NP], float beta, float (&o)[NP]) {
+  float dot[NP];
+#pragma unroll
+  for (int p = 0; p < NP; ++p) dot[p] = 0.f;
 #pragma unroll
   for (int i = 0; i < DK / 4; ++i) {
     const float4 gv = *reinterpret_cast<const float4*>(g + 32 * i + 4 * li);
     const float4 kv = *reinterpret_cast<const float4*>(k + 32 * i + 4 * li);
-    S[4 * i] *= gv.x; S[4 * i + 1] *= gv.y; S[4 * i + 2] *= gv.z; S[4 * i + 3] *= gv.w;
-    d0 = fmaf(S[4 * i], kv.x, d0); d1 = fmaf(S[4 * i + 1], kv.y, d1);
-    d0 = fmaf(S[4 * i + 2], kv.z, d0); d1 = fmaf(S[4 * i + 3], kv.w, d1);
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+      S[p][4 * i] *= gv.x; S[p][4 * i + 1] *= gv.y; S[p][4 * i + 2] *= gv.z; S[p][4 * i + 3] *= gv.w;
+      dot[p] = fmaf(S[p][4 * i], kv.x, dot[p]); dot[p] = fmaf(S[p][4 * i + 1], kv.y, dot[p]);
+      dot[p] = fmaf(S[p][4 * i + 2], kv.z, dot[p]); dot[p] = fmaf(S[p][4 * i + 3], kv.w, dot[p]);
+    }
   }
-  float dot = d0 + d1;
-  dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-  dot += __shfl_xor_sync(0xffffffffu, dot, 2);
-  dot += __shfl_xor_sync(0xffffffffu, dot, 4);
-  const float u = beta * (v - dot);
-  float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+  for (int p = 0; p < NP; ++p) {
+    dot[p] += __shfl_xor_sync(0xffffffffu, dot[p], 1);
+    dot[p] += __shfl_xor_sync(0xffffffffu, dot[p], 2);
+    dot[p] += __shfl_xor_sync(0xffffffffu, dot[p], 4);
+    dot[p] = beta * (v[p] - dot[p]);
+    o[p] = 0.f;
+  }
 #pragma unroll
   for (int i = 0; i < DK / 4; ++i) {
     const float4 kv = *reinterpret_cast<const float4*>(k + 32 * i + 4 * li);
     const float4 qv = *reinterpret_cast<const float4*>(q + 32 * i + 4 * li);
-    S[4 * i] = fmaf(kv.x, u, S[4 * i]); S[4 * i + 1] = fmaf(kv.y, u, S[4 * i + 1]);
-    S[4 * i + 2] = fmaf(kv.z, u, S[4 * i + 2]); S[4 * i + 3] = fmaf(kv.w, u, S[4 * i + 3]);
-    o0 = fmaf(S[4 * i], qv.x, o0); o1 = fmaf(S[4 * i + 1], qv.y, o1);
-    o0 = fmaf(S[4 * i + 2], qv.z, o0); o1 = fmaf(S[4 * i + 3], qv.w, o1);
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+      S[p][4 * i] = fmaf(kv.x, dot[p], S[p][4 * i]); S[p][4 * i + 1] = fmaf(kv.y, dot[p], S[p][4 * i + 1]);
+      S[p][4 * i + 2] = fmaf(kv.z, dot[p], S[p][4 * i + 2]); S[p][4 * i + 3] = fmaf(kv.w, dot[p], S[p][4 * i + 3]);
+      o[p] = fmaf(S[p][4 * i], qv.x, o[p]); o[p] = fmaf(S[p][4 * i + 1], qv.y, o[p]);
+      o[p] = fmaf(S[p][4 * i + 2], qv.z, o[p]); o[p] = fmaf(S[p][4 * i + 3], qv.w, o[p]);
+    }
   }
-  return o0 + o1;
 }
 
 // 4 or 16 bytes from global to shared memory, asynchronously
@@ -178,33 +210,115 @@ __device__ __forceinline__ void cp_async_f(float* s, const float* g) {
   else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(a), "l"(g));
 }
 
-// DK rows per lane (d <= 8 DK); VEC 4 when d and vd are multiples of 4.  grid (ceil(vd / 16), H, n_ent), 128 threads
-template <int DK, int VEC>
-__global__ void __launch_bounds__(128) delta_scan_kernel(DeltaRuleArgs a) {
-  constexpr int DP = 8 * DK, CT = DK > 16 ? 4 : 8;
-  __shared__ __align__(16) float s_q[2][CT][DP], s_k[2][CT][DP], s_g[2][CT][DP], s_v[2][CT][DR_COLS];
-  __shared__ float s_b[2][CT], s_o[CT][DR_COLS];
+// ---- the scan over new tokens --------------------------------------------------------------------------------------
+// Sixteen lanes share NC columns of the state, each with RPL rows of all of them, so that what a lane reads of q, k and g
+// serves NC columns.  The NC partial sums of a dot product are reduced by halving: after log2(NC) exchanges every lane is
+// left with one column's sum, the remaining exchanges complete it.  Rows are handled in pairs (two fp32 products or
+// sums in one instruction).  Register 4 i + e <-> row 64 i + 4 li + e.
+__device__ __forceinline__ unsigned long long f2_pack(float x, float y) {
+  unsigned long long r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ float f2_sum(unsigned long long v) {
+  float x, y;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v));
+  return x + y;
+}
+__device__ __forceinline__ unsigned long long f2_mul(unsigned long long a, unsigned long long b) {
+  unsigned long long r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ unsigned long long f2_fma(unsigned long long a, unsigned long long b, unsigned long long c) {
+  unsigned long long r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+// sum of v[c] over the sixteen lanes of a group: the lane returns the total of column delta_scan_col<NC>(li)
+template <int NC> __device__ __forceinline__ int delta_scan_col(int li) { return NC == 8 ? li >> 1 : li >> 2; }
+template <int NC>
+__device__ __forceinline__ float group_sum(float (&v)[NC], int li) {
+#pragma unroll
+  for (int half = NC / 2, bit = 8; half >= 1; half >>= 1, bit >>= 1) {
+    const bool up = li & bit;
+#pragma unroll
+    for (int c = 0; c < half; ++c) {
+      const float give = up ? v[c] : v[c + half], keep = up ? v[c + half] : v[c];
+      v[c] = keep + __shfl_xor_sync(0xffffffffu, give, bit);
+    }
+  }
+  float s = v[0];
+#pragma unroll
+  for (int bit = 8 / NC; bit >= 1; bit >>= 1) s += __shfl_xor_sync(0xffffffffu, s, bit);
+  return s;
+}
+
+// RPL rows per lane (d <= 16 RPL); NC columns per group; VEC 4 when d and vd are multiples of 4; W warps.
+// grid (ceil(vd / (2 NC W)), H, n_ent), 32 W threads
+template <int RPL, int NC, int VEC, int W>
+__global__ void __launch_bounds__(32 * W) delta_scan_kernel(DeltaRuleArgs a) {
+  constexpr int DP = 16 * RPL, CT = RPL > 8 ? 4 : 8, COLS = 2 * NC * W, THREADS = 32 * W;
+  typedef unsigned long long u64;
+  __shared__ __align__(16) float s_q[2][CT][DP], s_k[2][CT][DP], s_g[2][CT][DP], s_v[2][CT][COLS];
+  __shared__ float s_b[2][CT], s_o[CT][COLS];
   int slot, r0, n, start;
   a.rows.entry(blockIdx.z, &slot, &r0, &n, &start);
   if (n <= 0) return;
-  const int tid = threadIdx.x, h = blockIdx.y, kh = h / (a.H / a.KH), c0 = blockIdx.x * DR_COLS;
-  const int cl = tid >> 3, li = tid & 7;              // column of the CTA, lane of the column
-  const bool ok = c0 + cl < a.vd;
-  const int d = a.d, vd = a.vd, nv = min(DR_COLS, vd - c0);
-  for (int i = tid; i < 2 * CT * DP; i += 128) (&s_q[0][0][0])[i] = (&s_k[0][0][0])[i] = (&s_g[0][0][0])[i] = 0.f;
-  for (int i = tid; i < 2 * CT * DR_COLS; i += 128) (&s_v[0][0][0])[i] = 0.f;
+  const int tid = threadIdx.x, lane = tid & 31, h = blockIdx.y, kh = h / (a.H / a.KH), c0 = blockIdx.x * COLS;
+  const int li = lane & 15, gcol = (tid >> 4) * NC;    // lane of the group; the group's first column in the CTA
+  const int mine = gcol + delta_scan_col<NC>(li);      // the column whose sums this lane ends up with
+  const int d = a.d, vd = a.vd, nv = min(COLS, vd - c0);
+  for (int i = tid; i < 2 * CT * DP; i += THREADS) (&s_q[0][0][0])[i] = (&s_k[0][0][0])[i] = (&s_g[0][0][0])[i] = 0.f;
+  for (int i = tid; i < 2 * CT * COLS; i += THREADS) (&s_v[0][0][0])[i] = 0.f;
   __syncthreads();
-  float S[DK];
+  u64 S[NC][RPL / 2];
   const long long one = (long long)vd * d;
-  delta_col_load<DK>(a.state + (((long long)slot * a.R + start % a.R) * a.H + h) * one + (long long)(c0 + cl) * d, d, li,
-                     ok && start > 0, S);
-  auto store_state = [&](int p) {
-    if (ok) delta_col_store<DK>(a.state + (((long long)slot * a.R + p % a.R) * a.H + h) * one + (long long)(c0 + cl) * d, d, li, S);
+  const bool vec = (d & 3) == 0;
+  const float* st_in = a.state + (((long long)slot * a.R + start % a.R) * a.H + h) * one;
+#pragma unroll
+  for (int c = 0; c < NC; ++c)
+#pragma unroll
+    for (int i = 0; i < RPL / 4; ++i) {
+      const int r = 64 * i + 4 * li;
+      const float* p = st_in + (long long)(c0 + gcol + c) * d + r;
+      const bool ok = start > 0 && c0 + gcol + c < vd;
+      float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (ok && vec && r < d) t = *reinterpret_cast<const float4*>(p);
+      else if (ok) {
+        if (r < d) t.x = p[0];
+        if (r + 1 < d) t.y = p[1];
+        if (r + 2 < d) t.z = p[2];
+        if (r + 3 < d) t.w = p[3];
+      }
+      S[c][2 * i] = f2_pack(t.x, t.y);
+      S[c][2 * i + 1] = f2_pack(t.z, t.w);
+    }
+  auto store_state = [&](int pos) {
+    float* st = a.state + (((long long)slot * a.R + pos % a.R) * a.H + h) * one;
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+      for (int i = 0; i < RPL / 4; ++i) {
+        const int r = 64 * i + 4 * li;
+        if (c0 + gcol + c >= vd || r >= d) continue;
+        float* p = st + (long long)(c0 + gcol + c) * d + r;
+        float4 t;
+        asm("mov.b64 {%0, %1}, %2;" : "=f"(t.x), "=f"(t.y) : "l"(S[c][2 * i]));
+        asm("mov.b64 {%0, %1}, %2;" : "=f"(t.z), "=f"(t.w) : "l"(S[c][2 * i + 1]));
+        if (vec) *reinterpret_cast<float4*>(p) = t;
+        else {
+          p[0] = t.x;
+          if (r + 1 < d) p[1] = t.y;
+          if (r + 2 < d) p[2] = t.z;
+          if (r + 3 < d) p[3] = t.w;
+        }
+      }
   };
   auto fetch = [&](int t0, int buf) {
     const int m = min(CT, n - t0);
     const int per = d / VEC;
-    for (int i = tid; i < m * per; i += 128) {
+    for (int i = tid; i < m * per; i += THREADS) {
       const int t = i / per, j = (i % per) * VEC;
       const long long row = r0 + t0 + t;
       cp_async_f<VEC>(&s_q[buf][t][j], a.q + row * a.KH * d + kh * d + j);
@@ -212,7 +326,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaRuleArgs a) {
       cp_async_f<VEC>(&s_g[buf][t][j], a.g + row * a.H * d + h * d + j);
     }
     const int pv = nv / VEC;
-    for (int i = tid; i < m * pv; i += 128) {
+    for (int i = tid; i < m * pv; i += THREADS) {
       const int t = i / pv, j = (i % pv) * VEC;
       cp_async_f<VEC>(&s_v[buf][t][j], a.v + (long long)(r0 + t0 + t) * a.H * vd + h * vd + c0 + j);
     }
@@ -226,18 +340,78 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaRuleArgs a) {
     else mma_detail::cp_async_wait<0>();
     __syncthreads();
     const int m = min(CT, n - t0);
-#pragma unroll 2
-    for (int t = 0; t < m; ++t) {
-      float o = delta_col_step<DK>(S, s_q[buf][t], s_k[buf][t], s_g[buf][t], li, s_v[buf][t][cl], s_b[buf][t]);
-      o += __shfl_xor_sync(0xffffffffu, o, 1);
-      o += __shfl_xor_sync(0xffffffffu, o, 2);
-      o += __shfl_xor_sync(0xffffffffu, o, 4);
-      if (li == 0) s_o[t][cl] = o;
-      if (snap) store_state(start + t0 + t + 1);
+    // The read-out sums of a token are finished together with the next token's first sums, and the next token's operands
+    // are fetched under them: the recurrence itself (sum, exchange, update) is what is left on the critical path.
+    u64 gg[RPL / 2], kk[RPL / 2], qq[RPL / 2];
+    float part[NC], late[NC], vb, bb;
+    auto operands = [&](int t) {
+#pragma unroll
+      for (int i = 0; i < RPL / 4; ++i) {
+        const ulonglong2 g2 = *reinterpret_cast<const ulonglong2*>(&s_g[buf][t][64 * i + 4 * li]);
+        const ulonglong2 k2 = *reinterpret_cast<const ulonglong2*>(&s_k[buf][t][64 * i + 4 * li]);
+        const ulonglong2 q2 = *reinterpret_cast<const ulonglong2*>(&s_q[buf][t][64 * i + 4 * li]);
+        gg[2 * i] = g2.x; gg[2 * i + 1] = g2.y; kk[2 * i] = k2.x; kk[2 * i + 1] = k2.y; qq[2 * i] = q2.x; qq[2 * i + 1] = q2.y;
+      }
+      vb = s_v[buf][t][mine];
+      bb = s_b[buf][t];
+    };
+    operands(0);
+    auto token = [&](int t, bool has_late) {
+      {
+        u64 acc[NC];
+#pragma unroll
+        for (int i = 0; i < RPL / 2; ++i)
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            S[c][i] = f2_mul(S[c][i], gg[i]);
+            acc[c] = i ? f2_fma(S[c][i], kk[i], acc[c]) : f2_mul(S[c][0], kk[0]);
+          }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) part[c] = f2_sum(acc[c]);
+      }
+      const float dot = group_sum<NC>(part, li);
+      if (has_late) {
+        const float o = group_sum<NC>(late, li);
+        if ((li & (16 / NC - 1)) == 0) s_o[t - 1][mine] = o;
+      }
+      const float u = bb * (vb - dot);
+      u64 uc[NC], k0[RPL / 2], q0[RPL / 2];
+#pragma unroll
+      for (int i = 0; i < RPL / 2; ++i) { k0[i] = kk[i]; q0[i] = qq[i]; }
+      operands(min(t + 1, CT - 1));
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        const float x = __shfl_sync(0xffffffffu, u, (lane & 16) + c * (16 / NC));
+        uc[c] = f2_pack(x, x);
+      }
+      u64 acc[NC];
+#pragma unroll
+      for (int i = 0; i < RPL / 2; ++i)
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          S[c][i] = f2_fma(k0[i], uc[c], S[c][i]);
+          acc[c] = i ? f2_fma(S[c][i], q0[i], acc[c]) : f2_mul(S[c][0], q0[0]);
+        }
+#pragma unroll
+      for (int c = 0; c < NC; ++c) late[c] = f2_sum(acc[c]);
+    };
+    if (!snap && m == CT) {
+      token(0, false);
+#pragma unroll
+      for (int t = 1; t < CT; ++t) token(t, true);
+    } else {
+      for (int t = 0; t < m; ++t) {
+        token(t, t > 0);
+        if (snap) store_state(start + t0 + t + 1);
+      }
+    }
+    {
+      const float o = group_sum<NC>(late, li);
+      if ((li & (16 / NC - 1)) == 0) s_o[m - 1][mine] = o;
     }
     __syncthreads();
-    for (int i = tid; i < m * DR_COLS; i += 128) {
-      const int t = i / DR_COLS, j = i % DR_COLS;
+    for (int i = tid; i < m * COLS; i += THREADS) {
+      const int t = i / COLS, j = i % COLS;
       if (j < nv) a.o[(long long)(r0 + t0 + t) * a.H * vd + h * vd + c0 + j] = s_o[t][j];
     }
   }
@@ -264,6 +438,7 @@ template <typename T>
 __device__ __forceinline__ float low_rank_dot(const T* w, const float* s, int ld, int part, int parts) {
   float acc = 0.f;
   if (sizeof(T) == 2) {
+#pragma unroll 4
     for (int j = part * 8; j < ld; j += parts * 8) {
       const uint4 u = *reinterpret_cast<const uint4*>(w + j);
       const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
@@ -280,25 +455,28 @@ __device__ __forceinline__ float low_rank_dot(const T* w, const float* s, int ld
   return acc;
 }
 
-// shared memory: 3 DP + 2 vd + ra_ld + rg_ld floats.  grid (H, M)
-template <typename T, int DK>
+// NP: columns a lane takes at a time (the state of 32 NP columns is requested before anything else, so that it arrives
+// under the convolutions and the low-rank products).  Shared memory: 3 DP + 3 vd + ra_ld + rg_ld floats.  grid (H, M)
+template <typename T, int DK, int NP>
 __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepArgs<T> a) {
   constexpr int DP = 8 * DK;
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[8], s_misc[2];
   const DeltaIn& in = a.in;
   const int d = in.d, vd = in.vd, H = in.H, KH = in.KH;
-  float *s_q = sm, *s_k = s_q + DP, *s_g = s_k + DP, *s_a = s_g + DP, *s_w = s_a + in.ra_ld, *s_v = s_w + in.rg_ld, *s_o = s_v + vd;
+  float *s_q = sm, *s_k = s_q + DP, *s_g = s_k + DP, *s_a = s_g + DP, *s_w = s_a + in.ra_ld, *s_v = s_w + in.rg_ld,
+        *s_o = s_v + vd, *s_gate = s_o + vd;
   const int tid = threadIdx.x, h = blockIdx.x, row = blockIdx.y, kh = h / (H / KH);
   int slot, r0, n, start;
   in.rows.entry(in.rows.entry_of(row), &slot, &r0, &n, &start);
-  // this thread's first column of the state: requested before anything else
   const int cl = tid >> 3, li = tid & 7;
   const long long one = (long long)vd * d;
   const float* st_in = a.state + (((long long)slot * a.R + start % a.R) * H + h) * one;
   float* st_out = a.state + (((long long)slot * a.R + (start + 1) % a.R) * H + h) * one;
-  float S[DK];
-  delta_col_load<DK>(st_in + (long long)cl * d, d, li, start > 0 && cl < vd, S);
+  float S[NP][DK];
+#pragma unroll
+  for (int p = 0; p < NP; ++p)
+    delta_col_load<DK>(st_in + (long long)(cl + 32 * p) * d, d, li, start > 0 && cl + 32 * p < vd, S[p]);
   // inputs of this head
   const bool first = h % (H / KH) == 0;              // the group's first head keeps the shared q / k inputs
   for (int i = tid; i < 2 * DP + vd; i += 256) {
@@ -321,7 +499,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepArgs<T> a) {
   for (int j = tid; j < in.rg_ld; j += 256) s_w[j] = j < in.rg ? round_to<T>(in.src.get(row, in.col_g + j)) : 0.f;
   if (tid == 0) s_misc[0] = sigmoid_f(in.src.get(row, in.col_b + h));
   __syncthreads();
-  // unit norms: warp 0 takes q, warp 1 takes k; the others already start on the decays
+  // unit norms: warp 0 takes q, warp 1 takes k
   const int warp = tid >> 5, lane = tid & 31;
   if (warp < 2) {
     float* s = warp ? s_k : s_q;
@@ -331,41 +509,50 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepArgs<T> a) {
     if (!warp) f *= 1.f / sqrtf((float)d);
     for (int j = lane; j < d; j += 32) s[j] *= f;
   }
-  for (int j0 = 0; j0 < DP; j0 += 64) {               // four lanes per key channel
-    const int j = j0 + (tid >> 2);
-    float acc = j < d ? low_rank_dot<T>(a.w_a + (long long)(h * d + j) * in.ra_ld, s_a, in.ra_ld, tid & 3, 4) : 0.f;
+  // decays of the key channels, then gates of the value columns: four lanes per row of the low-rank matrices
+  const int nd = (DP + 63) & ~63;
+#pragma unroll 2
+  for (int j0 = 0; j0 < nd + vd; j0 += 64) {
+    const int jj = j0 + (tid >> 2);
+    const bool dec = j0 < nd;
+    const int j = dec ? jj : jj - nd;
+    float acc = 0.f;
+    if (dec && j < d) acc = low_rank_dot<T>(a.w_a + (long long)(h * d + j) * in.ra_ld, s_a, in.ra_ld, tid & 3, 4);
+    if (!dec && j < vd) acc = low_rank_dot<T>(a.w_g + (long long)(h * vd + j) * in.rg_ld, s_w, in.rg_ld, tid & 3, 4);
     acc += __shfl_xor_sync(0xffffffffu, acc, 1);
     acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-    if ((tid & 3) == 0 && j < DP)
-      s_g[j] = j < d ? expf(-a.decay_rate[h] * softplus_f(acc + a.dt_bias[h * d + j])) : 0.f;
-  }
-  __syncthreads();
-  const float beta = s_misc[0];
-  for (int c0 = 0; c0 < vd; c0 += 32) {
-    const int c = c0 + cl;
-    const bool ok = c < vd;
-    if (c0 > 0) delta_col_load<DK>(st_in + (long long)c * d, d, li, start > 0 && ok, S);
-    float o = delta_col_step<DK>(S, s_q, s_k, s_g, li, ok ? s_v[c] : 0.f, beta);
-    o += __shfl_xor_sync(0xffffffffu, o, 1);
-    o += __shfl_xor_sync(0xffffffffu, o, 2);
-    o += __shfl_xor_sync(0xffffffffu, o, 4);
-    if (ok) {
-      if (li == 0) s_o[c] = o;
-      delta_col_store<DK>(st_out + (long long)c * d, d, li, S);
+    if ((tid & 3) == 0) {
+      if (dec && j < DP) s_g[j] = j < d ? expf(-a.decay_rate[h] * softplus_f(acc + a.dt_bias[h * d + j])) : 0.f;
+      if (!dec && j < vd) s_gate[j] = sigmoid_f(acc);
     }
   }
   __syncthreads();
+  const float beta = s_misc[0];
   float ss = 0.f;
-  for (int j = tid; j < vd; j += 256) ss += s_o[j] * s_o[j];
-  const float r = sqrtf(block_sum256(ss, red) / (float)vd + a.eps);
-  for (int j0 = 0; j0 < vd; j0 += 64) {
-    const int j = j0 + (tid >> 2);
-    float acc = j < vd ? low_rank_dot<T>(a.w_g + (long long)(h * vd + j) * in.rg_ld, s_w, in.rg_ld, tid & 3, 4) : 0.f;
-    acc += __shfl_xor_sync(0xffffffffu, acc, 1);
-    acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-    if ((tid & 3) == 0 && j < vd)
-      a.out[(long long)row * H * vd + h * vd + j] = from_f<T>(s_o[j] / r * a.norm_w[j] * sigmoid_f(acc));
+  for (int c0 = 0; c0 < vd; c0 += 32 * NP) {
+    float v[NP], o[NP];
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+      const int c = c0 + cl + 32 * p;
+      if (c0 > 0) delta_col_load<DK>(st_in + (long long)c * d, d, li, start > 0 && c < vd, S[p]);
+      v[p] = c < vd ? s_v[c] : 0.f;
+    }
+    delta_cols_step<DK, NP>(S, s_q, s_k, s_g, li, v, beta, o);
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+      const int c = c0 + cl + 32 * p;
+      o[p] += __shfl_xor_sync(0xffffffffu, o[p], 1);
+      o[p] += __shfl_xor_sync(0xffffffffu, o[p], 2);
+      o[p] += __shfl_xor_sync(0xffffffffu, o[p], 4);
+      if (c < vd) {
+        if (li == 0) { s_o[c] = o[p]; ss += o[p] * o[p]; }
+        delta_col_store<DK>(st_out + (long long)c * d, d, li, S[p]);
+      }
+    }
   }
+  const float r = sqrtf(block_sum256(ss, red) / (float)vd + a.eps);     // its barrier also publishes s_o
+  for (int j = tid; j < vd; j += 256)
+    a.out[(long long)row * H * vd + h * vd + j] = from_f<T>(s_o[j] / r * a.norm_w[j] * s_gate[j]);
 }
 
 template <typename T> int32_t vn_delta_inputs(vn_ctx* ctx, const ConvIn<T>& conv, const DeltaIn& in);

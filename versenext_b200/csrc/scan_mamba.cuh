@@ -11,6 +11,7 @@
 // then is a change of the sequence's length and nothing else.
 #pragma once
 #include "rows.cuh"
+#include <type_traits>
 
 struct MambaArgs {
   const float* dt = nullptr;     // [M, inner] W_dt dt, before the bias (scan); unused by the step kernel
@@ -28,19 +29,41 @@ struct MambaArgs {
   Rows rows;
 };
 
-// convolution of the x half, copy of the z half.  grid (ceil(inner / 32), ceil(M / 8)), block (32, 8)
-template <typename T>
+// convolution of the x half, copy of the z half.  grid (ceil(inner / 32), ceil(M / (8 RB))), block (32, 8): a thread
+// takes one channel of RB rows (8 for prompts, 1 when every entry has one row)
+template <typename T, int RB>
 __global__ void __launch_bounds__(256) mamba_conv_kernel(ConvIn<T> in, Rows rows, T* __restrict__ xc, T* __restrict__ z,
                                                          int pending) {
-  const int c = blockIdx.x * 32 + threadIdx.x, row = blockIdx.y * 8 + threadIdx.y;
-  if (c >= in.C || row >= rows.M) return;
-  int slot, r0, n, start;
-  rows.entry(rows.entry_of(row), &slot, &r0, &n, &start);
-  float cur;
-  const float v = in.at(row, r0, start, slot, c, &cur);
-  if (n <= pending) in.keep(slot, start + row - r0, c, cur);
-  xc[(long long)row * in.C + c] = from_f<T>(v);
-  z[(long long)row * in.C + c] = from_f<T>(in.src.get(row, in.col0 + in.C + c));
+  const int c = blockIdx.x * 32 + threadIdx.x;
+  int row = (blockIdx.y * 8 + threadIdx.y) * RB;
+  const int last = min(row + RB, rows.M);
+  if (c >= in.C) return;
+  while (row < last) {                                 // stretches of one entry
+    int slot, r0, n, start;
+    rows.entry(rows.entry_of(row), &slot, &r0, &n, &start);
+    const int first = row, end = min(last, r0 + n);
+    float v[RB], zv[RB];
+    if (RB > 1 && in.taps <= 4) {
+      in.template run<RB>(first, end, r0, start, slot, c, v);
+    } else {
+#pragma unroll
+      for (int r = 0; r < RB; ++r) {
+        float cur;
+        v[r] = first + r < end ? in.at(first + r, r0, start, slot, c, &cur) : 0.f;
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < RB; ++r) zv[r] = first + r < end ? in.src.get(first + r, in.col0 + in.C + c) : 0.f;
+    if (n <= pending)
+      for (int r = first; r < end; ++r) in.keep(slot, start + r - r0, c, in.src.get(r, in.col0 + c));
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      if (first + r >= end) break;
+      xc[(long long)(first + r) * in.C + c] = from_f<T>(v[r]);
+      z[(long long)(first + r) * in.C + c] = from_f<T>(zv[r]);
+    }
+    row = end;
+  }
 }
 
 // the dt columns of W_x x as the operand of W_dt (padding columns zero).  grid M
@@ -51,13 +74,14 @@ __global__ void cast_cols_kernel(Src src, int col0, int n, T* __restrict__ out, 
 }
 
 constexpr int MAMBA_L = 4, MAMBA_CH = 32, MAMBA_CT = 16;
+constexpr float LOG2E = 1.4426950408889634f;       // exp(dt A) = 2^(dt (A log2 e))
 
 // NS: states per lane (nstate <= 4 NS).  grid (ceil(inner / 32), n_ent)
 template <typename T, int NS>
 __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
   constexpr int N4 = MAMBA_L * NS, CT = MAMBA_CT, CH = MAMBA_CH;
   __shared__ float s_dt[2][CT][CH], s_x[2][CT][CH], s_y[CT][CH];
-  __shared__ float s_b[2][CT][N4], s_c[2][CT][N4];
+  __shared__ __align__(16) float s_b[2][CT][N4], s_c[2][CT][N4];
   int slot, r0, n, start;
   a.rows.entry(blockIdx.y, &slot, &r0, &n, &start);
   if (n <= 0) return;
@@ -72,16 +96,16 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
   const float* st_in = a.state + ((long long)slot * a.R + start % a.R) * a.inner * a.nstate;
 #pragma unroll
   for (int j = 0; j < NS; ++j) {
-    const int i = j * MAMBA_L + l;
+    const int i = l * NS + j;
     const bool ok = c_ok && i < a.nstate;
-    A[j] = ok ? a.A[(long long)c * a.nstate + i] : 0.f;
+    A[j] = ok ? a.A[(long long)c * a.nstate + i] * LOG2E : 0.f;
     S[j] = (ok && start > 0) ? st_in[(long long)c * a.nstate + i] : 0.f;
   }
   auto store_state = [&](int p) {
     float* so = a.state + ((long long)slot * a.R + p % a.R) * a.inner * a.nstate;
 #pragma unroll
     for (int j = 0; j < NS; ++j) {
-      const int i = j * MAMBA_L + l;
+      const int i = l * NS + j;
       if (c_ok && i < a.nstate) so[(long long)c * a.nstate + i] = S[j];
     }
   };
@@ -132,18 +156,53 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
     __syncthreads();
     if (t0 + CT < n) fetch(t0 + CT);
     const int m = min(CT, n - t0);
-    for (int t = 0; t < m; ++t) {
-      const float d = s_dt[buf][t][ch], dx = d * s_x[buf][t][ch];
-      float y = 0.f;
+    // G tokens at a time: everything that does not depend on the state first
+    auto tokens = [&](int t, auto tag) {
+      constexpr int G = decltype(tag)::value;
+      __align__(16) float e[G][NS], bx[G][NS], cv[G][NS];
+      float y[G];
 #pragma unroll
-      for (int j = 0; j < NS; ++j) {
-        S[j] = fmaf(expf(d * A[j]), S[j], dx * s_b[buf][t][j * MAMBA_L + l]);
-        y = fmaf(S[j], s_c[buf][t][j * MAMBA_L + l], y);
+      for (int q = 0; q < G; ++q) {
+        const float d = s_dt[buf][t + q][ch], dx = d * s_x[buf][t + q][ch];
+        if (NS % 4 == 0) {
+#pragma unroll
+          for (int j = 0; j < NS; j += 4) {
+            *reinterpret_cast<float4*>(&bx[q][j]) = *reinterpret_cast<const float4*>(&s_b[buf][t + q][l * NS + j]);
+            *reinterpret_cast<float4*>(&cv[q][j]) = *reinterpret_cast<const float4*>(&s_c[buf][t + q][l * NS + j]);
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < NS; ++j) { bx[q][j] = s_b[buf][t + q][l * NS + j]; cv[q][j] = s_c[buf][t + q][l * NS + j]; }
+        }
+#pragma unroll
+        for (int j = 0; j < NS; ++j) { e[q][j] = exp2f(d * A[j]); bx[q][j] *= dx; }
       }
-      y += __shfl_xor_sync(0xffffffffu, y, 1);
-      y += __shfl_xor_sync(0xffffffffu, y, 2);
-      if (l == 0) s_y[t][ch] = y;
-      if (snap) store_state(start + t0 + t + 1);
+#pragma unroll
+      for (int q = 0; q < G; ++q) {
+        y[q] = 0.f;
+#pragma unroll
+        for (int j = 0; j < NS; ++j) {
+          S[j] = fmaf(e[q][j], S[j], bx[q][j]);
+          y[q] = fmaf(S[j], cv[q][j], y[q]);
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < G; ++q) y[q] += __shfl_xor_sync(0xffffffffu, y[q], 1);
+#pragma unroll
+      for (int q = 0; q < G; ++q) y[q] += __shfl_xor_sync(0xffffffffu, y[q], 2);
+      if (l == 0)
+#pragma unroll
+        for (int q = 0; q < G; ++q) s_y[t + q][ch] = y[q];
+    };
+    if (!snap && m == CT) {
+      constexpr int G = NS <= 4 ? 4 : NS <= 8 ? 2 : 1;
+#pragma unroll 1
+      for (int t = 0; t < CT; t += G) tokens(t, std::integral_constant<int, G>());
+    } else {
+      for (int t = 0; t < m; ++t) {
+        tokens(t, std::integral_constant<int, 1>());
+        if (snap) store_state(start + t0 + t + 1);
+      }
     }
     __syncthreads();
 #pragma unroll
@@ -152,7 +211,7 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
       if (t < m && tc_ok) {
         const float z = z_cur[k];
         const float y = s_y[t][tc] + Dc * s_x[buf][t][tc];
-        out[(long long)(r0 + t0 + t) * a.inner + c0 + tc] = from_f<T>(y * (z / (1.f + expf(-z))));
+        out[(long long)(r0 + t0 + t) * a.inner + c0 + tc] = from_f<T>(y * silu_as<T>(z));
       }
     }
   }
@@ -175,9 +234,9 @@ __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
   const float* st_in = a.state + ((long long)slot * a.R + start % a.R) * a.inner * a.nstate;
 #pragma unroll
   for (int j = 0; j < NS; ++j) {
-    const int i = j * MAMBA_L + l;
+    const int i = l * NS + j;
     const bool ok = c_ok && i < a.nstate;
-    A[j] = ok ? a.A[(long long)c * a.nstate + i] : 0.f;
+    A[j] = ok ? a.A[(long long)c * a.nstate + i] * LOG2E : 0.f;
     S[j] = (ok && start > 0) ? st_in[(long long)c * a.nstate + i] : 0.f;
   }
   const int np = a.dt_cols + 2 * a.nstate;
@@ -190,6 +249,7 @@ __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
   if (c_ok) {
     const T* w = reinterpret_cast<const T*>(a.w_dt) + (long long)c * a.dt_cols;
     if (sizeof(T) == 2) {                             // dt_cols is a multiple of 8: 16-byte loads
+#pragma unroll 4
       for (int j = l * 8; j < a.dt_cols; j += 32) {
         const uint4 u = *reinterpret_cast<const uint4*>(w + j);
         const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
@@ -215,16 +275,16 @@ __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
   float y = 0.f;
 #pragma unroll
   for (int j = 0; j < NS; ++j) {
-    const int i = j * MAMBA_L + l;
+    const int i = l * NS + j;
     if (i < a.nstate) {
-      S[j] = fmaf(expf(d * A[j]), S[j], d * x * s_p[a.dt_cols + i]);
+      S[j] = fmaf(exp2f(d * A[j]), S[j], d * x * s_p[a.dt_cols + i]);
       y = fmaf(S[j], s_p[a.dt_cols + a.nstate + i], y);
       so[(long long)c * a.nstate + i] = S[j];
     }
   }
   y += __shfl_xor_sync(grp, y, 1);
   y += __shfl_xor_sync(grp, y, 2);
-  if (l == 0) reinterpret_cast<T*>(a.out)[o] = from_f<T>((y + a.D[c] * x) * (z / (1.f + expf(-z))));
+  if (l == 0) reinterpret_cast<T*>(a.out)[o] = from_f<T>((y + a.D[c] * x) * silu_as<T>(z));
 }
 
 int32_t vn_mamba_scan(vn_ctx* ctx, const MambaArgs& a, bool bf16);
