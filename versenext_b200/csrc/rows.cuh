@@ -47,6 +47,18 @@ struct Src {
     for (; s < splits; ++s) a += q[s * pstride];
     return a;
   }
+  // rows row .. row + RB - 1 of a column (clamped to row_end - 1), loads independent of one another
+  template <int RB>
+  __device__ __forceinline__ void column(int row, int row_end, int col, float (&out)[RB]) const {
+    if (splits == 1) {
+      const float* q = p + (long long)row * ld + col;
+#pragma unroll
+      for (int i = 0; i < RB; ++i) out[i] = q[(long long)(min(row + i, row_end - 1) - row) * ld];
+    } else {
+#pragma unroll
+      for (int i = 0; i < RB; ++i) out[i] = get(min(row + i, row_end - 1), col);
+    }
+  }
 };
 
 __device__ __forceinline__ float warp_sum(float v) {
@@ -127,10 +139,18 @@ struct ConvIn {
     float wt[4], x[RB + 3];
 #pragma unroll
     for (int j = 0; j < 4; ++j) wt[j] = j < taps ? wc[taps - 1 - j] : 0.f;
+    if (src.splits == 1 && row - r0 >= 3) {            // inside an entry's rows: plain loads, all independent
+      const float* p = src.p + (long long)row * src.ld + col0 + c;
 #pragma unroll
-    for (int j = 1; j < 4; ++j) x[3 - j] = j < taps ? input(row, r0, start, slot, pos - j, c) : 0.f;
+      for (int i = 0; i < RB + 3; ++i) x[i] = p[(long long)(min(row + i - 3, row_end - 1) - row) * src.ld];
 #pragma unroll
-    for (int i = 0; i < RB; ++i) x[3 + i] = row + i < row_end ? round_to<T>(src.get(row + i, col0 + c)) : 0.f;
+      for (int i = 0; i < RB + 3; ++i) x[i] = round_to<T>(x[i]);
+    } else {
+#pragma unroll
+      for (int j = 1; j < 4; ++j) x[3 - j] = j < taps ? input(row, r0, start, slot, pos - j, c) : 0.f;
+#pragma unroll
+      for (int i = 0; i < RB; ++i) x[3 + i] = row + i < row_end ? round_to<T>(src.get(row + i, col0 + c)) : 0.f;
+    }
 #pragma unroll
     for (int i = 0; i < RB; ++i) {
       float acc = x[3 + i] * wt[0];

@@ -34,13 +34,14 @@ template int32_t vn_delta_step<__nv_bfloat16>(vn_ctx*, const DeltaStepArgs<__nv_
 int32_t vn_delta_scan(vn_ctx* ctx, const DeltaRuleArgs& a) {
   const int d = a.d;
   const bool vec = d % 4 == 0 && a.vd % 4 == 0;
-  // enough columns to fill the GPU with eight per group: fewer reads per column; else four per group, smaller CTAs
-  const bool wide = d <= 128 && (long long)a.rows.n_ent * a.H * ceil_div(a.vd, 64) >= 8 * ctx->sm_count;
+  // more columns per group: fewer reads per column; fewer: more warps.  The widest that leaves two warps per scheduler
+  const long long cols = (long long)a.rows.n_ent * a.H * a.vd;
+  const int nc = d > 128 ? 4 : cols >= 16 * 8 * ctx->sm_count ? 8 : cols >= 16 * 4 * ctx->sm_count ? 4 : 2;
 #define SCAN2(RPL, NC, VEC, W) do { const dim3 grid(ceil_div(a.vd, 2 * NC * W), a.H, a.rows.n_ent); \
     VN_LAUNCH_NAMED(ctx, "delta_scan_kernel", (delta_scan_kernel<RPL, NC, VEC, W>), grid, 32 * W, 0, a); } while (0)
 #define SCAN(RPL, NC, W) do { if (vec) SCAN2(RPL, NC, 4, W); else SCAN2(RPL, NC, 1, W); } while (0)
-  if (d <= 64) { if (wide) SCAN(4, 8, 4); else SCAN(4, 4, 2); }
-  else if (d <= 128) { if (wide) SCAN(8, 8, 4); else SCAN(8, 4, 2); }
+  if (d <= 64) { if (nc == 8) SCAN(4, 8, 4); else if (nc == 4) SCAN(4, 4, 2); else SCAN(4, 2, 2); }
+  else if (d <= 128) { if (nc == 8) SCAN(8, 8, 4); else if (nc == 4) SCAN(8, 4, 2); else SCAN(8, 2, 2); }
   else SCAN(16, 4, 2);
 #undef SCAN
 #undef SCAN2

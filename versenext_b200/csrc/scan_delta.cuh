@@ -236,7 +236,7 @@ __device__ __forceinline__ unsigned long long f2_fma(unsigned long long a, unsig
   return r;
 }
 // sum of v[c] over the sixteen lanes of a group: the lane returns the total of column delta_scan_col<NC>(li)
-template <int NC> __device__ __forceinline__ int delta_scan_col(int li) { return NC == 8 ? li >> 1 : li >> 2; }
+template <int NC> __device__ __forceinline__ int delta_scan_col(int li) { return li / (16 / NC); }
 template <int NC>
 __device__ __forceinline__ float group_sum(float (&v)[NC], int li) {
 #pragma unroll
@@ -441,13 +441,11 @@ __device__ __forceinline__ float low_rank_dot(const T* w, const float* s, int ld
 #pragma unroll 4
     for (int j = part * 8; j < ld; j += parts * 8) {
       const uint4 u = *reinterpret_cast<const uint4*>(w + j);
+      const float4 x = *reinterpret_cast<const float4*>(s + j), y = *reinterpret_cast<const float4*>(s + j + 4);
       const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-      for (int q = 0; q < 4; ++q) {
-        const float2 f = __bfloat1622float2(h[q]);
-        acc = fmaf(f.x, s[j + 2 * q], acc);
-        acc = fmaf(f.y, s[j + 2 * q + 1], acc);
-      }
+      const float2 f0 = __bfloat1622float2(h[0]), f1 = __bfloat1622float2(h[1]), f2 = __bfloat1622float2(h[2]), f3 = __bfloat1622float2(h[3]);
+      acc = fmaf(f0.x, x.x, acc); acc = fmaf(f0.y, x.y, acc); acc = fmaf(f1.x, x.z, acc); acc = fmaf(f1.y, x.w, acc);
+      acc = fmaf(f2.x, y.x, acc); acc = fmaf(f2.y, y.y, acc); acc = fmaf(f3.x, y.z, acc); acc = fmaf(f3.y, y.w, acc);
     }
   } else {
     for (int j = part; j < ld; j += parts) acc = fmaf(to_f<T>(w[j]), s[j], acc);
@@ -458,7 +456,7 @@ __device__ __forceinline__ float low_rank_dot(const T* w, const float* s, int ld
 // NP: columns a lane takes at a time (the state of 32 NP columns is requested before anything else, so that it arrives
 // under the convolutions and the low-rank products).  Shared memory: 3 DP + 3 vd + ra_ld + rg_ld floats.  grid (H, M)
 template <typename T, int DK, int NP>
-__global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepArgs<T> a) {
+__global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) {
   constexpr int DP = 8 * DK;
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[8], s_misc[2];
@@ -479,24 +477,34 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepArgs<T> a) {
     delta_col_load<DK>(st_in + (long long)(cl + 32 * p) * d, d, li, start > 0 && cl + 32 * p < vd, S[p]);
   // inputs of this head
   const bool first = h % (H / KH) == 0;              // the group's first head keeps the shared q / k inputs
-  for (int i = tid; i < 2 * DP + vd; i += 256) {
-    float cur, v = 0.f;
-    if (i < 2 * DP) {
-      const int j = i % DP;
-      if (j < d) {
-        const int c = (i < DP ? 0 : KH * d) + kh * d + j;
-        v = a.conv.at(row, r0, start, slot, c, &cur);
-        if (first) a.conv.keep(slot, start, c, cur);
-      }
-      (i < DP ? s_q : s_k)[j] = v;
-    } else {
-      const int c = 2 * KH * d + h * vd + (i - 2 * DP);
-      s_v[i - 2 * DP] = a.conv.at(row, r0, start, slot, c, &cur);
-      a.conv.keep(slot, start, c, cur);
+  // columns q | k | v (convolved) and a1 | g1 (as they are); one pass, small code: the kernel's instructions are fetched
+  // anew at every step of a large model
+  const int n_conv = 2 * d + vd, n_all = n_conv + in.ra + in.rg;
+  const int taps = a.conv.taps, C = a.conv.C, RC = a.conv.RC;
+  T* ring = a.conv.ring + (long long)slot * RC * C;
+  for (int i = tid; i < n_all; i += 256) {
+    int c;
+    float* dst;
+    if (i < d) { c = kh * d + i; dst = s_q + i; }
+    else if (i < 2 * d) { c = (KH + kh) * d + i - d; dst = s_k + i - d; }
+    else if (i < n_conv) { c = 2 * KH * d + h * vd + i - 2 * d; dst = s_v + i - 2 * d; }
+    else if (i < n_conv + in.ra) { c = in.col_a + i - n_conv; dst = s_a + i - n_conv; }
+    else { c = in.col_g + i - n_conv - in.ra; dst = s_w + i - n_conv - in.ra; }
+    float x = round_to<T>(in.src.get(row, c));
+    if (i < n_conv) {
+      const float* wc = a.conv.w + (long long)c * taps;
+      float acc = x * wc[taps - 1];
+      if (first || i >= 2 * d) ring[(long long)(start % RC) * C + c] = from_f<T>(x);
+#pragma unroll 3
+      for (int j = 1; j < taps; ++j)
+        acc = fmaf(start >= j ? to_f<T>(ring[(long long)((start - j) % RC) * C + c]) : 0.f, wc[taps - 1 - j], acc);
+      x = silu_as<T>(acc);
     }
+    *dst = x;
   }
-  for (int j = tid; j < in.ra_ld; j += 256) s_a[j] = j < in.ra ? round_to<T>(in.src.get(row, in.col_a + j)) : 0.f;
-  for (int j = tid; j < in.rg_ld; j += 256) s_w[j] = j < in.rg ? round_to<T>(in.src.get(row, in.col_g + j)) : 0.f;
+  for (int j = d + tid; j < DP; j += 256) s_q[j] = s_k[j] = 0.f;
+  for (int j = in.ra + tid; j < in.ra_ld; j += 256) s_a[j] = 0.f;
+  for (int j = in.rg + tid; j < in.rg_ld; j += 256) s_w[j] = 0.f;
   if (tid == 0) s_misc[0] = sigmoid_f(in.src.get(row, in.col_b + h));
   __syncthreads();
   // unit norms: warp 0 takes q, warp 1 takes k
@@ -511,14 +519,13 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaStepArgs<T> a) {
   }
   // decays of the key channels, then gates of the value columns: four lanes per row of the low-rank matrices
   const int nd = (DP + 63) & ~63;
-#pragma unroll 2
+#pragma unroll 1
   for (int j0 = 0; j0 < nd + vd; j0 += 64) {
     const int jj = j0 + (tid >> 2);
     const bool dec = j0 < nd;
     const int j = dec ? jj : jj - nd;
-    float acc = 0.f;
-    if (dec && j < d) acc = low_rank_dot<T>(a.w_a + (long long)(h * d + j) * in.ra_ld, s_a, in.ra_ld, tid & 3, 4);
-    if (!dec && j < vd) acc = low_rank_dot<T>(a.w_g + (long long)(h * vd + j) * in.rg_ld, s_w, in.rg_ld, tid & 3, 4);
+    const T* w = dec ? a.w_a + (long long)(h * d + j) * in.ra_ld : a.w_g + (long long)(h * vd + j) * in.rg_ld;
+    float acc = j < (dec ? d : vd) ? low_rank_dot<T>(w, dec ? s_a : s_w, dec ? in.ra_ld : in.rg_ld, tid & 3, 4) : 0.f;
     acc += __shfl_xor_sync(0xffffffffu, acc, 1);
     acc += __shfl_xor_sync(0xffffffffu, acc, 2);
     if ((tid & 3) == 0) {

@@ -5,23 +5,28 @@ namespace {
 
 template <typename T>
 int32_t scan(vn_ctx* ctx, const MambaArgs& a) {
-  const int ns = ceil_div(a.nstate, MAMBA_L);
   const dim3 grid(ceil_div(a.inner, MAMBA_CH), a.rows.n_ent);
-#define SCAN(NS) VN_LAUNCH_NAMED(ctx, "mamba_scan_kernel", (mamba_scan_kernel<T, NS>), grid, 128, 0, a)
-  if (ns <= 1) SCAN(1); else if (ns <= 2) SCAN(2); else if (ns <= 4) SCAN(4); else if (ns <= 6) SCAN(6);
-  else if (ns <= 8) SCAN(8); else if (ns <= 16) SCAN(16); else SCAN(32);
+#define SCAN(NS, L) VN_LAUNCH_NAMED(ctx, "mamba_scan_kernel", (mamba_scan_kernel<T, NS, L>), grid, 32 * L, 0, a)
+  // few sequences: eight lanes per channel, so that every scheduler has more than one warp
+  if (a.nstate >= 8 && a.nstate <= 32 && (long long)grid.x * grid.y <= 2 * ctx->sm_count) {
+    if (a.nstate <= 16) SCAN(2, 8); else SCAN(4, 8);
+    return VN_OK;
+  }
+  const int ns = ceil_div(a.nstate, 4);
+  if (ns <= 1) SCAN(1, 4); else if (ns <= 2) SCAN(2, 4); else if (ns <= 4) SCAN(4, 4); else if (ns <= 6) SCAN(6, 4);
+  else if (ns <= 8) SCAN(8, 4); else if (ns <= 16) SCAN(16, 4); else SCAN(32, 4);
 #undef SCAN
   return VN_OK;
 }
 
 template <typename T>
 int32_t step(vn_ctx* ctx, const MambaArgs& a) {
-  const int ns = ceil_div(a.nstate, MAMBA_L);
-  const dim3 grid(ceil_div(a.inner, 64), a.rows.M);
   const size_t smem = (size_t)(a.dt_cols + 2 * a.nstate) * 4;
-#define STEP(NS) VN_LAUNCH_NAMED(ctx, "mamba_step_kernel", (mamba_step_kernel<T, NS>), grid, 256, smem, a)
-  if (ns <= 1) STEP(1); else if (ns <= 2) STEP(2); else if (ns <= 4) STEP(4); else if (ns <= 6) STEP(6);
-  else if (ns <= 8) STEP(8); else if (ns <= 16) STEP(16); else STEP(32);
+#define STEP(NS, L) VN_LAUNCH_NAMED(ctx, "mamba_step_kernel", (mamba_step_kernel<T, NS, L>), \
+                                    dim3(ceil_div(a.inner, 256 / L), a.rows.M), 256, smem, a)
+  const int n = a.nstate;
+  if (n <= 4) STEP(2, 2); else if (n <= 8) STEP(4, 2); else if (n <= 16) STEP(8, 2); else if (n <= 24) STEP(6, 4);
+  else if (n <= 32) STEP(8, 4); else if (n <= 64) STEP(16, 4); else STEP(32, 4);
 #undef STEP
   return VN_OK;
 }

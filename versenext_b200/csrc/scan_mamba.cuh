@@ -2,9 +2,8 @@
 //
 //   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n ;  y_c = sum_n S[c, n] C_n + D_c x_c ;  out = y * silu(z)
 //
-// A recurrence runs over the tokens of one sequence; its parallelism is channels x sequences.  Four lanes share a
-// channel (each holds every fourth state in registers), a CTA of 128 threads takes 32 channels of one sequence and
-// stages the per-token inputs of CT tokens in shared memory while the next CT tokens are on their way.
+// A recurrence runs over the tokens of one sequence; its parallelism is channels x sequences.  A few lanes share a
+// channel (each holds some of its states in registers), a CTA takes 32 channels of one sequence and stages the per-token inputs of CT tokens in shared memory while the next CT tokens are on their way.
 //
 // State ring: the state after p tokens of slot s lives at ring index p mod R.  A forward of n rows leaves the state
 // after every row when n is small enough to be cut back (n <= R - 1), otherwise the last one only; committing k rows
@@ -43,6 +42,7 @@ __global__ void __launch_bounds__(256) mamba_conv_kernel(ConvIn<T> in, Rows rows
     rows.entry(rows.entry_of(row), &slot, &r0, &n, &start);
     const int first = row, end = min(last, r0 + n);
     float v[RB], zv[RB];
+    in.src.template column<RB>(first, end, in.col0 + in.C + c, zv);
     if (RB > 1 && in.taps <= 4) {
       in.template run<RB>(first, end, r0, start, slot, c, v);
     } else {
@@ -52,8 +52,6 @@ __global__ void __launch_bounds__(256) mamba_conv_kernel(ConvIn<T> in, Rows rows
         v[r] = first + r < end ? in.at(first + r, r0, start, slot, c, &cur) : 0.f;
       }
     }
-#pragma unroll
-    for (int r = 0; r < RB; ++r) zv[r] = first + r < end ? in.src.get(first + r, in.col0 + in.C + c) : 0.f;
     if (n <= pending)
       for (int r = first; r < end; ++r) in.keep(slot, start + r - r0, c, in.src.get(r, in.col0 + c));
 #pragma unroll
@@ -73,19 +71,19 @@ __global__ void cast_cols_kernel(Src src, int col0, int n, T* __restrict__ out, 
     out[(long long)blockIdx.x * ld + j] = from_f<T>(j < n ? src.get(blockIdx.x, col0 + j) : 0.f);
 }
 
-constexpr int MAMBA_L = 4, MAMBA_CH = 32, MAMBA_CT = 16;
+constexpr int MAMBA_CH = 32, MAMBA_CT = 16;
 constexpr float LOG2E = 1.4426950408889634f;       // exp(dt A) = 2^(dt (A log2 e))
 
-// NS: states per lane (nstate <= 4 NS).  grid (ceil(inner / 32), n_ent)
-template <typename T, int NS>
-__global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
-  constexpr int N4 = MAMBA_L * NS, CT = MAMBA_CT, CH = MAMBA_CH;
+// L lanes share a channel, NS states each (nstate <= L NS); 32 L threads.  grid (ceil(inner / 32), n_ent)
+template <typename T, int NS, int L>
+__global__ void __launch_bounds__(32 * L) mamba_scan_kernel(MambaArgs a) {
+  constexpr int N4 = L * NS, THREADS = 32 * L, CT = MAMBA_CT, CH = MAMBA_CH;
   __shared__ float s_dt[2][CT][CH], s_x[2][CT][CH], s_y[CT][CH];
   __shared__ __align__(16) float s_b[2][CT][N4], s_c[2][CT][N4];
   int slot, r0, n, start;
   a.rows.entry(blockIdx.y, &slot, &r0, &n, &start);
   if (n <= 0) return;
-  const int tid = threadIdx.x, ch = tid >> 2, l = tid & 3;
+  const int tid = threadIdx.x, ch = tid / L, l = tid % L;
   const int c0 = blockIdx.x * CH, c = c0 + ch;
   const bool c_ok = c < a.inner;
   const T* xc = reinterpret_cast<const T*>(a.xc);
@@ -110,16 +108,16 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
     }
   };
 
-  // staging: thread -> (token ti + 4 k, channel tc) for the per-channel inputs, flat indices for B and C
+  // staging: thread -> (token ti + L k, channel tc) for the per-channel inputs, flat indices for B and C
   const int tc = tid & 31, ti = tid >> 5;
   const bool tc_ok = c0 + tc < a.inner;
   const float bias = tc_ok ? a.dt_bias[c0 + tc] : 0.f, Dc = tc_ok ? a.D[c0 + tc] : 0.f;
-  constexpr int BI = (CT * N4 + 127) / 128;
-  float r_dt[CT / 4], r_x[CT / 4], r_z[CT / 4], z_cur[CT / 4], r_b[BI], r_c[BI];
+  constexpr int BI = (CT * N4 + THREADS - 1) / THREADS;
+  float r_dt[CT / L], r_x[CT / L], r_z[CT / L], z_cur[CT / L], r_b[BI], r_c[BI];
   auto fetch = [&](int t0) {
 #pragma unroll
-    for (int k = 0; k < CT / 4; ++k) {
-      const int t = t0 + ti + 4 * k;
+    for (int k = 0; k < CT / L; ++k) {
+      const int t = t0 + ti + L * k;
       r_dt[k] = r_x[k] = r_z[k] = 0.f;
       if (t < n && tc_ok) {
         const long long o = (long long)(r0 + t) * a.inner + c0 + tc;
@@ -128,7 +126,7 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
     }
 #pragma unroll
     for (int k = 0; k < BI; ++k) {
-      const int f = tid + k * 128, t = t0 + f / N4, i = f % N4;
+      const int f = tid + k * THREADS, t = t0 + f / N4, i = f % N4;
       r_b[k] = r_c[k] = 0.f;
       if (f < CT * N4 && t < n && i < a.nstate) {
         r_b[k] = a.p.get(r0 + t, a.dt_cols + i);
@@ -138,14 +136,14 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
   };
   auto stash = [&](int buf) {
 #pragma unroll
-    for (int k = 0; k < CT / 4; ++k) {
-      s_dt[buf][ti + 4 * k][tc] = softplus_f(r_dt[k] + bias);
-      s_x[buf][ti + 4 * k][tc] = r_x[k];
+    for (int k = 0; k < CT / L; ++k) {
+      s_dt[buf][ti + L * k][tc] = softplus_f(r_dt[k] + bias);
+      s_x[buf][ti + L * k][tc] = r_x[k];
       z_cur[k] = r_z[k];
     }
 #pragma unroll
     for (int k = 0; k < BI; ++k) {
-      const int f = tid + k * 128;
+      const int f = tid + k * THREADS;
       if (f < CT * N4) { s_b[buf][f / N4][f % N4] = r_b[k]; s_c[buf][f / N4][f % N4] = r_c[k]; }
     }
   };
@@ -187,9 +185,9 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
         }
       }
 #pragma unroll
-      for (int q = 0; q < G; ++q) y[q] += __shfl_xor_sync(0xffffffffu, y[q], 1);
+      for (int o = 1; o < L; o <<= 1)
 #pragma unroll
-      for (int q = 0; q < G; ++q) y[q] += __shfl_xor_sync(0xffffffffu, y[q], 2);
+        for (int q = 0; q < G; ++q) y[q] += __shfl_xor_sync(0xffffffffu, y[q], o);
       if (l == 0)
 #pragma unroll
         for (int q = 0; q < G; ++q) s_y[t + q][ch] = y[q];
@@ -206,8 +204,8 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
     }
     __syncthreads();
 #pragma unroll
-    for (int k = 0; k < CT / 4; ++k) {
-      const int t = ti + 4 * k;
+    for (int k = 0; k < CT / L; ++k) {
+      const int t = ti + L * k;
       if (t < m && tc_ok) {
         const float z = z_cur[k];
         const float y = s_y[t][tc] + Dc * s_x[buf][t][tc];
@@ -218,16 +216,16 @@ __global__ void __launch_bounds__(128) mamba_scan_kernel(MambaArgs a) {
   if (!snap) store_state(start + n);
 }
 
-// One new token per sequence: the dt projection, the state update and the gate in one kernel.  256 threads, 64 channels
-// of one row; grid (ceil(inner / 64), M), shared memory (dt_cols + 2 nstate) floats
-template <typename T, int NS>
+// One new token per sequence: the dt projection, the state update and the gate in one kernel.  256 threads, 256 / L
+// channels of one row; grid (ceil(inner / (256 / L)), M), shared memory (dt_cols + 2 nstate) floats
+template <typename T, int NS, int L>
 __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
-  extern __shared__ float s_p[];
+  extern __shared__ __align__(16) float s_p[];
   const int row = blockIdx.y;
   int slot, r0, n, start;
   a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
-  const int tid = threadIdx.x, ch = tid >> 2, l = tid & 3;
-  const int c = blockIdx.x * 64 + ch;
+  const int tid = threadIdx.x, ch = tid / L, l = tid % L;
+  const int c = blockIdx.x * (256 / L) + ch;
   const bool c_ok = c < a.inner;
   // the state and A do not depend on the projection: on their way while it is summed
   float S[NS], A[NS];
@@ -250,26 +248,23 @@ __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
     const T* w = reinterpret_cast<const T*>(a.w_dt) + (long long)c * a.dt_cols;
     if (sizeof(T) == 2) {                             // dt_cols is a multiple of 8: 16-byte loads
 #pragma unroll 4
-      for (int j = l * 8; j < a.dt_cols; j += 32) {
+      for (int j = l * 8; j < a.dt_cols; j += 8 * L) {
         const uint4 u = *reinterpret_cast<const uint4*>(w + j);
+        const float4 x = *reinterpret_cast<const float4*>(s_p + j), y = *reinterpret_cast<const float4*>(s_p + j + 4);
         const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          const float2 f = __bfloat1622float2(h[q]);
-          acc = fmaf(f.x, s_p[j + 2 * q], acc);
-          acc = fmaf(f.y, s_p[j + 2 * q + 1], acc);
-        }
+        const float2 f0 = __bfloat1622float2(h[0]), f1 = __bfloat1622float2(h[1]), f2 = __bfloat1622float2(h[2]), f3 = __bfloat1622float2(h[3]);
+        acc = fmaf(f0.x, x.x, acc); acc = fmaf(f0.y, x.y, acc); acc = fmaf(f1.x, x.z, acc); acc = fmaf(f1.y, x.w, acc);
+        acc = fmaf(f2.x, y.x, acc); acc = fmaf(f2.y, y.y, acc); acc = fmaf(f3.x, y.z, acc); acc = fmaf(f3.y, y.w, acc);
       }
     } else {
-      for (int j = l; j < a.dt_cols; j += 4) acc = fmaf(to_f<T>(w[j]), s_p[j], acc);
+      for (int j = l; j < a.dt_cols; j += L) acc = fmaf(to_f<T>(w[j]), s_p[j], acc);
     }
   }
-  acc += __shfl_xor_sync(0xffffffffu, acc, 1);
-  acc += __shfl_xor_sync(0xffffffffu, acc, 2);
-  if (!c_ok) return;                                  // whole groups of four lanes leave together
-  const unsigned grp = 0xfu << (tid & 28);
-  const float d = softplus_f(acc + a.dt_bias[c]);
-  const long long o = (long long)row * a.inner + c;
+#pragma unroll
+  for (int o = 1; o < L; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+  const int cc = c_ok ? c : a.inner - 1;               // lanes beyond the last channel go along without storing
+  const float d = softplus_f(acc + a.dt_bias[cc]);
+  const long long o = (long long)row * a.inner + cc;
   const float x = to_f<T>(reinterpret_cast<const T*>(a.xc)[o]), z = to_f<T>(reinterpret_cast<const T*>(a.z)[o]);
   float* so = a.state + ((long long)slot * a.R + (start + 1) % a.R) * a.inner * a.nstate;
   float y = 0.f;
@@ -279,12 +274,12 @@ __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
     if (i < a.nstate) {
       S[j] = fmaf(exp2f(d * A[j]), S[j], d * x * s_p[a.dt_cols + i]);
       y = fmaf(S[j], s_p[a.dt_cols + a.nstate + i], y);
-      so[(long long)c * a.nstate + i] = S[j];
+      if (c_ok) so[(long long)c * a.nstate + i] = S[j];
     }
   }
-  y += __shfl_xor_sync(grp, y, 1);
-  y += __shfl_xor_sync(grp, y, 2);
-  if (l == 0) reinterpret_cast<T*>(a.out)[o] = from_f<T>((y + a.D[c] * x) * silu_as<T>(z));
+#pragma unroll
+  for (int q = 1; q < L; q <<= 1) y += __shfl_xor_sync(0xffffffffu, y, q);
+  if (l == 0 && c_ok) reinterpret_cast<T*>(a.out)[o] = from_f<T>((y + a.D[c] * x) * silu_as<T>(z));
 }
 
 int32_t vn_mamba_scan(vn_ctx* ctx, const MambaArgs& a, bool bf16);
