@@ -145,6 +145,8 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
           float* c = reinterpret_cast<float*>(g.C) + crow + n;
           if (n < g.N) c[0] += v0;
           if (n + 1 < g.N) c[1] += v1;
+        } else if (g.c_bf16 && !g.bias && n + 1 < g.N && ((crow + n) & 1) == 0) {
+          *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(g.C) + crow + n) = __floats2bfloat162_rn(v0, v1);
         } else {
           if (n < g.N) store_out<float>(g.C, crow + n, v0 + (g.bias ? g.bias[n] : 0.f), g.c_bf16);
           if (n + 1 < g.N) store_out<float>(g.C, crow + n + 1, v1 + (g.bias ? g.bias[n + 1] : 0.f), g.c_bf16);

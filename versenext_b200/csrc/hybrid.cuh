@@ -523,6 +523,12 @@ int32_t mamba1(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, cons
   a.xc = b.xc; a.z = b.z; a.dt_cols = L.dtp; a.dt_rank = L.dt_rank; a.w_dt = L.w_uk; a.dt_bias = L.f_c; a.A = L.f_a; a.D = L.f_b;
   a.state = (float*)kv->v[run]; a.R = hc.ring; a.inner = n; a.nstate = L.nstate; a.out = b.mix; a.rows = rows;
   if (rows.max_n == 1) {
+    if (M >= 16 && a.p.splits > 1) {     // many rows: the slices are summed once, not by every CTA of a row
+      VN_LAUNCH(ctx, splitk_store_kernel, (unsigned)ceil_div((long long)M * L.n_x, 256ll), 256, 0, a.p.p, a.p.splits, a.p.pstride,
+                b.p, (long long)L.n_x, L.n_x, (long long)M * L.n_x);
+      a.p = Src();
+      a.p.p = b.p; a.p.ld = L.n_x;
+    }
     TRY(vn_mamba_step(ctx, a, m->cfg.bf16 != 0));
     return VN_OK;
   }

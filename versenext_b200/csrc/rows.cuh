@@ -137,12 +137,23 @@ struct ConvIn {
     const int pos = start + row - r0;
     const float* wc = w + (long long)c * taps;
     float wt[4], x[RB + 3];
+    if (taps == 4) {
+      const float4 t = *reinterpret_cast<const float4*>(wc);
+      wt[0] = t.w; wt[1] = t.z; wt[2] = t.y; wt[3] = t.x;
+    } else {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) wt[j] = j < taps ? wc[taps - 1 - j] : 0.f;
+      for (int j = 0; j < 4; ++j) wt[j] = j < taps ? wc[taps - 1 - j] : 0.f;
+    }
     if (src.splits == 1 && row - r0 >= 3) {            // inside an entry's rows: plain loads, all independent
       const float* p = src.p + (long long)row * src.ld + col0 + c;
+      if (row + RB <= row_end) {
+        p -= 3ll * src.ld;
 #pragma unroll
-      for (int i = 0; i < RB + 3; ++i) x[i] = p[(long long)(min(row + i - 3, row_end - 1) - row) * src.ld];
+        for (int i = 0; i < RB + 3; ++i, p += src.ld) x[i] = *p;
+      } else {
+#pragma unroll
+        for (int i = 0; i < RB + 3; ++i) x[i] = p[(long long)(min(row + i - 3, row_end - 1) - row) * src.ld];
+      }
 #pragma unroll
       for (int i = 0; i < RB + 3; ++i) x[i] = round_to<T>(x[i]);
     } else {

@@ -5,9 +5,9 @@ template <typename T>
 int32_t vn_delta_inputs(vn_ctx* ctx, const ConvIn<T>& conv, const DeltaIn& in) {
   const int nc = ceil_div(in.d > in.vd ? in.d : in.vd, 32);
   const bool many = in.rows.M >= 512 && nc <= 4;
-  const dim3 grid(2 * in.KH + in.H + 1, ceil_div(in.rows.M, many ? 32 : 8)), block(32, 8);
+  const dim3 grid(2 * in.KH + in.H + 1, ceil_div(in.rows.M, many ? 64 : 8)), block(32, 8);
 #define INPUTS(NC, RB) VN_LAUNCH_NAMED(ctx, "delta_inputs_kernel", (delta_inputs_kernel<T, NC, RB>), grid, block, 0, conv, in)
-  if (many) { if (nc <= 1) INPUTS(1, 4); else if (nc <= 2) INPUTS(2, 4); else INPUTS(4, 4); return VN_OK; }
+  if (many) { if (nc <= 1) INPUTS(1, 8); else if (nc <= 2) INPUTS(2, 8); else INPUTS(4, 8); return VN_OK; }
   if (nc <= 1) INPUTS(1, 1); else if (nc <= 2) INPUTS(2, 1); else if (nc <= 4) INPUTS(4, 1); else if (nc <= 8) INPUTS(8, 1); else INPUTS(16, 1);
 #undef INPUTS
   return VN_OK;
@@ -21,9 +21,10 @@ int32_t vn_delta_step(vn_ctx* ctx, const DeltaStepArgs<T>& a) {
   const int d = a.in.d;
   const int extra = 3 * a.in.vd + a.in.ra_ld + a.in.rg_ld;
   VN_REQUIRE(ctx, extra + 24 * 32 <= 12000, "low-rank factors too wide for the step kernel");
-#define STEP2(DK, NP) VN_LAUNCH_NAMED(ctx, "delta_step_kernel", (delta_step_kernel<T, DK, NP>), grid, 256, (size_t)(24 * DK + extra) * 4, a)
-#define STEP(DK) do { if (a.in.vd <= 32) STEP2(DK, 1); else if (a.in.vd <= 64) STEP2(DK, 2); else STEP2(DK, 4); } while (0)
-  if (d <= 32) STEP(4); else if (d <= 64) STEP(8); else if (d <= 96) STEP(12); else if (d <= 128) STEP(16); else STEP2(32, 2);
+#define STEP2(DK, NP) VN_LAUNCH_NAMED(ctx, "delta_step_kernel", (delta_step_kernel<T, DK, NP>), grid, DELTA_STEP_THREADS, \
+                                      (size_t)(24 * DK + extra) * 4, a)
+#define STEP(DK) do { if (a.in.vd <= 64) STEP2(DK, 1); else STEP2(DK, 2); } while (0)
+  if (d <= 32) STEP(4); else if (d <= 64) STEP(8); else if (d <= 96) STEP(12); else if (d <= 128) STEP(16); else STEP2(32, 1);
 #undef STEP2
 #undef STEP
   return VN_OK;

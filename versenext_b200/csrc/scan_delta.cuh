@@ -419,7 +419,7 @@ __global__ void __launch_bounds__(32 * W) delta_scan_kernel(DeltaRuleArgs a) {
 }
 
 // One new token per sequence, everything between the two projections in one kernel: convolutions, unit norms, beta,
-// both low-rank products, decay, state update, read-out, norm and gate.  One CTA (256 threads) per (row, head).
+// both low-rank products, decay, state update, read-out, norm and gate.  One CTA per (row, head).
 template <typename T>
 struct DeltaStepArgs {
   ConvIn<T> conv;
@@ -453,13 +453,14 @@ __device__ __forceinline__ float low_rank_dot(const T* w, const float* s, int ld
   return acc;
 }
 
-// NP: columns a lane takes at a time (the state of 32 NP columns is requested before anything else, so that it arrives
+// NP: columns a lane takes at a time (the state of 64 NP columns is requested before anything else, so that it arrives
 // under the convolutions and the low-rank products).  Shared memory: 3 DP + 3 vd + ra_ld + rg_ld floats.  grid (H, M)
+constexpr int DELTA_STEP_THREADS = 512;
 template <typename T, int DK, int NP>
-__global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) {
-  constexpr int DP = 8 * DK;
+__global__ void __launch_bounds__(DELTA_STEP_THREADS, 2) delta_step_kernel(DeltaStepArgs<T> a) {
+  constexpr int DP = 8 * DK, TH = DELTA_STEP_THREADS, CP = TH / 8, RP = TH / 4;   // columns, low-rank rows per pass
   extern __shared__ __align__(16) float sm[];
-  __shared__ float red[8], s_misc[2];
+  __shared__ float red[TH / 32], s_misc[2];
   const DeltaIn& in = a.in;
   const int d = in.d, vd = in.vd, H = in.H, KH = in.KH;
   float *s_q = sm, *s_k = s_q + DP, *s_g = s_k + DP, *s_a = s_g + DP, *s_w = s_a + in.ra_ld, *s_v = s_w + in.rg_ld,
@@ -474,7 +475,7 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) 
   float S[NP][DK];
 #pragma unroll
   for (int p = 0; p < NP; ++p)
-    delta_col_load<DK>(st_in + (long long)(cl + 32 * p) * d, d, li, start > 0 && cl + 32 * p < vd, S[p]);
+    delta_col_load<DK>(st_in + (long long)(cl + CP * p) * d, d, li, start > 0 && cl + CP * p < vd, S[p]);
   // inputs of this head
   const bool first = h % (H / KH) == 0;              // the group's first head keeps the shared q / k inputs
   // columns q | k | v (convolved) and a1 | g1 (as they are); one pass, small code: the kernel's instructions are fetched
@@ -482,7 +483,7 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) 
   const int n_conv = 2 * d + vd, n_all = n_conv + in.ra + in.rg;
   const int taps = a.conv.taps, C = a.conv.C, RC = a.conv.RC;
   T* ring = a.conv.ring + (long long)slot * RC * C;
-  for (int i = tid; i < n_all; i += 256) {
+  for (int i = tid; i < n_all; i += TH) {
     int c;
     float* dst;
     if (i < d) { c = kh * d + i; dst = s_q + i; }
@@ -490,21 +491,24 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) 
     else if (i < n_conv) { c = 2 * KH * d + h * vd + i - 2 * d; dst = s_v + i - 2 * d; }
     else if (i < n_conv + in.ra) { c = in.col_a + i - n_conv; dst = s_a + i - n_conv; }
     else { c = in.col_g + i - n_conv - in.ra; dst = s_w + i - n_conv - in.ra; }
-    float x = round_to<T>(in.src.get(row, c));
-    if (i < n_conv) {
+    float past = 0.f, w0 = 1.f;
+    if (i < n_conv) {                                // what came before is requested ahead of the projection's slices
       const float* wc = a.conv.w + (long long)c * taps;
-      float acc = x * wc[taps - 1];
-      if (first || i >= 2 * d) ring[(long long)(start % RC) * C + c] = from_f<T>(x);
+      w0 = wc[taps - 1];
 #pragma unroll 3
       for (int j = 1; j < taps; ++j)
-        acc = fmaf(start >= j ? to_f<T>(ring[(long long)((start - j) % RC) * C + c]) : 0.f, wc[taps - 1 - j], acc);
-      x = silu_as<T>(acc);
+        past = fmaf(start >= j ? to_f<T>(ring[(long long)((start - j) % RC) * C + c]) : 0.f, wc[taps - 1 - j], past);
+    }
+    float x = round_to<T>(in.src.get(row, c));
+    if (i < n_conv) {
+      if (first || i >= 2 * d) ring[(long long)(start % RC) * C + c] = from_f<T>(x);
+      x = silu_as<T>(fmaf(x, w0, past));
     }
     *dst = x;
   }
-  for (int j = d + tid; j < DP; j += 256) s_q[j] = s_k[j] = 0.f;
-  for (int j = in.ra + tid; j < in.ra_ld; j += 256) s_a[j] = 0.f;
-  for (int j = in.rg + tid; j < in.rg_ld; j += 256) s_w[j] = 0.f;
+  for (int j = d + tid; j < DP; j += TH) s_q[j] = s_k[j] = 0.f;
+  for (int j = in.ra + tid; j < in.ra_ld; j += TH) s_a[j] = 0.f;
+  for (int j = in.rg + tid; j < in.rg_ld; j += TH) s_w[j] = 0.f;
   if (tid == 0) s_misc[0] = sigmoid_f(in.src.get(row, in.col_b + h));
   __syncthreads();
   // unit norms: warp 0 takes q, warp 1 takes k
@@ -518,9 +522,9 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) 
     for (int j = lane; j < d; j += 32) s[j] *= f;
   }
   // decays of the key channels, then gates of the value columns: four lanes per row of the low-rank matrices
-  const int nd = (DP + 63) & ~63;
+  const int nd = (DP + RP - 1) / RP * RP;
 #pragma unroll 1
-  for (int j0 = 0; j0 < nd + vd; j0 += 64) {
+  for (int j0 = 0; j0 < nd + vd; j0 += RP) {
     const int jj = j0 + (tid >> 2);
     const bool dec = j0 < nd;
     const int j = dec ? jj : jj - nd;
@@ -536,18 +540,18 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) 
   __syncthreads();
   const float beta = s_misc[0];
   float ss = 0.f;
-  for (int c0 = 0; c0 < vd; c0 += 32 * NP) {
+  for (int c0 = 0; c0 < vd; c0 += CP * NP) {
     float v[NP], o[NP];
 #pragma unroll
     for (int p = 0; p < NP; ++p) {
-      const int c = c0 + cl + 32 * p;
+      const int c = c0 + cl + CP * p;
       if (c0 > 0) delta_col_load<DK>(st_in + (long long)c * d, d, li, start > 0 && c < vd, S[p]);
       v[p] = c < vd ? s_v[c] : 0.f;
     }
     delta_cols_step<DK, NP>(S, s_q, s_k, s_g, li, v, beta, o);
 #pragma unroll
     for (int p = 0; p < NP; ++p) {
-      const int c = c0 + cl + 32 * p;
+      const int c = c0 + cl + CP * p;
       o[p] += __shfl_xor_sync(0xffffffffu, o[p], 1);
       o[p] += __shfl_xor_sync(0xffffffffu, o[p], 2);
       o[p] += __shfl_xor_sync(0xffffffffu, o[p], 4);
@@ -557,8 +561,14 @@ __global__ void __launch_bounds__(256, 2) delta_step_kernel(DeltaStepArgs<T> a) 
       }
     }
   }
-  const float r = sqrtf(block_sum256(ss, red) / (float)vd + a.eps);     // its barrier also publishes s_o
-  for (int j = tid; j < vd; j += 256)
+  ss = warp_sum(ss);
+  if (lane == 0) red[warp] = ss;
+  __syncthreads();                                   // also publishes s_o
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < TH / 32; ++i) ss += red[i];
+  const float r = sqrtf(ss / (float)vd + a.eps);
+  for (int j = tid; j < vd; j += TH)
     a.out[(long long)row * H * vd + h * vd + j] = from_f<T>(s_o[j] / r * a.norm_w[j] * s_gate[j]);
 }
 

@@ -227,6 +227,9 @@ __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
   const int tid = threadIdx.x, ch = tid / L, l = tid % L;
   const int c = blockIdx.x * (256 / L) + ch;
   const bool c_ok = c < a.inner;
+  const int cc = c_ok ? c : a.inner - 1;               // lanes beyond the last channel go along without storing
+  const long long o = (long long)row * a.inner + cc;
+  const float x = to_f<T>(reinterpret_cast<const T*>(a.xc)[o]), z = to_f<T>(reinterpret_cast<const T*>(a.z)[o]);
   // the state and A do not depend on the projection: on their way while it is summed
   float S[NS], A[NS];
   const float* st_in = a.state + ((long long)slot * a.R + start % a.R) * a.inner * a.nstate;
@@ -262,10 +265,7 @@ __global__ void __launch_bounds__(256) mamba_step_kernel(MambaArgs a) {
   }
 #pragma unroll
   for (int o = 1; o < L; o <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-  const int cc = c_ok ? c : a.inner - 1;               // lanes beyond the last channel go along without storing
   const float d = softplus_f(acc + a.dt_bias[cc]);
-  const long long o = (long long)row * a.inner + cc;
-  const float x = to_f<T>(reinterpret_cast<const T*>(a.xc)[o]), z = to_f<T>(reinterpret_cast<const T*>(a.z)[o]);
   float* so = a.state + ((long long)slot * a.R + (start + 1) % a.R) * a.inner * a.nstate;
   float y = 0.f;
 #pragma unroll
