@@ -28,12 +28,22 @@ struct GemmArgs {
   int epi = EPI_STORE;
   int c_bf16 = 0;
   int act = 0;                    // gate activation of EPI_SWIGLU: 0 silu, 1 gelu (tanh form)
+  int post = 0;                   // EPI_STORE: function of columns [0, post_n): 0 none, POST_SILU, POST_RELU2
+  int post_n = 0;
   const char* tag = nullptr;      // name of the call site in the per-kernel timing report (string literal)
   // weight-only quantisation: W points at INT8 / packed INT4 bytes, ldw and w_stride stay in ELEMENTS
   int wq = 0;                     // 0 dense, 1 int8, 2 int4 per output row, 3 int4 with one scale per 128 inputs
   const float* w_scale = nullptr; // [N] (wq 1, 2) or [N, K/128] (wq 3)
   long long ws_stride = 0;        // scales between consecutive segments
 };
+
+enum GemmPost { POST_SILU = 1, POST_RELU2 = 2 };
+// `fast`: the result is kept in 16 bits
+__device__ __forceinline__ float post_act(float x, int post, bool fast) {
+  if (post == POST_RELU2) { x = fmaxf(x, 0.f); return x * x; }
+  if (post == POST_SILU) return fast ? __fdividef(x, 1.0f + __expf(-x)) : x / (1.0f + expf(-x));
+  return x;
+}
 
 __device__ __forceinline__ float ld_f(const float* p) { return *p; }
 __device__ __forceinline__ float ld_f(const __nv_bfloat16* p) { return __bfloat162float(*p); }
@@ -124,6 +134,7 @@ __global__ void __launch_bounds__(256) gemm_nt_simt_kernel(GemmArgs g) {
         if (n >= g.N) continue;
         float v = acc[i][j];
         if (g.bias) v += g.bias[n];
+        if (n < g.post_n) v = post_act(v, g.post, g.c_bf16);
         const long long idx = c_base + crow * g.ldc + n;
         if (g.epi == EPI_ADD) reinterpret_cast<float*>(g.C)[idx] += v;
         else store_out<float>(g.C, idx, v, g.c_bf16);

@@ -138,7 +138,9 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int n = n0 + wn * 32 + j * 8 + (lane & 3) * 2;
-        const float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
+        float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
+        if (n < g.post_n) v0 = post_act(v0, g.post, g.c_bf16);       // no bias goes with it
+        if (n + 1 < g.post_n) v1 = post_act(v1, g.post, g.c_bf16);
         if (g.epi == EPI_SWIGLU) {
           if (n + 1 < g.N) store_out<float>(g.C, crow + (n >> 1), glu_act(v0, g.act) * v1, g.c_bf16);
         } else if (g.epi == EPI_ADD) {

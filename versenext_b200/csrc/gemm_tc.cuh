@@ -66,6 +66,7 @@ struct TcArgs {
   int tma_out;             // fp32 output rows leave through TMA stores (dense PARTIAL / STORE only)
   int out_bufs;            // 16 KB staging tiles per epilogue group for that
   int kb_per_split;        // k blocks (of 64) per blockIdx.y
+  int post, post_n;        // 16-bit TC_STORE only: GemmArgs::post
   int epi, c_bf16;
   int act;                 // TC_SWIGLU: activation of the gate (GemmArgs::act)
   const int* seg_off;      // segmented mode (blockIdx.z = segment)
@@ -381,9 +382,10 @@ __device__ __forceinline__ void tc_epilogue_chunk(const TcArgs& g, const unsigne
         const long long at = (long long)(row0 + m0) * g.ldc + n;
         if (g.c_bf16) {
           __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + at;
+          const int post = n < g.post_n ? g.post : 0;
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (i < mrem) dst[(long long)i * g.ldc] = __float2bfloat16_rn(__uint_as_float(r[i]) + bias);
+            if (i < mrem) dst[(long long)i * g.ldc] = __float2bfloat16_rn(post_act(__uint_as_float(r[i]) + bias, post, true));
         } else {
           float* dst = reinterpret_cast<float*>(g.C) + at;
 #pragma unroll
@@ -1037,7 +1039,7 @@ inline int32_t launch_gemm_tc(vn_ctx* ctx, const GemmArgs& g, long long a_rows_t
   budget = std::max(budget, 2 * stage_bytes);
   budget = std::max<size_t>(budget, 64 * 1024);       // the epilogue stages four 16 KB tiles in the freed stage memory
   a.smem_budget = (unsigned)budget;
-  a.epi = g.epi; a.c_bf16 = g.c_bf16; a.act = g.act;
+  a.epi = g.epi; a.c_bf16 = g.c_bf16; a.act = g.act; a.post = g.post; a.post_n = g.post_n;
   a.seg_off = g.seg_off; a.seg_cnt = g.seg_cnt;
   a.w_rows_per_seg = g.seg_cnt ? g.w_stride / g.ldw : 0;
   a.seg_w = g.seg_w;

@@ -517,7 +517,7 @@ int32_t mamba1(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, cons
   else
     VN_LAUNCH(ctx, (mamba_conv_kernel<T, 8>), dim3(ceil_div(n, 32), ceil_div(M, 64)), dim3(32, 8), 0, cv, rows, (T*)b.xc, (T*)b.z, hc.pending);
   if (rows.max_n > hc.pending)
-    VN_LAUNCH(ctx, conv_tail_kernel<T>, dim3(ceil_div(n, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
+    VN_LAUNCH(ctx, (conv_tail_kernel<T, Src, true>), dim3(ceil_div(n, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
   MambaArgs a;
   TRY(project(m, gemm_args(b.xc, n, L.w_uv, L.n_x, n, M, "gemm_mamba_x"), b.p, &a.p));
   a.xc = b.xc; a.z = b.z; a.dt_cols = L.dtp; a.dt_rank = L.dt_rank; a.w_dt = L.w_uk; a.dt_bias = L.f_c; a.A = L.f_a; a.D = L.f_b;
@@ -561,7 +561,7 @@ int32_t channel_delta(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int ru
   }
   TRY(vn_delta_inputs(ctx, cv, in));
   if (rows.max_n > hc.pending)
-    VN_LAUNCH(ctx, conv_tail_kernel<T>, dim3(ceil_div(cv.C, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
+    VN_LAUNCH(ctx, (conv_tail_kernel<T, Src, true>), dim3(ceil_div(cv.C, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
   GemmArgs g = gemm_args(b.low_a, L.rap, L.w_uk, H * d, L.rap, M, "gemm_delta_a2");
   g.C = b.g; g.ldc = H * d;
   TRY(linear(m, g));

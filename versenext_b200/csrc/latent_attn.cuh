@@ -11,8 +11,6 @@
 #include "rows.cuh"
 #include <math_constants.h>
 
-constexpr int KV_PAGE = 64;
-
 struct LatentArgs {
   const void* qc = nullptr;       // [M, H, Rp] queries in the latent space, storage dtype
   const void* plane = nullptr;    // latent cache of this layer run, storage dtype

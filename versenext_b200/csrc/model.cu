@@ -398,7 +398,7 @@ int32_t linear(vn_model* m, GemmArgs g) {
     const char* pe = getenv("VN_PREFILL_TC");
     if (m->use_tc && !(pe && pe[0] == '0') && g.M > 256 && !g.seg_cnt && !g.a_rows && g.nseg == 1 && !g.bias &&
         g.K % tc_detail::BK == 0 && g.N >= tc_detail::BF && g.ldw_k == 1 && tc_detail::encode_fn() != nullptr &&
-        (g.epi == EPI_STORE || g.epi == EPI_ADD || g.epi == EPI_SWIGLU)) {
+        (g.epi == EPI_STORE || g.epi == EPI_ADD || g.epi == EPI_SWIGLU) && (!g.post || g.c_bf16)) {
       const int nseg = ceil_div(g.M, 256);
       if (nseg <= m->row_seg_cap) {
       VN_LAUNCH(ctx, row_segments_kernel, ceil_div(nseg, 128), 128, 0, m->row_seg, m->row_seg + m->row_seg_cap, nseg, g.M);

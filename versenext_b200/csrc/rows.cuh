@@ -11,6 +11,8 @@ template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
+constexpr int KV_PAGE = 64;      // tokens of a cache page
+
 // Rows of a forward.  Either a uniform batch (T > 0: entry e = sequence slot0 + e, rows [e*T, e*T + T)) or a ragged
 // one (T == 0: tables).  Row r of an entry that starts at row row0 has position lens[slot] + off + (r - row0).
 struct Rows {
@@ -28,6 +30,13 @@ struct Rows {
     *start = lens[*s] + off;
   }
 };
+
+// sum of split-K slices of one value, out of line: for code that needs many such values on a rare path
+static __device__ __noinline__ float sum_slices(const float* q, int splits, long long pstride) {
+  float a = 0.f;
+  for (int s = 0; s < splits; ++s) a += q[s * pstride];
+  return a;
+}
 
 // the fp32 result of a projection: one matrix, or split-K slices that the reader sums in slice order
 struct Src {
@@ -47,6 +56,7 @@ struct Src {
     for (; s < splits; ++s) a += q[s * pstride];
     return a;
   }
+  __device__ __forceinline__ float get_rare(long long row, int col) const { return sum_slices(p + row * ld + col, splits, pstride); }
   // rows row .. row + RB - 1 of a column (clamped to row_end - 1), loads independent of one another
   template <int RB>
   __device__ __forceinline__ void column(int row, int row_end, int col, float (&out)[RB]) const {
@@ -60,6 +70,44 @@ struct Src {
     }
   }
 };
+
+// the same as a matrix in the storage dtype (many rows of a 16-bit model: half the bytes)
+template <typename T>
+struct Mat {
+  const T* p = nullptr;
+  int ld = 0;
+  static constexpr int splits = 1;
+  __device__ __forceinline__ float get(long long row, int col) const { return to_f<T>(p[row * ld + col]); }
+  __device__ __forceinline__ float get_rare(long long row, int col) const { return get(row, col); }
+};
+
+// four neighbouring columns (16-byte aligned fp32, 8-byte aligned 16-bit)
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+  uint2 u;
+  *reinterpret_cast<__nv_bfloat162*>(&u.x) = __floats2bfloat162_rn(v.x, v.y);
+  *reinterpret_cast<__nv_bfloat162*>(&u.y) = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+__device__ __forceinline__ float4 get4(const Src& s, long long row, int col) {
+  const float* q = s.p + row * s.ld + col;
+  float4 a = load4(q);
+#pragma unroll 4
+  for (int i = 1; i < s.splits; ++i) {
+    const float4 t = load4(q + (long long)i * s.pstride);
+    a.x += t.x; a.y += t.y; a.z += t.z; a.w += t.w;
+  }
+  return a;
+}
+template <typename T>
+__device__ __forceinline__ float4 get4(const Mat<T>& s, long long row, int col) { return load4(s.p + row * s.ld + col); }
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -90,21 +138,23 @@ __device__ __forceinline__ float block_sum256(float v, float* sm8) {
 // others are inputs of positions that are appended and not committed yet (a rejected suffix is simply overwritten).
 // An input is rounded to the storage dtype before it is used, so that it does not matter whether it came from this
 // forward or from the ring.
-template <typename T>
+// S: where this forward's rows come from.  ACT: silu behind the sum, or nothing.
+template <typename T, typename S = Src, bool ACT = true>
 struct ConvIn {
-  Src src;                 // projection rows of this forward
+  S src;                   // projection rows of this forward
   int col0 = 0;            // first convolved column
   T* ring = nullptr;
   int RC = 1, C = 0, taps = 1;
   const float* w = nullptr;      // [C, taps]
   const float* bias = nullptr;   // [C] or null
 
+  template <bool RARE = false>
   __device__ __forceinline__ float input(int row, int r0, int start, int slot, int pos, int c) const {
-    if (pos >= start) return round_to<T>(src.get(r0 + pos - start, col0 + c));
+    if (pos >= start) return round_to<T>(RARE ? src.get_rare(r0 + pos - start, col0 + c) : src.get(r0 + pos - start, col0 + c));
     if (pos < 0) return 0.f;
     return to_f<T>(ring[((long long)slot * RC + pos % RC) * C + c]);
   }
-  // silu(conv) of channel c at `row`; *cur receives the row's own input
+  // the activated sum of channel c at `row`; *cur receives the row's own input
   __device__ __forceinline__ float at(int row, int r0, int start, int slot, int c, float* cur) const {
     const int pos = start + row - r0;
     const float* wc = w + (long long)c * taps;
@@ -128,7 +178,7 @@ struct ConvIn {
   }
   __device__ __forceinline__ float activate(float acc, int c) const {
     if (bias) acc += bias[c];
-    return silu_as<T>(acc);
+    return ACT ? silu_as<T>(acc) : acc;
   }
   // The same for rows row, row + 1, .. row + RB - 1 (those below row_end, all of one entry): every input is read once.
   // taps <= 4.  Nothing is stored here, so that the loads of several calls can be in flight together.
@@ -145,22 +195,22 @@ struct ConvIn {
       for (int j = 0; j < 4; ++j) wt[j] = j < taps ? wc[taps - 1 - j] : 0.f;
     }
     if (src.splits == 1 && row - r0 >= 3) {            // inside an entry's rows: plain loads, all independent
-      const float* p = src.p + (long long)row * src.ld + col0 + c;
+      const auto* p = src.p + (long long)row * src.ld + col0 + c;
       if (row + RB <= row_end) {
         p -= 3ll * src.ld;
 #pragma unroll
-        for (int i = 0; i < RB + 3; ++i, p += src.ld) x[i] = *p;
+        for (int i = 0; i < RB + 3; ++i, p += src.ld) x[i] = to_f(*p);
       } else {
 #pragma unroll
-        for (int i = 0; i < RB + 3; ++i) x[i] = p[(long long)(min(row + i - 3, row_end - 1) - row) * src.ld];
+        for (int i = 0; i < RB + 3; ++i) x[i] = to_f(p[(long long)(min(row + i - 3, row_end - 1) - row) * src.ld]);
       }
 #pragma unroll
       for (int i = 0; i < RB + 3; ++i) x[i] = round_to<T>(x[i]);
     } else {
 #pragma unroll
-      for (int j = 1; j < 4; ++j) x[3 - j] = j < taps ? input(row, r0, start, slot, pos - j, c) : 0.f;
+      for (int j = 1; j < 4; ++j) x[3 - j] = j < taps ? input<true>(row, r0, start, slot, pos - j, c) : 0.f;
 #pragma unroll
-      for (int i = 0; i < RB; ++i) x[3 + i] = row + i < row_end ? round_to<T>(src.get(row + i, col0 + c)) : 0.f;
+      for (int i = 0; i < RB; ++i) x[3 + i] = row + i < row_end ? round_to<T>(src.get_rare(row + i, col0 + c)) : 0.f;
     }
 #pragma unroll
     for (int i = 0; i < RB; ++i) {

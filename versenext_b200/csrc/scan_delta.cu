@@ -4,7 +4,7 @@
 template <typename T>
 int32_t vn_delta_inputs(vn_ctx* ctx, const ConvIn<T>& conv, const DeltaIn& in) {
   const int nc = ceil_div(in.d > in.vd ? in.d : in.vd, 32);
-  const bool many = in.rows.M >= 512 && nc <= 4;
+  const bool many = in.rows.M >= 512 && nc <= 4 && conv.taps <= 4;
   const dim3 grid(2 * in.KH + in.H + 1, ceil_div(in.rows.M, many ? 64 : 8)), block(32, 8);
 #define INPUTS(NC, RB) VN_LAUNCH_NAMED(ctx, "delta_inputs_kernel", (delta_inputs_kernel<T, NC, RB>), grid, block, 0, conv, in)
   if (many) { if (nc <= 1) INPUTS(1, 8); else if (nc <= 2) INPUTS(2, 8); else INPUTS(4, 8); return VN_OK; }

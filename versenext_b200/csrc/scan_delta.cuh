@@ -61,21 +61,18 @@ __global__ void __launch_bounds__(256) delta_inputs_kernel(ConvIn<T> in, DeltaIn
     a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
     const int first = row, end = min(last, r0 + n);
     float val[RB][NC];
-#pragma unroll
+#pragma unroll (NC > 4 ? 1 : NC)             // wide heads: the convolution's code once
     for (int i = 0; i < NC; ++i) {
       const int j = lane + 32 * i;
       float v[RB];
 #pragma unroll
       for (int r = 0; r < RB; ++r) v[r] = 0.f;
       if (j < w) {
-        if (RB > 1 && in.taps <= 4) {
+        if constexpr (RB > 1) {                  // filters of at most four taps
           in.template run<RB>(first, end, r0, start, slot, c0 + j, v);
         } else {
-#pragma unroll
-          for (int r = 0; r < RB; ++r) {
-            float cur;
-            if (first + r < end) v[r] = in.at(first + r, r0, start, slot, c0 + j, &cur);
-          }
+          float cur;
+          v[0] = in.at(first, r0, start, slot, c0 + j, &cur);
         }
       }
 #pragma unroll

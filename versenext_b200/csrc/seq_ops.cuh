@@ -87,6 +87,38 @@ __global__ void __launch_bounds__(256) rmsnorm_pick_kernel(const float* __restri
   }
 }
 
+// sum of split-K slices [M, N]: columns below n_act through a function (GemmPost) to `act` [M, ld_act] in the storage dtype,
+// the others as they are to `rest` [M, N - n_act] in fp32 (or, with rest null, to `act` too).  N % 4 == n_act % 4 == 0.
+template <typename T>
+__global__ void __launch_bounds__(256) slices_act_kernel(Src src, int N, int n_act, int post, T* __restrict__ act, int ld_act,
+                                                         float* __restrict__ rest, long long total4) {
+  pdl_trigger();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= total4) return;
+  const long long row = i / (N / 4);
+  const int c = (int)(i % (N / 4)) * 4;
+  float4 v = get4(src, row, c);
+  if (c >= n_act && rest) {
+    store4(rest + row * (N - n_act) + c - n_act, v);
+    return;
+  }
+  if (c < n_act) {
+    constexpr bool fast = sizeof(T) == 2;
+    v = make_float4(post_act(v.x, post, fast), post_act(v.y, post, fast), post_act(v.z, post, fast), post_act(v.w, post, fast));
+  }
+  store4(act + row * ld_act + c, v);
+}
+// the same one column at a time: columns [0, N) of the source's rows to a matrix [M, N], any sizes
+template <typename T>
+__global__ void __launch_bounds__(256) slices_act1_kernel(Src src, int N, int n_act, int post, T* __restrict__ act, long long total) {
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= total) return;
+  const int c = (int)(i % N);
+  const float v = src.get(i / N, c);
+  act[i] = from_f<T>(c < n_act ? post_act(v, post, sizeof(T) == 2) : v);
+}
+
 // lens[slot] += rows of the entry (a step that keeps everything it appended)
 __global__ void rows_advance_kernel(Rows rows, int* __restrict__ lens) {
   const int e = blockIdx.x * blockDim.x + threadIdx.x;
@@ -96,8 +128,8 @@ __global__ void rows_advance_kernel(Rows rows, int* __restrict__ lens) {
 
 // inputs of long entries (more rows than the ring keeps apart): the last taps - 1 positions, after every reader of
 // the older ones has finished.  grid (ceil(C / 256), n_ent)
-template <typename T>
-__global__ void __launch_bounds__(256) conv_tail_kernel(ConvIn<T> in, Rows rows, int pending) {
+template <typename T, typename S, bool ACT>
+__global__ void __launch_bounds__(256) conv_tail_kernel(ConvIn<T, S, ACT> in, Rows rows, int pending) {
   int slot, r0, n, start;
   rows.entry(blockIdx.y, &slot, &r0, &n, &start);
   const int c = blockIdx.x * 256 + threadIdx.x;
