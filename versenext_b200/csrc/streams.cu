@@ -1,0 +1,211 @@
+// Kernels of streams.cuh.
+#include "streams.cuh"
+
+namespace {
+
+template <int V> struct Vec { float v[V]; };
+template <int V, typename P> __device__ __forceinline__ Vec<V> vload(const P* p) {
+  Vec<V> r;
+  if constexpr (V == 4) { const float4 t = load4(p); r.v[0] = t.x; r.v[1] = t.y; r.v[2] = t.z; r.v[3] = t.w; }
+  else r.v[0] = to_f(*p);
+  return r;
+}
+template <int V, typename S> __device__ __forceinline__ Vec<V> vget(const S& s, long long row, int d) {
+  Vec<V> r;
+  if constexpr (V == 4) { const float4 t = get4(s, row, d); r.v[0] = t.x; r.v[1] = t.y; r.v[2] = t.z; r.v[3] = t.w; }
+  else r.v[0] = s.get(row, d);
+  return r;
+}
+template <int V, typename P> __device__ __forceinline__ void vstore(P* p, const Vec<V>& r) {
+  if constexpr (V == 4) store4(p, make_float4(r.v[0], r.v[1], r.v[2], r.v[3]));
+  else *p = from_f<P>(r.v[0]);
+}
+
+// One CTA per row.  Shared memory: D floats (u).
+template <typename T, typename S, int NS, int V>
+__global__ void __launch_bounds__(256) streams_kernel(StreamArgs<T, S> a) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float s_u[];
+  __shared__ float s_mix[NS * NS], s_out[NS], s_in[NS], red[3][8];
+  const int tid = threadIdx.x, D = a.D;
+  if (tid < NS * NS) s_mix[tid] = a.mix ? a.mix[tid] : (tid / NS == tid % NS ? 1.f : 0.f);
+  if (tid < NS) { s_out[tid] = a.out ? a.out[tid] : 1.f; s_in[tid] = a.in ? a.in[tid] : 1.f; }
+  pdl_wait();
+  const long long row = a.pick ? a.pick[blockIdx.x] : (long long)blockIdx.x * a.mul + a.add;
+  const bool write = a.y.p != nullptr, gated = a.gate.p != nullptr;
+  float ysc = 1.f;
+  if (a.ss) {
+    float v = 0.f;
+    for (int i = tid; i < a.n_ss; i += 256) v += a.ss[row * a.n_ss + i];
+    ysc = 1.f / sqrtf(block_sum256(v, red[0]) / a.ss_count + a.eps);   // the sum's barrier also publishes the weights
+  } else {
+    __syncthreads();
+  }
+  float* x = a.x + row * NS * D;
+  const float* first = a.first ? a.first + row * D : nullptr;
+  float sum = 0.f;
+  for (int d = tid * V; d < D; d += 256 * V) {
+    Vec<V> xs[NS], u;
+    if (first) {
+      xs[0] = vload<V>(first + d);
+#pragma unroll
+      for (int s = 1; s < NS; ++s) xs[s] = xs[0];
+    } else {
+#pragma unroll
+      for (int s = 0; s < NS; ++s) xs[s] = vload<V>(x + (long long)s * D + d);
+    }
+    if (write) {
+      Vec<V> y = vget<V>(a.y, row, d), n[NS];
+      if (gated) {
+        const Vec<V> g = vget<V>(a.gate, row, d);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y.v[e] *= sigmoid_f(g.v[e] + (a.gate_b ? a.gate_b[d + e] : 0.f));
+      }
+#pragma unroll
+      for (int t = 0; t < NS; ++t) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          float v = s_out[t] * (y.v[e] * ysc);
+#pragma unroll
+          for (int s = 0; s < NS; ++s) v = fmaf(s_mix[s * NS + t], xs[s].v[e], v);
+          n[t].v[e] = v;
+        }
+        vstore<V>(x + (long long)t * D + d, n[t]);
+      }
+#pragma unroll
+      for (int t = 0; t < NS; ++t) xs[t] = n[t];
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      u.v[e] = 0.f;
+#pragma unroll
+      for (int s = 0; s < NS; ++s) u.v[e] = fmaf(s_in[s], xs[s].v[e], u.v[e]);
+      sum += a.layer_norm ? u.v[e] : u.v[e] * u.v[e];
+    }
+    vstore<V>(s_u + d, u);
+  }
+  if (!a.norm_w) return;
+  float mean = 0.f, r;
+  const float tot = block_sum256(sum, red[1]);
+  if (a.layer_norm) {
+    mean = tot / (float)D;
+    float v = 0.f;
+    for (int d = tid * V; d < D; d += 256 * V)
+#pragma unroll
+      for (int e = 0; e < V; ++e) { const float t = s_u[d + e] - mean; v = fmaf(t, t, v); }
+    r = sqrtf(block_sum256(v, red[2]) / (float)D + a.eps);
+  } else {
+    r = sqrtf(tot / (float)D + a.eps);
+  }
+  int slot = 0, r0, n, pos = 0;
+  if (a.hc) a.rows.entry(a.rows.entry_of((int)row), &slot, &r0, &n, &pos);
+  const long long orow = blockIdx.x;
+  for (int d = tid * V; d < D; d += 256 * V) {
+    Vec<V> v = vload<V>(s_u + d);
+    const Vec<V> w = vload<V>(a.norm_w + d);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v.v[e] = (v.v[e] - mean) / r * w.v[e];
+    if (a.h) vstore<V>(a.h + orow * D + d, v);
+    if (a.h32) vstore<V>(a.h32 + orow * D + d, v);
+    if (a.hc) {
+      T* ring = a.ring + (long long)slot * a.RC * D + d;
+      Vec<V> acc;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        v.v[e] = round_to<T>(v.v[e]);
+        acc.v[e] = v.v[e] * a.conv_w[(long long)(d + e) * a.taps + a.taps - 1];
+      }
+#pragma unroll 3
+      for (int j = 1; j < a.taps; ++j) {
+        if (j > pos) break;
+        const Vec<V> old = vload<V>(ring + (long long)((pos - j) % a.RC) * D);
+#pragma unroll
+        for (int e = 0; e < V; ++e) acc.v[e] = fmaf(old.v[e], a.conv_w[(long long)(d + e) * a.taps + a.taps - 1 - j], acc.v[e]);
+      }
+      if (a.taps > 1) vstore<V>(ring + (long long)(pos % a.RC) * D, v);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc.v[e] += v.v[e];
+      vstore<V>(a.hc + orow * D + d, acc);
+    }
+  }
+}
+
+__global__ void __launch_bounds__(256) streams_sum_kernel(const float* __restrict__ x, float* __restrict__ out, int ns, int D) {
+  const long long row = blockIdx.x;
+  for (int d = threadIdx.x; d < D; d += 256) {
+    float v = 0.f;
+    for (int s = 0; s < ns; ++s) v += x[(row * ns + s) * D + d];
+    out[row * D + d] = v;
+  }
+}
+
+// RB rows of one channel per thread (RB > 1: filters of at most four taps).  grid (ceil(D / 256), ceil(M / RB))
+template <typename T, int RB>
+__global__ void __launch_bounds__(256) input_conv_kernel(ConvIn<T, Mat<T>, false> in, Rows rows, int pending, T* __restrict__ hc) {
+  const int c = blockIdx.x * 256 + threadIdx.x, D = in.C;
+  if (c >= D) return;
+  int row = blockIdx.y * RB;
+  const int last = min(row + RB, rows.M);
+  while (row < last) {                                  // stretches of one entry
+    int slot, r0, n, start;
+    rows.entry(rows.entry_of(row), &slot, &r0, &n, &start);
+    const int end = min(last, r0 + n);
+    float v[RB];
+    if constexpr (RB > 1) {
+      in.template run<RB>(row, end, r0, start, slot, c, v);
+    } else {
+      float cur;
+      v[0] = in.at(row, r0, start, slot, c, &cur);
+    }
+#pragma unroll
+    for (int i = 0; i < RB; ++i)
+      if (row + i < end) {
+        const float h = in.src.get(row + i, c);
+        hc[(long long)(row + i) * D + c] = from_f<T>(h + v[i]);
+        if (n <= pending && in.taps > 1) in.keep(slot, start + row + i - r0, c, h);
+      }
+    row = end;
+  }
+}
+
+template <typename T, typename S, int V>
+int32_t launch(vn_ctx* ctx, const StreamArgs<T, S>& a, int n_rows) {
+  const size_t smem = (size_t)a.D * 4;
+#define CASE(NS) case NS: \
+  if (smem > 40000) VN_CUDA(ctx, cudaFuncSetAttribute((streams_kernel<T, S, NS, V>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+  VN_LAUNCH_PDL_LEVEL(ctx, (vn_pdl_mask() & 4) ? 1 : 2, "streams_kernel", (streams_kernel<T, S, NS, V>), n_rows, 256, smem, a); break;
+  switch (a.ns) {
+    CASE(1) CASE(2) CASE(3) CASE(4) CASE(5) CASE(6) CASE(7) CASE(8)
+    default: return vn_fail(ctx, VN_ERR_UNSUPPORTED, "%d residual streams", a.ns);
+  }
+#undef CASE
+  return VN_OK;
+}
+
+}  // namespace
+
+template <typename T, typename S>
+int32_t vn_streams(vn_ctx* ctx, const StreamArgs<T, S>& a, int n_rows) {
+  if (a.D % 4 == 0 && a.y.ld % 4 == 0 && a.gate.ld % 4 == 0 && ((uintptr_t)a.gate.p & 15) == 0) return launch<T, S, 4>(ctx, a, n_rows);
+  return launch<T, S, 1>(ctx, a, n_rows);
+}
+template int32_t vn_streams(vn_ctx*, const StreamArgs<float, Src>&, int);
+template int32_t vn_streams(vn_ctx*, const StreamArgs<__nv_bfloat16, Src>&, int);
+template int32_t vn_streams(vn_ctx*, const StreamArgs<__nv_bfloat16, Mat<__nv_bfloat16>>&, int);
+
+int32_t vn_streams_sum(vn_ctx* ctx, const float* x, float* out, int M, int ns, int D) {
+  VN_LAUNCH(ctx, streams_sum_kernel, M, 256, 0, x, out, ns, D);
+  return VN_OK;
+}
+
+template <typename T>
+int32_t vn_input_conv(vn_ctx* ctx, const ConvIn<T, Mat<T>, false>& in, const Rows& rows, int pending, T* hc) {
+  if (in.taps <= 4)
+    VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv_kernel<T, 8>), dim3(ceil_div(in.C, 256), ceil_div(rows.M, 8)), 256, 0, in, rows,
+                    pending, hc);
+  else
+    VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv_kernel<T, 1>), dim3(ceil_div(in.C, 256), rows.M), 256, 0, in, rows, pending, hc);
+  return VN_OK;
+}
+template int32_t vn_input_conv(vn_ctx*, const ConvIn<float, Mat<float>, false>&, const Rows&, int, float*);
+template int32_t vn_input_conv(vn_ctx*, const ConvIn<__nv_bfloat16, Mat<__nv_bfloat16>, false>&, const Rows&, int, __nv_bfloat16*);
