@@ -1,0 +1,289 @@
+// The one-token kernel of paged_attn.cuh.
+//
+// CTA = (key range, key/value head and tile of 16 query heads, sequence).  It convolves and rotates its query heads; the
+// CTA of the last range does the same for the new key and value and appends them.  Each of four warps streams chunks of 16
+// keys through its own cp.async ring; the warps, then the CTAs of a sequence (the last one to finish), merge.
+#include "ldmatrix.cuh"
+#include "paged_attn.cuh"
+
+namespace {
+
+using bf16 = __nv_bfloat16;
+constexpr int WARPS = 4;
+template <int P> constexpr int stages() { return P > 128 ? 2 : 3; }
+template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2; }
+
+template <int P>
+__global__ void __launch_bounds__(32 * WARPS) attn_step_kernel(ConvIn<bf16, Src, false> in, PagedAttnArgs a) {
+  using namespace mma_detail;
+  constexpr int LD = P + 8, ST = stages<P>(), TH = 32 * WARPS, CH = P / 8, TILE = 16 * LD;
+  extern __shared__ __align__(16) unsigned char raw[];
+  bf16* ring = reinterpret_cast<bf16*>(raw);                          // [warp][stage][K, V][16][LD]
+  bf16* sQ = ring + WARPS * ST * 2 * TILE;                            // [16][LD]
+  bf16* sNew = sQ + TILE;                                             // [2][P] key and value of the new token
+  __shared__ int s_last;
+  __shared__ float s_ml[WARPS][16][2], s_f[WARPS][16];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = blockIdx.z;
+  const int hg = a.H / a.KH, tiles = (hg + 15) / 16, g = blockIdx.y / tiles, q0 = (blockIdx.y % tiles) * 16, nq = min(16, hg - q0);
+  int slot, r0, n, pos;
+  a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &pos);
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int c_lo = lo / 16, c_hi = pos / 16 + 1, per = (c_hi - c_lo + a.splits - 1) / a.splits;
+  const int c0 = min(c_hi, c_lo + (int)blockIdx.x * per), c1 = min(c_hi, c0 + per);
+  const bool fresh = a.own_kv && c0 < c1 && c1 == c_hi;               // this range ends with the new token
+  const int* tab = a.table + (long long)slot * a.max_pages;
+  const long long ldp = (long long)a.KH * P;
+  const bf16 *kp = reinterpret_cast<const bf16*>(a.kplane) + (long long)g * P, *vp = reinterpret_cast<const bf16*>(a.vplane) + (long long)g * P;
+  bf16* mine = ring + warp * ST * 2 * TILE;
+  auto fetch = [&](int c, int st) {
+    if (c < c1) {
+      const long long base = ((long long)tab[16 * c / KV_PAGE] * KV_PAGE + 16 * c % KV_PAGE) * ldp;
+      const int valid = min(16, pos + (fresh ? 0 : 1) - 16 * c);      // the new token's row comes from shared memory
+      for (int i = lane; i < 16 * CH; i += 32) {
+        const int r = i / CH, x = (i % CH) * 8;
+        const bool ok = r < valid;
+        const long long at = base + (ok ? r : 0) * ldp + x;
+        cp_async16(mine + st * 2 * TILE + r * LD + x, kp + at, ok);
+        cp_async16(mine + st * 2 * TILE + TILE + r * LD + x, vp + at, ok);
+      }
+    }
+    cp_async_commit();
+  };
+#pragma unroll
+  for (int s = 0; s < ST - 1; ++s) fetch(c0 + warp + s * WARPS, s);
+  // queries; the new key and value
+  {
+    const int np = a.rd / 2, qi = np + a.d - a.rd, nqi = nq * qi, nk = fresh ? qi : 0, nv = fresh ? a.vd : 0;
+    const float2* rope = a.rope + (long long)pos * np;
+    const bool keep_q = blockIdx.x == 0, keep_kv = q0 == 0;
+#pragma unroll 1
+    for (int i = tid; i < nqi + nk + nv; i += TH) {
+      // a pair of channels of a query or key head, one unrotated channel of either, or one of the value
+      int c, x = 0;
+      bf16* dst;
+      bool keep, pair = false;
+      if (i < nqi + nk) {
+        const bool q = i < nqi;
+        const int head = q ? i / qi : 0;
+        x = q ? i % qi : i - nqi;
+        pair = x < np;
+        if (!pair) x += np;
+        c = (q ? (g * hg + q0 + head) * a.d : (a.H + g) * a.d) + x;
+        keep = q ? keep_q : keep_kv;
+        dst = (q ? sQ + head * LD : sNew) + x;
+      } else {
+        x = i - nqi - nk;
+        c = (a.H + a.KH) * a.d + g * a.vd + x;
+        keep = keep_kv;
+        dst = sNew + P + x;
+      }
+      float cur, u = in.at(row, r0, pos, slot, c, &cur);
+      if (keep && in.taps > 1) in.keep(slot, pos, c, cur);
+      if (pair) {
+        const float v = in.at(row, r0, pos, slot, c + np, &cur);
+        if (keep && in.taps > 1) in.keep(slot, pos, c + np, cur);
+        const float2 cs = rope[x];
+        dst[np] = __float2bfloat16_rn(v * cs.x + u * cs.y);
+        u = u * cs.x - v * cs.y;
+      }
+      *dst = __float2bfloat16_rn(u);
+    }
+    const bf16 zero = __float2bfloat16_rn(0.f);
+    for (int i = tid; i < 16 * P; i += TH) {
+      const int r = i / P, c = i % P;
+      if (r >= nq || c >= a.d) sQ[r * LD + c] = zero;
+    }
+    if (fresh) {
+      for (int c = a.d + tid; c < P; c += TH) sNew[c] = zero;
+      for (int c = a.vd + tid; c < P; c += TH) sNew[P + c] = zero;
+    }
+  }
+  __syncthreads();
+  if (fresh && q0 == 0) {
+    const long long at = (((long long)tab[pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.KH + g) * P;
+    for (int c = tid; c < P; c += TH) {
+      reinterpret_cast<bf16*>(a.kplane)[at + c] = sNew[c];
+      reinterpret_cast<bf16*>(a.vplane)[at + c] = sNew[P + c];
+    }
+  }
+  float acc[P / 8][4];
+#pragma unroll
+  for (int j = 0; j < P / 8; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+  float m_run[2] = {-CUDART_INF_F, -CUDART_INF_F}, l_run[2] = {0.f, 0.f};
+  const float sc = a.scale * 1.4426950408889634f;
+  const bf16* q_at = sQ + (lane & 15) * LD + ((lane >> 4) << 3);
+  int st = 0;
+  for (int c = c0 + warp; c < c1; c += WARPS) {
+    fetch(c + (ST - 1) * WARPS, st == 0 ? ST - 1 : st - 1);
+    cp_async_wait<ST - 1>();
+    __syncwarp();
+    bf16 *K = mine + st * 2 * TILE, *V = K + TILE;
+    if (fresh && c == pos / 16) {
+      for (int x = lane; x < P; x += 32) { K[(pos & 15) * LD + x] = sNew[x]; V[(pos & 15) * LD + x] = sNew[P + x]; }
+      __syncwarp();
+    }
+    float s[2][4];
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
+#pragma unroll
+    for (int k = 0; k < P / 16; ++k) {
+      unsigned af[4], b0[2], b1[2];
+      ldmatrix_x4(af[0], af[1], af[2], af[3], q_at + 16 * k);
+      ldmatrix_x4(b0[0], b0[1], b1[0], b1[1], K + ((lane & 7) + ((lane >> 4) << 3)) * LD + 16 * k + (((lane >> 3) & 1) << 3));
+      mma_bf16(s[0], af, b0);
+      mma_bf16(s[1], af, b1);
+    }
+    float mx[2] = {m_run[0], m_run[1]};
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const int key = 16 * c + 8 * j + (lane & 3) * 2 + (x & 1);
+        s[j][x] = key >= lo && key <= pos ? s[j][x] * sc : -CUDART_INF_F;
+        mx[x >> 1] = fmaxf(mx[x >> 1], s[j][x]);
+      }
+    float f[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
+      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
+      f[e] = exp2f(m_run[e] - mx[e]);                     // a chunk has a visible key, so mx is finite
+      m_run[e] = mx[e];
+      l_run[e] *= f[e];
+    }
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        s[j][x] = exp2f(s[j][x] - mx[x >> 1]);
+        l_run[x >> 1] += s[j][x];
+      }
+    const unsigned af[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]), pack_bf16(s[1][2], s[1][3])};
+#pragma unroll
+    for (int j = 0; j < P / 16; ++j) {
+      unsigned b0[2], b1[2];
+      ldmatrix_x4_t(b0[0], b0[1], b1[0], b1[1], V + ((lane & 7) + (((lane >> 3) & 1) << 3)) * LD + 16 * j + ((lane >> 4) << 3));
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        acc[2 * j + y][0] *= f[0]; acc[2 * j + y][1] *= f[0]; acc[2 * j + y][2] *= f[1]; acc[2 * j + y][3] *= f[1];
+      }
+      mma_bf16(acc[2 * j], af, b0);
+      mma_bf16(acc[2 * j + 1], af, b1);
+    }
+    __syncwarp();
+    st = st + 1 == ST ? 0 : st + 1;
+  }
+  cp_async_wait<0>();
+  __syncthreads();                                        // the rings are free: outputs of the warps [warp][16][P]
+  float* sO = reinterpret_cast<float*>(raw);
+  static_assert(WARPS * 16 * P * 4 <= WARPS * ST * 2 * TILE * 2, "outputs fit where the rings were");
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    float l = l_run[e];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    const int r = (lane >> 2) + 8 * e;
+    if ((lane & 3) == 0) { s_ml[warp][r][0] = m_run[e]; s_ml[warp][r][1] = l; }
+#pragma unroll
+    for (int j = 0; j < P / 8; ++j)
+      *reinterpret_cast<float2*>(sO + (warp * 16 + r) * P + 8 * j + (lane & 3) * 2) = make_float2(acc[j][2 * e], acc[j][2 * e + 1]);
+  }
+  __syncthreads();
+  // factors of the warps, and the range's own maximum and sum
+  if (tid < 16) {
+    float m = -CUDART_INF_F, l = 0.f;
+#pragma unroll
+    for (int w = 0; w < WARPS; ++w) m = fmaxf(m, s_ml[w][tid][0]);
+#pragma unroll
+    for (int w = 0; w < WARPS; ++w) {
+      const float f = s_ml[w][tid][0] == -CUDART_INF_F ? 0.f : exp2f(s_ml[w][tid][0] - m);
+      s_f[w][tid] = f;
+      l += f * s_ml[w][tid][1];
+    }
+    s_ml[0][tid][0] = m;
+    s_ml[0][tid][1] = l;
+  }
+  __syncthreads();
+  auto finish = [&](int r, int c, float o, float l) {
+    const int h = g * hg + q0 + r;
+    if (c < a.vd) {
+      const float gate = a.col_g >= 0 ? sigmoid_f(in.src.get(row, a.col_g + h * a.vd + c)) : 1.f;
+      reinterpret_cast<bf16*>(a.out)[((long long)row * a.H + h) * a.vd + c] = __float2bfloat16_rn(o / l * gate);
+    }
+  };
+  const long long n_rh = (long long)a.rows.M * a.H, rh0 = (long long)row * a.H + g * hg + q0;
+  for (int i = tid; i < nq * P; i += TH) {
+    const int r = i / P, c = i % P;
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < WARPS; ++w) o = fmaf(s_f[w][r], sO[(w * 16 + r) * P + c], o);
+    if (a.splits == 1) finish(r, c, o, s_ml[0][r][1]);
+    else a.part_o[((long long)blockIdx.x * n_rh + rh0 + r) * P + c] = o;
+  }
+  if (a.splits == 1) return;
+  if (tid < nq) {
+    float* ml = a.part_ml + ((long long)blockIdx.x * n_rh + rh0 + tid) * 2;
+    ml[0] = s_ml[0][tid][0];
+    ml[1] = s_ml[0][tid][1];
+  }
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) {
+    int* t = a.tickets + (long long)row * gridDim.y + blockIdx.y;
+    s_last = atomicAdd(t, 1) == a.splits - 1;
+    if (s_last) *t = 0;
+  }
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+  // merge the ranges: weight of range s for head r in shared memory (lane s holds range s), then the heads' sums
+  float* sW = reinterpret_cast<float*>(raw);              // [32][16], then [16]
+  for (int r = warp; r < nq; r += WARPS) {
+    const float* ml = a.part_ml + ((long long)lane * n_rh + rh0 + r) * 2;
+    const float m = lane < a.splits ? __ldcg(ml) : -CUDART_INF_F, l = lane < a.splits ? __ldcg(ml + 1) : 0.f;
+    float top = m;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+    const float f = m == -CUDART_INF_F ? 0.f : exp2f(m - top);
+    const float sum = warp_sum(f * l);
+    sW[lane * 16 + r] = f;
+    if (lane == 0) sW[512 + r] = sum;
+  }
+  __syncthreads();
+  for (int i = tid; i < nq * P; i += TH) {
+    const int r = i / P, c = i % P;
+    float o = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < a.splits; ++s) o = fmaf(sW[s * 16 + r], __ldcg(a.part_o + ((long long)s * n_rh + rh0 + r) * P + c), o);
+    finish(r, c, o, sW[512 + r]);
+  }
+}
+
+}  // namespace
+
+int32_t vn_attn_step(vn_ctx* ctx, const ConvIn<bf16, Src, false>& conv, const PagedAttnArgs& a) {
+  const dim3 grid(a.splits, a.KH * ceil_div(a.H / a.KH, 16), a.rows.M);
+  VN_REQUIRE(ctx, a.splits >= 1 && a.splits <= 32 && (a.splits == 1 || (long long)grid.y * grid.z <= VN_TICKETS), "key ranges of the one-token kernel");
+#define STEP(P) do { \
+    static unsigned long long done = 0; \
+    if (!((done >> (ctx->device & 63)) & 1ull)) { \
+      VN_CUDA(ctx, cudaFuncSetAttribute(attn_step_kernel<P>, cudaFuncAttributeMaxDynamicSharedMemorySize, step_smem<P>())); \
+      done |= 1ull << (ctx->device & 63); \
+    } \
+    VN_LAUNCH_NAMED(ctx, "attn_step_kernel", attn_step_kernel<P>, grid, 32 * WARPS, step_smem<P>(), conv, a); } while (0)
+  switch (a.P) {
+    case 32: STEP(32); break;
+    case 64: STEP(64); break;
+    case 96: STEP(96); break;
+    case 128: STEP(128); break;
+    case 192: STEP(192); break;
+    case 256: STEP(256); break;
+    default: return vn_fail(ctx, VN_ERR_UNSUPPORTED, "key pitch %d", a.P);
+  }
+#undef STEP
+  return VN_OK;
+}
