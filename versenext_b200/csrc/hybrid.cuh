@@ -1,45 +1,71 @@
-// Composed models: a list of layers of different kinds (latent attention, selective scan, gated delta rule), each with
-// an optional gated feed-forward, and optionally a block of layers that is run several times with the same weights.
-// Weights, the per-sequence cache (paged latents, rings of convolution inputs and of recurrent states), and the forward
-// over new rows of a uniform or a ragged batch.  Included by model.cu: it uses that file's GEMM helpers.
+// Composed models: a list of layers of different kinds (latent attention, grouped-query attention, selective scan, gated
+// delta rule, lightning attention), each with an optional feed-forward, and optionally a block of layers that is run several
+// times with the same weights.  The residual is one stream that sublayers add to, or an arrangement of several (streams.cuh).
+// Weights, the per-sequence cache (paged latents, keys and values, rings of convolution inputs and of recurrent states), and
+// the forward over new rows of a uniform or a ragged batch.  Included by model.cu: it uses that file's GEMM helpers.
 //
 // One forward serves prompts, portions of prompts, single tokens and mixtures.  Projections of at most 256 rows of a
 // bf16 model are split-K tcgen05 GEMMs whose slices are summed by the kernel that needs them; longer ones go through
 // the tcgen05 segment kernel; an fp32 model uses the fp32 GEMM.  When every entry brings one token, a mixer's
-// recurrence and what surrounds it is one kernel (mamba_step_kernel, delta_step_kernel).
+// recurrence or attention and what surrounds it is one kernel (mamba_step_kernel, delta_step_kernel, attn_step_kernel,
+// lightning_scan_kernel).
 #pragma once
 #include "json_value.h"
 #include "latent_attn.cuh"
+#include "lightning.cuh"
+#include "paged_attn.cuh"
 #include "scan_delta.cuh"
 #include "scan_mamba.cuh"
 #include "seq_ops.cuh"
+#include "streams.cuh"
 
 namespace hybrid {
 
-enum Kind { LATENT = 0, MAMBA1 = 1, DELTA = 2 };
+enum Kind { LATENT = 0, MAMBA1 = 1, DELTA = 2, ATTENTION = 3, LIGHTNING = 4 };
 
 struct HLayer {
   int kind = 0;
   // latent: H, d, vd, R (kv_rank), window, scale.  mamba: inner, dt_rank, nstate, taps.  delta: H, KH, d, vd, taps, ra, rg
   int H = 0, KH = 0, d = 0, vd = 0, R = 0, window = 0, taps = 1, inner = 0, dt_rank = 0, nstate = 0, ra = 0, rg = 0;
   float scale = 1.f;
-  int ff = 0, act = 0;             // feed-forward width (0: none), activation
+  // attention: H, KH, d, vd, taps, window, scale and the line below (conv_named: the convolutions are in the checkpoint).
+  // lightning: H, d, vd, decay
+  int kv_from = -1, gated = 0, P = 0, rd = 0, rope = -1, conv_named = 0;
+  std::vector<double> decay;
+  int ff = 0, act = 0;             // feed-forward width (0: none), activation of its gate: 0 silu, 1 gelu
+  int ff_plain = 0;                // no gate: squared relu
   int dp = 0, Rp = 0, dtp = 0, rap = 0, rgp = 0, n_in = 0, n_x = 0, ffp = 0;    // padded sizes
   float* norm1 = nullptr; float* norm2 = nullptr;                               // 1 + stored weight
   void* w_in = nullptr;            // first projection, all its parts stacked [n_in, D]
   void* w_o = nullptr;
   void* w_uk = nullptr;            // latent: per head W_uk^T [H][Rp][dp];  delta: a2 [H d, rap];  mamba: dt [inner, dtp]
   void* w_uv = nullptr;            // latent: [H][vd][Rp];                  delta: g2 [H vd, rgp];  mamba: x [n_x, inner]
-  float* f_a = nullptr;            // latent: norm of the latent;  delta: norm [vd];         mamba: A = -exp(A_log)
-  float* f_b = nullptr;            // latent: sink [H];            delta: exp(A_log) [H];    mamba: D
-  float* f_c = nullptr;            //                              delta: dt_bias [H d];     mamba: dt bias
+  float* f_a = nullptr;            // latent: norm of the latent;  delta: norm [vd];       mamba: A = -exp(A_log);  lightning: norm [H vd]
+  float* f_b = nullptr;            // latent: sink [H];            delta: exp(A_log) [H];  mamba: D;                lightning: decay [H][2]
+  float* f_c = nullptr;            //                              delta: dt_bias [H d];   mamba: dt bias;          lightning: powers [H][65]
+  // residual arrangement, per sublayer (0 mixer, 1 feed-forward)
+  float *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
+  void* w_rg[2] = {nullptr, nullptr};     // gate of the sublayer's result; of a plain feed-forward: the rows behind w_gu's
+  float* rg_b[2] = {nullptr, nullptr};
+  float* in_conv = nullptr;               // [D, taps] convolution of what the mixer reads
   float* conv = nullptr; float* conv_b = nullptr;
   void* w_gu = nullptr; void* w_down = nullptr;
-  int conv_ch() const { return kind == MAMBA1 ? inner : 2 * KH * d + H * vd; }
+  int conv_ch() const {
+    if (kind == MAMBA1) return inner;
+    if (kind == ATTENTION) return H * d + (kv_from < 0 ? KH * (d + vd) : 0);
+    return 2 * KH * d + H * vd;
+  }
   long long state_elems() const { return kind == MAMBA1 ? (long long)inner * nstate : (long long)H * d * vd; }
 };
 
-struct Run { int layer; int pass; };      // pass: -1 outside the loop
+struct Run { int layer; int pass; int kv_run; };      // pass: -1 outside the loop; kv_run: the run whose keys it reads
+
+struct Rope {                      // frequencies of the rotated pairs, amplitude of cos and sin
+  std::vector<double> freq;
+  float amp = 1.f;
+  float2* table = nullptr;         // [rows][pairs]
+  int rows = 0;
+};
 
 struct Model {
   int D = 0, vocab = 0, sinusoidal = 0;
@@ -54,6 +80,15 @@ struct Model {
   float* x0 = nullptr; void* cat = nullptr; char* ws = nullptr; size_t ws_bytes = 0;
   int* meta = nullptr; int meta_cap = 0;
   float* probe = nullptr;          // residual stream after every layer run, [runs][M][D], or null
+  // arrangement of the residual
+  int layer_norm = 0, streams = 0, in_taps = 0, res_gate = 0;     // streams 0: one stream that sublayers add to
+  bool arranged = false;           // the forward goes through streams.cuh
+  std::vector<Rope> ropes;
+  std::vector<void*> retired;      // tables replaced by longer ones (a captured graph may still read them)
+  void* hc = nullptr;              // [rows, D] what the mixer reads
+  float *gate = nullptr, *y = nullptr;                            // [rows, D] raw gates; result of a sublayer
+  float* gate_ws = nullptr; size_t gate_ws_bytes = 0;             // split-K slices of a gate
+  float* seg = nullptr; size_t seg_bytes = 0;                     // LightningArgs::seg_state
 };
 
 // what a cache of such a model keeps besides the lengths; owned by the root cache, shared by its views
@@ -64,6 +99,7 @@ struct Cache {
   int* table_dev = nullptr;
   std::vector<int> table, used;    // [slots][max_pages]; pages held by each slot
   std::vector<int> free_pages;
+  std::vector<void*> ring, in_ring;   // per layer run: inputs of the mixer's convolutions (attention), of the input convolution
 };
 
 inline int up8(int n) { return (n + 7) & ~7; }
@@ -93,12 +129,13 @@ struct Buffers {
   void *xc = nullptr, *z = nullptr, *dtb = nullptr; float *p = nullptr, *dt = nullptr;       // mamba
   float *dq = nullptr, *dk = nullptr, *dv = nullptr, *beta = nullptr, *g = nullptr, *gg = nullptr, *o = nullptr;   // delta
   void *low_a = nullptr, *low_g = nullptr;
+  void* lin = nullptr; float* ss = nullptr;      // lightning
 };
 constexpr int SPLIT_ROWS = 64, MAX_SPLITS = 16;   // key splits of the latent attention: forwards of few rows
 
 inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& A, Buffers& b) {
   A.off = 0;
-  A.take(&b.proj, M * std::max(L.n_in, hm.D) * 4);
+  A.take(&b.proj, M * std::max(std::max(L.n_in, hm.D), L.ff_plain ? L.ffp + hm.D : 0) * 4);
   A.take(&b.mix, M * (size_t)(L.kind == MAMBA1 ? L.inner : L.H * L.vd) * e);
   if (L.ff) A.take(&b.act, M * L.ffp * e);
   if (L.kind == LATENT) {
@@ -116,6 +153,15 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
     A.take(&b.dtb, M * L.dtp * e);
     A.take(&b.p, M * L.n_x * 4);
     A.take(&b.dt, M * L.inner * 4);
+  } else if (L.kind == ATTENTION) {
+    A.take(&b.q, M * L.H * L.P * e);
+    if (M <= SPLIT_ROWS) {
+      A.take(&b.part_o, (size_t)MAX_SPLITS * M * L.H * L.P * 4);
+      A.take(&b.part_ml, (size_t)MAX_SPLITS * M * L.H * 2 * 4);
+    }
+  } else if (L.kind == LIGHTNING) {
+    A.take(&b.lin, M * L.n_in * e);
+    A.take(&b.ss, M * L.H * ceil_div(L.vd, 64) * 4 * 4);
   } else {
     A.take(&b.dq, M * L.KH * L.d * 4);
     A.take(&b.dk, M * L.KH * L.d * 4);
@@ -127,6 +173,27 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
     A.take(&b.low_a, M * L.rap * e);
     A.take(&b.low_g, M * L.rgp * e);
   }
+}
+
+// Rotary frequencies f_i = base^(-2 i / dims).  With scaling (YaRN), pairs that turn slowly over the original context are
+// divided by `factor`, those that turn fast are kept, with a linear ramp between the two.
+inline Rope make_rope(const JsonValue& r) {
+  Rope out;
+  const int dims = (int)r.number("dims", 0);
+  const double base = r.number("base", 10000.0);
+  for (int i = 0; i < dims / 2; ++i) out.freq.push_back(pow(base, -2.0 * i / dims));
+  const JsonValue* s = r.find("scaling");
+  if (!s || s->kind != JsonValue::OBJ) return out;
+  const double factor = s->number("factor", 1), original = s->number("original", 1);
+  auto dim_of = [&](double turns) { return dims * log(original / (2 * M_PI * turns)) / (2 * log(base)); };
+  const double lo = std::max(floor(dim_of(s->number("fast", 32))), 0.0);
+  const double hi = std::min(ceil(dim_of(s->number("slow", 1))), dims - 1.0);
+  for (int i = 0; i < dims / 2; ++i) {
+    const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+    out.freq[i] = out.freq[i] / factor * ramp + out.freq[i] * (1 - ramp);
+  }
+  out.amp = (float)(0.1 * log(factor) + 1.0);
+  return out;
 }
 
 // ---- configuration ---------------------------------------------------------------------------------------------
@@ -141,6 +208,14 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
   hm->D = c->dim; hm->vocab = c->vocab;
   hm->eps = (float)j.number("norm_eps", 1e-6);
   hm->sinusoidal = j.text("positions") == "sinusoidal";
+  const std::string norm = j.text("norm");
+  VN_REQUIRE(ctx, norm.empty() || norm == "rms" || norm == "layer", "norm %s unknown (rms | layer)", norm.c_str());
+  hm->layer_norm = norm == "layer";
+  hm->streams = (int)j.number("streams", 0);
+  hm->in_taps = (int)j.number("input_conv", 0);
+  hm->res_gate = j.number("residual_gate", 0) != 0;
+  VN_REQUIRE(ctx, hm->streams >= 0 && hm->streams <= MAX_STREAMS && hm->in_taps >= 0, "streams (at most %d) or input_conv out of range", MAX_STREAMS);
+  hm->arranged = hm->layer_norm || hm->streams || hm->in_taps || hm->res_gate;
   const JsonValue* ls = j.find("layers");
   VN_REQUIRE(ctx, c->vocab > 0 && c->dim > 0 && ls && ls->kind == JsonValue::ARR && !ls->arr.empty(),
              "a composed model needs vocab_size, dim and layers");
@@ -149,12 +224,15 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
     HLayer L;
     const std::string t = l.text("mixer");
     auto I = [&](const char* k, int dflt = 0) { return (int)l.number(k, dflt); };
-    L.kind = t == "latent_attention" ? LATENT : t == "mamba1" ? MAMBA1 : t == "channel_delta" ? DELTA : -1;
-    VN_REQUIRE(ctx, L.kind >= 0, "layer %zu: mixer %s unknown (latent_attention | mamba1 | channel_delta)", i, t.c_str());
+    L.kind = t == "latent_attention" ? LATENT : t == "mamba1" ? MAMBA1 : t == "channel_delta" ? DELTA : t == "attention" ? ATTENTION
+             : t == "lightning" ? LIGHTNING : -1;
+    VN_REQUIRE(ctx, L.kind >= 0, "layer %zu: mixer %s unknown (latent_attention | attention | mamba1 | channel_delta | lightning)", i, t.c_str());
     L.ff = I("mlp_hidden");
     const std::string act = l.text("mlp_act");
-    VN_REQUIRE(ctx, !L.ff || act == "gelu_tanh" || act == "silu", "layer %zu: activation %s unknown (gelu_tanh | silu)", i, act.c_str());
+    VN_REQUIRE(ctx, !L.ff || act == "gelu_tanh" || act == "silu" || act == "relu2", "layer %zu: activation %s unknown (gelu_tanh | silu | relu2)", i, act.c_str());
     L.act = act == "gelu_tanh";
+    L.ff_plain = act == "relu2";
+    if (L.ff_plain || L.kind == LIGHTNING) hm->arranged = true;
     L.ffp = up8(L.ff);
     L.H = I("heads"); L.d = I("dim"); L.vd = I("vdim"); L.taps = I("conv", 1);
     if (L.kind == LATENT) {
@@ -168,6 +246,34 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
       L.dtp = up8(L.dt_rank);
       L.n_in = 2 * L.inner;
       L.n_x = up8(L.dtp + 2 * L.nstate);
+    } else if (L.kind == ATTENTION) {
+      L.KH = I("kv_heads"); L.window = I("window"); L.scale = (float)l.number("scale", 0); L.kv_from = I("kv_from", -1);
+      L.gated = l.number("output_gate", 0) != 0;
+      L.conv_named = l.find("conv") && l.find("conv")->kind == JsonValue::NUM;
+      if (const JsonValue* r = l.find("rope"))
+        if (r->kind == JsonValue::OBJ) {
+          const Rope rope = make_rope(*r);
+          L.rd = 2 * (int)rope.freq.size();
+          for (size_t k = 0; k < hm->ropes.size() && L.rope < 0; ++k)
+            if (hm->ropes[k].freq == rope.freq && hm->ropes[k].amp == rope.amp) L.rope = (int)k;
+          if (L.rope < 0) { L.rope = (int)hm->ropes.size(); hm->ropes.push_back(rope); }
+        }
+      VN_REQUIRE(ctx, L.H > 0 && L.KH > 0 && L.H % L.KH == 0 && L.d > 0 && L.vd > 0 && L.d <= 1024 && L.vd <= 1024 && L.rd <= L.d &&
+                 L.window >= 0 && L.taps >= 1, "layer %zu: attention sizes", i);
+      if (L.kv_from >= 0) {
+        VN_REQUIRE(ctx, L.kv_from < (int)i, "layer %zu: keys and values of layer %d, which does not run before it", i, L.kv_from);
+        const HLayer& src = hm->layers[L.kv_from];
+        VN_REQUIRE(ctx, src.kind == ATTENTION && src.kv_from < 0 && src.KH == L.KH && src.d == L.d && src.vd == L.vd,
+                   "layer %zu: keys and values of layer %d have other sizes, or are not its own", i, L.kv_from);
+      }
+      L.P = attn_pitch(std::max(L.d, L.vd));
+      L.n_in = up8(L.conv_ch() + (L.gated ? L.H * L.vd : 0));
+    } else if (L.kind == LIGHTNING) {
+      const JsonValue* dec = l.find("decay");
+      VN_REQUIRE(ctx, L.H > 0 && L.d > 0 && L.d <= 512 && L.vd > 0 && dec && dec->kind == JsonValue::ARR && (int)dec->arr.size() == L.H,
+                 "layer %zu: lightning attention sizes, or not one decay per head", i);
+      for (auto& v : dec->arr) L.decay.push_back(v.num);
+      L.n_in = up8(2 * L.H * (L.d + L.vd));
     } else {
       L.KH = I("kv_heads"); L.ra = I("decay_rank"); L.rg = I("gate_rank");
       VN_REQUIRE(ctx, L.H > 0 && L.KH > 0 && L.H % L.KH == 0 && L.d > 0 && L.d <= 256 && L.vd > 0 && L.vd <= 512 && L.ra > 0 &&
@@ -188,10 +294,17 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
     }
   }
   const int a = hm->loop_times ? hm->loop_start : n, b = hm->loop_times ? hm->loop_stop : n;
-  for (int i = 0; i < a; ++i) hm->runs.push_back({i, -1});
+  std::vector<int> last(n, -1);           // latest run of a layer
+  auto run = [&](int i, int t) {
+    const int from = hm->layers[i].kv_from;
+    last[i] = (int)hm->runs.size();
+    hm->runs.push_back({i, t, from < 0 ? last[i] : last[from]});
+  };
+  for (int i = 0; i < a; ++i) run(i, -1);
   for (int t = 0; t < hm->loop_times; ++t)
-    for (int i = a; i < b; ++i) hm->runs.push_back({i, t});
-  for (int i = b; i < n; ++i) hm->runs.push_back({i, -1});
+    for (int i = a; i < b; ++i) run(i, t);
+  for (int i = b; i < n; ++i) run(i, -1);
+  VN_REQUIRE(ctx, !hm->arranged || !hm->loop_times, "a looped block needs the plain residual");
   return VN_OK;
 }
 
@@ -239,6 +352,32 @@ int32_t alloc(vn_model* m) {
       TRY(F(&L.f_a, L.R));
       TRY(F(&L.f_b, L.H));
       need({"mix.q", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv", "mix.sink", "mix.g"});
+    } else if (L.kind == ATTENTION) {
+      TRY(W(&L.w_o, D * L.H * L.vd));
+      TRY(F(&L.conv, (size_t)L.conv_ch() * L.taps));
+      if (!L.conv_named) {                                 // one tap of weight 1: the projection itself
+        const std::vector<float> unit(L.conv_ch(), 1.f);
+        TRY(upload(m, unit.data(), L.conv, 1, L.conv_ch(), L.conv_ch(), 1, 0, true));
+      }
+      need({"mix.q"});
+      if (L.kv_from < 0) need({"mix.k", "mix.v"});
+      if (L.gated) need({"mix.g"});
+      if (L.conv_named) need({"mix.q.conv"});
+      if (L.conv_named && L.kv_from < 0) need({"mix.k.conv", "mix.v.conv"});
+    } else if (L.kind == LIGHTNING) {
+      TRY(W(&L.w_o, D * L.H * L.vd));
+      TRY(F(&L.f_a, (size_t)L.H * L.vd));
+      TRY(F(&L.f_b, (size_t)2 * L.H));
+      TRY(F(&L.f_c, (size_t)65 * L.H));
+      std::vector<float> dec, pw;
+      for (double v : L.decay) {
+        dec.push_back((float)v);
+        dec.push_back((float)(v - (double)dec.back()));
+        for (int k = 0; k <= 64; ++k) pw.push_back((float)pow(v, k));
+      }
+      TRY(upload(m, dec.data(), L.f_b, 1, (long long)dec.size(), (long long)dec.size(), 1, 0, true));
+      TRY(upload(m, pw.data(), L.f_c, 1, (long long)pw.size(), (long long)pw.size(), 1, 0, true));
+      need({"mix.q", "mix.k", "mix.v", "mix.g", "mix.norm"});
     } else if (L.kind == MAMBA1) {
       TRY(W(&L.w_uk, (size_t)L.inner * L.dtp));
       TRY(W(&L.w_uv, (size_t)L.n_x * L.inner));
@@ -261,10 +400,32 @@ int32_t alloc(vn_model* m) {
             "mix.a2", "mix.dt_bias", "mix.g1", "mix.g2"});
     }
     if (L.ff) {
+      const bool stacked = L.ff_plain && hm.res_gate;          // up | gate of the result: both read the same rows
       TRY(F(&L.norm2, D));
-      TRY(W(&L.w_gu, (size_t)2 * L.ffp * D));
+      TRY(W(&L.w_gu, (size_t)(L.ff_plain ? L.ffp + (stacked ? D : 0) : 2 * L.ffp) * D));
       TRY(W(&L.w_down, D * L.ffp));
-      need({"norm2", "mlp.gate", "mlp.up", "mlp.down"});
+      need({"norm2", "mlp.up", "mlp.down"});
+      if (!L.ff_plain) need({"mlp.gate"});
+      if (stacked) L.w_rg[1] = (char*)L.w_gu + (size_t)L.ffp * D * e;
+    }
+    for (int q = 0; q < (L.ff ? 2 : 1); ++q) {
+      const std::string k = std::to_string(q + 1);
+      if (hm.streams) {
+        TRY(F(&L.hc_in[q], hm.streams));
+        TRY(F(&L.hc_out[q], hm.streams));
+        TRY(F(&L.hc_mix[q], hm.streams * hm.streams));
+        for (const char* part : {".in", ".out", ".mix"}) hm.want.insert(p + "hc" + k + part);
+      }
+      if (hm.res_gate) {
+        if (!L.w_rg[q]) TRY(W(&L.w_rg[q], D * D));
+        TRY(F(&L.rg_b[q], D));
+        hm.want.insert(p + "rg" + k);
+        hm.want.insert(p + "rg" + k + ".b");
+      }
+    }
+    if (hm.in_taps) {
+      TRY(F(&L.in_conv, D * hm.in_taps));
+      need({"canon1"});
     }
   }
   return VN_OK;
@@ -276,9 +437,14 @@ void destroy(vn_model* m) {
   Model& hm = *m->hyb;
   for (auto& L : hm.layers) {
     F(L.norm1); F(L.norm2); F(L.w_in); F(L.w_o); F(L.w_uk); F(L.w_uv); F(L.f_a); F(L.f_b); F(L.f_c); F(L.conv); F(L.conv_b);
-    F(L.w_gu); F(L.w_down);
+    if (!(L.ff_plain && hm.res_gate)) F(L.w_rg[1]);            // else part of w_gu
+    F(L.w_gu); F(L.w_down); F(L.w_rg[0]); F(L.in_conv);
+    for (int q = 0; q < 2; ++q) { F(L.hc_in[q]); F(L.hc_out[q]); F(L.hc_mix[q]); F(L.rg_b[q]); }
   }
+  for (Rope& r : hm.ropes) F(r.table);
+  for (void* t : hm.retired) F(t);
   F(hm.w_loop); F(hm.loop_step); F(hm.freq); F(hm.x0); F(hm.cat); F(hm.ws); F(hm.meta);
+  F(hm.hc); F(hm.gate); F(hm.y); F(hm.gate_ws); F(hm.seg);
   delete m->hyb;
   m->hyb = nullptr;
 }
