@@ -475,21 +475,52 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
   auto rate = [](float a) { return expf(a); };
   auto neg_rate = [](float a) { return -expf(a); };
   if (!hm.want.count(n)) return vn_fail(ctx, VN_ERR_INVALID, "unexpected tensor %s", n.c_str());
+  auto weight = [&](float* dst, long long count) {        // a norm's: around zero (rms) or plain (layer)
+    return hm.layer_norm ? f32(data, dst, count) : mapped(dst, count, one_plus);
+  };
 #define PUT(er, ec, expr) do { if (!shape((er), (ec))) return st; TRY(expr); return VN_OK; } while (0)
   if (n == "embed") PUT(hm.vocab, D, rows(m->emb, D));
   if (n == "head") PUT(hm.vocab, D, rows(m->head, D));
-  if (n == "final.norm") PUT(D, 1, mapped(m->norm_f, D, one_plus));
+  if (n == "final.norm") PUT(D, 1, weight(m->norm_f, D));
   if (n == "loop.in") PUT(D, 2 * D, rows(hm.w_loop, 2 * D));
   if (n == "loop.step") PUT(hm.loop_times, D, f32(data, hm.loop_step, r * cl));
   const size_t dot = n.find('.');
   HLayer& L = hm.layers[atoi(n.substr(1, dot - 1).c_str())];      // the name is in `want`: the layer exists
   const std::string s = n.substr(dot + 1);
-  if (s == "norm1") PUT(D, 1, mapped(L.norm1, D, one_plus));
-  if (s == "norm2") PUT(D, 1, mapped(L.norm2, D, one_plus));
+  if (s == "norm1") PUT(D, 1, weight(L.norm1, D));
+  if (s == "norm2") PUT(D, 1, weight(L.norm2, D));
   if (s == "mlp.gate") PUT(L.ff, D, rows(L.w_gu, D, 0, 2));
+  if (s == "mlp.up" && L.ff_plain) PUT(L.ff, D, rows(L.w_gu, D));
   if (s == "mlp.up") PUT(L.ff, D, rows(L.w_gu, D, 1, 2));
   if (s == "mlp.down") PUT(D, L.ff, rows(L.w_down, L.ffp));
-  if (L.kind == LATENT) {
+  if (s == "canon1") PUT(D, hm.in_taps, f32(data, L.in_conv, r * cl));
+  for (int q = 0; q < 2; ++q) {
+    const std::string k = std::to_string(q + 1);
+    if (s == "hc" + k + ".in") PUT(hm.streams, 1, f32(data, L.hc_in[q], r));
+    if (s == "hc" + k + ".out") PUT(hm.streams, 1, f32(data, L.hc_out[q], r));
+    if (s == "hc" + k + ".mix") PUT(hm.streams, hm.streams, f32(data, L.hc_mix[q], r * cl));
+    if (s == "rg" + k) PUT(D, D, rows(L.w_rg[q], D));
+    if (s == "rg" + k + ".b") PUT(D, 1, f32(data, L.rg_b[q], D));
+  }
+  if (L.kind == ATTENTION) {
+    const long long qd = (long long)L.H * L.d, kd = (long long)L.KH * L.d, vd = (long long)L.KH * L.vd, hv = (long long)L.H * L.vd;
+    if (s == "mix.q") PUT(qd, D, rows(L.w_in, D));
+    if (s == "mix.k") PUT(kd, D, rows(L.w_in, D, qd));
+    if (s == "mix.v") PUT(vd, D, rows(L.w_in, D, qd + kd));
+    if (s == "mix.g") PUT(hv, D, rows(L.w_in, D, L.conv_ch()));
+    if (s == "mix.q.conv") PUT(qd, L.taps, f32(data, L.conv, r * cl));
+    if (s == "mix.k.conv") PUT(kd, L.taps, f32(data, L.conv + qd * L.taps, r * cl));
+    if (s == "mix.v.conv") PUT(vd, L.taps, f32(data, L.conv + (qd + kd) * L.taps, r * cl));
+    if (s == "mix.o") PUT(D, hv, rows(L.w_o, hv));
+  } else if (L.kind == LIGHTNING) {
+    const long long qd = (long long)L.H * L.d, hv = (long long)L.H * L.vd;
+    if (s == "mix.q") PUT(qd, D, rows(L.w_in, D));
+    if (s == "mix.k") PUT(qd, D, rows(L.w_in, D, qd));
+    if (s == "mix.v") PUT(hv, D, rows(L.w_in, D, 2 * qd));
+    if (s == "mix.g") PUT(hv, D, rows(L.w_in, D, 2 * qd + hv));
+    if (s == "mix.norm") PUT(hv, 1, f32(data, L.f_a, r));
+    if (s == "mix.o") PUT(D, hv, rows(L.w_o, hv));
+  } else if (L.kind == LATENT) {
     const long long hd = (long long)L.H * L.d, hv = (long long)L.H * L.vd;
     if (s == "mix.q") PUT(hd, D, rows(L.w_in, D));
     if (s == "mix.dkv") PUT(L.R, D, rows(L.w_in, D, hd));
@@ -556,14 +587,19 @@ int32_t ensure(vn_model* m, int M) {
   Model& hm = *m->hyb;
   VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
   m->cap_rows = 0;
-  void** bufs[] = {(void**)&m->x, &m->h, (void**)&m->row_seg, (void**)&hm.x0, &hm.cat, (void**)&hm.ws};
+  void** bufs[] = {(void**)&m->x, &m->h, (void**)&m->row_seg, (void**)&hm.x0, &hm.cat, (void**)&hm.ws, &hm.hc, (void**)&hm.gate, (void**)&hm.y};
   for (void** b : bufs) { if (*b) cudaFree(*b); *b = nullptr; }
   const size_t R = (size_t)M + (M >> 2) + 32, D = hm.D, e = m->esz;
-  TRY(dev_alloc(ctx, (void**)&m->x, R * D * 4));
+  TRY(dev_alloc(ctx, (void**)&m->x, R * D * 4 * std::max(1, hm.streams)));
   TRY(dev_alloc(ctx, &m->h, R * D * e));
   m->row_seg_cap = (int)(R / 256 + 2);
   TRY(dev_alloc(ctx, (void**)&m->row_seg, (size_t)2 * m->row_seg_cap * sizeof(int)));
   TRY(dev_alloc(ctx, (void**)&hm.x0, R * D * 4));
+  if (hm.arranged) {
+    TRY(dev_alloc(ctx, &hm.hc, R * D * e));
+    TRY(dev_alloc(ctx, (void**)&hm.gate, R * D * 4));
+    TRY(dev_alloc(ctx, (void**)&hm.y, R * D * 4));
+  }
   if (hm.loop_times) TRY(dev_alloc(ctx, &hm.cat, R * 2 * D * e));
   size_t need = 0;
   for (auto& L : hm.layers)
@@ -589,17 +625,27 @@ GemmArgs gemm_args(const void* A, int lda, const void* W, int N, int K, int M, c
   return g;
 }
 // out = A W^T in fp32: split-K slices in the workspace, or the matrix `direct`
-int32_t project(vn_model* m, GemmArgs g, float* direct, Src* out) {
+int32_t project(vn_model* m, GemmArgs g, float* direct, Src* out, bool gate = false) {
   *out = Src();
   out->ld = g.N;
   if (tc_rows(m, g)) {
     int sp = 1;
-    TRY(tc_partial(m, g, g.M, g.M, &sp));
+    // a gate's slices outlive the projections that follow it: they have a workspace of their own
+    auto other = [&] { if (gate) { std::swap(m->partial, m->hyb->gate_ws); std::swap(m->partial_bytes, m->hyb->gate_ws_bytes); } };
+    other();
+    const int32_t st = tc_partial(m, g, g.M, g.M, &sp);
     out->p = m->partial; out->splits = sp; out->pstride = (long long)g.M * g.N;
-    return VN_OK;
+    other();
+    return st;
   }
   g.C = direct; g.ldc = g.N;
   out->p = direct;
+  return linear(m, g);
+}
+// the same in 16 bits (many rows), with the GEMM's own function on some columns
+int32_t project(vn_model* m, GemmArgs g, float* direct, Mat<__nv_bfloat16>* out, bool = false) {
+  g.C = direct; g.ldc = g.N; g.c_bf16 = 1;
+  out->p = (const __nv_bfloat16*)direct; out->ld = g.N;
   return linear(m, g);
 }
 // x += A W^T; then h = RMSNorm(x) * next_norm when given
@@ -634,13 +680,13 @@ int32_t batched(vn_model* m, const GemmArgs& g) {
   return launch_gemm_simt<float, float>(m->ctx, g);
 }
 
-// ---- mixers: m->h -> the input of the output projection -----------------------------------------------------------
+// ---- mixers: normalised rows -> the input of the output projection -----------------------------------------------------------
 template <typename T>
-int32_t latent_attention(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+int32_t latent_attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
   vn_ctx* ctx = m->ctx;
   const int M = rows.M, D = m->hyb->D, H = L.H;
   Src s;
-  TRY(project(m, gemm_args(m->h, D, L.w_in, L.n_in, D, M, "gemm_latent_in"), b.proj, &s));
+  TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_latent_in"), b.proj, &s));
   VN_LAUNCH(ctx, latent_append_kernel<T>, M, 256, (size_t)L.R * 4, s, H, L.d, L.dp, L.R, L.Rp, L.f_a, m->hyb->eps, (T*)b.q,
             b.gate, (T*)kv->k[run], hc.table_dev, hc.max_pages, rows);
   GemmArgs g = gemm_args(b.q, H * L.dp, L.w_uk, L.Rp, L.dp, M, "gemm_latent_uk");
@@ -672,11 +718,11 @@ ConvIn<T> conv_in(const HLayer& L, const Cache& hc, const Src& s, void* ring) {
 }
 
 template <typename T>
-int32_t mamba1(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+int32_t mamba1(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
   vn_ctx* ctx = m->ctx;
   const int M = rows.M, D = m->hyb->D, n = L.inner;
   Src s;
-  TRY(project(m, gemm_args(m->h, D, L.w_in, L.n_in, D, M, "gemm_mamba_in"), b.proj, &s));
+  TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_mamba_in"), b.proj, &s));
   const ConvIn<T> cv = conv_in<T>(L, hc, s, kv->k[run]);
   if (rows.max_n == 1)
     VN_LAUNCH(ctx, (mamba_conv_kernel<T, 1>), dim3(ceil_div(n, 32), ceil_div(M, 8)), dim3(32, 8), 0, cv, rows, (T*)b.xc, (T*)b.z, hc.pending);
@@ -707,11 +753,11 @@ int32_t mamba1(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, cons
 }
 
 template <typename T>
-int32_t channel_delta(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+int32_t channel_delta(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
   vn_ctx* ctx = m->ctx;
   const int M = rows.M, D = m->hyb->D, H = L.H, KH = L.KH, d = L.d, vd = L.vd;
   Src s;
-  TRY(project(m, gemm_args(m->h, D, L.w_in, L.n_in, D, M, "gemm_delta_in"), b.proj, &s));
+  TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_delta_in"), b.proj, &s));
   const ConvIn<T> cv = conv_in<T>(L, hc, s, kv->k[run]);
   DeltaIn in;
   in.src = s; in.H = H; in.KH = KH; in.d = d; in.vd = vd; in.ra = L.ra; in.rg = L.rg; in.ra_ld = L.rap; in.rg_ld = L.rgp;
@@ -743,6 +789,82 @@ int32_t channel_delta(vn_model* m, vn_kv* kv, Cache& hc, const HLayer& L, int ru
   const long long nh = (long long)M * H;
   VN_LAUNCH(ctx, delta_out_kernel<T>, (unsigned)ceil_div(nh, 8ll), 256, 0, b.o, b.gg, L.f_a, (T*)b.mix, nh, vd, m->hyb->eps);
   return VN_OK;
+}
+
+// Grouped-query attention.  S: Src, or the 16-bit matrix of a forward of many rows
+template <typename T, typename S>
+int32_t attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+  vn_ctx* ctx = m->ctx;
+  const Model& hm = *m->hyb;
+  const int M = rows.M, D = hm.D, from = hm.runs[run].kv_run;
+  ConvIn<T, S, false> cv;
+  TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_attn_in"), b.proj, &cv.src));
+  cv.ring = (T*)hc.ring[run]; cv.RC = L.taps - 1 + hc.pending; cv.C = L.conv_ch(); cv.taps = L.taps; cv.w = L.conv;
+  PagedAttnArgs a;
+  a.H = L.H; a.KH = L.KH; a.d = L.d; a.vd = L.vd; a.P = L.P; a.window = L.window; a.scale = L.scale; a.rd = L.rd;
+  a.rope = L.rope >= 0 ? hm.ropes[L.rope].table : nullptr;
+  a.own_kv = from == run;
+  a.kplane = kv->k[from]; a.vplane = kv->v[from]; a.table = hc.table_dev; a.max_pages = hc.max_pages;
+  a.col_g = L.gated ? L.conv_ch() : -1;
+  a.q = b.q; a.out = b.mix; a.pending = hc.pending; a.rows = rows;
+  const bool mma = m->cfg.bf16 && attn_mma_ok(L.P) && !m->force_simt_attn;
+  if constexpr (std::is_same<T, __nv_bfloat16>::value && std::is_same<S, Src>::value) {
+    if (mma && rows.max_n == 1) {
+      const int ctas = L.KH * ceil_div(L.H / L.KH, 16) * M, keys = L.window > 0 ? std::min(L.window, kv->max_seq) : kv->max_seq;
+      a.splits = M > SPLIT_ROWS ? 1 : std::max(1, std::min(std::min(MAX_SPLITS, ceil_div(keys, 64)), 2 * ctx->sm_count / ctas));
+      a.part_o = b.part_o; a.part_ml = b.part_ml;
+      TRY(vn_tickets(ctx, &a.tickets));
+      return vn_attn_step(ctx, cv, a);
+    }
+  }
+  TRY(vn_attn_inputs(ctx, cv, a));
+  if (rows.max_n > hc.pending && L.taps > 1)
+    VN_LAUNCH(ctx, (conv_tail_kernel<T, S, false>), dim3(ceil_div(cv.C, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
+  return vn_paged_attention<T, S>(ctx, cv.src, a, mma);
+}
+
+// Lightning attention; its output still has to be divided by the root mean square that b.ss [M, *n_ss] gives
+template <typename T, typename S>
+int32_t lightning(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b, int* n_ss) {
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  const int M = rows.M, D = hm.D, n_act = L.H * (2 * L.d + L.vd);
+  const LightningPlan plan = vn_lightning_plan(ctx, m->cfg.bf16 != 0, L.H, L.d, L.vd, rows, hc.pending);
+  LightningArgs a;
+  a.H = L.H; a.d = L.d; a.vd = L.vd; a.decay = L.f_b; a.powers = L.f_c; a.norm_w = L.f_a; a.state = (float*)kv->v[run]; a.R = hc.ring_len;
+  a.out = b.mix; a.ss = b.ss; a.n_ss = *n_ss = plan.n_ss; a.segments = plan.segments; a.seg_len = plan.seg_len; a.rows = rows;
+  if (plan.seg_bytes > hm.seg_bytes) {
+    VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    if (hm.seg) cudaFree(hm.seg);
+    hm.seg = nullptr; hm.seg_bytes = 0;
+    TRY(dev_alloc(ctx, (void**)&hm.seg, plan.seg_bytes));
+    hm.seg_bytes = plan.seg_bytes;
+  }
+  a.seg_state = hm.seg;
+  GemmArgs g = gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_lightning_in");
+  S s;
+  if constexpr (std::is_same<S, Src>::value) {
+    TRY(project(m, g, b.proj, &s));
+    if constexpr (std::is_same<T, __nv_bfloat16>::value) {
+      if (plan.chunked) {
+        Mat<T> act;
+        act.p = (const T*)b.lin; act.ld = L.n_in;
+        const long long total4 = (long long)M * L.n_in / 4;
+        if (n_act % 4 == 0)
+          VN_LAUNCH(ctx, slices_act_kernel<T>, (unsigned)ceil_div(total4, 256ll), 256, 0, s, L.n_in, n_act, (int)POST_SILU, (T*)b.lin, L.n_in,
+                    (float*)nullptr, total4);
+        else
+          VN_LAUNCH(ctx, slices_act1_kernel<T>, (unsigned)ceil_div(total4 * 4, 256ll), 256, 0, s, L.n_in, n_act, (int)POST_SILU, (T*)b.lin, total4 * 4);
+        return vn_lightning_chunks(ctx, act, a);
+      }
+    }
+    return vn_lightning_scan<T, S>(ctx, s, a);
+  } else {
+    g.post = POST_SILU; g.post_n = n_act;
+    TRY(project(m, g, b.proj, &s));
+    a.activated = 1;
+    return plan.chunked ? vn_lightning_chunks(ctx, s, a) : vn_lightning_scan<T, S>(ctx, s, a);
+  }
 }
 
 // ---- the forward ---------------------------------------------------------------------------------------------------
