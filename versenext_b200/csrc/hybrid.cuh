@@ -93,7 +93,7 @@ struct Model {
 
 // what a cache of such a model keeps besides the lengths; owned by the root cache, shared by its views
 struct Cache {
-  int pending = 1, ring = 2;       // rows that can be appended and cut back; state snapshots per sequence
+  int pending = 1, ring_len = 2;   // rows that can be appended and cut back; state snapshots per sequence
   bool pooled = false;
   int max_pages = 0, n_pages = 0, slots = 0;
   int* table_dev = nullptr;
@@ -733,7 +733,7 @@ int32_t mamba1(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLa
   MambaArgs a;
   TRY(project(m, gemm_args(b.xc, n, L.w_uv, L.n_x, n, M, "gemm_mamba_x"), b.p, &a.p));
   a.xc = b.xc; a.z = b.z; a.dt_cols = L.dtp; a.dt_rank = L.dt_rank; a.w_dt = L.w_uk; a.dt_bias = L.f_c; a.A = L.f_a; a.D = L.f_b;
-  a.state = (float*)kv->v[run]; a.R = hc.ring; a.inner = n; a.nstate = L.nstate; a.out = b.mix; a.rows = rows;
+  a.state = (float*)kv->v[run]; a.R = hc.ring_len; a.inner = n; a.nstate = L.nstate; a.out = b.mix; a.rows = rows;
   if (rows.max_n == 1) {
     if (M >= 16 && a.p.splits > 1) {     // many rows: the slices are summed once, not by every CTA of a row
       VN_LAUNCH(ctx, splitk_store_kernel, (unsigned)ceil_div((long long)M * L.n_x, 256ll), 256, 0, a.p.p, a.p.splits, a.p.pstride,
@@ -767,7 +767,7 @@ int32_t channel_delta(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, co
   if (rows.max_n == 1) {
     DeltaStepArgs<T> a;
     a.conv = cv; a.in = in; a.w_a = (const T*)L.w_uk; a.w_g = (const T*)L.w_uv; a.decay_rate = L.f_b; a.dt_bias = L.f_c;
-    a.norm_w = L.f_a; a.state = (float*)kv->v[run]; a.R = hc.ring; a.eps = m->hyb->eps; a.out = (T*)b.mix;
+    a.norm_w = L.f_a; a.state = (float*)kv->v[run]; a.R = hc.ring_len; a.eps = m->hyb->eps; a.out = (T*)b.mix;
     TRY(vn_delta_step(ctx, a));
     return VN_OK;
   }
@@ -784,7 +784,7 @@ int32_t channel_delta(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, co
   TRY(linear(m, g));
   DeltaRuleArgs a;
   a.q = b.dq; a.k = b.dk; a.v = b.dv; a.g = b.g; a.beta = b.beta; a.o = b.o; a.state = (float*)kv->v[run];
-  a.R = hc.ring; a.H = H; a.KH = KH; a.d = d; a.vd = vd; a.rows = rows;
+  a.R = hc.ring_len; a.H = H; a.KH = KH; a.d = d; a.vd = vd; a.rows = rows;
   TRY(vn_delta_scan(ctx, a));
   const long long nh = (long long)M * H;
   VN_LAUNCH(ctx, delta_out_kernel<T>, (unsigned)ceil_div(nh, 8ll), 256, 0, b.o, b.gg, L.f_a, (T*)b.mix, nh, vd, m->hyb->eps);
@@ -871,6 +871,161 @@ int32_t lightning(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const 
 // where the output rows come from: all rows, the entries' last rows of a uniform batch, or a list (device)
 struct Pick { const int* list = nullptr; int n = 0, mul = 1, add = 0; };
 
+// final norm's rows in m->h -> logits
+int32_t head(vn_model* m, int n_rows, float* out_logits) {
+  const Model& hm = *m->hyb;
+  GemmArgs g = gemm_args(m->h, hm.D, m->head, hm.vocab, hm.D, n_rows, "gemm_head");
+  g.C = out_logits; g.ldc = hm.vocab;
+  if (tc_rows(m, g)) {
+    TcPlan direct;
+    direct.error_flag = m->tc_error;
+    return tc_launch(m->ctx, g, n_rows, direct);
+  }
+  return linear(m, g);
+}
+
+// act = f(h W_gate^T) * (h W_up^T) of a gated feed-forward
+template <typename T>
+int32_t gated_up(vn_model* m, const HLayer& L, int M, const Buffers& b) {
+  vn_ctx* ctx = m->ctx;
+  const int D = m->hyb->D;
+  GemmArgs g = gemm_args(m->h, D, L.w_gu, 2 * L.ffp, D, M, "gemm_ff_gateup");
+  if (tc_rows(m, g)) {
+    int sp = 1;
+    TRY(tc_partial(m, g, M, M, &sp));
+    const long long pairs = (long long)M * L.ffp;
+    VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp,
+                      (long long)M * 2 * L.ffp, (T*)b.act, 2 * L.ffp, pairs, L.act);
+    return VN_OK;
+  }
+  g.C = b.act; g.ldc = L.ffp; g.epi = EPI_SWIGLU; g.act = L.act; g.c_bf16 = m->cfg.bf16;
+  return linear(m, g);
+}
+
+// act = relu(h W_up^T)^2, and the raw gate of the result beside it when the model has one
+template <typename T>
+int32_t plain_up(vn_model* m, const HLayer& L, int M, const Buffers& b, Src* gate) {
+  vn_ctx* ctx = m->ctx;
+  const Model& hm = *m->hyb;
+  const int D = hm.D, n = L.ffp + (hm.res_gate ? D : 0);
+  Src s;
+  TRY(project(m, gemm_args(m->h, D, L.w_gu, n, D, M, "gemm_ff_up"), b.proj, &s));
+  if (n % 4 == 0) {
+    const long long total4 = (long long)M * n / 4;
+    VN_LAUNCH_PDL_BIT(ctx, 8, slices_act_kernel<T>, (unsigned)ceil_div(total4, 256ll), 256, 0, s, n, L.ffp, (int)POST_RELU2, (T*)b.act,
+                      L.ffp, hm.gate, total4);
+    if (hm.res_gate) { *gate = Src(); gate->p = hm.gate; gate->ld = D; }
+  } else {                                               // a plain matrix: the gate is read where it stands
+    const long long total = (long long)M * L.ffp;
+    VN_LAUNCH(ctx, slices_act1_kernel<T>, (unsigned)ceil_div(total, 256ll), 256, 0, s, L.ffp, L.ffp, (int)POST_RELU2, (T*)b.act, total);
+    *gate = s;
+    gate->p = s.p + L.ffp;
+  }
+  return VN_OK;
+}
+template <typename T>
+int32_t plain_up(vn_model* m, const HLayer& L, int M, const Buffers& b, Mat<__nv_bfloat16>* gate) {
+  const Model& hm = *m->hyb;
+  GemmArgs g = gemm_args(m->h, hm.D, L.w_gu, L.ffp, hm.D, M, "gemm_ff_up");
+  g.C = b.act; g.ldc = L.ffp; g.c_bf16 = 1; g.post = POST_RELU2; g.post_n = L.ffp;
+  TRY(linear(m, g));
+  return hm.res_gate ? project(m, gemm_args(m->h, hm.D, L.w_rg[1], hm.D, hm.D, M, "gemm_result_gate"), hm.gate, gate) : VN_OK;
+}
+
+// The forward over an arrangement of residual streams.  S: type of the projections' results
+template <typename T, typename S>
+int32_t forward_arranged(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows, const Pick& pick, float* out_hidden,
+                         float* out_logits) {
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  Cache& hc = *kv->hyb;
+  const int M = rows.M, D = hm.D, n_runs = (int)hm.runs.size();
+  const bool single = rows.max_n == 1;
+  struct Sub { int run, q; };
+  std::vector<Sub> subs;
+  for (int i = 0; i < n_runs; ++i) {
+    subs.push_back({i, 0});
+    if (hm.layers[hm.runs[i].layer].ff) subs.push_back({i, 1});
+  }
+  VN_LAUNCH(ctx, embed_pos_kernel<T>, M, 256, 0, (const long long*)tokens, (const T*)m->emb, hm.freq, m->x, hm.x0, rows, D,
+            hm.vocab, m->status);
+  StreamArgs<T, S> base;
+  base.x = m->x; base.ns = std::max(1, hm.streams); base.D = D; base.layer_norm = hm.layer_norm; base.eps = hm.eps; base.rows = rows;
+  // what a pass over the streams reads off for the next sublayer, or for the head when all rows go there in order
+  const bool all_out = pick.n == M && !pick.list && pick.mul == 1 && pick.add == 0;
+  auto next = [&](StreamArgs<T, S>& a, size_t k) {
+    if (k < subs.size()) {
+      const HLayer& L = hm.layers[hm.runs[subs[k].run].layer];
+      const int q = subs[k].q;
+      a.in = L.hc_in[q]; a.norm_w = q ? L.norm2 : L.norm1; a.h = (T*)m->h;
+      if (!q && hm.in_taps && single) {
+        a.hc = (T*)hm.hc; a.ring = (T*)hc.in_ring[subs[k].run]; a.conv_w = L.in_conv; a.taps = hm.in_taps;
+        a.RC = hm.in_taps - 1 + hc.pending;
+      }
+    } else if (all_out) {
+      a.norm_w = m->norm_f; a.h = (T*)m->h; a.h32 = out_hidden;
+    }
+  };
+  {
+    StreamArgs<T, S> a = base;
+    a.first = hm.x0;
+    next(a, 0);
+    TRY(vn_streams(ctx, a, M));
+  }
+  for (size_t k = 0; k < subs.size(); ++k) {
+    const int i = subs[k].run, q = subs[k].q;
+    const HLayer& L = hm.layers[hm.runs[i].layer];
+    Arena A;
+    Buffers b;
+    A.base = hm.ws;
+    layout(hm, L, M, m->esz, A, b);
+    StreamArgs<T, S> a = base;
+    if (k == 0) a.first = hm.x0;
+    if (hm.res_gate && !(q && L.ff_plain))
+      TRY(project(m, gemm_args(m->h, D, L.w_rg[q], D, D, M, "gemm_result_gate"), hm.gate, &a.gate, true));
+    GemmArgs out;
+    if (!q) {
+      const void* in_rows = m->h;
+      if (hm.in_taps) {
+        in_rows = hm.hc;
+        if (!single) {
+          ConvIn<T, Mat<T>, false> cv;
+          cv.src.p = (const T*)m->h; cv.src.ld = D; cv.ring = (T*)hc.in_ring[i]; cv.RC = hm.in_taps - 1 + hc.pending; cv.C = D;
+          cv.taps = hm.in_taps; cv.w = L.in_conv;
+          TRY(vn_input_conv(ctx, cv, rows, hc.pending, (T*)hm.hc));
+          if (rows.max_n > hc.pending && hm.in_taps > 1)
+            VN_LAUNCH(ctx, (conv_tail_kernel<T, Mat<T>, false>), dim3(ceil_div(D, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
+        }
+      }
+      if (L.kind == LATENT) TRY(latent_attention<T>(m, in_rows, kv, hc, L, i, rows, b));
+      else if (L.kind == MAMBA1) TRY(mamba1<T>(m, in_rows, kv, hc, L, i, rows, b));
+      else if (L.kind == DELTA) TRY(channel_delta<T>(m, in_rows, kv, hc, L, i, rows, b));
+      else if (L.kind == ATTENTION) TRY((attention<T, S>(m, in_rows, kv, hc, L, i, rows, b)));
+      else {
+        TRY((lightning<T, S>(m, in_rows, kv, hc, L, i, rows, b, &a.n_ss)));
+        a.ss = b.ss; a.ss_count = (float)(L.H * L.vd);
+      }
+      const int width = L.kind == MAMBA1 ? L.inner : L.H * L.vd;
+      out = gemm_args(b.mix, width, L.w_o, D, width, M, "gemm_mix_out");
+    } else {
+      if (L.ff_plain) TRY(plain_up<T>(m, L, M, b, &a.gate)); else TRY(gated_up<T>(m, L, M, b));
+      out = gemm_args(b.act, L.ffp, L.w_down, D, L.ffp, M, "gemm_ff_down");
+    }
+    TRY(project(m, out, hm.y, &a.y));
+    a.gate_b = L.rg_b[q]; a.mix = L.hc_mix[q]; a.out = L.hc_out[q];
+    next(a, k + 1);
+    TRY(vn_streams(ctx, a, M));
+    if (hm.probe && (k + 1 == subs.size() || subs[k + 1].run != i)) TRY(vn_streams_sum(ctx, m->x, hm.probe + (size_t)i * M * D, M, base.ns, D));
+  }
+  if (pick.n == 0) return VN_OK;
+  if (!all_out) {
+    StreamArgs<T, S> a = base;
+    a.pick = pick.list; a.mul = pick.mul; a.add = pick.add; a.norm_w = m->norm_f; a.h = (T*)m->h; a.h32 = out_hidden;
+    TRY(vn_streams(ctx, a, pick.n));
+  }
+  return out_logits ? head(m, pick.n, out_logits) : VN_OK;
+}
+
 template <typename T>
 int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows, const Pick& pick, float* out_hidden,
                 float* out_logits) {
@@ -879,6 +1034,11 @@ int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows,
   Cache& hc = *kv->hyb;
   const int M = rows.M, D = hm.D, n_runs = (int)hm.runs.size();
   TRY(ensure_partial(m, 1024));
+  if (hm.arranged) {
+    if constexpr (std::is_same<T, __nv_bfloat16>::value)
+      if (M > 256) return forward_arranged<T, Mat<T>>(m, kv, tokens, rows, pick, out_hidden, out_logits);
+    return forward_arranged<T, Src>(m, kv, tokens, rows, pick, out_hidden, out_logits);
+  }
   VN_LAUNCH(ctx, embed_pos_kernel<T>, M, 256, 0, (const long long*)tokens, (const T*)m->emb, hm.freq, m->x, hm.x0, rows, D,
             hm.vocab, m->status);
   auto enters_pass = [&](int i) { return i < n_runs && hm.runs[i].pass >= 0 && hm.runs[i].layer == hm.loop_start; };
@@ -899,23 +1059,14 @@ int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows,
       VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, L.norm1, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
     }
     const float* next_norm = i + 1 < n_runs && !enters_pass(i + 1) ? hm.layers[hm.runs[i + 1].layer].norm1 : nullptr;
-    if (L.kind == LATENT) TRY(latent_attention<T>(m, kv, hc, L, i, rows, b));
-    else if (L.kind == MAMBA1) TRY(mamba1<T>(m, kv, hc, L, i, rows, b));
-    else TRY(channel_delta<T>(m, kv, hc, L, i, rows, b));
+    if (L.kind == LATENT) TRY(latent_attention<T>(m, m->h, kv, hc, L, i, rows, b));
+    else if (L.kind == MAMBA1) TRY(mamba1<T>(m, m->h, kv, hc, L, i, rows, b));
+    else if (L.kind == DELTA) TRY(channel_delta<T>(m, m->h, kv, hc, L, i, rows, b));
+    else TRY((attention<T, Src>(m, m->h, kv, hc, L, i, rows, b)));
     const int width = L.kind == MAMBA1 ? L.inner : L.H * L.vd;
     TRY(close_block<T>(m, gemm_args(b.mix, width, L.w_o, D, width, M, "gemm_mix_out"), L.ff ? L.norm2 : next_norm));
     if (L.ff) {
-      GemmArgs g = gemm_args(m->h, D, L.w_gu, 2 * L.ffp, D, M, "gemm_ff_gateup");
-      if (tc_rows(m, g)) {
-        int sp = 1;
-        TRY(tc_partial(m, g, M, M, &sp));
-        const long long pairs = (long long)M * L.ffp;
-        VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp,
-                          (long long)M * 2 * L.ffp, (T*)b.act, 2 * L.ffp, pairs, L.act);
-      } else {
-        g.C = b.act; g.ldc = L.ffp; g.epi = EPI_SWIGLU; g.act = L.act; g.c_bf16 = m->cfg.bf16;
-        TRY(linear(m, g));
-      }
+      TRY(gated_up<T>(m, L, M, b));
       TRY(close_block<T>(m, gemm_args(b.act, L.ffp, L.w_down, D, L.ffp, M, "gemm_ff_down"), next_norm));
     }
     if (hm.probe)
@@ -926,17 +1077,7 @@ int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows,
     VN_LAUNCH(ctx, rmsnorm_pick_kernel<T>, pick.n, 256, 0, m->x, m->norm_f, (T*)m->h, out_hidden, pick.list, 1, 0, D, hm.eps);
   else
     VN_LAUNCH(ctx, rmsnorm_kernel<T>, pick.n, 256, 0, m->x, m->norm_f, (T*)m->h, out_hidden, pick.mul, pick.add, D, hm.eps);
-  if (out_logits) {
-    GemmArgs g = gemm_args(m->h, D, m->head, hm.vocab, D, pick.n, "gemm_head");
-    g.C = out_logits; g.ldc = hm.vocab;
-    if (tc_rows(m, g)) {
-      TcPlan direct;
-      direct.error_flag = m->tc_error;
-      return tc_launch(ctx, g, pick.n, direct);
-    }
-    return linear(m, g);
-  }
-  return VN_OK;
+  return out_logits ? head(m, pick.n, out_logits) : VN_OK;
 }
 
 // ---- cache -----------------------------------------------------------------------------------------------------------
@@ -946,12 +1087,33 @@ int32_t push_table(vn_ctx* ctx, Cache& hc, int slot) {
   return VN_OK;
 }
 
+// rotation tables for at least `rows` positions
+int32_t ensure_ropes(vn_model* m, int rows) {
+  vn_ctx* ctx = m->ctx;
+  for (Rope& r : m->hyb->ropes) {
+    if (r.rows >= rows || r.freq.empty()) continue;
+    const int n = std::max(rows, 2 * r.rows), pairs = (int)r.freq.size();
+    float2* t = nullptr;
+    double* f = nullptr;
+    TRY(dev_alloc(ctx, (void**)&t, (size_t)n * pairs * sizeof(float2)));
+    TRY(dev_alloc(ctx, (void**)&f, (size_t)pairs * 8));
+    VN_CUDA(ctx, cudaMemcpyAsync(f, r.freq.data(), (size_t)pairs * 8, cudaMemcpyHostToDevice, ctx->stream));
+    const int32_t st = vn_rope_table(ctx, f, pairs, r.amp, n, t);
+    VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+    cudaFree(f);
+    if (r.table) m->hyb->retired.push_back(r.table);
+    r.table = t; r.rows = n;
+    TRY(st);
+  }
+  return VN_OK;
+}
+
 int32_t cache_create(vn_model* m, vn_kv* kv, int pool_tokens, int pending) {
   vn_ctx* ctx = m->ctx;
   Model& hm = *m->hyb;
   Cache* hc = kv->hyb = new Cache();
   hc->pending = pending;
-  hc->ring = pending + 1;
+  hc->ring_len = pending + 1;
   hc->slots = kv->max_batch;
   hc->max_pages = ceil_div(kv->max_seq, KV_PAGE);
   hc->pooled = pool_tokens > 0;
@@ -966,15 +1128,28 @@ int32_t cache_create(vn_model* m, vn_kv* kv, int pool_tokens, int pending) {
   }
   TRY(dev_alloc(ctx, (void**)&hc->table_dev, hc->table.size() * 4));
   VN_CUDA(ctx, cudaMemcpyAsync(hc->table_dev, hc->table.data(), hc->table.size() * 4, cudaMemcpyHostToDevice, ctx->stream));
-  for (const Run& r : hm.runs) {
+  TRY(ensure_ropes(m, kv->max_seq));
+  for (size_t i = 0; i < hm.runs.size(); ++i) {
+    const Run& r = hm.runs[i];
     const HLayer& L = hm.layers[r.layer];
-    void *a = nullptr, *b = nullptr;
-    int32_t st;
-    if (L.kind == LATENT) {
+    void *a = nullptr, *b = nullptr, *c = nullptr, *in = nullptr;
+    int32_t st = VN_OK;
+    if (hm.in_taps) st = dev_alloc(ctx, &in, (size_t)hc->slots * (hm.in_taps - 1 + pending) * hm.D * m->esz);
+    hc->in_ring.push_back(in);
+    if (st == VN_OK && L.kind == ATTENTION) st = dev_alloc(ctx, &c, (size_t)hc->slots * (L.taps - 1 + pending) * L.conv_ch() * m->esz);
+    hc->ring.push_back(c);
+    if (st != VN_OK) return st;
+    if (L.kind == ATTENTION) {
+      const size_t plane = (size_t)hc->n_pages * KV_PAGE * L.KH * L.P * m->esz;
+      if (r.kv_run == (int)i) st = dev_alloc(ctx, &a, plane);
+      if (st == VN_OK && a) st = dev_alloc(ctx, &b, plane);
+    } else if (L.kind == LIGHTNING) {
+      st = dev_alloc(ctx, &b, (size_t)hc->slots * hc->ring_len * L.state_elems() * 4);
+    } else if (L.kind == LATENT) {
       st = dev_alloc(ctx, &a, (size_t)hc->n_pages * KV_PAGE * L.Rp * m->esz);
     } else {
       st = dev_alloc(ctx, &a, (size_t)hc->slots * (L.taps - 1 + pending) * L.conv_ch() * m->esz);
-      if (st == VN_OK) st = dev_alloc(ctx, &b, (size_t)hc->slots * hc->ring * L.state_elems() * 4);
+      if (st == VN_OK) st = dev_alloc(ctx, &b, (size_t)hc->slots * hc->ring_len * L.state_elems() * 4);
     }
     kv->k.push_back(a); kv->v.push_back(b);
     TRY(st);
@@ -986,6 +1161,8 @@ int32_t cache_create(vn_model* m, vn_kv* kv, int pool_tokens, int pending) {
 void cache_free(vn_kv* kv) {
   if (!kv->hyb || kv->parent) return;
   if (kv->hyb->table_dev) cudaFree(kv->hyb->table_dev);
+  for (void* p : kv->hyb->ring) if (p) cudaFree(p);
+  for (void* p : kv->hyb->in_ring) if (p) cudaFree(p);
   delete kv->hyb;
   kv->hyb = nullptr;
 }
