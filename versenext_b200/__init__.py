@@ -4,7 +4,7 @@ Public surface (names follow the reference):
   SpeculativeDecoder                      verse_nex/speculative.py:55
   VerseNexLM (= CometSparkNexLM), KVCache verse_nex/cometspark.py:294, kv_cache_parallel.py:42
   build_verse_delta_pattern               verse_nex/delta_attention.py:1218 (layer kinds vda / dsa / kda / gmla)
-  ComposedLM, FuzudraLM                   models composed of latent attention, selective scan and delta rule layers
+  ComposedLM, FuzudraLM, MusutarLM        models composed of attention, latent attention, scan, delta rule, lightning layers
   load_model                              a model by the architecture its config.json names
   BatchEngine, StepRunner                 ragged batches: portions of prompts beside single tokens, slots and pages reused
   SpecEngine                              batched draft -> verify -> accept -> commit loop
@@ -28,6 +28,7 @@ from .model import VerseNexLM, CometSparkNexLM, KVCache, build_verse_delta_patte
 from .engine import SpecEngine
 from .composed import ComposedLM
 from .fuzudra import FuzudraLM
+from .musutar import MusutarLM
 from .serving import BatchEngine, StepRunner
 from .registry import load_model
 from .tree_engine import TreeSpecEngine
@@ -38,6 +39,6 @@ from . import sampling
 from . import quant
 
 __all__ = ["Context", "DeviceArray", "as_device", "DeviceBackend", "B200Backend", "get_backend",
-           "clear_backend_cache", "SpeculativeDecoder", "Tensor", "no_grad", "sampling", "quant", "VerseNexLM", "CometSparkNexLM", "KVCache", "ComposedLM", "FuzudraLM", "load_model", "BatchEngine",
-           "StepRunner", "build_verse_delta_pattern", "SpecEngine", "TreeSpecEngine",
+           "clear_backend_cache", "SpeculativeDecoder", "Tensor", "no_grad", "sampling", "quant", "VerseNexLM", "CometSparkNexLM", "KVCache", "ComposedLM", "FuzudraLM", "MusutarLM",
+           "load_model", "BatchEngine", "StepRunner", "build_verse_delta_pattern", "SpecEngine", "TreeSpecEngine",
            "ShardedSpecEngine", "Comm", "rank_seed", "VNFileReader", "load_vn"]

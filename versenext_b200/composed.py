@@ -1,23 +1,34 @@
 """Models composed of layers of different kinds: the device's `"family": "composed"` configurations.
 
 `ComposedLM` takes the neutral configuration the library reads (a list of layers, each a mixer with its sizes and an
-optional gated feed-forward; an optional looped block; the norm's eps; the kind of positions) and offers what every model
-of the package offers: weight loading, caches, uniform and ragged steps, generation, speculative decoding as target or
-draft.  A named design is a subclass that translates its own config.json (see fuzudra.py).
+optional feed-forward; an optional looped block; the norm and its eps; the kind of positions; the arrangement of the
+residual) and offers what every model of the package offers: weight loading, caches, uniform and ragged steps, generation,
+speculative decoding as target or draft.  A named design is a subclass of `DesignLM` that translates its own config.json
+(see fuzudra.py, musutar.py).
 
-Mixers: "latent_attention" (heads, dim, vdim, kv_rank, scale, window), "mamba1" (inner, state, dt_rank, conv),
-"channel_delta" (heads, kv_heads, dim, vdim, conv, decay_rank, gate_rank).
+Mixers: "latent_attention" (heads, dim, vdim, kv_rank, scale, window), "attention" (heads, kv_heads, dim, vdim, scale,
+window, conv, rope {dims, base, scaling {factor, original, fast, slow}}, output_gate, kv_from), "mamba1" (inner, state,
+dt_rank, conv), "channel_delta" (heads, kv_heads, dim, vdim, conv, decay_rank, gate_rank), "lightning" (heads, dim, vdim,
+decay).
+
+Feed-forwards: mlp_hidden with mlp_act "silu" or "gelu_tanh" (gated) or "relu2" (plain).
+
+Model-wide: norm "rms" (weights stored around zero) or "layer" (plain weights); streams (residual streams, hyper-connections);
+input_conv (taps of the convolution that a mixer's input gets); residual_gate (sigmoid gate on every sublayer's result).
 """
 
 from __future__ import annotations
 
 import ctypes as C
-from typing import Optional
+import json
+import os
+from typing import Dict, Optional, Tuple
 
 import numpy as np
 
 from .device import as_device
 from .model import DeviceLM, KVCache, _ptr
+from .safetensors_file import SafetensorsFile
 
 
 class ComposedLM(DeviceLM):
@@ -95,3 +106,37 @@ class ComposedLM(DeviceLM):
         from .serving import BatchEngine
         eng = BatchEngine(self, max_batch=len(prompts), max_seq=max(map(len, prompts)) + max_new_tokens)
         return eng.run(prompts, max_new_tokens, temperature=temperature, top_k=top_k or 0, eos_id=eos_id, seed=seed)
+
+
+class DesignLM(ComposedLM):
+    """A named design: `ARCHITECTURE` and `composed_config(config, shapes)` make it a `ComposedLM`.  `config`: config.json's
+    contents; `shapes`: tensor name -> shape."""
+
+    ARCHITECTURE = ""
+
+    @staticmethod
+    def composed_config(config: dict, shapes: Dict[str, Tuple[int, ...]]) -> dict:
+        raise NotImplementedError
+
+    def __init__(self, config: dict, shapes: Dict[str, Tuple[int, ...]], dtype: str = "bf16", device: str = "cuda",
+                 max_seq_len: int = 4096):
+        self.source_config = config
+        super().__init__(dict(self.composed_config(config, shapes), max_seq_len=max_seq_len), dtype=dtype, device=device)
+
+    @classmethod
+    def from_state_dict(cls, config: dict, sd: dict, **kw):
+        model = cls(config, {n: tuple(a.shape) for n, a in sd.items()}, **kw)
+        model.load_state_dict(sd)
+        return model
+
+    @classmethod
+    def from_pretrained(cls, path: str, dtype: str = "bf16", device: str = "cuda", **kw):
+        """A directory with config.json and model.safetensors; tensors stream to the device one at a time."""
+        with open(os.path.join(path, "config.json")) as f:
+            config = json.load(f)
+        with SafetensorsFile(os.path.join(path, "model.safetensors")) as st:
+            model = cls(config, st.shapes(), dtype=dtype, device=device, **kw)
+            for name, arr in st:
+                model.load_tensor(name, arr)
+        model.finalize()
+        return model

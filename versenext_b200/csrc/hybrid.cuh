@@ -474,7 +474,16 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
   auto one_plus = [](float w) { return 1.0f + w; };
   auto rate = [](float a) { return expf(a); };
   auto neg_rate = [](float a) { return -expf(a); };
-  if (!hm.want.count(n)) return vn_fail(ctx, VN_ERR_INVALID, "unexpected tensor %s", n.c_str());
+  if (!hm.want.count(n)) {
+    // a layer without a feed-forward has no use for its second sublayer's tensors
+    const size_t at = n.find('.');
+    const int i = n[0] == 'l' && at != std::string::npos ? atoi(n.substr(1, at - 1).c_str()) : -1;
+    const std::string part = at != std::string::npos ? n.substr(at + 1) : "";
+    if (i >= 0 && i < (int)hm.layers.size() && !hm.layers[i].ff && n.substr(0, at) == "l" + std::to_string(i) &&
+        (part == "norm2" || part.compare(0, 4, "hc2.") == 0 || part == "rg2" || part == "rg2.b"))
+      return VN_OK;
+    return vn_fail(ctx, VN_ERR_INVALID, "unexpected tensor %s", n.c_str());
+  }
   auto weight = [&](float* dst, long long count) {        // a norm's: around zero (rms) or plain (layer)
     return hm.layer_norm ? f32(data, dst, count) : mapped(dst, count, one_plus);
   };

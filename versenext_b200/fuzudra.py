@@ -7,12 +7,9 @@ Weights are bfloat16 in `model.safetensors`, named as the library takes them.
 
 from __future__ import annotations
 
-import json
-import os
 from typing import Dict, Tuple
 
-from .composed import ComposedLM
-from .safetensors_file import SafetensorsFile
+from .composed import DesignLM
 
 _MIXER_KEYS = {
     "latent_attention": ("heads", "dim", "vdim", "kv_rank", "scale"),
@@ -47,28 +44,6 @@ def composed_config(config: dict, shapes: Dict[str, Tuple[int, ...]]) -> dict:
     return out
 
 
-class FuzudraLM(ComposedLM):
+class FuzudraLM(DesignLM):
     ARCHITECTURE = "Fuzudra"
-
-    def __init__(self, config: dict, shapes: Dict[str, Tuple[int, ...]], dtype: str = "bf16", device: str = "cuda",
-                 max_seq_len: int = 4096):
-        self.source_config = config
-        super().__init__(dict(composed_config(config, shapes), max_seq_len=max_seq_len), dtype=dtype, device=device)
-
-    @classmethod
-    def from_state_dict(cls, config: dict, sd: dict, **kw) -> "FuzudraLM":
-        model = cls(config, {n: tuple(a.shape) for n, a in sd.items()}, **kw)
-        model.load_state_dict(sd)
-        return model
-
-    @classmethod
-    def from_pretrained(cls, path: str, dtype: str = "bf16", device: str = "cuda", **kw) -> "FuzudraLM":
-        """A directory with config.json and model.safetensors; tensors stream to the device one at a time."""
-        with open(os.path.join(path, "config.json")) as f:
-            config = json.load(f)
-        with SafetensorsFile(os.path.join(path, "model.safetensors")) as st:
-            model = cls(config, st.shapes(), dtype=dtype, device=device, **kw)
-            for name, arr in st:
-                model.load_tensor(name, arr)
-        model.finalize()
-        return model
+    composed_config = staticmethod(composed_config)

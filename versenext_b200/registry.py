@@ -7,6 +7,7 @@ import os
 
 from .fuzudra import FuzudraLM
 from .model import DeviceLM, VerseNexLM
+from .musutar import MusutarLM
 
 _DESIGNS: dict = {}
 
@@ -39,5 +40,6 @@ def load_model(path: str, dtype: str = "bf16", device: str = "cuda", **kw) -> De
 
 
 register(FuzudraLM.ARCHITECTURE, FuzudraLM)
+register(MusutarLM.ARCHITECTURE, MusutarLM)
 register("VerseNexLM", VerseNexLM)
 register("CometSparkNexLM", VerseNexLM)
