@@ -118,12 +118,14 @@ class Expected:
     """Logits of one sequence and what rounding costs there: fp32 a fixed fraction of their spread; bf16 a multiple of the
     error of the restatement itself when it stores what the device stores in 16 bits."""
 
+    oracle = OF
+
     def __init__(self, sd, cfg, toks):
         self.runs = []
-        self.logits = OF.forward(sd, cfg, toks, self.runs)
+        self.logits = self.oracle.forward(sd, cfg, toks, self.runs)
         rough = []
         with OF.rounded():
-            r = OF.forward(sd, cfg, toks, rough)
+            r = self.oracle.forward(sd, cfg, toks, rough)
         self.tol = {"f32": 3e-5, "bf16": 4 * max(err(r, self.logits), 2e-3)}
         self.run_tol = [{"f32": 3e-5, "bf16": 4 * max(err(a, b), 2e-3)} for a, b in zip(rough, self.runs)]
         self.spread = np.std(self.logits)
