@@ -1027,8 +1027,8 @@ def run_layer(args):
         dist.destroy_process_group()
 
 
-FUZUDRA_WIDTHS = (1024, 2048)
-FUZUDRA_CTX, FUZUDRA_DECODE_B, FUZUDRA_PREFILL = 1024, (1, 32, 128), ((1, 4096), (8, 1024))
+COMPOSED_WIDTHS = (1024, 2048)
+COMPOSED_CTX, COMPOSED_DECODE_B, COMPOSED_PREFILL = 1024, (1, 32, 128), ((1, 4096), (8, 1024))
 
 
 def _decode_ms(m, ctx, B, T0, V, steps, profile=False):
@@ -1119,20 +1119,23 @@ def _prefill_ms(m, ctx, B, T, V, steps, profile=False):
     return statistics.median(times), prof
 
 
-def run_fuzudra(args):
-    """Prefill and decode of the Fuzudra design (random weights, 4 layers) beside VerseNexLM models of the same width,
-    depth, feed-forward, window and vocabulary: all TriSparse, and all GMLA (a latent behind K and V), the closest layers."""
+def run_composed(args):
+    """Prefill and decode of a composed design (random weights, 4 layers) beside VerseNexLM models of the same width, depth,
+    feed-forward weights, window and vocabulary: all TriSparse, and all GMLA (a latent behind K and V); with Musutar also
+    Fuzudra, the other composed design."""
     import versenext_b200 as vn
     from versenext_b200 import synthetic as S
+    design = args.workload
     world, rank, local, dist = dist_setup(args.gpus)
     ctx = vn.Context.get(local)
     V = 32000
     clocks = ClockSampler(local).start() if rank == 0 else None
     rows, profs, l0 = [], {}, ctx.launch_count()
     steps = min(max(args.steps, 5), 20)
-    for D in FUZUDRA_WIDTHS:
-        def composed():
-            return S.random_fuzudra(S.fuzudra_config(D, V), dtype="bf16", device=f"cuda:{local}")
+    for D in COMPOSED_WIDTHS:
+        def composed(name):
+            make, config = getattr(S, f"random_{name}"), getattr(S, f"{name}_config")
+            return make(config(D, V), dtype="bf16", device=f"cuda:{local}")
 
         def verse(kind):
             kw = dict(vocab_size=V, dim=D, n_layer=4, n_head=D // 64, layer_pattern=[kind] * 4, window_size=1024,
@@ -1140,16 +1143,18 @@ def run_fuzudra(args):
             m = vn.VerseNexLM(dtype="bf16", device=f"cuda:{local}", **kw)
             S.load_random(m, kw, seed=3)
             return m
-        for name, make in (("fuzudra", composed), ("trisparse", lambda: verse("trisparse")), ("gmla", lambda: verse("gmla"))):
-            m = make()
+        for name in ([design, "fuzudra"] if design != "fuzudra" else [design]) + ["trisparse", "gmla"]:
+            if args.only and name not in args.only.split(","):
+                continue
+            m = verse(name) if name in ("trisparse", "gmla") else composed(name)
             row = {"model": name, "width": D, "param_mb": round(m.param_bytes() / 1e6, 1)}
-            for B in FUZUDRA_DECODE_B:
-                ms, prof = _decode_ms(m, ctx, B, FUZUDRA_CTX, V, steps, profile=args.kernels)
+            for B in COMPOSED_DECODE_B:
+                ms, prof = _decode_ms(m, ctx, B, COMPOSED_CTX, V, steps, profile=args.kernels)
                 row[f"decode_B{B}_tok_s"] = round(B / ms * 1e3, 1)
                 row[f"decode_B{B}_ms"] = round(ms, 4)
                 if prof:
                     profs[f"{name}.{D}.decode_B{B}"] = prof
-            for B, T in FUZUDRA_PREFILL:
+            for B, T in COMPOSED_PREFILL:
                 ms, prof = _prefill_ms(m, ctx, B, T, V, steps, profile=args.kernels)
                 row[f"prefill_{B}x{T}_tok_s"] = round(B * T / ms * 1e3, 1)
                 row[f"prefill_{B}x{T}_ms"] = round(ms, 4)
@@ -1159,11 +1164,11 @@ def run_fuzudra(args):
             del m
     clk = clocks.stop() if clocks else None
     if rank == 0:
-        head = next(r for r in rows if r["model"] == "fuzudra" and r["width"] == FUZUDRA_WIDTHS[-1])
+        head = next(r for r in rows if r["model"] in (design, args.only) and r["width"] == COMPOSED_WIDTHS[-1])
         line = {"metric": "composed-model decode throughput", "value": head["decode_B32_tok_s"], "unit": "tokens/s",
                 "n_gpus": world, "steps": steps, "warmup": 3, "ms_per_step": head["decode_B32_ms"], "higher_is_better": True,
                 "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-                "config": {"workload": f"fuzudra: 4 layers, widths {FUZUDRA_WIDTHS}, V={V}, context {FUZUDRA_CTX}, L2 flushed "
+                "config": {"workload": f"{design}: 4 layers, widths {COMPOSED_WIDTHS}, V={V}, context {COMPOSED_CTX}, L2 flushed "
                                        "between steps, decode replayed from a CUDA graph"},
                 "rows": rows, "clocks": clk, "gpu_launches": ctx.launch_count() - l0}
         if profs:
@@ -1387,7 +1392,7 @@ def main():
     ap.add_argument("--steps", type=int, default=32)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--workload", default="spec", choices=["spec", "accept", "sharded", "tree", "small", "layer", "delta", "fuzudra"])
+    ap.add_argument("--workload", default="spec", choices=["spec", "accept", "sharded", "tree", "small", "layer", "delta", "fuzudra", "musutar"])
     ap.add_argument("--weak", action="store_true",
                     help="spec workload: 32 requests on every rank (default: the configuration's 32 split over the ranks)")
     ap.add_argument("--no-weak", action="store_true", help="N > 1: skip the extra 32-per-GPU measurement")
@@ -1396,7 +1401,8 @@ def main():
                     help="spec workload: quantise the target's linear weights (not the default benchmark line)")
     ap.add_argument("--pattern", default="mod,trisparse", help="layer workload: comma-separated layer kinds")
     ap.add_argument("--context", type=int, default=1100, help="layer workload: cached positions (a multiple of 220)")
-    ap.add_argument("--kernels", action="store_true", help="fuzudra workload: per-kernel times of every case")
+    ap.add_argument("--kernels", action="store_true", help="fuzudra / musutar workloads: per-kernel times of every case")
+    ap.add_argument("--only", default=None, help="fuzudra / musutar workloads: these models only (comma-separated)")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU-baseline leg")
     ap.add_argument("--no-sampler", action="store_true", help="spec workload: skip the sampler GB/s measurement")
     args = ap.parse_args()
@@ -1404,7 +1410,7 @@ def main():
         {"accept": run_reference, "small": run_reference_small}.get(args.workload, run_reference_spec)(args)
     else:
         {"spec": run_spec, "accept": run_accept, "sharded": run_sharded, "tree": run_tree,
-         "small": run_small, "layer": run_layer, "delta": run_delta, "fuzudra": run_fuzudra}[args.workload](args)
+         "small": run_small, "layer": run_layer, "delta": run_delta, "fuzudra": run_composed, "musutar": run_composed}[args.workload](args)
 
 
 if __name__ == "__main__":

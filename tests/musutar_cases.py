@@ -51,14 +51,14 @@ def weights(cfg, seed=0):
         for q in (1, 2) if L["mlp"] else (1,):
             put(p + f"norm{q}", (D,), 0.3, 1.0)
             put(p + f"hc{q}.in", (ns,), 0.4, 0.5)
-            put(p + f"hc{q}.out", (ns,), 0.4, 0.8)
-            sd[p + f"hc{q}.mix"] = bf16((np.eye(ns) * 0.8 + 0.2 * rng.standard_normal((ns, ns))).astype(np.float32))
+            put(p + f"hc{q}.out", (ns,), 0.3, 0.5)
+            sd[p + f"hc{q}.mix"] = bf16((np.eye(ns) * 0.9 + 0.1 * rng.standard_normal((ns, ns))).astype(np.float32))
             lin(p + f"rg{q}", D, D, 1.5)
             put(p + f"rg{q}.b", (D,), 0.5, 0.5)
         put(p + "canon1", (D, cfg["canon"]["taps"]), 0.4)
         H, d, vd = m["heads"], m["dim"], m["vdim"]
         if L["type"] == "attention":
-            parts = [("q", H * d, 2.0)] + ([("k", m["kv_heads"] * d, 2.0), ("v", m["kv_heads"] * vd, 2.0)] if m.get("kv_from") is None else [])
+            parts = [("q", H * d, 1.5)] + ([("k", m["kv_heads"] * d, 1.5), ("v", m["kv_heads"] * vd, 2.0)] if m.get("kv_from") is None else [])
             for t, w, gain in parts:
                 lin(p + "mix." + t, w, D, gain)
                 put(p + f"mix.{t}.conv", (w, m["conv"]), 0.6)

@@ -162,22 +162,79 @@ def fuzudra_shapes(cfg: dict) -> dict:
     return s
 
 
+def musutar_config(width: int, vocab: int = 32000, n_layer: int = 4) -> dict:
+    """config.json contents: lightning attention and sliding-window attention in turn, every second attention layer with
+    the keys and values of the one before it; four residual streams; heads of 128 (64 below width 2048), four query heads
+    per key head, a window of 1024; feed-forwards with as many weights as VerseNexLM's gated ones."""
+    hd = 128 if width >= 2048 else 64
+    heads = width // hd
+    mlp = {"kind": "dense", "ff": 4 * width}
+    decay = [float(1 - 2.0 ** (-1 - 7.0 * i / max(heads - 1, 1))) for i in range(heads)]
+    layers = []
+    for i in range(n_layer):
+        if i % 2 == 0:
+            layers.append({"type": "lightning", "mlp": mlp, "mixer": {"heads": heads, "dim": hd, "vdim": hd, "decay": decay}})
+            continue
+        m = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "conv": 4, "scale": hd ** -0.5, "mask": {"size": 1024},
+             "rot": {"base": 10000.0, "dims": hd, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        if i % 4 == 3:
+            m["kv_from"] = i - 2
+        layers.append({"type": "attention", "mlp": mlp, "mixer": m})
+    return {"architecture": "Musutar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "streams": 4, "canon": {"taps": 4}, "layers": layers}
+
+
+def musutar_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape."""
+    D, V, n = cfg["width"], cfg["vocab"], cfg["streams"]
+    s = {"embed": (V, D), "head": (V, D), "final.norm": (D,)}
+    for i, L in enumerate(cfg["layers"]):
+        m = L["mixer"]
+        H, d, v = m["heads"], m["dim"], m["vdim"]
+        t = {"canon1": (D, cfg["canon"]["taps"]), "mix.q": (H * d, D), "mix.g": (H * v, D), "mix.o": (D, H * v)}
+        if L["type"] == "attention":
+            G = m["kv_heads"]
+            t["mix.q.conv"] = (H * d, m["conv"])
+            if m.get("kv_from") is None:
+                t.update({"mix.k": (G * d, D), "mix.v": (G * v, D), "mix.k.conv": (G * d, m["conv"]), "mix.v.conv": (G * v, m["conv"])})
+        else:
+            t.update({"mix.k": (H * d, D), "mix.v": (H * v, D), "mix.norm": (H * v,)})
+        for q in (1, 2) if L["mlp"] else (1,):
+            t.update({f"norm{q}": (D,), f"hc{q}.in": (n,), f"hc{q}.out": (n,), f"hc{q}.mix": (n, n), f"rg{q}": (D, D), f"rg{q}.b": (D,)})
+        if L["mlp"]:
+            t.update({"mlp.up": (L["mlp"]["ff"], D), "mlp.down": (D, L["mlp"]["ff"])})
+        s.update({f"l{i}.{k}": x for k, x in t.items()})
+    return s
+
+
 def random_fuzudra(cfg: dict, seed: int = 0, **kw):
     """A FuzudraLM with seeded random weights, tensor by tensor."""
     from .fuzudra import FuzudraLM
-    shapes = fuzudra_shapes(cfg)
-    model = FuzudraLM(cfg, shapes, **kw)
+    return _random_design(FuzudraLM, cfg, fuzudra_shapes(cfg), seed, **kw)
+
+
+def random_musutar(cfg: dict, seed: int = 0, **kw):
+    """A MusutarLM with seeded random weights, tensor by tensor."""
+    from .musutar import MusutarLM
+    return _random_design(MusutarLM, cfg, musutar_shapes(cfg), seed, **kw)
+
+
+# (name's end, standard deviation, mean) of the tensors that are not plain linear weights or norms around zero
+_SPECIAL = (("mix.A_log", 1.0, -1.0), ("mix.dt_bias", 1.0, -2.0), ("mix.dt.b", 1.0, -3.0), ("mix.D", 0.1, 1.0), ("mix.sink", 1.0, 0.0),
+            (".conv", 0.4, 0.0), ("canon1", 0.3, 0.0), ("mix.norm", 0.1, 1.0), ("dkv.norm", 0.1, 1.0), ("hc1.in", 0.1, 0.25), ("hc2.in", 0.1, 0.25),
+            ("hc1.out", 0.1, 1.0), ("hc2.out", 0.1, 1.0))
+
+
+def _random_design(cls, cfg: dict, shapes: dict, seed: int, **kw):
+    model = cls(cfg, shapes, **kw)
     rng = np.random.default_rng(seed)
-    special = {"A_log": (1.0, -1.0), "dt_bias": (1.0, -2.0), "dt.b": (1.0, -3.0), "D": (0.1, 1.0), "sink": (1.0, 0.0)}
     for name, shape in shapes.items():
         std, mean = (0.02, 0.0) if len(shape) == 2 else (0.1, 0.0)
-        for end, sm in special.items():
-            if name.endswith("mix." + end):
-                std, mean = sm
-        if name.endswith(".conv"):
-            std = 0.4
-        if name.endswith("mix.norm") or name.endswith("dkv.norm"):
-            mean = 1.0
-        model.load_tensor(name, mean + std * rng.standard_normal(shape, dtype=np.float32))
+        for end, s, m in _SPECIAL:
+            if name.endswith(end):
+                std, mean = s, m
+        if cfg["architecture"] == "Musutar" and name.split(".")[-1] in ("norm", "norm1", "norm2"):
+            mean = 1.0                                     # layer norms: plain weights
+        w = mean + std * rng.standard_normal(shape, dtype=np.float32)
+        model.load_tensor(name, w + np.eye(shape[0], dtype=np.float32) if name.endswith(".mix") else w)
     model.finalize()
     return model
