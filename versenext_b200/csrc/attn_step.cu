@@ -14,7 +14,7 @@ template <int P> constexpr int stages() { return P > 128 ? 2 : 3; }
 template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2; }
 
 template <int P>
-__global__ void __launch_bounds__(32 * WARPS) attn_step_kernel(ConvIn<bf16, Src, false> in, PagedAttnArgs a) {
+__global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(ConvIn<bf16, Src, false> in, PagedAttnArgs a) {
   using namespace mma_detail;
   constexpr int LD = P + 8, ST = stages<P>(), TH = 32 * WARPS, CH = P / 8, TILE = 16 * LD;
   extern __shared__ __align__(16) unsigned char raw[];
@@ -56,37 +56,53 @@ __global__ void __launch_bounds__(32 * WARPS) attn_step_kernel(ConvIn<bf16, Src,
     const int np = a.rd / 2, qi = np + a.d - a.rd, nqi = nq * qi, nk = fresh ? qi : 0, nv = fresh ? a.vd : 0;
     const float2* rope = a.rope + (long long)pos * np;
     const bool keep_q = blockIdx.x == 0, keep_kv = q0 == 0;
-#pragma unroll 1
-    for (int i = tid; i < nqi + nk + nv; i += TH) {
-      // a pair of channels of a query or key head, one unrotated channel of either, or one of the value
-      int c, x = 0;
-      bf16* dst;
-      bool keep, pair = false;
+    // a pair of channels of a query or key head, one unrotated channel of either, or one of the value.  Everything that an
+    // item reads is requested before anything is stored, for two items at a time.
+    struct Item { int c, x; bf16* dst; bool keep, pair, on; float u, v, cu, cv; };
+    auto locate = [&](int i, Item& t) {
+      t.on = i < nqi + nk + nv;
+      t.pair = false;
+      t.c = t.x = 0;
+      if (!t.on) return;
       if (i < nqi + nk) {
         const bool q = i < nqi;
         const int head = q ? i / qi : 0;
-        x = q ? i % qi : i - nqi;
-        pair = x < np;
-        if (!pair) x += np;
-        c = (q ? (g * hg + q0 + head) * a.d : (a.H + g) * a.d) + x;
-        keep = q ? keep_q : keep_kv;
-        dst = (q ? sQ + head * LD : sNew) + x;
+        t.x = q ? i % qi : i - nqi;
+        t.pair = t.x < np;
+        if (!t.pair) t.x += np;
+        t.c = (q ? (g * hg + q0 + head) * a.d : (a.H + g) * a.d) + t.x;
+        t.keep = q ? keep_q : keep_kv;
+        t.dst = (q ? sQ + head * LD : sNew) + t.x;
       } else {
-        x = i - nqi - nk;
-        c = (a.H + a.KH) * a.d + g * a.vd + x;
-        keep = keep_kv;
-        dst = sNew + P + x;
+        t.x = i - nqi - nk;
+        t.c = (a.H + a.KH) * a.d + g * a.vd + t.x;
+        t.keep = keep_kv;
+        t.dst = sNew + P + t.x;
       }
-      float cur, u = in.at(row, r0, pos, slot, c, &cur);
-      if (keep && in.taps > 1) in.keep(slot, pos, c, cur);
-      if (pair) {
-        const float v = in.at(row, r0, pos, slot, c + np, &cur);
-        if (keep && in.taps > 1) in.keep(slot, pos, c + np, cur);
-        const float2 cs = rope[x];
-        dst[np] = __float2bfloat16_rn(v * cs.x + u * cs.y);
-        u = u * cs.x - v * cs.y;
+    };
+#pragma unroll 1
+    for (int i = tid; i < nqi + nk + nv; i += 2 * TH) {
+      Item t[2];
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        locate(i + y * TH, t[y]);
+        if (t[y].on) t[y].u = in.at(row, r0, pos, slot, t[y].c, &t[y].cu);
+        if (t[y].pair) t[y].v = in.at(row, r0, pos, slot, t[y].c + np, &t[y].cv);
       }
-      *dst = __float2bfloat16_rn(u);
+#pragma unroll
+      for (int y = 0; y < 2; ++y) {
+        if (!t[y].on) continue;
+        float u = t[y].u;
+        const bool keep = t[y].keep && in.taps > 1;
+        if (t[y].pair) {
+          const float2 cs = rope[t[y].x];
+          t[y].dst[np] = __float2bfloat16_rn(t[y].v * cs.x + u * cs.y);
+          u = u * cs.x - t[y].v * cs.y;
+          if (keep) in.keep(slot, pos, t[y].c + np, t[y].cv);
+        }
+        *t[y].dst = __float2bfloat16_rn(u);
+        if (keep) in.keep(slot, pos, t[y].c, t[y].cu);
+      }
     }
     const bf16 zero = __float2bfloat16_rn(0.f);
     for (int i = tid; i < 16 * P; i += TH) {

@@ -242,8 +242,28 @@ __global__ void __launch_bounds__(32 * CW) lightning_chunk_kernel(LightningArgs 
       for (int s = 0; s < seg; ++s) load_state(piece(s), keep);
     }
   }
+  float nw[2][2];                                                // norm weights of the columns this lane finishes
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int c = 16 * warp + 8 * j + l2 + x;
+      nw[j][x] = !LOCAL && c < nv ? a.norm_w[h * vd + cb + c] : 0.f;
+    }
 #pragma unroll 1
   for (int t0 = t_lo, buf = 0; t0 < t_hi; t0 += CH, buf ^= 1) {
+    unsigned gate[LOCAL || !VEC ? 1 : 4][2][2];                  // raw gates of this lane's outputs: requested ahead of the products
+    if (!LOCAL && VEC)
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const int t = t0 + 16 * i + g4 + 8 * e, c = 16 * warp + 8 * j + l2;
+            if (t < t_hi && c < nv)
+              gate[LOCAL || !VEC ? 0 : i][e][j] = *reinterpret_cast<const unsigned*>(proj.p + (long long)(r0 + t) * proj.ld + kg + h * vd + cb + c);
+          }
     if (t0 + CH < t_hi) { fetch(t0 + CH, buf ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
     __syncthreads();
     const int m = min(CH, t_hi - t0);
@@ -351,13 +371,15 @@ __global__ void __launch_bounds__(32 * CW) lightning_chunk_kernel(LightningArgs 
             for (int j = 0; j < 2; ++j) {
               const int c = 16 * warp + 8 * j + l2;
               float v[2];
+              float2 gv = make_float2(0.f, 0.f);
+              if (VEC) gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[LOCAL || !VEC ? 0 : i][e][j]));
 #pragma unroll
               for (int x = 0; x < 2; ++x) {
                 v[x] = o[i][j][2 * e + x];
                 ss = fmaf(v[x], v[x], ss);
                 if (c + x < nv) {
                   const int col = h * vd + cb + c + x;
-                  v[x] *= a.norm_w[col] * sigmoid_f(proj.get(row, kg + col));
+                  v[x] *= nw[j][x] * sigmoid_f(VEC ? (x ? gv.y : gv.x) : proj.get(row, kg + col));
                   if (!VEC) reinterpret_cast<bf16*>(a.out)[row * a.H * vd + col] = __float2bfloat16_rn(v[x]);
                 }
               }

@@ -1,6 +1,8 @@
 // Kernels of paged_attn.cuh for prompts and mixed batches; the one-token kernel is in attn_step.cu.
-#include "paged_attn.cuh"
+#include <type_traits>
+
 #include "ldmatrix.cuh"
+#include "paged_attn.cuh"
 
 namespace {
 
@@ -67,6 +69,63 @@ __global__ void __launch_bounds__(256) attn_inputs_kernel(ConvIn<T, S, false> in
     }
     for (int j = w + lane; j < a.P; j += 32)
       for (int r = first; r < end; ++r) dest(r)[j] = from_f<T>(0.f);
+    row = end;
+  }
+}
+
+// The same for many rows: a thread takes four channels of RB rows, with the four they are rotated with.  Filters of at most
+// four taps; d, vd, rd / 2 and the source's pitch multiples of 4.  grid (ceil(items / 256), ceil(M / RB)): items of a row
+// are the rotated quads of all heads, the unrotated ones, the values'
+template <typename T, int RB>
+__global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, false> in, PagedAttnArgs a, int qk_heads, int items) {
+  const int it = blockIdx.x * 256 + threadIdx.x;
+  if (it >= items) return;
+  const int np = a.rd / 2, nr = np / 4, nu = (a.d - a.rd) / 4, nv = a.vd / 4;
+  int head, c;                                             // head of q | k | v; first channel in it
+  const bool pair = it < qk_heads * nr;
+  bool is_v = false;
+  if (pair) { head = it / nr; c = it % nr * 4; }
+  else if (it < qk_heads * (nr + nu)) { const int i = it - qk_heads * nr; head = i / nu; c = a.rd + i % nu * 4; }
+  else { const int i = it - qk_heads * (nr + nu); is_v = true; head = i / nv; c = i % nv * 4; }
+  const int col = is_v ? (a.H + a.KH) * a.d + head * a.vd + c : head * a.d + c;
+  int row = blockIdx.y * RB;
+  const int last = min(row + RB, a.rows.M);
+  while (row < last) {                                     // stretches of one entry
+    int slot, r0, n, start;
+    a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
+    const int end = min(last, r0 + n);
+    float4 u[RB], v[RB];
+    in.template run4<RB>(row, end, r0, start, slot, col, u);
+    if (pair) in.template run4<RB>(row, end, r0, start, slot, col + np, v);
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      if (row + r >= end) break;
+      const int pos = start + row + r - r0;
+      T* dst;
+      if (!is_v && head < a.H) {
+        dst = reinterpret_cast<T*>(a.q) + ((long long)(row + r) * a.H + head) * a.P + c;
+      } else {
+        const int g = is_v ? head : head - a.H;
+        dst = reinterpret_cast<T*>(is_v ? a.vplane : a.kplane) +
+              (((long long)a.table[(long long)slot * a.max_pages + pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.KH + g) * a.P + c;
+      }
+      if (pair) {
+        const float4* cs = reinterpret_cast<const float4*>(a.rope + (long long)pos * np + c);   // two pairs each
+        const float4 p0 = cs[0], p1 = cs[1], x = u[r], y = v[r];
+        store4(dst, make_float4(x.x * p0.x - y.x * p0.y, x.y * p0.z - y.y * p0.w, x.z * p1.x - y.z * p1.y, x.w * p1.z - y.w * p1.w));
+        store4(dst + np, make_float4(y.x * p0.x + x.x * p0.y, y.y * p0.z + x.y * p0.w, y.z * p1.x + x.z * p1.y, y.w * p1.z + x.w * p1.w));
+      } else {
+        store4(dst, u[r]);
+      }
+      const int w = is_v ? a.vd : a.d;
+      if (c + 4 == w || (pair && np + c + 4 == w))         // the last quad of a head also pads it
+        for (int j = w - (pair ? np + c : c); j < a.P - (pair ? np + c : c); j += 4) store4((pair ? dst + np : dst) + j, make_float4(0.f, 0.f, 0.f, 0.f));
+      if (n <= a.pending && in.taps > 1)
+        for (int e = 0; e < 4; ++e) {
+          in.keep(slot, pos, col + e, in.src.get(row + r, in.col0 + col + e));
+          if (pair) in.keep(slot, pos, col + np + e, in.src.get(row + r, in.col0 + col + np + e));
+        }
+    }
     row = end;
   }
 }
@@ -345,6 +404,13 @@ template <typename T, typename S>
 int32_t vn_attn_inputs(vn_ctx* ctx, const ConvIn<T, S, false>& conv, const PagedAttnArgs& a) {
   const int units = a.H + (a.own_kv ? 2 * a.KH : 0);
   const dim3 block(32, 8);
+  if constexpr (std::is_same<S, Mat<T>>::value) {
+    if (conv.taps <= 4 && a.d % 4 == 0 && a.vd % 4 == 0 && a.rd % 8 == 0 && conv.src.ld % 4 == 0) {
+      const int qk = a.H + (a.own_kv ? a.KH : 0), items = qk * (a.d - a.rd / 2) / 4 + (a.own_kv ? a.KH * a.vd / 4 : 0);
+      VN_LAUNCH_NAMED(ctx, "attn_inputs_kernel", (attn_inputs4_kernel<T, 4>), dim3(ceil_div(items, 256), ceil_div(a.rows.M, 4)), 256, 0, conv, a, qk, items);
+      return VN_OK;
+    }
+  }
   if (a.rows.M >= 512 && conv.taps <= 4)
     VN_LAUNCH_NAMED(ctx, "attn_inputs_kernel", (attn_inputs_kernel<T, S, 8>), dim3(units, ceil_div(a.rows.M, 64)), block, 0, conv, a);
   else

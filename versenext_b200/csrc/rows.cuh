@@ -220,6 +220,52 @@ struct ConvIn {
       out[i] = activate(acc, c);
     }
   }
+  // The same for channels c .. c + 3 of a source of plain rows (splits 1; col0 + c, the pitch and c multiples of 4).
+  template <int RB>
+  __device__ __forceinline__ void run4(int row, int row_end, int r0, int start, int slot, int c, float4 (&out)[RB]) const {
+    float wt[4][4];                                     // [tap back][channel]
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float* wc = w + (long long)(c + e) * taps;
+      if (taps == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(wc);
+        wt[0][e] = t.w; wt[1][e] = t.z; wt[2][e] = t.y; wt[3][e] = t.x;
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) wt[j][e] = j < taps ? wc[taps - 1 - j] : 0.f;
+      }
+    }
+    float4 x[RB + 3];
+    const auto* p = src.p + (long long)row * src.ld + col0 + c;
+#pragma unroll
+    for (int i = 0; i < RB; ++i) x[3 + i] = load4(p + (long long)(min(row + i, row_end - 1) - row) * src.ld);
+    if (row - r0 >= 3) {
+#pragma unroll
+      for (int i = 0; i < 3; ++i) x[i] = load4(p + (long long)(i - 3) * src.ld);
+    } else {
+      const int pos = start + row - r0;
+#pragma unroll
+      for (int j = 1; j < 4; ++j) {
+        x[3 - j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < taps)
+          x[3 - j] = make_float4(input(row, r0, start, slot, pos - j, c), input(row, r0, start, slot, pos - j, c + 1),
+                                 input(row, r0, start, slot, pos - j, c + 2), input(row, r0, start, slot, pos - j, c + 3));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < RB; ++i) {
+      float a[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        auto at = [&](const float4& v) { return round_to<T>(e == 0 ? v.x : e == 1 ? v.y : e == 2 ? v.z : v.w); };
+        a[e] = at(x[3 + i]) * wt[0][e];
+#pragma unroll
+        for (int j = 1; j < 4; ++j) a[e] = fmaf(at(x[3 + i - j]), wt[j][e], a[e]);
+        a[e] = activate(a[e], c + e);
+      }
+      out[i] = make_float4(a[0], a[1], a[2], a[3]);
+    }
+  }
   __device__ __forceinline__ void keep(int slot, int pos, int c, float v) const {
     ring[((long long)slot * RC + pos % RC) * C + c] = from_f<T>(v);
   }

@@ -168,6 +168,33 @@ __global__ void __launch_bounds__(256) input_conv_kernel(ConvIn<T, Mat<T>, false
   }
 }
 
+// four channels per thread, filters of at most four taps.  grid (ceil(D / 1024), ceil(M / RB))
+template <typename T, int RB>
+__global__ void __launch_bounds__(256) input_conv4_kernel(ConvIn<T, Mat<T>, false> in, Rows rows, int pending, T* __restrict__ hc) {
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4, D = in.C;
+  if (c >= D) return;
+  int row = blockIdx.y * RB;
+  const int last = min(row + RB, rows.M);
+  while (row < last) {                                  // stretches of one entry
+    int slot, r0, n, start;
+    rows.entry(rows.entry_of(row), &slot, &r0, &n, &start);
+    const int end = min(last, r0 + n);
+    float4 v[RB];
+    in.template run4<RB>(row, end, r0, start, slot, c, v);
+#pragma unroll
+    for (int i = 0; i < RB; ++i)
+      if (row + i < end) {
+        const float4 h = load4(in.src.p + (long long)(row + i) * in.src.ld + c);
+        store4(hc + (long long)(row + i) * D + c, make_float4(h.x + v[i].x, h.y + v[i].y, h.z + v[i].z, h.w + v[i].w));
+        if (n <= pending && in.taps > 1) {
+          const int pos = start + row + i - r0;
+          in.keep(slot, pos, c, h.x); in.keep(slot, pos, c + 1, h.y); in.keep(slot, pos, c + 2, h.z); in.keep(slot, pos, c + 3, h.w);
+        }
+      }
+    row = end;
+  }
+}
+
 template <typename T, typename S, int V>
 int32_t launch(vn_ctx* ctx, const StreamArgs<T, S>& a, int n_rows) {
   const size_t smem = (size_t)a.D * 4;
@@ -200,7 +227,10 @@ int32_t vn_streams_sum(vn_ctx* ctx, const float* x, float* out, int M, int ns, i
 
 template <typename T>
 int32_t vn_input_conv(vn_ctx* ctx, const ConvIn<T, Mat<T>, false>& in, const Rows& rows, int pending, T* hc) {
-  if (in.taps <= 4)
+  if (in.taps <= 4 && in.C % 4 == 0)
+    VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv4_kernel<T, 4>), dim3(ceil_div(in.C, 1024), ceil_div(rows.M, 4)), 256, 0, in, rows,
+                    pending, hc);
+  else if (in.taps <= 4)
     VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv_kernel<T, 8>), dim3(ceil_div(in.C, 256), ceil_div(rows.M, 8)), 256, 0, in, rows,
                     pending, hc);
   else
