@@ -11,7 +11,7 @@ namespace {
 using bf16 = __nv_bfloat16;
 constexpr int WARPS = 4;
 template <int P> constexpr int stages() { return P > 128 ? 2 : 3; }
-template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2; }
+template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2 + 18 * P * 4; }
 
 template <int P>
 __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(ConvIn<bf16, Src, false> in, PagedAttnArgs a) {
@@ -21,6 +21,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
   bf16* ring = reinterpret_cast<bf16*>(raw);                          // [warp][stage][K, V][16][LD]
   bf16* sQ = ring + WARPS * ST * 2 * TILE;                            // [16][LD]
   bf16* sNew = sQ + TILE;                                             // [2][P] key and value of the new token
+  float* sConv = reinterpret_cast<float*>(sNew + 2 * P);              // [18][P] convolved channels: query heads, key, value
   __shared__ int s_last;
   __shared__ float s_ml[WARPS][16][2], s_f[WARPS][16];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = blockIdx.z;
@@ -53,65 +54,79 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
   for (int s = 0; s < ST - 1; ++s) fetch(c0 + warp + s * WARPS, s);
   // queries; the new key and value
   {
-    const int np = a.rd / 2, qi = np + a.d - a.rd, nqi = nq * qi, nk = fresh ? qi : 0, nv = fresh ? a.vd : 0;
-    const float2* rope = a.rope + (long long)pos * np;
-    const bool keep_q = blockIdx.x == 0, keep_kv = q0 == 0;
-    // a pair of channels of a query or key head, one unrotated channel of either, or one of the value.  Everything that an
-    // item reads is requested before anything is stored, for two items at a time.
-    struct Item { int c, x; bf16* dst; bool keep, pair, on; float u, v, cu, cv; };
-    auto locate = [&](int i, Item& t) {
-      t.on = i < nqi + nk + nv;
-      t.pair = false;
-      t.c = t.x = 0;
-      if (!t.on) return;
-      if (i < nqi + nk) {
-        const bool q = i < nqi;
-        const int head = q ? i / qi : 0;
-        t.x = q ? i % qi : i - nqi;
-        t.pair = t.x < np;
-        if (!t.pair) t.x += np;
-        t.c = (q ? (g * hg + q0 + head) * a.d : (a.H + g) * a.d) + t.x;
-        t.keep = q ? keep_q : keep_kv;
-        t.dst = (q ? sQ + head * LD : sNew) + t.x;
-      } else {
-        t.x = i - nqi - nk;
-        t.c = (a.H + a.KH) * a.d + g * a.vd + t.x;
-        t.keep = keep_kv;
-        t.dst = sNew + P + t.x;
-      }
+    const int d = a.d, vd = a.vd, taps = in.taps, C = in.C, n_qk = (nq + (fresh ? 1 : 0)) * d, n_all = n_qk + (fresh ? vd : 0);
+    // channel i of this CTA's list (query heads, key, value) -> column of the projection, place in sConv
+    auto place = [&](int i, int& c, float*& dst, bool& keep) {
+      const int head = i < n_qk ? i / d : nq + 1, x = i < n_qk ? i - head * d : i - n_qk;
+      c = head < nq ? (g * hg + q0 + head) * d + x : head == nq ? (a.H + g) * d + x : (a.H + a.KH) * d + g * vd + x;
+      dst = sConv + (head < nq ? head : head == nq ? 16 : 17) * P + x;
+      keep = head < nq ? blockIdx.x == 0 : q0 == 0;
     };
+    bf16* inputs = in.ring + (long long)slot * in.RC * C;
+    int c;
+    float* dst;
+    bool keep;
+    if (d % 4 == 0 && vd % 4 == 0 && in.src.ld % 4 == 0 && C % 4 == 0 && taps <= 4) {
+      // four channels at a time; one copy of the code, which is fetched anew at every step of a large model
 #pragma unroll 1
-    for (int i = tid; i < nqi + nk + nv; i += 2 * TH) {
-      Item t[2];
+      for (int i = tid * 4; i < n_all; i += TH * 4) {
+        place(i, c, dst, keep);
+        float4 x[4];
 #pragma unroll
-      for (int y = 0; y < 2; ++y) {
-        locate(i + y * TH, t[y]);
-        if (t[y].on) t[y].u = in.at(row, r0, pos, slot, t[y].c, &t[y].cu);
-        if (t[y].pair) t[y].v = in.at(row, r0, pos, slot, t[y].c + np, &t[y].cv);
-      }
-#pragma unroll
-      for (int y = 0; y < 2; ++y) {
-        if (!t[y].on) continue;
-        float u = t[y].u;
-        const bool keep = t[y].keep && in.taps > 1;
-        if (t[y].pair) {
-          const float2 cs = rope[t[y].x];
-          t[y].dst[np] = __float2bfloat16_rn(t[y].v * cs.x + u * cs.y);
-          u = u * cs.x - t[y].v * cs.y;
-          if (keep) in.keep(slot, pos, t[y].c + np, t[y].cv);
+        for (int j = 1; j < 4; ++j) {
+          x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+          if (j < taps && j <= pos) x[j] = load4(inputs + (long long)((pos - j) % in.RC) * C + c);
         }
-        *t[y].dst = __float2bfloat16_rn(u);
-        if (keep) in.keep(slot, pos, t[y].c, t[y].cu);
+        x[0] = get4(in.src, row, c);
+        if (keep && taps > 1) store4(inputs + (long long)(pos % in.RC) * C + c, x[0]);
+        x[0] = make_float4(round_to<bf16>(x[0].x), round_to<bf16>(x[0].y), round_to<bf16>(x[0].z), round_to<bf16>(x[0].w));
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float* w = in.w + (long long)c * taps + taps - 1;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (j < taps) {
+            acc.x = fmaf(x[j].x, w[-j], acc.x); acc.y = fmaf(x[j].y, w[taps - j], acc.y);
+            acc.z = fmaf(x[j].z, w[2 * taps - j], acc.z); acc.w = fmaf(x[j].w, w[3 * taps - j], acc.w);
+          }
+        store4(dst, acc);
+      }
+    } else {
+#pragma unroll 1
+      for (int i = tid; i < n_all; i += TH) {
+        place(i, c, dst, keep);
+        float cur;
+        *dst = in.at(row, r0, pos, slot, c, &cur);
+        if (keep && taps > 1) in.keep(slot, pos, c, cur);
       }
     }
+    __syncthreads();
+    // rotation of the queries and the key
+    const int np = a.rd / 2, half = np + d - a.rd;
+    const float2* rope = a.rope + (long long)pos * np;
+#pragma unroll 1
+    for (int i = tid; i < (nq + (fresh ? 1 : 0)) * half; i += TH) {
+      const int head = i / half, x = i - head * half;
+      const float* src = sConv + (head < nq ? head : 16) * P;
+      bf16* to = head < nq ? sQ + head * LD : sNew;
+      if (x < np) {
+        const float2 cs = rope[x];
+        const float u = src[x], v = src[np + x];
+        to[x] = __float2bfloat16_rn(u * cs.x - v * cs.y);
+        to[np + x] = __float2bfloat16_rn(v * cs.x + u * cs.y);
+      } else {
+        to[np + x] = __float2bfloat16_rn(src[np + x]);
+      }
+    }
+    if (fresh)
+      for (int x = tid; x < vd; x += TH) sNew[P + x] = __float2bfloat16_rn(sConv[17 * P + x]);
     const bf16 zero = __float2bfloat16_rn(0.f);
     for (int i = tid; i < 16 * P; i += TH) {
       const int r = i / P, c = i % P;
-      if (r >= nq || c >= a.d) sQ[r * LD + c] = zero;
+      if (r >= nq || c >= d) sQ[r * LD + c] = zero;
     }
     if (fresh) {
-      for (int c = a.d + tid; c < P; c += TH) sNew[c] = zero;
-      for (int c = a.vd + tid; c < P; c += TH) sNew[P + c] = zero;
+      for (int c = d + tid; c < P; c += TH) sNew[c] = zero;
+      for (int c = vd + tid; c < P; c += TH) sNew[P + c] = zero;
     }
   }
   __syncthreads();

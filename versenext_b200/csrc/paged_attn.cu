@@ -341,14 +341,38 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
       *reinterpret_cast<float2*>(sO + ((lane >> 2) + 8 * e) * P + 8 * j + (lane & 3) * 2) = make_float2(acc[j][2 * e] * inv, acc[j][2 * e + 1] * inv);
   }
   __syncwarp();
+  const int fw = f0 + 16 * warp;
+  if (a.vd % 4 == 0 && (a.col_g < 0 || (a.col_g % 4 == 0 && proj.ld % 4 == 0))) {
+    // four columns per lane, eight rows' gates requested at a time
+#pragma unroll 1
+    for (int c = lane * 4; c < a.vd; c += 128)
+#pragma unroll 1
+      for (int r = 0; r < 16; r += 8) {
+        float4 gt[8];
+#pragma unroll
+        for (int y = 0; y < 8; ++y) {
+          const int f = min(fw + r + y, nf - 1);
+          if (a.col_g >= 0) gt[y] = get4(proj, r0 + f / hg, a.col_g + (g * hg + f % hg) * a.vd + c);
+        }
+#pragma unroll
+        for (int y = 0; y < 8; ++y) {
+          const int f = fw + r + y;
+          if (f >= nf) break;
+          float4 v = load4(sO + (r + y) * P + c);
+          if (a.col_g >= 0) { v.x *= sigmoid_f(gt[y].x); v.y *= sigmoid_f(gt[y].y); v.z *= sigmoid_f(gt[y].z); v.w *= sigmoid_f(gt[y].w); }
+          store4(reinterpret_cast<bf16*>(a.out) + ((long long)(r0 + f / hg) * a.H + g * hg + f % hg) * a.vd + c, v);
+        }
+      }
+    return;
+  }
   for (int r = 0; r < 16; ++r) {
-    const int f = f0 + 16 * warp + r;
+    const int f = fw + r;
     if (f >= nf) break;
     const long long row = r0 + f / hg;
     const int h = g * hg + f % hg;
     bf16* o = reinterpret_cast<bf16*>(a.out) + (row * a.H + h) * a.vd;
     for (int c = lane; c < a.vd; c += 32)
-      o[c] = __float2bfloat16_rn(sO[r * P + c] * (a.col_g >= 0 ? sigmoid_f(proj.get(row, a.col_g + h * a.vd + c)) : 1.f));
+      o[c] = __float2bfloat16_rn(sO[r * P + c] * (a.col_g >= 0 ? sigmoid_f(proj.get_rare(row, a.col_g + h * a.vd + c)) : 1.f));
   }
 }
 

@@ -130,6 +130,139 @@ __global__ void __launch_bounds__(256) streams_kernel(StreamArgs<T, S> a) {
   }
 }
 
+// The same for few rows and D <= 2048 (a multiple of 4): a thread keeps its four columns of everything in registers, so that
+// all loads are in flight together; weights are fetched ahead of the wait on the preceding kernel; one block reduction, of
+// counts, means and squared deviations.  D / 4 threads, rounded up to whole warps.
+struct Moments { float n, mean, m2; };
+__device__ __forceinline__ Moments merge(const Moments& a, const Moments& b) {
+  const float n = a.n + b.n;
+  if (n == 0.f) return a;
+  const float d = b.mean - a.mean, f = b.n / n;
+  return {n, fmaf(d, f, a.mean), a.m2 + b.m2 + d * d * a.n * f};
+}
+
+template <typename T, typename S, int NS>
+__global__ void __launch_bounds__(512) streams_row_kernel(StreamArgs<T, S> a) {
+  pdl_trigger();
+  __shared__ float s_mix[NS * NS], s_out[NS], s_in[NS];
+  __shared__ Moments s_mom[16];
+  const int tid = threadIdx.x, lane = tid & 31, D = a.D, d = tid * 4;
+  const bool on = d < D;
+  if (tid < NS * NS) s_mix[tid] = a.mix ? a.mix[tid] : (tid / NS == tid % NS ? 1.f : 0.f);
+  if (tid < NS) { s_out[tid] = a.out ? a.out[tid] : 1.f; s_in[tid] = a.in ? a.in[tid] : 1.f; }
+  const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
+  const float4 wn = on && a.norm_w ? load4(a.norm_w + d) : zero4, gb = on && a.gate_b ? load4(a.gate_b + d) : zero4;
+  float4 cw[4] = {zero4, zero4, zero4, zero4};              // filter of channel d + e, the current token's tap last
+  const int taps = a.hc ? a.taps : 0;
+  if (on && taps == 4) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) cw[e] = load4(a.conv_w + (long long)(d + e) * 4);
+  }
+  __syncthreads();
+  pdl_wait();
+  const long long row = a.pick ? a.pick[blockIdx.x] : (long long)blockIdx.x * a.mul + a.add;
+  const bool write = a.y.p != nullptr, gated = a.gate.p != nullptr;
+  int slot = 0, r0, n, pos = 0;
+  if (a.hc) a.rows.entry(a.rows.entry_of((int)row), &slot, &r0, &n, &pos);
+  float* x = a.x + row * NS * D + d;
+  float4 xs[NS], y = zero4;
+  float ysc = 1.f;
+  if (on) {
+    if (a.first) {
+      xs[0] = load4(a.first + row * D + d);
+#pragma unroll
+      for (int s = 1; s < NS; ++s) xs[s] = xs[0];
+    } else {
+#pragma unroll
+      for (int s = 0; s < NS; ++s) xs[s] = load4(x + (long long)s * D);
+    }
+    if (write) y = get4(a.y, row, d);
+    if (write && gated) {
+      const float4 g = get4(a.gate, row, d);
+      y.x *= sigmoid_f(g.x + gb.x); y.y *= sigmoid_f(g.y + gb.y); y.z *= sigmoid_f(g.z + gb.z); y.w *= sigmoid_f(g.w + gb.w);
+    }
+  }
+  if (a.ss) {                                               // every warp sums the row's parts
+    float v = 0.f;
+    for (int i = lane; i < a.n_ss; i += 32) v += a.ss[row * a.n_ss + i];
+    ysc = 1.f / sqrtf(warp_sum(v) / a.ss_count + a.eps);
+  }
+  float4 u = zero4;
+  if (on) {
+    if (write) {
+      y.x *= ysc; y.y *= ysc; y.z *= ysc; y.w *= ysc;
+      float4 nx[NS];
+#pragma unroll
+      for (int t = 0; t < NS; ++t) {
+        const float o = s_out[t];
+        nx[t] = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+#pragma unroll
+        for (int s = 0; s < NS; ++s) {
+          const float m = s_mix[s * NS + t];
+          nx[t].x = fmaf(m, xs[s].x, nx[t].x); nx[t].y = fmaf(m, xs[s].y, nx[t].y);
+          nx[t].z = fmaf(m, xs[s].z, nx[t].z); nx[t].w = fmaf(m, xs[s].w, nx[t].w);
+        }
+        store4(x + (long long)t * D, nx[t]);
+      }
+#pragma unroll
+      for (int t = 0; t < NS; ++t) xs[t] = nx[t];
+    }
+#pragma unroll
+    for (int s = 0; s < NS; ++s) {
+      const float m = s_in[s];
+      u.x = fmaf(m, xs[s].x, u.x); u.y = fmaf(m, xs[s].y, u.y); u.z = fmaf(m, xs[s].z, u.z); u.w = fmaf(m, xs[s].w, u.w);
+    }
+  }
+  if (!a.norm_w) return;
+  Moments mo = {0.f, 0.f, 0.f};
+  if (on) {
+    if (a.layer_norm) {
+      const float mean = (u.x + u.y + u.z + u.w) * 0.25f, p = u.x - mean, q = u.y - mean, v = u.z - mean, w = u.w - mean;
+      mo = {4.f, mean, p * p + q * q + v * v + w * w};
+    } else {
+      mo = {4.f, 0.f, u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w};
+    }
+  }
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1)
+    mo = merge(mo, {__shfl_xor_sync(0xffffffffu, mo.n, o), __shfl_xor_sync(0xffffffffu, mo.mean, o), __shfl_xor_sync(0xffffffffu, mo.m2, o)});
+  if (lane == 0) s_mom[tid >> 5] = mo;
+  __syncthreads();
+  mo = s_mom[0];
+  for (int w = 1; w < (int)blockDim.x / 32; ++w) mo = merge(mo, s_mom[w]);
+  if (!on) return;
+  const float r = sqrtf(mo.m2 / (float)D + a.eps);
+  float v[4] = {(u.x - mo.mean) / r * wn.x, (u.y - mo.mean) / r * wn.y, (u.z - mo.mean) / r * wn.z, (u.w - mo.mean) / r * wn.w};
+  const long long at = (long long)blockIdx.x * D + d;
+  if (a.h) store4(a.h + at, make_float4(v[0], v[1], v[2], v[3]));
+  if (a.h32) store4(a.h32 + at, make_float4(v[0], v[1], v[2], v[3]));
+  if (!a.hc) return;
+  T* ring = a.ring + (long long)slot * a.RC * D + d;
+  float acc[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) v[e] = round_to<T>(v[e]);
+  if (taps == 4) {
+    float4 old[3] = {zero4, zero4, zero4};
+#pragma unroll
+    for (int j = 1; j < 4; ++j)
+      if (j <= pos) old[j - 1] = load4(ring + (long long)((pos - j) % a.RC) * D);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      auto of = [&](const float4& t) { return e == 0 ? t.x : e == 1 ? t.y : e == 2 ? t.z : t.w; };
+      acc[e] = fmaf(of(old[2]), cw[e].x, fmaf(of(old[1]), cw[e].y, fmaf(of(old[0]), cw[e].z, v[e] * cw[e].w)));
+    }
+  } else {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float* w = a.conv_w + (long long)(d + e) * taps;
+      acc[e] = v[e] * w[taps - 1];
+      for (int j = 1; j < taps && j <= pos; ++j) acc[e] = fmaf(to_f<T>(ring[(long long)((pos - j) % a.RC) * D + e]), w[taps - 1 - j], acc[e]);
+    }
+  }
+  if (taps > 1) store4(ring + (long long)(pos % a.RC) * D, make_float4(v[0], v[1], v[2], v[3]));
+  store4(a.hc + at, make_float4(v[0] + acc[0], v[1] + acc[1], v[2] + acc[2], v[3] + acc[3]));
+}
+
 __global__ void __launch_bounds__(256) streams_sum_kernel(const float* __restrict__ x, float* __restrict__ out, int ns, int D) {
   const long long row = blockIdx.x;
   for (int d = threadIdx.x; d < D; d += 256) {
@@ -198,7 +331,12 @@ __global__ void __launch_bounds__(256) input_conv4_kernel(ConvIn<T, Mat<T>, fals
 template <typename T, typename S, int V>
 int32_t launch(vn_ctx* ctx, const StreamArgs<T, S>& a, int n_rows) {
   const size_t smem = (size_t)a.D * 4;
+  const bool few = V == 4 && a.D <= 2048 && n_rows <= 1024;
+  const int block = (a.D / 4 + 31) & ~31;
 #define CASE(NS) case NS: \
+  if constexpr (V == 4) { \
+    if (few) { VN_LAUNCH_PDL_LEVEL(ctx, (vn_pdl_mask() & 4) ? 1 : 2, "streams_row_kernel", (streams_row_kernel<T, S, NS>), n_rows, block, 0, a); break; } \
+  } \
   if (smem > 40000) VN_CUDA(ctx, cudaFuncSetAttribute((streams_kernel<T, S, NS, V>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
   VN_LAUNCH_PDL_LEVEL(ctx, (vn_pdl_mask() & 4) ? 1 : 2, "streams_kernel", (streams_kernel<T, S, NS, V>), n_rows, 256, smem, a); break;
   switch (a.ns) {
