@@ -11,7 +11,7 @@ namespace {
 using bf16 = __nv_bfloat16;
 constexpr int WARPS = 4;
 template <int P> constexpr int stages() { return P > 128 ? 2 : 3; }
-template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2 + 18 * P * 4; }
+template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2; }
 
 template <int P>
 __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(ConvIn<bf16, Src, false> in, PagedAttnArgs a) {
@@ -21,7 +21,8 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
   bf16* ring = reinterpret_cast<bf16*>(raw);                          // [warp][stage][K, V][16][LD]
   bf16* sQ = ring + WARPS * ST * 2 * TILE;                            // [16][LD]
   bf16* sNew = sQ + TILE;                                             // [2][P] key and value of the new token
-  float* sConv = reinterpret_cast<float*>(sNew + 2 * P);              // [18][P] convolved channels: query heads, key, value
+  // convolved channels: query heads 0 .. 15, key (16), value (17); they lie in ring stages that no prefetch has reached yet
+  auto sConv = [&](int r) { return reinterpret_cast<float*>(ring + ((r < 16 ? 0 : ST * 2) + (ST - 1) * 2) * TILE) + (r < 16 ? r : r - 16) * P; };
   __shared__ int s_last;
   __shared__ float s_ml[WARPS][16][2], s_f[WARPS][16];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = blockIdx.z;
@@ -52,6 +53,8 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
   };
 #pragma unroll
   for (int s = 0; s < ST - 1; ++s) fetch(c0 + warp + s * WARPS, s);
+  if (tid < (a.rd / 2 + 15) / 16)                                     // the rotation's row is needed two barriers from here
+    asm volatile("prefetch.global.L2 [%0];" ::"l"(a.rope + (long long)pos * (a.rd / 2) + 16 * tid));
   // queries; the new key and value
   {
     const int d = a.d, vd = a.vd, taps = in.taps, C = in.C, n_qk = (nq + (fresh ? 1 : 0)) * d, n_all = n_qk + (fresh ? vd : 0);
@@ -59,7 +62,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
     auto place = [&](int i, int& c, float*& dst, bool& keep) {
       const int head = i < n_qk ? i / d : nq + 1, x = i < n_qk ? i - head * d : i - n_qk;
       c = head < nq ? (g * hg + q0 + head) * d + x : head == nq ? (a.H + g) * d + x : (a.H + a.KH) * d + g * vd + x;
-      dst = sConv + (head < nq ? head : head == nq ? 16 : 17) * P + x;
+      dst = sConv(head < nq ? head : head == nq ? 16 : 17) + x;
       keep = head < nq ? blockIdx.x == 0 : q0 == 0;
     };
     bf16* inputs = in.ring + (long long)slot * in.RC * C;
@@ -106,7 +109,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
 #pragma unroll 1
     for (int i = tid; i < (nq + (fresh ? 1 : 0)) * half; i += TH) {
       const int head = i / half, x = i - head * half;
-      const float* src = sConv + (head < nq ? head : 16) * P;
+      const float* src = sConv(head < nq ? head : 16);
       bf16* to = head < nq ? sQ + head * LD : sNew;
       if (x < np) {
         const float2 cs = rope[x];
@@ -118,7 +121,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
       }
     }
     if (fresh)
-      for (int x = tid; x < vd; x += TH) sNew[P + x] = __float2bfloat16_rn(sConv[17 * P + x]);
+      for (int x = tid; x < vd; x += TH) sNew[P + x] = __float2bfloat16_rn(sConv(17)[x]);
     const bf16 zero = __float2bfloat16_rn(0.f);
     for (int i = tid; i < 16 * P; i += TH) {
       const int r = i / P, c = i % P;
@@ -239,21 +242,40 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
     s_ml[0][tid][1] = l;
   }
   __syncthreads();
-  auto finish = [&](int r, int c, float o, float l) {
-    const int h = g * hg + q0 + r;
-    if (c < a.vd) {
-      const float gate = a.col_g >= 0 ? sigmoid_f(in.src.get(row, a.col_g + h * a.vd + c)) : 1.f;
-      reinterpret_cast<bf16*>(a.out)[((long long)row * a.H + h) * a.vd + c] = __float2bfloat16_rn(o / l * gate);
-    }
+  // four columns of a head: divided by the sum, gated, stored
+  const bool vec = a.vd % 4 == 0 && a.col_g % 4 == 0 && in.src.ld % 4 == 0;
+  auto gates = [&](int r, int c) {
+    const int col = a.col_g + (g * hg + q0 + r) * a.vd + c;
+    if (a.col_g < 0 || c >= a.vd) return make_float4(0.f, 0.f, 0.f, 0.f);
+    if (vec) return get4(in.src, row, col);
+    const int last = a.vd - 1 - c;
+    return make_float4(in.src.get_rare(row, col), in.src.get_rare(row, col + min(1, last)), in.src.get_rare(row, col + min(2, last)),
+                       in.src.get_rare(row, col + min(3, last)));
+  };
+  auto finish = [&](int r, int c, float4 o, float l, float4 gt) {
+    if (c >= a.vd) return;
+    const float inv = 1.f / l;
+    float v[4] = {o.x * inv, o.y * inv, o.z * inv, o.w * inv};
+    if (a.col_g >= 0) { v[0] *= sigmoid_f(gt.x); v[1] *= sigmoid_f(gt.y); v[2] *= sigmoid_f(gt.z); v[3] *= sigmoid_f(gt.w); }
+    bf16* out = reinterpret_cast<bf16*>(a.out) + ((long long)row * a.H + g * hg + q0 + r) * a.vd + c;
+    if (vec) store4(out, make_float4(v[0], v[1], v[2], v[3]));
+    else
+      for (int e = 0; e < 4 && c + e < a.vd; ++e) out[e] = __float2bfloat16_rn(v[e]);
   };
   const long long n_rh = (long long)a.rows.M * a.H, rh0 = (long long)row * a.H + g * hg + q0;
-  for (int i = tid; i < nq * P; i += TH) {
-    const int r = i / P, c = i % P;
-    float o = 0.f;
+#pragma unroll 1
+  for (int i = tid; i < nq * (P / 4); i += TH) {
+    const int r = i / (P / 4), c = i % (P / 4) * 4;
+    float4 gt, o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (a.splits == 1) gt = gates(r, c);
 #pragma unroll
-    for (int w = 0; w < WARPS; ++w) o = fmaf(s_f[w][r], sO[(w * 16 + r) * P + c], o);
-    if (a.splits == 1) finish(r, c, o, s_ml[0][r][1]);
-    else a.part_o[((long long)blockIdx.x * n_rh + rh0 + r) * P + c] = o;
+    for (int w = 0; w < WARPS; ++w) {
+      const float4 t = load4(sO + (w * 16 + r) * P + c);
+      const float f = s_f[w][r];
+      o.x = fmaf(f, t.x, o.x); o.y = fmaf(f, t.y, o.y); o.z = fmaf(f, t.z, o.z); o.w = fmaf(f, t.w, o.w);
+    }
+    if (a.splits == 1) finish(r, c, o, s_ml[0][r][1], gt);
+    else store4(a.part_o + ((long long)blockIdx.x * n_rh + rh0 + r) * P + c, o);
   }
   if (a.splits == 1) return;
   if (tid < nq) {
@@ -285,12 +307,19 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
     if (lane == 0) sW[512 + r] = sum;
   }
   __syncthreads();
-  for (int i = tid; i < nq * P; i += TH) {
-    const int r = i / P, c = i % P;
-    float o = 0.f;
-#pragma unroll 4
-    for (int s = 0; s < a.splits; ++s) o = fmaf(sW[s * 16 + r], __ldcg(a.part_o + ((long long)s * n_rh + rh0 + r) * P + c), o);
-    finish(r, c, o, sW[512 + r]);
+#pragma unroll 1
+  for (int i = tid; i < nq * (P / 4); i += TH) {
+    const int r = i / (P / 4), c = i % (P / 4) * 4;
+    const float4 gt = gates(r, c);
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float* part = a.part_o + (rh0 + r) * P + c;
+#pragma unroll 8
+    for (int s = 0; s < a.splits; ++s) {
+      const float4 t = __ldcg(reinterpret_cast<const float4*>(part + s * n_rh * P));
+      const float f = sW[s * 16 + r];
+      o.x = fmaf(f, t.x, o.x); o.y = fmaf(f, t.y, o.y); o.z = fmaf(f, t.z, o.z); o.w = fmaf(f, t.w, o.w);
+    }
+    finish(r, c, o, sW[512 + r], gt);
   }
 }
 
