@@ -220,7 +220,7 @@ struct ConvIn {
       out[i] = activate(acc, c);
     }
   }
-  // The same for channels c .. c + 3 of a source of plain rows (splits 1; col0 + c, the pitch and c multiples of 4).
+  // The same for channels c .. c + 3 of a matrix in the storage dtype (col0 + c, the pitch and c multiples of 4).
   template <int RB>
   __device__ __forceinline__ void run4(int row, int row_end, int r0, int start, int slot, int c, float4 (&out)[RB]) const {
     float wt[4][4];                                     // [tap back][channel]
@@ -257,7 +257,7 @@ struct ConvIn {
       float a[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        auto at = [&](const float4& v) { return round_to<T>(e == 0 ? v.x : e == 1 ? v.y : e == 2 ? v.z : v.w); };
+        auto at = [&](const float4& v) { return e == 0 ? v.x : e == 1 ? v.y : e == 2 ? v.z : v.w; };
         a[e] = at(x[3 + i]) * wt[0][e];
 #pragma unroll
         for (int j = 1; j < 4; ++j) a[e] = fmaf(at(x[3 + i - j]), wt[j][e], a[e]);

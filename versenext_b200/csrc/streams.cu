@@ -366,7 +366,7 @@ int32_t vn_streams_sum(vn_ctx* ctx, const float* x, float* out, int M, int ns, i
 template <typename T>
 int32_t vn_input_conv(vn_ctx* ctx, const ConvIn<T, Mat<T>, false>& in, const Rows& rows, int pending, T* hc) {
   if (in.taps <= 4 && in.C % 4 == 0)
-    VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv4_kernel<T, 4>), dim3(ceil_div(in.C, 1024), ceil_div(rows.M, 4)), 256, 0, in, rows,
+    VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv4_kernel<T, 8>), dim3(ceil_div(in.C, 1024), ceil_div(rows.M, 8)), 256, 0, in, rows,
                     pending, hc);
   else if (in.taps <= 4)
     VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv_kernel<T, 8>), dim3(ceil_div(in.C, 256), ceil_div(rows.M, 8)), 256, 0, in, rows,
