@@ -73,11 +73,11 @@ __global__ void __launch_bounds__(256) attn_inputs_kernel(ConvIn<T, S, false> in
   }
 }
 
-// The same for many rows: a thread takes four channels of RB rows, with the four they are rotated with.  Filters of at most
-// four taps; d, vd, rd / 2 and the source's pitch multiples of 4.  grid (ceil(items / 256), ceil(M / RB)): items of a row
-// are the rotated quads of all heads, the unrotated ones, the values'
+// The same for many rows: a thread takes four channels of `rep` times RB rows, with the four they are rotated with.
+// Filters of at most four taps; d, vd, rd / 2 and the source's pitch multiples of 4.  grid (ceil(items / 256),
+// ceil(M / (rep RB))): items of a row are the rotated quads of all heads, the unrotated ones, the values'
 template <typename T, int RB>
-__global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, false> in, PagedAttnArgs a, int qk_heads, int items) {
+__global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, false> in, PagedAttnArgs a, int qk_heads, int items, int rep) {
   const int it = blockIdx.x * 256 + threadIdx.x;
   if (it >= items) return;
   const int np = a.rd / 2, nr = np / 4, nu = (a.d - a.rd) / 4, nv = a.vd / 4;
@@ -88,15 +88,19 @@ __global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, fal
   else if (it < qk_heads * (nr + nu)) { const int i = it - qk_heads * nr; head = i / nu; c = a.rd + i % nu * 4; }
   else { const int i = it - qk_heads * (nr + nu); is_v = true; head = i / nv; c = i % nv * 4; }
   const int col = is_v ? (a.H + a.KH) * a.d + head * a.vd + c : head * a.d + c;
-  int row = blockIdx.y * RB;
-  const int last = min(row + RB, a.rows.M);
+  int row = blockIdx.y * rep * RB;
+  const int last = min(row + rep * RB, a.rows.M);
+  float wu[4][4], wv[4][4];
+  in.filters4(col, wu);
+  in.filters4(pair ? col + np : col, wv);
+#pragma unroll 1
   while (row < last) {                                     // stretches of one entry
     int slot, r0, n, start;
     a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
-    const int end = min(last, r0 + n);
+    const int end = min(min(last, row + RB), r0 + n);
     float4 u[RB], v[RB];
-    in.template run4<RB>(row, end, r0, start, slot, col, u);
-    if (pair) in.template run4<RB>(row, end, r0, start, slot, col + np, v);
+    in.template run4<RB>(row, end, r0, start, slot, col, wu, u);
+    if (pair) in.template run4<RB>(row, end, r0, start, slot, col + np, wv, v);
 #pragma unroll
     for (int r = 0; r < RB; ++r) {
       if (row + r >= end) break;
@@ -430,8 +434,9 @@ int32_t vn_attn_inputs(vn_ctx* ctx, const ConvIn<T, S, false>& conv, const Paged
   const dim3 block(32, 8);
   if constexpr (std::is_same<S, Mat<T>>::value) {
     if (conv.taps <= 4 && a.d % 4 == 0 && a.vd % 4 == 0 && a.rd % 8 == 0 && conv.src.ld % 4 == 0) {
+      const int rep = a.rows.M >= 2048 ? 4 : 1;
       const int qk = a.H + (a.own_kv ? a.KH : 0), items = qk * (a.d - a.rd / 2) / 4 + (a.own_kv ? a.KH * a.vd / 4 : 0);
-      VN_LAUNCH_NAMED(ctx, "attn_inputs_kernel", (attn_inputs4_kernel<T, 4>), dim3(ceil_div(items, 256), ceil_div(a.rows.M, 4)), 256, 0, conv, a, qk, items);
+      VN_LAUNCH_NAMED(ctx, "attn_inputs_kernel", (attn_inputs4_kernel<T, 4>), dim3(ceil_div(items, 256), ceil_div(a.rows.M, 4 * rep)), 256, 0, conv, a, qk, items, rep);
       return VN_OK;
     }
   }

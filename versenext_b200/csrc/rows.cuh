@@ -221,9 +221,8 @@ struct ConvIn {
     }
   }
   // The same for channels c .. c + 3 of a matrix in the storage dtype (col0 + c, the pitch and c multiples of 4).
-  template <int RB>
-  __device__ __forceinline__ void run4(int row, int row_end, int r0, int start, int slot, int c, float4 (&out)[RB]) const {
-    float wt[4][4];                                     // [tap back][channel]
+  // wt: filters4(c), [tap back][channel].
+  __device__ __forceinline__ void filters4(int c, float (&wt)[4][4]) const {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float* wc = w + (long long)(c + e) * taps;
@@ -235,6 +234,10 @@ struct ConvIn {
         for (int j = 0; j < 4; ++j) wt[j][e] = j < taps ? wc[taps - 1 - j] : 0.f;
       }
     }
+  }
+  template <int RB>
+  __device__ __forceinline__ void run4(int row, int row_end, int r0, int start, int slot, int c, const float (&wt)[4][4],
+                                       float4 (&out)[RB]) const {
     float4 x[RB + 3];
     const auto* p = src.p + (long long)row * src.ld + col0 + c;
 #pragma unroll

@@ -301,19 +301,22 @@ __global__ void __launch_bounds__(256) input_conv_kernel(ConvIn<T, Mat<T>, false
   }
 }
 
-// four channels per thread, filters of at most four taps.  grid (ceil(D / 1024), ceil(M / RB))
+// four channels per thread, `rep` times RB rows, filters of at most four taps.  grid (ceil(D / 1024), ceil(M / (rep RB)))
 template <typename T, int RB>
-__global__ void __launch_bounds__(256) input_conv4_kernel(ConvIn<T, Mat<T>, false> in, Rows rows, int pending, T* __restrict__ hc) {
+__global__ void __launch_bounds__(256) input_conv4_kernel(ConvIn<T, Mat<T>, false> in, Rows rows, int pending, int rep, T* __restrict__ hc) {
   const int c = (blockIdx.x * 256 + threadIdx.x) * 4, D = in.C;
   if (c >= D) return;
-  int row = blockIdx.y * RB;
-  const int last = min(row + RB, rows.M);
+  int row = blockIdx.y * rep * RB;
+  const int last = min(row + rep * RB, rows.M);
+  float wt[4][4];
+  in.filters4(c, wt);
+#pragma unroll 1
   while (row < last) {                                  // stretches of one entry
     int slot, r0, n, start;
     rows.entry(rows.entry_of(row), &slot, &r0, &n, &start);
-    const int end = min(last, r0 + n);
+    const int end = min(min(last, row + RB), r0 + n);
     float4 v[RB];
-    in.template run4<RB>(row, end, r0, start, slot, c, v);
+    in.template run4<RB>(row, end, r0, start, slot, c, wt, v);
 #pragma unroll
     for (int i = 0; i < RB; ++i)
       if (row + i < end) {
@@ -365,9 +368,10 @@ int32_t vn_streams_sum(vn_ctx* ctx, const float* x, float* out, int M, int ns, i
 
 template <typename T>
 int32_t vn_input_conv(vn_ctx* ctx, const ConvIn<T, Mat<T>, false>& in, const Rows& rows, int pending, T* hc) {
+  const int rep = rows.M >= 2048 ? 2 : 1;
   if (in.taps <= 4 && in.C % 4 == 0)
-    VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv4_kernel<T, 8>), dim3(ceil_div(in.C, 1024), ceil_div(rows.M, 8)), 256, 0, in, rows,
-                    pending, hc);
+    VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv4_kernel<T, 8>), dim3(ceil_div(in.C, 1024), ceil_div(rows.M, 8 * rep)), 256, 0, in,
+                    rows, pending, rep, hc);
   else if (in.taps <= 4)
     VN_LAUNCH_NAMED(ctx, "input_conv_kernel", (input_conv_kernel<T, 8>), dim3(ceil_div(in.C, 256), ceil_div(rows.M, 8)), 256, 0, in, rows,
                     pending, hc);
