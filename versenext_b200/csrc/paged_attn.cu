@@ -134,10 +134,10 @@ __global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, fal
   }
 }
 
-// ---- one warp per (row, head), any dtype; NR = values per lane (P <= 32 NR).  grid (ceil(H / 8), M) --------------------
+// ---- one warp per (row, head), any dtype; NR = values per lane (P <= 32 NR).  grid (M, ceil(H / 8)) --------------------
 template <typename T, typename S, int NR>
 __global__ void __launch_bounds__(256) paged_attn_kernel(PagedAttnArgs a, S proj) {
-  const int h = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, row = blockIdx.y;
+  const int h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, row = blockIdx.x;
   if (h >= a.H) return;
   int slot, r0, n, start;
   a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
@@ -394,7 +394,7 @@ int32_t launch_mma(vn_ctx* ctx, const PagedAttnArgs& a, const S& proj) {
 
 template <typename T, typename S>
 int32_t launch_simt(vn_ctx* ctx, const PagedAttnArgs& a, const S& proj) {
-  const dim3 grid(ceil_div(a.H, 8), a.rows.M);
+  const dim3 grid(a.rows.M, ceil_div(a.H, 8));
   const int nr = a.P / 32;
 #define PA(NR) VN_LAUNCH_NAMED(ctx, "paged_attn_kernel", (paged_attn_kernel<T, S, NR>), grid, 256, 0, a, proj)
   if (nr <= 2) PA(2); else if (nr <= 4) PA(4); else if (nr <= 8) PA(8); else PA(32);
