@@ -291,7 +291,7 @@ int32_t vn_model_status(vn_model* m, int32_t* bad_token, int32_t* wait_timeout);
  * its latents. */
 int32_t vn_kv_create(vn_model* m, int32_t max_batch, int32_t max_seq, vn_kv** out);
 /* The same with the cache of a composed model (a configuration with "family": "composed", see vn_model_create) sized
- * explicitly.  pool_tokens > 0: latents live in a pool of pages for that many tokens (rounded up to pages of 64) shared
+ * explicitly.  pool_tokens > 0: latents, keys and values live in a pool of pages for that many tokens (rounded up to pages of 64) shared
  * by all sequences; a sequence takes pages as it grows and gives them back when it is reset.  0: every sequence owns
  * the pages of max_seq positions.  max_pending: rows a sequence may append and cut back with vn_kv_commit; the cache
  * keeps that many recurrent states besides the committed one.  A longer append (a prompt) can only be kept whole. */
