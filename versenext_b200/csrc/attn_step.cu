@@ -24,12 +24,12 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
   // convolved channels: query heads 0 .. 15, key (16), value (17); they lie in ring stages that no prefetch has reached yet
   auto sConv = [&](int r) { return reinterpret_cast<float*>(ring + ((r < 16 ? 0 : ST * 2) + (ST - 1) * 2) * TILE) + (r < 16 ? r : r - 16) * P; };
   __shared__ int s_last;
-  __shared__ float s_ml[WARPS][16][2], s_f[WARPS][16];
+  __shared__ float s_ml[WARPS][16][2], s_f[WARPS][16], s_norm[17];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = blockIdx.z;
   const int hg = a.H / a.KH, tiles = (hg + 15) / 16, g = blockIdx.y / tiles, q0 = (blockIdx.y % tiles) * 16, nq = min(16, hg - q0);
   int slot, r0, n, pos;
   a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &pos);
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = a.first_key(pos);
   const int c_lo = lo / 16, c_hi = pos / 16 + 1, per = (c_hi - c_lo + a.splits - 1) / a.splits;
   const int c0 = min(c_hi, c_lo + (int)blockIdx.x * per), c1 = min(c_hi, c0 + per);
   const bool fresh = a.own_kv && c0 < c1 && c1 == c_hi;               // this range ends with the new token
@@ -91,6 +91,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
             acc.x = fmaf(x[j].x, w[-j], acc.x); acc.y = fmaf(x[j].y, w[taps - j], acc.y);
             acc.z = fmaf(x[j].z, w[2 * taps - j], acc.z); acc.w = fmaf(x[j].w, w[3 * taps - j], acc.w);
           }
+        if (in.bias) { const float4 b = load4(in.bias + c); acc.x += b.x; acc.y += b.y; acc.z += b.z; acc.w += b.w; }
         store4(dst, acc);
       }
     } else {
@@ -103,6 +104,17 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
       }
     }
     __syncthreads();
+    if (a.qn) {                                                       // factors of the heads' norms
+#pragma unroll 1
+      for (int head = warp; head < nq + (fresh ? 1 : 0); head += WARPS) {
+        const float* src = sConv(head < nq ? head : 16);
+        float ss = 0.f;
+        for (int x = lane; x < d; x += 32) ss = fmaf(src[x], src[x], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) s_norm[head] = 1.f / sqrtf(ss / (float)d + a.eps);
+      }
+      __syncthreads();
+    }
     // rotation of the queries and the key
     const int np = a.rd / 2, half = np + d - a.rd;
     const float2* rope = a.rope + (long long)pos * np;
@@ -111,14 +123,16 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
       const int head = i / half, x = i - head * half;
       const float* src = sConv(head < nq ? head : 16);
       bf16* to = head < nq ? sQ + head * LD : sNew;
-      if (x < np) {
-        const float2 cs = rope[x];
-        const float u = src[x], v = src[np + x];
-        to[x] = __float2bfloat16_rn(u * cs.x - v * cs.y);
-        to[np + x] = __float2bfloat16_rn(v * cs.x + u * cs.y);
-      } else {
-        to[np + x] = __float2bfloat16_rn(src[np + x]);
+      const int cu = x >= np ? np + x : a.interleaved ? 2 * x : x, cv = x >= np ? cu : a.interleaved ? 2 * x + 1 : np + x;
+      float u = src[cu], v = src[cv];
+      if (a.qn) {
+        const float* nw = head < nq ? a.qn : a.kn;
+        u *= s_norm[head] * nw[cu];
+        v *= s_norm[head] * nw[cv];
       }
+      const float2 cs = x < np ? rope[x] : make_float2(1.f, 0.f);
+      to[cu] = __float2bfloat16_rn(u * cs.x - v * cs.y);
+      if (x < np) to[cv] = __float2bfloat16_rn(v * cs.x + u * cs.y);
     }
     if (fresh)
       for (int x = tid; x < vd; x += TH) sNew[P + x] = __float2bfloat16_rn(sConv(17)[x]);
@@ -177,7 +191,8 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int key = 16 * c + 8 * j + (lane & 3) * 2 + (x & 1);
-        s[j][x] = key >= lo && key <= pos ? s[j][x] * sc : -CUDART_INF_F;
+        const float v = a.softcap > 0.f ? softcap_log2(s[j][x] * a.scale, a.softcap) : s[j][x] * sc;
+        s[j][x] = key >= lo && key <= pos ? v : -CUDART_INF_F;
         mx[x >> 1] = fmaxf(mx[x >> 1], s[j][x]);
       }
     float f[2];

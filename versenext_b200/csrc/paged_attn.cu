@@ -1,4 +1,5 @@
 // Kernels of paged_attn.cuh for prompts and mixed batches; the one-token kernel is in attn_step.cu.
+#include <algorithm>
 #include <type_traits>
 
 #include "ldmatrix.cuh"
@@ -51,19 +52,20 @@ __global__ void __launch_bounds__(256) attn_inputs_kernel(ConvIn<T, S, false> in
     };
     for (int i = lane; i < items; i += 32) {
       const bool pair = i < np;
+      const int cu = !pair ? np + i : a.interleaved ? 2 * i : i, cv = a.interleaved ? 2 * i + 1 : np + i;
       float u[RB], v[RB];
-      convolve(pair ? i : np + i, u);
-      if (pair) convolve(np + i, v);
+      convolve(cu, u);
+      if (pair) convolve(cv, v);
 #pragma unroll
       for (int r = 0; r < RB; ++r) {
         if (first + r >= end) break;
         T* dst = dest(first + r);
         if (pair) {
           const float2 cs = a.rope[(long long)(start + first + r - r0) * np + i];
-          dst[i] = from_f<T>(u[r] * cs.x - v[r] * cs.y);
-          dst[np + i] = from_f<T>(v[r] * cs.x + u[r] * cs.y);
+          dst[cu] = from_f<T>(u[r] * cs.x - v[r] * cs.y);
+          dst[cv] = from_f<T>(v[r] * cs.x + u[r] * cs.y);
         } else {
-          dst[np + i] = from_f<T>(u[r]);
+          dst[cu] = from_f<T>(u[r]);
         }
       }
     }
@@ -134,6 +136,97 @@ __global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, fal
   }
 }
 
+// Heads with a norm (or interleaved pairs), without convolutions: bias, norm, rotation.  One warp per (row, unit) with the
+// head staged in shared memory; units as above.  grid (units, ceil(M / 8)), block (32, 8), 8 max(d, vd) floats
+template <typename T, typename S>
+__global__ void __launch_bounds__(256) attn_heads_kernel(ConvIn<T, S, false> in, PagedAttnArgs a) {
+  extern __shared__ __align__(16) float s_head[];
+  const int lane = threadIdx.x, unit = blockIdx.x, row = blockIdx.y * 8 + threadIdx.y;
+  if (row >= a.rows.M) return;
+  float* s = s_head + threadIdx.y * max(a.d, a.vd);
+  const bool is_q = unit < a.H, is_v = unit >= a.H + a.KH;
+  const int head = is_q ? unit : is_v ? unit - a.H - a.KH : unit - a.H, w = is_v ? a.vd : a.d, np = is_v ? 0 : a.rd / 2;
+  const int c0 = is_v ? (a.H + a.KH) * a.d + head * a.vd : unit * a.d;
+  const float* nw = is_v ? nullptr : is_q ? a.qn : a.kn;
+  int slot, r0, n, start;
+  a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
+  const int pos = start + row - r0;
+  float ss = 0.f;
+  for (int c = lane; c < w; c += 32) {
+    const float v = round_to<T>(in.src.get(row, in.col0 + c0 + c)) + (in.bias ? in.bias[c0 + c] : 0.f);
+    s[c] = v;
+    ss += v * v;
+  }
+  const float r = nw ? 1.f / sqrtf(warp_sum(ss) / (float)w + a.eps) : 1.f;
+  __syncwarp();
+  T* dst = is_q ? reinterpret_cast<T*>(a.q) + ((long long)row * a.H + head) * a.P
+                : reinterpret_cast<T*>(is_v ? a.vplane : a.kplane) +
+                      (((long long)a.table[(long long)slot * a.max_pages + pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.KH + head) * a.P;
+  auto value = [&](int c) { return nw ? s[c] * r * nw[c] : s[c]; };
+  for (int i = lane; i < w - np; i += 32) {
+    if (i < np) {
+      const int cu = a.interleaved ? 2 * i : i, cv = a.interleaved ? 2 * i + 1 : np + i;
+      const float u = value(cu), v = value(cv);
+      const float2 cs = a.rope[(long long)pos * np + i];
+      dst[cu] = from_f<T>(u * cs.x - v * cs.y);
+      dst[cv] = from_f<T>(v * cs.x + u * cs.y);
+    } else {
+      dst[np + i] = from_f<T>(value(np + i));
+    }
+  }
+  for (int c = w + lane; c < a.P; c += 32) dst[c] = from_f<T>(0.f);
+}
+
+// The same for interleaved pairs and heads of at most 128: W lanes take a head, four channels each, of RB rows at once.
+// d, vd, rd and the source's pitch multiples of 4.  grid (ceil(units / (32 / W)), ceil(M / (8 RB))), block (32, 8)
+template <typename T, typename S, int W, int RB>
+__global__ void __launch_bounds__(256) attn_heads4_kernel(ConvIn<T, S, false> in, PagedAttnArgs a, int units) {
+  const int l = threadIdx.x % W, unit = blockIdx.x * (32 / W) + threadIdx.x / W, row0 = (blockIdx.y * 8 + threadIdx.y) * RB;
+  if (row0 >= a.rows.M) return;
+  const bool live = unit < units, is_q = unit < a.H, is_v = unit >= a.H + a.KH;
+  const int head = is_q ? unit : is_v ? unit - a.H - a.KH : unit - a.H, w = is_v ? a.vd : a.d, np = is_v ? 0 : a.rd / 2, c = 4 * l;
+  const int c0 = (is_v ? (a.H + a.KH) * a.d + head * a.vd : unit * a.d) + c;
+  const float* nw = is_v ? nullptr : is_q ? a.qn : a.kn;
+  const bool mine = live && c < w;
+  float4 x[RB], b = make_float4(0.f, 0.f, 0.f, 0.f), wt = make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll
+  for (int r = 0; r < RB; ++r)
+    x[r] = mine ? get4(in.src, min(row0 + r, a.rows.M - 1), in.col0 + c0) : make_float4(0.f, 0.f, 0.f, 0.f);
+  if (mine && in.bias) b = load4(in.bias + c0);
+  if (mine && nw) wt = load4(nw + c);
+  float ss[RB];
+#pragma unroll
+  for (int r = 0; r < RB; ++r) {
+    x[r] = make_float4(round_to<T>(x[r].x) + b.x, round_to<T>(x[r].y) + b.y, round_to<T>(x[r].z) + b.z, round_to<T>(x[r].w) + b.w);
+    ss[r] = x[r].x * x[r].x + x[r].y * x[r].y + x[r].z * x[r].z + x[r].w * x[r].w;
+  }
+#pragma unroll
+  for (int o = W / 2; o > 0; o >>= 1)
+#pragma unroll
+    for (int r = 0; r < RB; ++r) ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], o);
+#pragma unroll
+  for (int r = 0; r < RB; ++r) {
+    const int row = row0 + r;
+    if (row >= a.rows.M || !live || c >= a.P) break;
+    int slot, r0, n, start;
+    a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
+    const int pos = start + row - r0;
+    T* dst = is_q ? reinterpret_cast<T*>(a.q) + ((long long)row * a.H + head) * a.P
+                  : reinterpret_cast<T*>(is_v ? a.vplane : a.kplane) +
+                        (((long long)a.table[(long long)slot * a.max_pages + pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.KH + head) * a.P;
+    float4 v = x[r];
+    if (nw) {
+      const float f = 1.f / sqrtf(ss[r] / (float)w + a.eps);
+      v = make_float4(v.x * f * wt.x, v.y * f * wt.y, v.z * f * wt.z, v.w * f * wt.w);
+    }
+    if (c < 2 * np) {
+      const float4 cs = *reinterpret_cast<const float4*>(a.rope + (long long)pos * np + 2 * l);
+      v = make_float4(v.x * cs.x - v.y * cs.y, v.y * cs.x + v.x * cs.y, v.z * cs.z - v.w * cs.w, v.w * cs.z + v.z * cs.w);
+    }
+    store4(dst + c, v);                                    // pads too: their quads are zero
+  }
+}
+
 // ---- one warp per (row, head), any dtype; NR = values per lane (P <= 32 NR).  grid (M, ceil(H / 8)) --------------------
 template <typename T, typename S, int NR>
 __global__ void __launch_bounds__(256) paged_attn_kernel(PagedAttnArgs a, S proj) {
@@ -142,7 +235,7 @@ __global__ void __launch_bounds__(256) paged_attn_kernel(PagedAttnArgs a, S proj
   int slot, r0, n, start;
   a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
   const int pos = start + row - r0, g = h / (a.H / a.KH);
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = a.first_key(pos);
   const T* q = reinterpret_cast<const T*>(a.q) + ((long long)row * a.H + h) * a.P;
   const int* tab = a.table + (long long)slot * a.max_pages;
   float qv[NR], acc[NR];
@@ -165,6 +258,7 @@ __global__ void __launch_bounds__(256) paged_attn_kernel(PagedAttnArgs a, S proj
       vv[i] = j < a.vd ? to_f<T>(v[j]) : 0.f;
     }
     s = warp_sum(s) * a.scale;
+    if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
     const float m2 = fmaxf(m, s), f = expf(m - m2), e = expf(s - m2);
     l = l * f + e;
 #pragma unroll
@@ -205,7 +299,7 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int f_last = min(f0 + ROWS, nf) - 1;
   const int p_lo = start + f0 / hg, p_hi = start + f_last / hg;
-  const int pg0 = (a.window > 0 ? max(0, p_lo - a.window + 1) : 0) / KV_PAGE, pg1 = p_hi / KV_PAGE + 1;
+  const int pg0 = a.first_key(p_lo) / KV_PAGE, pg1 = p_hi / KV_PAGE + 1;
   const int* tab = a.table + (long long)slot * a.max_pages;
   const long long ldp = (long long)a.KH * P;
   const bf16 *kp = reinterpret_cast<const bf16*>(a.kplane) + (long long)g * P, *vp = reinterpret_cast<const bf16*>(a.vplane) + (long long)g * P;
@@ -243,21 +337,23 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
   float m_run[2] = {-CUDART_INF_F, -CUDART_INF_F}, l_run[2] = {0.f, 0.f};
-  int rp[2];                                              // positions of rows lane / 4 and lane / 4 + 8; -1 beyond the entry
+  int rp[2], rk[2];                                       // positions of rows lane / 4 and lane / 4 + 8 (-1 beyond the entry), their first keys
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
     const int f = f0 + 16 * warp + (lane >> 2) + 8 * e;
     rp[e] = f < nf ? start + f / hg : -1;
+    rk[e] = f < nf ? a.first_key(rp[e]) : 0;
   }
   const int w_lo = start + min(f0 + 16 * warp, nf - 1) / hg, w_hi = start + min(f0 + 16 * warp + 15, nf - 1) / hg;
+  const int k_lo = a.first_key(w_lo), k_hi = a.first_key(w_hi);
   const float sc = a.scale * 1.4426950408889634f;
   fetch(pg0, 0);
   for (int pg = pg0, buf = 0; pg < pg1; ++pg, buf ^= 1) {
     if (pg + 1 < pg1) { fetch(pg + 1, buf ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
     __syncthreads();
     const bf16 *K = sK + buf * KV_PAGE * LD, *V = sV + buf * KV_PAGE * LD;
-    // nothing of this page is visible to the warp's rows: keys all later, or all out of the window
-    const bool skip = pg * KV_PAGE > w_hi || (a.window > 0 && pg * KV_PAGE + KV_PAGE - 1 <= w_lo - a.window);
+    // nothing of this page is visible to the warp's rows: keys all later, or all before the first one
+    const bool skip = pg * KV_PAGE > w_hi || pg * KV_PAGE + KV_PAGE <= k_lo;
     if (!skip) {
       float s[8][4];
 #pragma unroll
@@ -282,17 +378,17 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
           mma_bf16(s[2 * j + 1], af, b1);
         }
       }
-      const bool whole = pg * KV_PAGE + KV_PAGE - 1 <= w_lo && (a.window <= 0 || w_hi - pg * KV_PAGE < a.window);
+      const bool whole = pg * KV_PAGE + KV_PAGE - 1 <= w_lo && pg * KV_PAGE >= k_hi;
       float mx[2] = {m_run[0], m_run[1]};
 #pragma unroll
       for (int j = 0; j < 8; ++j)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
           const int e = x >> 1;
-          float v = s[j][x] * sc;
+          float v = a.softcap > 0.f ? softcap_log2(s[j][x] * a.scale, a.softcap) : s[j][x] * sc;
           if (!whole) {
-            const int dist = rp[e] - (pg * KV_PAGE + 8 * j + (lane & 3) * 2 + (x & 1));
-            if (dist < 0 || (a.window > 0 && dist >= a.window)) v = -CUDART_INF_F;
+            const int key = pg * KV_PAGE + 8 * j + (lane & 3) * 2 + (x & 1);
+            if (key > rp[e] || key < rk[e]) v = -CUDART_INF_F;
           }
           s[j][x] = v;
           mx[e] = fmaxf(mx[e], v);
@@ -432,8 +528,24 @@ template <typename T, typename S>
 int32_t vn_attn_inputs(vn_ctx* ctx, const ConvIn<T, S, false>& conv, const PagedAttnArgs& a) {
   const int units = a.H + (a.own_kv ? 2 * a.KH : 0);
   const dim3 block(32, 8);
+  if (a.qn || conv.bias) {
+    VN_REQUIRE(ctx, conv.taps == 1, "norms and biases of the heads stand without convolutions");
+    const int w = std::max(a.d, a.vd);
+    if (a.d % 4 == 0 && a.vd % 4 == 0 && a.rd % 4 == 0 && conv.src.ld % 4 == 0 && w <= 128 && (a.interleaved || !a.rd)) {
+      const bool many = a.rows.M >= 512;
+#define HEADS(W, RB) VN_LAUNCH_NAMED(ctx, "attn_heads_kernel", (attn_heads4_kernel<T, S, W, RB>), \
+                                     dim3(ceil_div(units, 32 / W), ceil_div(a.rows.M, 8 * RB)), block, 0, conv, a, units)
+#define HEADS1(W) do { if (many) HEADS(W, 4); else HEADS(W, 1); } while (0)
+      if (w <= 32) HEADS1(8); else if (w <= 64) HEADS1(16); else HEADS1(32);
+#undef HEADS1
+#undef HEADS
+      return VN_OK;
+    }
+    VN_LAUNCH_NAMED(ctx, "attn_heads_kernel", (attn_heads_kernel<T, S>), dim3(units, ceil_div(a.rows.M, 8)), block, (size_t)8 * w * 4, conv, a);
+    return VN_OK;
+  }
   if constexpr (std::is_same<S, Mat<T>>::value) {
-    if (conv.taps <= 4 && a.d % 4 == 0 && a.vd % 4 == 0 && a.rd % 8 == 0 && conv.src.ld % 4 == 0) {
+    if (conv.taps <= 4 && a.d % 4 == 0 && a.vd % 4 == 0 && a.rd % 8 == 0 && conv.src.ld % 4 == 0 && !a.interleaved) {
       const int rep = a.rows.M >= 2048 ? 4 : 1;
       const int qk = a.H + (a.own_kv ? a.KH : 0), items = qk * (a.d - a.rd / 2) / 4 + (a.own_kv ? a.KH * a.vd / 4 : 0);
       VN_LAUNCH_NAMED(ctx, "attn_inputs_kernel", (attn_inputs4_kernel<T, 4>), dim3(ceil_div(items, 256), ceil_div(a.rows.M, 4 * rep)), 256, 0, conv, a, qk, items, rep);
