@@ -30,6 +30,7 @@ struct GemmArgs {
   int act = 0;                    // gate activation of EPI_SWIGLU: 0 silu, 1 gelu (tanh form)
   int post = 0;                   // EPI_STORE: function of columns [0, post_n): 0 none, POST_SILU, POST_RELU2
   int post_n = 0;
+  const void* mul = nullptr;      // EPI_STORE, plain and batched modes: factors of the results, laid out and typed as C
   const char* tag = nullptr;      // name of the call site in the per-kernel timing report (string literal)
   // weight-only quantisation: W points at INT8 / packed INT4 bytes, ldw and w_stride stay in ELEMENTS
   int wq = 0;                     // 0 dense, 1 int8, 2 int4 per output row, 3 int4 with one scale per 128 inputs
@@ -56,6 +57,10 @@ __device__ __forceinline__ float gelu_tanh(float x) {
   return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
 }
 __device__ __forceinline__ float glu_act(float x, int act) { return act ? gelu_tanh(x) : silu_ref(x); }
+
+__device__ __forceinline__ float mul_at(const GemmArgs& g, long long idx) {
+  return g.c_bf16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(g.mul)[idx]) : reinterpret_cast<const float*>(g.mul)[idx];
+}
 
 template <typename T>
 __device__ __forceinline__ void store_out(void* C, long long idx, float v, int c_bf16) {
@@ -136,6 +141,7 @@ __global__ void __launch_bounds__(256) gemm_nt_simt_kernel(GemmArgs g) {
         if (g.bias) v += g.bias[n];
         if (n < g.post_n) v = post_act(v, g.post, g.c_bf16);
         const long long idx = c_base + crow * g.ldc + n;
+        if (g.mul) v *= mul_at(g, idx);
         if (g.epi == EPI_ADD) reinterpret_cast<float*>(g.C)[idx] += v;
         else store_out<float>(g.C, idx, v, g.c_bf16);
       }

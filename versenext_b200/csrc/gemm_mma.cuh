@@ -141,12 +141,16 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
         float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
         if (n < g.post_n) v0 = post_act(v0, g.post, g.c_bf16);       // no bias goes with it
         if (n + 1 < g.post_n) v1 = post_act(v1, g.post, g.c_bf16);
+        if (g.mul) {                                                 // nor with this
+          if (n < g.N) v0 *= mul_at(g, crow + n);
+          if (n + 1 < g.N) v1 *= mul_at(g, crow + n + 1);
+        }
         if (g.epi == EPI_SWIGLU) {
           if (n + 1 < g.N) store_out<float>(g.C, crow + (n >> 1), glu_act(v0, g.act) * v1, g.c_bf16);
         } else if (g.epi == EPI_ADD) {
           float* c = reinterpret_cast<float*>(g.C) + crow + n;
-          if (n < g.N) c[0] += v0;
-          if (n + 1 < g.N) c[1] += v1;
+          if (n < g.N) c[0] += v0 + (g.bias ? g.bias[n] : 0.f);
+          if (n + 1 < g.N) c[1] += v1 + (g.bias ? g.bias[n + 1] : 0.f);
         } else if (g.c_bf16 && !g.bias && n + 1 < g.N && ((crow + n) & 1) == 0) {
           *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(g.C) + crow + n) = __floats2bfloat162_rn(v0, v1);
         } else {

@@ -372,9 +372,10 @@ __device__ __forceinline__ void tc_epilogue_chunk(const TcArgs& g, const unsigne
     } else if (MODE == TC_ADD) {
       if (n < g.N) {
         float* dst = reinterpret_cast<float*>(g.C) + (long long)(row0 + m0) * g.ldc + n;
+        const float bias = g.bias ? g.bias[n] : 0.f;
 #pragma unroll
         for (int i = 0; i < 32; ++i)
-          if (i < mrem) dst[(long long)i * g.ldc] += __uint_as_float(r[i]);
+          if (i < mrem) dst[(long long)i * g.ldc] += __uint_as_float(r[i]) + bias;
       }
     } else {
       if (n < g.N) {

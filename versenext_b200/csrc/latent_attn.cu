@@ -47,8 +47,10 @@ int32_t vn_latent_attention(vn_ctx* ctx, const LatentArgs& a, bool bf16, bool mm
     case 4: st = launch_rows<4>(ctx, a); break;
     case 6: st = launch_rows<6>(ctx, a); break;
     case 8: st = launch_rows<8>(ctx, a); break;
+    case 10: st = launch_rows<10>(ctx, a); break;
     case 12: st = launch_rows<12>(ctx, a); break;
     case 16: st = launch_rows<16>(ctx, a); break;
+    case 18: st = launch_rows<18>(ctx, a); break;
     default: return vn_fail(ctx, VN_ERR_UNSUPPORTED, "latent pitch %d", a.Rp);
   }
   if (st != VN_OK || a.splits <= 1) return st;

@@ -3,7 +3,8 @@
 // With k_h = W_uk,h c and v_h = W_uv,h c the score (q_h . k_h) equals (W_uk,h^T q_h) . c and the output W_uv,h (sum_j p_j
 // c_j), so the queries are carried into the latent space once and attention runs on c itself (all heads share the keys:
 // heads and tokens together are the rows of one matrix product).  Sliding window, a learned sink per head in the
-// denominator, an output gate per head; scores, soft-max and gate in fp32.
+// denominator, an output gate per head; scores, soft-max and gate in fp32.  A key may have a rotated part that all heads
+// share: it stands behind the latent in the cached row, the query's rotated part behind the carried query.
 //
 // Cache: pages of KV_PAGE tokens, plane[page * KV_PAGE + pos % KV_PAGE][Rp]; table[slot * max_pages + pos / KV_PAGE].
 #pragma once
@@ -28,15 +29,28 @@ struct LatentArgs {
   Rows rows;
 };
 
-// latent of the row: RMS norm with a plain weight, appended to its page; queries to the storage dtype (head pitch dp);
-// sigmoid of the gates.  src columns: q [H d] | latent [R] | gate [H].  grid M
+// Inputs of the attention.  src columns: q [H][d | rr] | latent [R] | rotated key [rr] | gates [n_gate]
+struct LatentIn {
+  int H = 0, d = 0, dp = 0, rr = 0, R = 0, Rp = 0;
+  const float2* rope = nullptr;    // [positions][rr / 2]: pairs of neighbours
+  const float* norm_w = nullptr;
+  float eps = 0.f;
+  int n_gate = 0;
+  float* gate = nullptr;           // [M, n_gate] sigmoid of the gates, or null
+  void* gate_t = nullptr;          // the same in the storage dtype, or null
+  void* q = nullptr;               // [M, H, dp] storage dtype
+  void* qc = nullptr;              // [M, H, Rp]: columns from R on (rr > 0)
+  void* plane = nullptr;
+  const int* table = nullptr;
+  int max_pages = 0;
+};
+
+// latent of the row: RMS norm with a plain weight, appended to its page with the rotated key; queries to the storage dtype
+// (head pitch dp), their rotated parts to their places behind the carried queries; sigmoid of the gates.  grid M
 template <typename T>
-__global__ void __launch_bounds__(256) latent_append_kernel(Src src, int H, int d, int dp, int R, int Rp,
-                                                            const float* __restrict__ norm_w, float eps,
-                                                            T* __restrict__ q, float* __restrict__ gate,
-                                                            T* __restrict__ plane, const int* __restrict__ table,
-                                                            int max_pages, Rows rows) {
+__global__ void __launch_bounds__(256) latent_append_kernel(Src src, LatentIn a, Rows rows) {
   __shared__ float sm[8];
+  const int H = a.H, d = a.d, dp = a.dp, rr = a.rr, R = a.R, Rp = a.Rp, max_pages = a.max_pages, qd = d + rr, np = rr / 2;
   extern __shared__ float s_c[];
   const int row = blockIdx.x;
   int slot, r0, n, start;
@@ -44,22 +58,50 @@ __global__ void __launch_bounds__(256) latent_append_kernel(Src src, int H, int 
   const int pos = start + row - r0;
   float ss = 0.f;
   for (int j = threadIdx.x; j < R; j += 256) {
-    const float v = src.get(row, H * d + j);
+    const float v = src.get(row, H * qd + j);
     s_c[j] = v;
     ss += v * v;
   }
-  const float r = sqrtf(block_sum256(ss, sm) / (float)R + eps);
+  const float2* rope = a.rope + (long long)pos * np;
+  // pair i of the rr values from column c on, rotated by the row's position
+  auto rotated = [&](int c, int i) {
+    const float u = src.get(row, c + 2 * i), v = src.get(row, c + 2 * i + 1);
+    const float2 cs = rope[i];
+    return make_float2(u * cs.x - v * cs.y, v * cs.x + u * cs.y);
+  };
+  const float r = sqrtf(block_sum256(ss, sm) / (float)R + a.eps);
   const int pg = pos / KV_PAGE;
   if (pg < max_pages) {
-    T* dst = plane + ((long long)table[(long long)slot * max_pages + pg] * KV_PAGE + pos % KV_PAGE) * Rp;
-    for (int j = threadIdx.x; j < Rp; j += 256) dst[j] = from_f<T>(j < R ? s_c[j] / r * norm_w[j] : 0.f);
+    T* dst = reinterpret_cast<T*>(a.plane) + ((long long)a.table[(long long)slot * max_pages + pg] * KV_PAGE + pos % KV_PAGE) * Rp;
+    for (int j = threadIdx.x; j < Rp; j += 256)
+      if (j < R || j >= R + rr) dst[j] = from_f<T>(j < R ? s_c[j] / r * a.norm_w[j] : 0.f);
+    for (int i = threadIdx.x; i < np; i += 256) {
+      const float2 v = rotated(H * qd + R, i);
+      dst[R + 2 * i] = from_f<T>(v.x);
+      dst[R + 2 * i + 1] = from_f<T>(v.y);
+    }
   }
+  T* q = reinterpret_cast<T*>(a.q) + (long long)row * H * dp;
   for (int i = threadIdx.x; i < H * dp; i += 256) {
     const int h = i / dp, j = i % dp;
-    q[(long long)row * H * dp + i] = from_f<T>(j < d ? src.get(row, h * d + j) : 0.f);
+    q[i] = from_f<T>(j < d ? src.get(row, h * qd + j) : 0.f);
   }
-  if (gate)
-    for (int h = threadIdx.x; h < H; h += 256) gate[(long long)row * H + h] = sigmoid_f(src.get(row, H * d + R + h));
+  if (rr) {
+    T* qc = reinterpret_cast<T*>(a.qc) + (long long)row * H * Rp;
+    for (int i = threadIdx.x; i < H * np; i += 256) {
+      const int h = i / np, j = i % np;
+      const float2 v = rotated(h * qd + d, j);
+      qc[h * Rp + R + 2 * j] = from_f<T>(v.x);
+      qc[h * Rp + R + 2 * j + 1] = from_f<T>(v.y);
+    }
+    const int pad = Rp - R - rr;
+    for (int i = threadIdx.x; i < H * pad; i += 256) qc[(i / pad) * Rp + R + rr + i % pad] = from_f<T>(0.f);
+  }
+  for (int i = threadIdx.x; i < a.n_gate; i += 256) {
+    const float v = sigmoid_f(src.get(row, H * qd + R + rr + i));
+    if (a.gate) a.gate[(long long)row * a.n_gate + i] = v;
+    if (a.gate_t) reinterpret_cast<T*>(a.gate_t)[(long long)row * a.n_gate + i] = from_f<T>(v);
+  }
 }
 
 // ---- one warp per (row, head), any dtype; NR = values per lane (Rp <= 32 NR).  grid (ceil(H / 8), M) -------------
