@@ -115,18 +115,7 @@ int scan_np(const vn_ctx* ctx, int H, int vd, int d, int n_ent) {
 //
 // CTA = four warps, 64 columns of v of one head; warp w keeps the state of columns 16 w .. 16 w + 15 transposed in its
 // accumulators [vd 16][d], which is also the layout its pieces have as the B operand of q S.
-constexpr int CH = 64, CW = 4, VB = 16 * CW, PIECES = 3;
-
-// two fp32 values -> PIECES packed pairs of bf16 that sum up to them
-__device__ __forceinline__ void split2(float x, float y, unsigned (&p)[PIECES]) {
-#pragma unroll
-  for (int i = 0; i < PIECES; ++i) {
-    p[i] = pack_bf16(x, y);
-    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&p[i]));
-    x -= f.x;
-    y -= f.y;
-  }
-}
+constexpr int CH = 64, CW = 4, VB = 16 * CW;
 
 template <int DT> constexpr int chunk_smem(bool local) {
   const int q = 2 * CH * (DT + 8) * 2, v = 2 * CH * (VB + 8) * 2, p = CH * (CH + 4) * 4;
