@@ -1,27 +1,31 @@
-// Composed models: a list of layers of different kinds (latent attention, grouped-query attention, selective scan, gated
-// delta rule, lightning attention), each with an optional feed-forward, and optionally a block of layers that is run several
-// times with the same weights.  The residual is one stream that sublayers add to, or an arrangement of several (streams.cuh).
+// Composed models: a list of layers of different kinds (latent attention, grouped-query attention, selective scan, state-space
+// duality, gated delta rule, lightning attention), each with an optional feed-forward or mixture of experts and an optional
+// input of its own for every token, and optionally a block of layers that is run several times with the same weights.  The
+// residual is one stream that sublayers add to, or an arrangement of several (streams.cuh).
 // Weights, the per-sequence cache (paged latents, keys and values, rings of convolution inputs and of recurrent states), and
 // the forward over new rows of a uniform or a ragged batch.  Included by model.cu: it uses that file's GEMM helpers.
 //
 // One forward serves prompts, portions of prompts, single tokens and mixtures.  Projections of at most 256 rows of a
 // bf16 model are split-K tcgen05 GEMMs whose slices are summed by the kernel that needs them; longer ones go through
 // the tcgen05 segment kernel; an fp32 model uses the fp32 GEMM.  When every entry brings one token, a mixer's
-// recurrence or attention and what surrounds it is one kernel (mamba_step_kernel, delta_step_kernel, attn_step_kernel,
-// lightning_scan_kernel).
+// recurrence or attention and what surrounds it is one kernel (mamba_step_kernel, ssd_step_kernel, delta_step_kernel,
+// attn_step_kernel, lightning_scan_kernel).
 #pragma once
 #include "json_value.h"
 #include "latent_attn.cuh"
 #include "lightning.cuh"
 #include "paged_attn.cuh"
+#include "router.cuh"
 #include "scan_delta.cuh"
 #include "scan_mamba.cuh"
 #include "seq_ops.cuh"
+#include "ssd.cuh"
 #include "streams.cuh"
 
 namespace hybrid {
 
-enum Kind { LATENT = 0, MAMBA1 = 1, DELTA = 2, ATTENTION = 3, LIGHTNING = 4 };
+enum Kind { LATENT = 0, MAMBA1 = 1, DELTA = 2, ATTENTION = 3, LIGHTNING = 4, MAMBA2 = 5 };
+enum Gate { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
 
 struct HLayer {
   int kind = 0;
@@ -31,8 +35,15 @@ struct HLayer {
   // attention: H, KH, d, vd, taps, window, scale and the line below (conv_named: the convolutions are in the checkpoint).
   // lightning: H, d, vd, decay
   int kv_from = -1, gated = 0, P = 0, rd = 0, rope = -1, conv_named = 0;
+  int chunk = 0, qk_norm = 0, bias = 0, interleaved = 0;
+  float softcap = 0.f;
+  // latent, besides: rotated dimensions rr, what the output gate multiplies, sink.  mamba2: H, vd, nstate, taps, groups, norm_groups
+  int rr = 0, gate = GATE_HEAD, sinks = 1, groups = 1, norm_groups = 1;
   std::vector<double> decay;
   int ff = 0, act = 0;             // feed-forward width (0: none), activation of its gate: 0 silu, 1 gelu
+  // mixture: n_exp experts of width ff and n_id identity experts (0: a dense feed-forward), of which a row uses `top`, out of
+  // the `keep` best of exp_groups groups
+  int n_exp = 0, n_id = 0, top = 0, exp_groups = 1, keep = 1, corrected = 0;
   int ff_plain = 0;                // no gate: squared relu
   int dp = 0, Rp = 0, dtp = 0, rap = 0, rgp = 0, n_in = 0, n_x = 0, ffp = 0;    // padded sizes
   float* norm1 = nullptr; float* norm2 = nullptr;                               // 1 + stored weight
@@ -49,13 +60,20 @@ struct HLayer {
   float* rg_b[2] = {nullptr, nullptr};
   float* in_conv = nullptr;               // [D, taps] convolution of what the mixer reads
   float* conv = nullptr; float* conv_b = nullptr;
-  void* w_gu = nullptr; void* w_down = nullptr;
+  void* w_gu = nullptr; void* w_down = nullptr;                                 // of a mixture: per expert
+  float* f_d = nullptr;                   // mamba2: -exp(A_log) [H]
+  float* o_b = nullptr;                   // bias of the output projection
+  void* w_router = nullptr; float* correction = nullptr;                        // [n_exp + n_id, D], [n_exp + n_id]
+  void *w_sgate = nullptr, *w_sproj = nullptr; float* s_norm = nullptr;         // the token's own input
+  int n_out() const { return n_exp + n_id; }
+  int n_gate() const { return gate == GATE_HEAD ? H : gate == GATE_ELEMENT ? H * vd : 0; }      // latent
   int conv_ch() const {
     if (kind == MAMBA1) return inner;
+    if (kind == MAMBA2) return inner + 2 * groups * nstate;
     if (kind == ATTENTION) return H * d + (kv_from < 0 ? KH * (d + vd) : 0);
     return 2 * KH * d + H * vd;
   }
-  long long state_elems() const { return kind == MAMBA1 ? (long long)inner * nstate : (long long)H * d * vd; }
+  long long state_elems() const { return kind == MAMBA1 || kind == MAMBA2 ? (long long)inner * nstate : (long long)H * d * vd; }
 };
 
 struct Run { int layer; int pass; int kv_run; };      // pass: -1 outside the loop; kv_run: the run whose keys it reads
@@ -83,12 +101,17 @@ struct Model {
   // arrangement of the residual
   int layer_norm = 0, streams = 0, in_taps = 0, res_gate = 0;     // streams 0: one stream that sublayers add to
   bool arranged = false;           // the forward goes through streams.cuh
+  bool plain_norm = false;         // norm weights are stored as they are, not around zero
+  int side = 0, sidep = 0;         // width of the tokens' own inputs per layer (0: none), padded
+  void* side_embed = nullptr;      // [V, layers * side]
+  int *exp_count = nullptr, *exp_cur = nullptr, *exp_off = nullptr;    // per expert: rows (zero between forwards), fill level, first row
+  int max_out = 0;
   std::vector<Rope> ropes;
   std::vector<void*> retired;      // tables replaced by longer ones (a captured graph may still read them)
   void* hc = nullptr;              // [rows, D] what the mixer reads
   float *gate = nullptr, *y = nullptr;                            // [rows, D] raw gates; result of a sublayer
   float* gate_ws = nullptr; size_t gate_ws_bytes = 0;             // split-K slices of a gate
-  float* seg = nullptr; size_t seg_bytes = 0;                     // LightningArgs::seg_state
+  float* seg = nullptr; size_t seg_bytes = 0;                     // LightningArgs::seg_state, SsdArgs::seg_state and seg_decay
 };
 
 // what a cache of such a model keeps besides the lengths; owned by the root cache, shared by its views
@@ -106,7 +129,7 @@ inline int up8(int n) { return (n + 7) & ~7; }
 inline int up4(int n) { return (n + 3) & ~3; }
 // latent rows are padded to a multiple of 32 that the tensor-core kernel has an instance for
 inline int latent_pitch(int R) {
-  static const int tiles[] = {1, 2, 3, 4, 6, 8, 12, 16};
+  static const int tiles[] = {1, 2, 3, 4, 6, 8, 10, 12, 16, 18};
   for (int t : tiles)
     if (R <= 32 * t) return 32 * t;
   return (R + 31) & ~31;
@@ -130,6 +153,14 @@ struct Buffers {
   float *dq = nullptr, *dk = nullptr, *dv = nullptr, *beta = nullptr, *g = nullptr, *gg = nullptr, *o = nullptr;   // delta
   void *low_a = nullptr, *low_g = nullptr;
   void* lin = nullptr; float* ss = nullptr;      // lightning
+  void* gate_t = nullptr;                        // latent: output gates in the storage dtype
+  void *xbc = nullptr, *u = nullptr;             // mamba2
+  // mixture of experts
+  float *logits = nullptr, *slot_w = nullptr;
+  int *slot_expert = nullptr, *slot_pos = nullptr, *sorted_row = nullptr, *sub_seg = nullptr;
+  void *hs = nullptr, *ey = nullptr;
+  int sub_cap = 0;
+  void* side_act = nullptr;
 };
 constexpr int SPLIT_ROWS = 64, MAX_SPLITS = 16;   // key splits of the latent attention: forwards of few rows
 
@@ -137,12 +168,26 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
   A.off = 0;
   A.take(&b.proj, M * std::max(std::max(L.n_in, hm.D), L.ff_plain ? L.ffp + hm.D : 0) * 4);
   A.take(&b.mix, M * (size_t)(L.kind == MAMBA1 ? L.inner : L.H * L.vd) * e);
-  if (L.ff) A.take(&b.act, M * L.ffp * e);
+  if (L.ff) A.take(&b.act, M * std::max(1, L.top) * L.ffp * e);
+  if (L.n_exp) {
+    const size_t slots = M * L.top;
+    A.take(&b.logits, M * L.n_out() * 4);
+    A.take(&b.slot_w, slots * 4);
+    A.take(&b.slot_expert, slots * 4);
+    A.take(&b.slot_pos, slots * 4);
+    A.take(&b.sorted_row, slots * 4);
+    A.take(&b.hs, slots * hm.D * e);
+    A.take(&b.ey, slots * hm.D * e);
+    b.sub_cap = (int)(L.n_exp + slots / 256 + 1);
+    A.take(&b.sub_seg, (size_t)3 * b.sub_cap * 4);
+  }
+  if (hm.side) A.take(&b.side_act, M * hm.sidep * e);
   if (L.kind == LATENT) {
     A.take(&b.q, M * L.H * L.dp * e);
     A.take(&b.qc, M * L.H * L.Rp * e);
     A.take(&b.oc, M * L.H * L.Rp * e);
-    A.take(&b.gate, M * L.H * 4);
+    if (L.gate == GATE_HEAD) A.take(&b.gate, M * L.H * 4);
+    if (L.gate == GATE_ELEMENT) A.take(&b.gate_t, M * L.H * L.vd * e);
     if (M <= SPLIT_ROWS) {
       A.take(&b.part_o, (size_t)MAX_SPLITS * M * L.H * L.Rp * 4);
       A.take(&b.part_ml, (size_t)MAX_SPLITS * M * L.H * 2 * 4);
@@ -153,6 +198,10 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
     A.take(&b.dtb, M * L.dtp * e);
     A.take(&b.p, M * L.n_x * 4);
     A.take(&b.dt, M * L.inner * 4);
+  } else if (L.kind == MAMBA2) {
+    A.take(&b.xbc, M * up8(L.conv_ch()) * e);
+    A.take(&b.dt, M * L.H * 4);
+    A.take(&b.u, M * L.inner * e);
   } else if (L.kind == ATTENTION) {
     A.take(&b.q, M * L.H * L.P * e);
     if (M <= SPLIT_ROWS) {
@@ -175,8 +224,8 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
   }
 }
 
-// Rotary frequencies f_i = base^(-2 i / dims).  With scaling (YaRN), pairs that turn slowly over the original context are
-// divided by `factor`, those that turn fast are kept, with a linear ramp between the two.
+// Rotary frequencies f_i = base^(-2 i / dims).  Linear scaling divides them all by `factor`; YaRN divides those of pairs that
+// turn slowly over the original context, keeps those that turn fast, with a linear ramp between the two.
 inline Rope make_rope(const JsonValue& r) {
   Rope out;
   const int dims = (int)r.number("dims", 0);
@@ -185,6 +234,10 @@ inline Rope make_rope(const JsonValue& r) {
   const JsonValue* s = r.find("scaling");
   if (!s || s->kind != JsonValue::OBJ) return out;
   const double factor = s->number("factor", 1), original = s->number("original", 1);
+  if (s->text("kind") == "linear") {
+    for (double& f : out.freq) f /= factor;
+    return out;
+  }
   auto dim_of = [&](double turns) { return dims * log(original / (2 * M_PI * turns)) / (2 * log(base)); };
   const double lo = std::max(floor(dim_of(s->number("fast", 32))), 0.0);
   const double hi = std::min(ceil(dim_of(s->number("slow", 1))), dims - 1.0);
@@ -216,6 +269,12 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
   hm->res_gate = j.number("residual_gate", 0) != 0;
   VN_REQUIRE(ctx, hm->streams >= 0 && hm->streams <= MAX_STREAMS && hm->in_taps >= 0, "streams (at most %d) or input_conv out of range", MAX_STREAMS);
   hm->arranged = hm->layer_norm || hm->streams || hm->in_taps || hm->res_gate;
+  const std::string nw = j.text("norm_weight");
+  VN_REQUIRE(ctx, nw.empty() || nw == "plain" || nw == "around_zero", "norm_weight %s unknown (plain | around_zero)", nw.c_str());
+  hm->plain_norm = hm->layer_norm || nw == "plain";
+  hm->side = (int)j.number("token_side", 0);
+  hm->sidep = up8(hm->side);
+  VN_REQUIRE(ctx, hm->side >= 0, "token_side out of range");
   const JsonValue* ls = j.find("layers");
   VN_REQUIRE(ctx, c->vocab > 0 && c->dim > 0 && ls && ls->kind == JsonValue::ARR && !ls->arr.empty(),
              "a composed model needs vocab_size, dim and layers");
@@ -225,40 +284,70 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
     const std::string t = l.text("mixer");
     auto I = [&](const char* k, int dflt = 0) { return (int)l.number(k, dflt); };
     L.kind = t == "latent_attention" ? LATENT : t == "mamba1" ? MAMBA1 : t == "channel_delta" ? DELTA : t == "attention" ? ATTENTION
-             : t == "lightning" ? LIGHTNING : -1;
-    VN_REQUIRE(ctx, L.kind >= 0, "layer %zu: mixer %s unknown (latent_attention | attention | mamba1 | channel_delta | lightning)", i, t.c_str());
+             : t == "lightning" ? LIGHTNING : t == "mamba2" ? MAMBA2 : -1;
+    VN_REQUIRE(ctx, L.kind >= 0, "layer %zu: mixer %s unknown (latent_attention | attention | mamba1 | mamba2 | channel_delta | lightning)", i, t.c_str());
+    auto rope = [&](int dims) -> int32_t {       // the layer's rotation, at most `dims` dimensions
+      const JsonValue* r = l.find("rope");
+      if (!r || r->kind != JsonValue::OBJ) return VN_OK;
+      const Rope made = make_rope(*r);
+      L.rd = 2 * (int)made.freq.size();
+      VN_REQUIRE(ctx, L.rd <= dims, "layer %zu: %d of %d dimensions rotated", i, L.rd, dims);
+      for (size_t k = 0; k < hm->ropes.size() && L.rope < 0; ++k)
+        if (hm->ropes[k].freq == made.freq && hm->ropes[k].amp == made.amp) L.rope = (int)k;
+      if (L.rope < 0) { L.rope = (int)hm->ropes.size(); hm->ropes.push_back(made); }
+      L.interleaved = r->number("interleaved", 0) != 0;
+      return VN_OK;
+    };
     L.ff = I("mlp_hidden");
     const std::string act = l.text("mlp_act");
     VN_REQUIRE(ctx, !L.ff || act == "gelu_tanh" || act == "silu" || act == "relu2", "layer %zu: activation %s unknown (gelu_tanh | silu | relu2)", i, act.c_str());
     L.act = act == "gelu_tanh";
     L.ff_plain = act == "relu2";
+    if (const JsonValue* x = l.find("experts"))
+      if (x->kind == JsonValue::OBJ) {
+        L.n_exp = (int)x->number("count", 0); L.n_id = (int)x->number("identity", 0); L.top = (int)x->number("top", 0);
+        L.exp_groups = (int)x->number("groups", 1); L.keep = (int)x->number("keep", L.exp_groups);
+        L.corrected = x->number("correction", 0) != 0;
+        const int n = L.n_out();
+        VN_REQUIRE(ctx, L.ff > 0 && !L.ff_plain && L.n_exp > 0 && L.n_id >= 0 && n <= 1024 && L.exp_groups >= 1 && n % L.exp_groups == 0 &&
+                   L.keep >= 1 && L.keep <= L.exp_groups && L.top >= 1 && L.top <= MAX_CHOSEN && L.top <= L.keep * (n / L.exp_groups),
+                   "layer %zu: mixture of %d experts and %d identities in %d groups, %d kept, %d chosen", i, L.n_exp, L.n_id, L.exp_groups, L.keep, L.top);
+        hm->max_out = std::max(hm->max_out, n);
+      }
     if (L.ff_plain || L.kind == LIGHTNING) hm->arranged = true;
     L.ffp = up8(L.ff);
     L.H = I("heads"); L.d = I("dim"); L.vd = I("vdim"); L.taps = I("conv", 1);
     if (L.kind == LATENT) {
       L.R = I("kv_rank"); L.window = I("window"); L.scale = (float)l.number("scale", 0);
-      VN_REQUIRE(ctx, L.H > 0 && L.d > 0 && L.vd > 0 && L.R > 0 && L.R <= 1024 && L.window >= 0, "layer %zu: latent attention sizes", i);
-      L.dp = up8(L.d); L.Rp = latent_pitch(L.R);
-      L.n_in = up8(L.H * L.d + L.R + L.H);
+      L.rr = I("rot_dim"); L.sinks = l.number("sink", 1) != 0;
+      const std::string gate = l.text("output_gate");
+      VN_REQUIRE(ctx, gate.empty() || gate == "head" || gate == "element" || gate == "none", "layer %zu: output gate %s unknown (head | element | none)", i, gate.c_str());
+      L.gate = gate == "none" ? GATE_NONE : gate == "element" ? GATE_ELEMENT : GATE_HEAD;
+      VN_REQUIRE(ctx, L.H > 0 && L.d > 0 && L.vd > 0 && L.R > 0 && L.rr >= 0 && L.rr % 2 == 0 && L.R + L.rr <= 1024 && L.window >= 0, "layer %zu: latent attention sizes", i);
+      TRY(rope(L.rr));
+      VN_REQUIRE(ctx, L.rd == L.rr && (!L.rr || L.interleaved), "layer %zu: the rotated part of %d dimensions needs a rotation of as many interleaved ones", i, L.rr);
+      L.dp = up8(L.d); L.Rp = latent_pitch(L.R + L.rr);
+      L.n_in = up8(L.H * (L.d + L.rr) + L.R + L.rr + L.n_gate());
     } else if (L.kind == MAMBA1) {
       L.inner = I("inner"); L.dt_rank = I("dt_rank"); L.nstate = I("state");
       VN_REQUIRE(ctx, L.inner > 0 && L.dt_rank > 0 && L.nstate > 0 && L.nstate <= 128 && L.taps >= 1, "layer %zu: selective scan sizes", i);
       L.dtp = up8(L.dt_rank);
       L.n_in = 2 * L.inner;
       L.n_x = up8(L.dtp + 2 * L.nstate);
+    } else if (L.kind == MAMBA2) {
+      L.inner = L.H * L.vd; L.nstate = I("state"); L.groups = I("groups", 1); L.norm_groups = I("norm_groups", 1);
+      VN_REQUIRE(ctx, L.H > 0 && L.vd > 0 && L.nstate > 0 && L.nstate <= 512 && L.groups > 0 && L.H % L.groups == 0 && L.norm_groups > 0 &&
+                 L.inner % L.norm_groups == 0 && L.taps >= 1, "layer %zu: state-space sizes", i);
+      L.n_in = up8(2 * L.inner + 2 * L.groups * L.nstate + L.H);
     } else if (L.kind == ATTENTION) {
       L.KH = I("kv_heads"); L.window = I("window"); L.scale = (float)l.number("scale", 0); L.kv_from = I("kv_from", -1);
+      L.chunk = I("chunk"); L.softcap = (float)l.number("softcap", 0); L.qk_norm = l.number("qk_norm", 0) != 0; L.bias = l.number("bias", 0) != 0;
       L.gated = l.number("output_gate", 0) != 0;
       L.conv_named = l.find("conv") && l.find("conv")->kind == JsonValue::NUM;
-      if (const JsonValue* r = l.find("rope"))
-        if (r->kind == JsonValue::OBJ) {
-          const Rope rope = make_rope(*r);
-          L.rd = 2 * (int)rope.freq.size();
-          for (size_t k = 0; k < hm->ropes.size() && L.rope < 0; ++k)
-            if (hm->ropes[k].freq == rope.freq && hm->ropes[k].amp == rope.amp) L.rope = (int)k;
-          if (L.rope < 0) { L.rope = (int)hm->ropes.size(); hm->ropes.push_back(rope); }
-        }
-      VN_REQUIRE(ctx, L.H > 0 && L.KH > 0 && L.H % L.KH == 0 && L.d > 0 && L.vd > 0 && L.d <= 1024 && L.vd <= 1024 && L.rd <= L.d &&
+      TRY(rope(L.d));
+      VN_REQUIRE(ctx, !(L.conv_named && (L.qk_norm || L.bias)) && !(L.kv_from >= 0 && L.qk_norm), "layer %zu: norms and biases of the heads together with "
+                 "convolutions, or norms of another layer's keys", i);
+      VN_REQUIRE(ctx, L.chunk >= 0 && L.softcap >= 0.f && L.H > 0 && L.KH > 0 && L.H % L.KH == 0 && L.d > 0 && L.vd > 0 && L.d <= 1024 && L.vd <= 1024 && L.rd <= L.d &&
                  L.window >= 0 && L.taps >= 1, "layer %zu: attention sizes", i);
       if (L.kv_from >= 0) {
         VN_REQUIRE(ctx, L.kv_from < (int)i, "layer %zu: keys and values of layer %d, which does not run before it", i, L.kv_from);
@@ -305,6 +394,10 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
     for (int i = a; i < b; ++i) run(i, t);
   for (int i = b; i < n; ++i) run(i, -1);
   VN_REQUIRE(ctx, !hm->arranged || !hm->loop_times, "a looped block needs the plain residual");
+  VN_REQUIRE(ctx, !hm->side || !hm->loop_times, "tokens' own inputs do not go with a looped block");
+  if (hm->arranged)
+    for (const HLayer& L : hm->layers)
+      VN_REQUIRE(ctx, !L.n_exp && !hm->side && L.kind != MAMBA2 && !L.bias, "mixtures, state-space layers, biases and tokens' own inputs need the plain residual");
   return VN_OK;
 }
 
@@ -331,6 +424,15 @@ int32_t alloc(vn_model* m) {
     TRY(F(&hm.loop_step, hm.loop_times * D));
     hm.want.insert("loop.in"); hm.want.insert("loop.step");
   }
+  if (hm.side) {
+    TRY(W(&hm.side_embed, (size_t)hm.vocab * hm.layers.size() * hm.side));
+    hm.want.insert("side.embed");
+  }
+  if (hm.max_out) {
+    void* p[3] = {nullptr, nullptr, nullptr};
+    for (void*& q : p) TRY(zalloc(m, &q, (size_t)hm.max_out * 4));
+    hm.exp_count = (int*)p[0]; hm.exp_cur = (int*)p[1]; hm.exp_off = (int*)p[2];
+  }
   if (hm.sinusoidal) {
     std::vector<double> f((D + 1) / 2);
     for (size_t i = 0; i < f.size(); ++i) f[i] = pow(10000.0, -2.0 * (double)i / (double)D);
@@ -351,7 +453,9 @@ int32_t alloc(vn_model* m) {
       TRY(W(&L.w_o, D * L.H * L.vd));
       TRY(F(&L.f_a, L.R));
       TRY(F(&L.f_b, L.H));
-      need({"mix.q", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv", "mix.sink", "mix.g"});
+      need({"mix.q", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv"});
+      if (L.sinks) need({"mix.sink"});
+      if (L.gate) need({"mix.g"});
     } else if (L.kind == ATTENTION) {
       TRY(W(&L.w_o, D * L.H * L.vd));
       TRY(F(&L.conv, (size_t)L.conv_ch() * L.taps));
@@ -362,6 +466,17 @@ int32_t alloc(vn_model* m) {
       need({"mix.q"});
       if (L.kv_from < 0) need({"mix.k", "mix.v"});
       if (L.gated) need({"mix.g"});
+      if (L.qk_norm) {
+        TRY(F(&L.f_a, L.d));
+        TRY(F(&L.f_b, L.d));
+        need({"mix.q.norm", "mix.k.norm"});
+      }
+      if (L.bias) {
+        TRY(F(&L.f_c, L.conv_ch()));
+        TRY(F(&L.o_b, D));
+        need({"mix.q.b", "mix.o.b"});
+        if (L.kv_from < 0) need({"mix.k.b", "mix.v.b"});
+      }
       if (L.conv_named) need({"mix.q.conv"});
       if (L.conv_named && L.kv_from < 0) need({"mix.k.conv", "mix.v.conv"});
     } else if (L.kind == LIGHTNING) {
@@ -378,6 +493,15 @@ int32_t alloc(vn_model* m) {
       TRY(upload(m, dec.data(), L.f_b, 1, (long long)dec.size(), (long long)dec.size(), 1, 0, true));
       TRY(upload(m, pw.data(), L.f_c, 1, (long long)pw.size(), (long long)pw.size(), 1, 0, true));
       need({"mix.q", "mix.k", "mix.v", "mix.g", "mix.norm"});
+    } else if (L.kind == MAMBA2) {
+      TRY(W(&L.w_o, D * L.inner));
+      TRY(F(&L.f_a, L.inner));
+      TRY(F(&L.f_b, L.H));
+      TRY(F(&L.f_c, L.H));
+      TRY(F(&L.f_d, L.H));
+      TRY(F(&L.conv, (size_t)L.conv_ch() * L.taps));
+      TRY(F(&L.conv_b, L.conv_ch()));
+      need({"mix.in", "mix.conv", "mix.conv.b", "mix.dt_bias", "mix.A_log", "mix.D", "mix.norm"});
     } else if (L.kind == MAMBA1) {
       TRY(W(&L.w_uk, (size_t)L.inner * L.dtp));
       TRY(W(&L.w_uv, (size_t)L.n_x * L.inner));
@@ -401,12 +525,28 @@ int32_t alloc(vn_model* m) {
     }
     if (L.ff) {
       const bool stacked = L.ff_plain && hm.res_gate;          // up | gate of the result: both read the same rows
+      const size_t n = std::max(1, L.n_exp);
       TRY(F(&L.norm2, D));
-      TRY(W(&L.w_gu, (size_t)(L.ff_plain ? L.ffp + (stacked ? D : 0) : 2 * L.ffp) * D));
-      TRY(W(&L.w_down, D * L.ffp));
-      need({"norm2", "mlp.up", "mlp.down"});
-      if (!L.ff_plain) need({"mlp.gate"});
+      TRY(W(&L.w_gu, n * (L.ff_plain ? L.ffp + (stacked ? D : 0) : 2 * L.ffp) * D));
+      TRY(W(&L.w_down, n * D * L.ffp));
+      need({"norm2"});
+      if (L.n_exp) {
+        TRY(W(&L.w_router, (size_t)L.n_out() * D));
+        need({"mlp.router"});
+        if (L.corrected) { TRY(F(&L.correction, L.n_out())); need({"mlp.correction"}); }
+        for (int x = 0; x < L.n_exp; ++x)
+          for (const char* part : {".gate", ".up", ".down"}) hm.want.insert(p + "mlp.e" + std::to_string(x) + part);
+      } else {
+        need({"mlp.up", "mlp.down"});
+        if (!L.ff_plain) need({"mlp.gate"});
+      }
       if (stacked) L.w_rg[1] = (char*)L.w_gu + (size_t)L.ffp * D * e;
+    }
+    if (hm.side) {
+      TRY(W(&L.w_sgate, (size_t)up4(hm.side) * D));
+      TRY(W(&L.w_sproj, D * hm.sidep));
+      TRY(F(&L.s_norm, D));
+      need({"side.gate", "side.proj", "side.norm"});
     }
     for (int q = 0; q < (L.ff ? 2 : 1); ++q) {
       const std::string k = std::to_string(q + 1);
@@ -439,12 +579,14 @@ void destroy(vn_model* m) {
     F(L.norm1); F(L.norm2); F(L.w_in); F(L.w_o); F(L.w_uk); F(L.w_uv); F(L.f_a); F(L.f_b); F(L.f_c); F(L.conv); F(L.conv_b);
     if (!(L.ff_plain && hm.res_gate)) F(L.w_rg[1]);            // else part of w_gu
     F(L.w_gu); F(L.w_down); F(L.w_rg[0]); F(L.in_conv);
+    F(L.f_d); F(L.o_b); F(L.w_router); F(L.correction); F(L.w_sgate); F(L.w_sproj); F(L.s_norm);
     for (int q = 0; q < 2; ++q) { F(L.hc_in[q]); F(L.hc_out[q]); F(L.hc_mix[q]); F(L.rg_b[q]); }
   }
   for (Rope& r : hm.ropes) F(r.table);
   for (void* t : hm.retired) F(t);
   F(hm.w_loop); F(hm.loop_step); F(hm.freq); F(hm.x0); F(hm.cat); F(hm.ws); F(hm.meta);
   F(hm.hc); F(hm.gate); F(hm.y); F(hm.gate_ws); F(hm.seg);
+  F(hm.side_embed); F(hm.exp_count); F(hm.exp_cur); F(hm.exp_off);
   delete m->hyb;
   m->hyb = nullptr;
 }
@@ -484,13 +626,14 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
       return VN_OK;
     return vn_fail(ctx, VN_ERR_INVALID, "unexpected tensor %s", n.c_str());
   }
-  auto weight = [&](float* dst, long long count) {        // a norm's: around zero (rms) or plain (layer)
-    return hm.layer_norm ? f32(data, dst, count) : mapped(dst, count, one_plus);
+  auto weight = [&](float* dst, long long count) {        // a norm's: around zero or plain
+    return hm.plain_norm ? f32(data, dst, count) : mapped(dst, count, one_plus);
   };
 #define PUT(er, ec, expr) do { if (!shape((er), (ec))) return st; TRY(expr); return VN_OK; } while (0)
   if (n == "embed") PUT(hm.vocab, D, rows(m->emb, D));
   if (n == "head") PUT(hm.vocab, D, rows(m->head, D));
   if (n == "final.norm") PUT(D, 1, weight(m->norm_f, D));
+  if (n == "side.embed") PUT(hm.vocab, (long long)hm.layers.size() * hm.side, rows(hm.side_embed, cl));
   if (n == "loop.in") PUT(D, 2 * D, rows(hm.w_loop, 2 * D));
   if (n == "loop.step") PUT(hm.loop_times, D, f32(data, hm.loop_step, r * cl));
   const size_t dot = n.find('.');
@@ -502,6 +645,20 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
   if (s == "mlp.up" && L.ff_plain) PUT(L.ff, D, rows(L.w_gu, D));
   if (s == "mlp.up") PUT(L.ff, D, rows(L.w_gu, D, 1, 2));
   if (s == "mlp.down") PUT(D, L.ff, rows(L.w_down, L.ffp));
+  if (s == "mlp.router") PUT(L.n_out(), D, rows(L.w_router, D));
+  if (s == "mlp.correction") PUT(L.n_out(), 1, f32(data, L.correction, r));
+  if (s.compare(0, 5, "mlp.e") == 0) {
+    const size_t end = s.find('.', 4);
+    const long long x = atoll(s.substr(5, end - 5).c_str());
+    const std::string part = s.substr(end + 1);
+    void* gu = (char*)L.w_gu + x * 2 * L.ffp * D * m->esz;
+    if (part == "gate") PUT(L.ff, D, rows(gu, D, 0, 2));
+    if (part == "up") PUT(L.ff, D, rows(gu, D, 1, 2));
+    PUT(D, L.ff, rows((char*)L.w_down + x * D * L.ffp * m->esz, L.ffp));
+  }
+  if (s == "side.gate") PUT(hm.side, D, rows(L.w_sgate, D));
+  if (s == "side.proj") PUT(D, hm.side, rows(L.w_sproj, hm.sidep));
+  if (s == "side.norm") PUT(D, 1, f32(data, L.s_norm, r));
   if (s == "canon1") PUT(D, hm.in_taps, f32(data, L.in_conv, r * cl));
   for (int q = 0; q < 2; ++q) {
     const std::string k = std::to_string(q + 1);
@@ -517,6 +674,12 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
     if (s == "mix.k") PUT(kd, D, rows(L.w_in, D, qd));
     if (s == "mix.v") PUT(vd, D, rows(L.w_in, D, qd + kd));
     if (s == "mix.g") PUT(hv, D, rows(L.w_in, D, L.conv_ch()));
+    if (s == "mix.q.norm") PUT(L.d, 1, f32(data, L.f_a, r));
+    if (s == "mix.k.norm") PUT(L.d, 1, f32(data, L.f_b, r));
+    if (s == "mix.q.b") PUT(qd, 1, f32(data, L.f_c, r));
+    if (s == "mix.k.b") PUT(kd, 1, f32(data, L.f_c + qd, r));
+    if (s == "mix.v.b") PUT(vd, 1, f32(data, L.f_c + qd + kd, r));
+    if (s == "mix.o.b") PUT(D, 1, f32(data, L.o_b, r));
     if (s == "mix.q.conv") PUT(qd, L.taps, f32(data, L.conv, r * cl));
     if (s == "mix.k.conv") PUT(kd, L.taps, f32(data, L.conv + qd * L.taps, r * cl));
     if (s == "mix.v.conv") PUT(vd, L.taps, f32(data, L.conv + (qd + kd) * L.taps, r * cl));
@@ -530,10 +693,10 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
     if (s == "mix.norm") PUT(hv, 1, f32(data, L.f_a, r));
     if (s == "mix.o") PUT(D, hv, rows(L.w_o, hv));
   } else if (L.kind == LATENT) {
-    const long long hd = (long long)L.H * L.d, hv = (long long)L.H * L.vd;
-    if (s == "mix.q") PUT(hd, D, rows(L.w_in, D));
-    if (s == "mix.dkv") PUT(L.R, D, rows(L.w_in, D, hd));
-    if (s == "mix.g") PUT(L.H, D, rows(L.w_in, D, hd + L.R));
+    const long long hd = (long long)L.H * L.d, hv = (long long)L.H * L.vd, hq = hd + (long long)L.H * L.rr;
+    if (s == "mix.q") PUT(hq, D, rows(L.w_in, D));
+    if (s == "mix.dkv") PUT(L.R + L.rr, D, rows(L.w_in, D, hq));
+    if (s == "mix.g") PUT(L.n_gate(), D, rows(L.w_in, D, hq + L.R + L.rr));
     if (s == "mix.dkv.norm") PUT(L.R, 1, f32(data, L.f_a, L.R));
     if (s == "mix.sink") PUT(L.H, 1, f32(data, L.f_b, L.H));
     if (s == "mix.uv") PUT(hv, L.R, rows(L.w_uv, L.Rp));
@@ -546,6 +709,16 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
           for (long long c = 0; c < L.R; ++c) tmp[(h * L.Rp + c) * L.dp + i] = data[(h * L.d + i) * L.R + c];
       return upload(m, tmp.data(), L.w_uk, (long long)L.H * L.Rp, L.dp, L.dp);
     }
+  } else if (L.kind == MAMBA2) {
+    const long long C = L.conv_ch();
+    if (s == "mix.in") PUT(L.inner + C + L.H, D, rows(L.w_in, D));
+    if (s == "mix.conv") PUT(C, L.taps, f32(data, L.conv, r * cl));
+    if (s == "mix.conv.b") PUT(C, 1, f32(data, L.conv_b, r));
+    if (s == "mix.dt_bias") PUT(L.H, 1, f32(data, L.f_c, r));
+    if (s == "mix.A_log") PUT(L.H, 1, mapped(L.f_d, r, neg_rate));
+    if (s == "mix.D") PUT(L.H, 1, f32(data, L.f_b, r));
+    if (s == "mix.norm") PUT(L.inner, 1, f32(data, L.f_a, r));
+    if (s == "mix.o") PUT(D, L.inner, rows(L.w_o, L.inner));
   } else if (L.kind == MAMBA1) {
     if (s == "mix.in") PUT(2ll * L.inner, D, rows(L.w_in, D));
     if (s == "mix.conv") PUT(L.inner, L.taps, f32(data, L.conv, r * cl));
@@ -657,15 +830,36 @@ int32_t project(vn_model* m, GemmArgs g, float* direct, Mat<__nv_bfloat16>* out,
   out->p = (const __nv_bfloat16*)direct; out->ld = g.N;
   return linear(m, g);
 }
-// x += A W^T; then h = RMSNorm(x) * next_norm when given
+// what m->h holds behind a sublayer: RMSNorm(x) * norm_w, x itself, or nothing
+struct Next { const float* norm_w = nullptr; bool cast = false; };
+
+// x += y (or y over its root mean square times own_norm), and what the next product reads, in one pass over the rows
+template <typename T, typename Y>
+int32_t close_rows(vn_model* m, const Y& y, int M, const float* own_norm, const Next& next) {
+  vn_ctx* ctx = m->ctx;
+  const int D = m->hyb->D;
+  const float eps = m->hyb->eps;
+#define RESIDUAL(NV) VN_LAUNCH_PDL_LEVEL(ctx, 1, "residual_kernel", (residual_kernel<T, Y, NV>), M, 256, 0, y, m->x, own_norm, next.norm_w, (int)next.cast, (T*)m->h, D, eps)
+  if (D % 4 || D > 8192) RESIDUAL(0); else if (D <= 1024) RESIDUAL(1); else if (D <= 2048) RESIDUAL(2); else if (D <= 4096) RESIDUAL(4); else RESIDUAL(8);
+#undef RESIDUAL
+  return VN_OK;
+}
+
+// x += A W^T (+ bias); then m->h as `next` says
 template <typename T>
-int32_t close_block(vn_model* m, GemmArgs g, const float* next_norm) {
+int32_t close_block(vn_model* m, GemmArgs g, const float* bias, const Next& next) {
   vn_ctx* ctx = m->ctx;
   const Model& hm = *m->hyb;
   const int D = hm.D, M = g.M;
+  const float* next_norm = next.norm_w;
   if (tc_rows(m, g)) {
     int sp = 1;
     TRY(tc_partial(m, g, M, M, &sp));
+    if (bias || next.cast) {
+      AddRows<Src> y;
+      y.y.p = m->partial; y.y.splits = sp; y.y.pstride = (long long)M * D; y.y.ld = D; y.bias = bias;
+      return close_rows<T>(m, y, M, nullptr, next);
+    }
     if (D % 4 == 0 && D <= 2048) {
       VN_LAUNCH_PDL_BIT(ctx, 4, splitk_add_norm_kernel<T>, M, 256, 0, m->partial, sp, (long long)M * D, m->x, next_norm,
                         (T*)m->h, (float*)nullptr, D, hm.eps);
@@ -676,8 +870,12 @@ int32_t close_block(vn_model* m, GemmArgs g, const float* next_norm) {
     }
     return VN_OK;
   }
-  g.C = m->x; g.ldc = D; g.epi = EPI_ADD;
+  g.C = m->x; g.ldc = D; g.epi = EPI_ADD; g.bias = bias;
   TRY(linear(m, g));
+  if (next.cast) {
+    const long long n = (long long)M * D;
+    VN_LAUNCH(ctx, cast_rows_kernel<T>, (unsigned)ceil_div(n, 256ll), 256, 0, m->x, (T*)m->h, n);
+  }
   if (next_norm)
     VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, next_norm, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
   return VN_OK;
@@ -696,16 +894,19 @@ int32_t latent_attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc,
   const int M = rows.M, D = m->hyb->D, H = L.H;
   Src s;
   TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_latent_in"), b.proj, &s));
-  VN_LAUNCH(ctx, latent_append_kernel<T>, M, 256, (size_t)L.R * 4, s, H, L.d, L.dp, L.R, L.Rp, L.f_a, m->hyb->eps, (T*)b.q,
-            b.gate, (T*)kv->k[run], hc.table_dev, hc.max_pages, rows);
-  GemmArgs g = gemm_args(b.q, H * L.dp, L.w_uk, L.Rp, L.dp, M, "gemm_latent_uk");
+  LatentIn in;
+  in.H = H; in.d = L.d; in.dp = L.dp; in.rr = L.rr; in.R = L.R; in.Rp = L.Rp; in.rope = L.rope >= 0 ? m->hyb->ropes[L.rope].table : nullptr;
+  in.norm_w = L.f_a; in.eps = m->hyb->eps; in.n_gate = L.n_gate(); in.gate = b.gate; in.gate_t = b.gate_t;
+  in.q = b.q; in.qc = b.qc; in.plane = kv->k[run]; in.table = hc.table_dev; in.max_pages = hc.max_pages;
+  VN_LAUNCH(ctx, latent_append_kernel<T>, M, 256, (size_t)L.R * 4, s, in, rows);
+  GemmArgs g = gemm_args(b.q, H * L.dp, L.w_uk, L.rr ? L.R : L.Rp, L.dp, M, "gemm_latent_uk");
   g.C = b.qc; g.ldc = (long long)H * L.Rp; g.c_bf16 = m->cfg.bf16;
   g.nseg = H; g.a_stride = L.dp; g.w_stride = (long long)L.Rp * L.dp; g.c_stride = L.Rp;
   TRY(batched(m, g));
   LatentArgs a;
   a.qc = b.qc; a.plane = kv->k[run]; a.table = hc.table_dev; a.max_pages = hc.max_pages; a.Rp = L.Rp; a.H = H;
-  a.window = L.window; a.scale = L.scale; a.sink = L.f_b; a.gate = b.gate; a.out = b.oc; a.rows = rows;
-  const bool mma = m->cfg.bf16 && L.Rp <= 512 && !m->force_simt_attn;
+  a.window = L.window; a.scale = L.scale; a.sink = L.sinks ? L.f_b : nullptr; a.gate = b.gate; a.out = b.oc; a.rows = rows;
+  const bool mma = m->cfg.bf16 && L.Rp <= 576 && !m->force_simt_attn;
   if (mma && M <= SPLIT_ROWS) {       // few rows: several CTAs share a tile's key pages
     const int tile = latent_tile_rows(L.Rp, rows.max_n * H), tiles = rows.n_ent * ceil_div(rows.max_n * H, tile);
     const int pages = L.window > 0 ? std::min(hc.max_pages, (L.window + rows.max_n) / KV_PAGE + 2) : hc.max_pages;
@@ -715,7 +916,7 @@ int32_t latent_attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc,
   TRY(vn_latent_attention(ctx, a, m->cfg.bf16 != 0, mma));
   g = gemm_args(b.oc, H * L.Rp, L.w_uv, L.vd, L.Rp, M, "gemm_latent_uv");
   g.C = b.mix; g.ldc = (long long)H * L.vd; g.c_bf16 = m->cfg.bf16;
-  g.nseg = H; g.a_stride = L.Rp; g.w_stride = (long long)L.vd * L.Rp; g.c_stride = L.vd;
+  g.nseg = H; g.a_stride = L.Rp; g.w_stride = (long long)L.vd * L.Rp; g.c_stride = L.vd; g.mul = b.gate_t;
   return batched(m, g);
 }
 
@@ -724,6 +925,17 @@ ConvIn<T> conv_in(const HLayer& L, const Cache& hc, const Src& s, void* ring) {
   ConvIn<T> c;
   c.src = s; c.ring = (T*)ring; c.RC = L.taps - 1 + hc.pending; c.C = L.conv_ch(); c.taps = L.taps; c.w = L.conv; c.bias = L.conv_b;
   return c;
+}
+
+int32_t ensure_segments(vn_model* m, size_t bytes) {
+  Model& hm = *m->hyb;
+  if (bytes <= hm.seg_bytes) return VN_OK;
+  VN_CUDA(m->ctx, cudaStreamSynchronize(m->ctx->stream));
+  if (hm.seg) cudaFree(hm.seg);
+  hm.seg = nullptr; hm.seg_bytes = 0;
+  TRY(dev_alloc(m->ctx, (void**)&hm.seg, bytes));
+  hm.seg_bytes = bytes;
+  return VN_OK;
 }
 
 template <typename T>
@@ -759,6 +971,42 @@ int32_t mamba1(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLa
   TRY(linear(m, g));
   a.dt = b.dt;
   return vn_mamba_scan(ctx, a, m->cfg.bf16 != 0);
+}
+
+// S: Src, or the 16-bit matrix of a forward of many rows
+template <typename T, typename S>
+int32_t mamba2(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  const int M = rows.M, D = hm.D;
+  ConvIn<T, S> cv;
+  TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_ssd_in"), b.proj, &cv.src));
+  cv.col0 = L.inner; cv.ring = (T*)kv->k[run]; cv.RC = L.taps - 1 + hc.pending; cv.C = L.conv_ch(); cv.taps = L.taps; cv.w = L.conv; cv.bias = L.conv_b;
+  SsdArgs a;
+  a.H = L.H; a.P = L.vd; a.N = L.nstate; a.G = L.groups; a.xbc = b.xbc; a.ld = up8(L.conv_ch()); a.dt = b.dt; a.dt_bias = L.f_c; a.A = L.f_d; a.D = L.f_b;
+  a.state = (float*)kv->v[run]; a.R = hc.ring_len; a.pending = hc.pending; a.u = b.u; a.rows = rows;
+  bool step = false;
+  if constexpr (std::is_same<S, Src>::value) {
+    step = rows.max_n == 1;
+    if (step) TRY(vn_ssd_step<T>(ctx, cv, a));
+  }
+  if (!step) {
+    TRY((vn_ssd_inputs<T, S>(ctx, cv, a)));
+    if (rows.max_n > hc.pending && L.taps > 1)
+      VN_LAUNCH(ctx, (conv_tail_kernel<T, S, true>), dim3(ceil_div(cv.C, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
+    const SsdPlan plan = vn_ssd_plan(ctx, m->cfg.bf16 != 0, L.H, L.nstate, L.vd, rows, hc.pending);
+    if (plan.chunked) {
+      if constexpr (std::is_same<T, __nv_bfloat16>::value) {
+        TRY(ensure_segments(m, plan.seg_bytes));
+        a.segments = plan.segments; a.seg_len = plan.seg_len; a.seg_state = hm.seg;
+        a.seg_decay = hm.seg + (long long)rows.n_ent * plan.segments * L.H * L.nstate * L.vd;
+        TRY(vn_ssd_chunks(ctx, cv.src, a));
+      }
+    } else {
+      TRY((vn_ssd_scan<T, S>(ctx, cv.src, a)));
+    }
+  }
+  return vn_ssd_norm<T>(ctx, (const T*)b.u, L.f_a, (T*)b.mix, M, L.inner, L.norm_groups, hm.eps);
 }
 
 template <typename T>
@@ -810,7 +1058,9 @@ int32_t attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const 
   TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_attn_in"), b.proj, &cv.src));
   cv.ring = (T*)hc.ring[run]; cv.RC = L.taps - 1 + hc.pending; cv.C = L.conv_ch(); cv.taps = L.taps; cv.w = L.conv;
   PagedAttnArgs a;
-  a.H = L.H; a.KH = L.KH; a.d = L.d; a.vd = L.vd; a.P = L.P; a.window = L.window; a.scale = L.scale; a.rd = L.rd;
+  a.H = L.H; a.KH = L.KH; a.d = L.d; a.vd = L.vd; a.P = L.P; a.window = L.window; a.chunk = L.chunk; a.scale = L.scale; a.softcap = L.softcap; a.rd = L.rd;
+  a.interleaved = L.interleaved; a.qn = L.f_a; a.kn = L.f_b; a.eps = hm.eps;
+  cv.bias = L.f_c;
   a.rope = L.rope >= 0 ? hm.ropes[L.rope].table : nullptr;
   a.own_kv = from == run;
   a.kplane = kv->k[from]; a.vplane = kv->v[from]; a.table = hc.table_dev; a.max_pages = hc.max_pages;
@@ -819,7 +1069,9 @@ int32_t attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const 
   const bool mma = m->cfg.bf16 && attn_mma_ok(L.P) && !m->force_simt_attn;
   if constexpr (std::is_same<T, __nv_bfloat16>::value && std::is_same<S, Src>::value) {
     if (mma && rows.max_n == 1) {
-      const int ctas = L.KH * ceil_div(L.H / L.KH, 16) * M, keys = L.window > 0 ? std::min(L.window, kv->max_seq) : kv->max_seq;
+      const int ctas = L.KH * ceil_div(L.H / L.KH, 16) * M;
+      int keys = kv->max_seq;
+      for (int reach : {L.window, L.chunk}) if (reach > 0) keys = std::min(keys, reach);
       a.splits = M > SPLIT_ROWS ? 1 : std::max(1, std::min(std::min(MAX_SPLITS, ceil_div(keys, 64)), 2 * ctx->sm_count / ctas));
       a.part_o = b.part_o; a.part_ml = b.part_ml;
       TRY(vn_tickets(ctx, &a.tickets));
@@ -842,13 +1094,7 @@ int32_t lightning(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const 
   LightningArgs a;
   a.H = L.H; a.d = L.d; a.vd = L.vd; a.decay = L.f_b; a.powers = L.f_c; a.norm_w = L.f_a; a.state = (float*)kv->v[run]; a.R = hc.ring_len;
   a.out = b.mix; a.ss = b.ss; a.n_ss = *n_ss = plan.n_ss; a.segments = plan.segments; a.seg_len = plan.seg_len; a.rows = rows;
-  if (plan.seg_bytes > hm.seg_bytes) {
-    VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    if (hm.seg) cudaFree(hm.seg);
-    hm.seg = nullptr; hm.seg_bytes = 0;
-    TRY(dev_alloc(ctx, (void**)&hm.seg, plan.seg_bytes));
-    hm.seg_bytes = plan.seg_bytes;
-  }
+  TRY(ensure_segments(m, plan.seg_bytes));
   a.seg_state = hm.seg;
   GemmArgs g = gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_lightning_in");
   S s;
@@ -909,6 +1155,99 @@ int32_t gated_up(vn_model* m, const HLayer& L, int M, const Buffers& b) {
   }
   g.C = b.act; g.ldc = L.ffp; g.epi = EPI_SWIGLU; g.act = L.act; g.c_bf16 = m->cfg.bf16;
   return linear(m, g);
+}
+
+// Mixture of experts: x += the weighted results of each row's experts, m->h as `next` says.  The rows are copied into expert
+// order; few rows go as one segment per expert through split-K GEMMs, many as pieces of 256 rows.
+template <typename T>
+int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Next& next) {
+  vn_ctx* ctx = m->ctx;
+  Model& hm = *m->hyb;
+  const int D = hm.D, n = L.n_out(), S = L.top, F = L.ffp;
+  const bool bf = m->cfg.bf16;
+  RouteIn r;
+  TRY(project(m, gemm_args(m->h, D, L.w_router, n, D, M, "gemm_router"), b.logits, &r.z));
+  r.correction = L.correction; r.M = M; r.E = n; r.top = S; r.groups = L.exp_groups; r.keep = L.keep;
+  r.slot_expert = b.slot_expert; r.slot_w = b.slot_w; r.count = hm.exp_count;
+  VN_LAUNCH_PDL_LEVEL(ctx, 1, "route_kernel", route_kernel, ceil_div(M, ROUTE_WARPS), 32 * ROUTE_WARPS, (size_t)ROUTE_WARPS * (2 * n + L.exp_groups) * 4, r);
+  AddExperts<T, Src> few;
+  few.h = (const T*)m->h; few.slot_pos = b.slot_pos; few.slot_expert = b.slot_expert; few.slot_w = b.slot_w; few.top = S; few.n_real = L.n_exp; few.D = D;
+  few.count = hm.exp_count; few.cursor = hm.exp_cur; few.n_count = n;
+  few.y.ld = D;
+  GemmArgs up, down;
+  up.A = b.hs; up.lda = D; up.W = L.w_gu; up.ldw = D; up.w_stride = (long long)2 * F * D; up.N = 2 * F; up.K = D; up.tag = "gemm_expert_gateup";
+  up.C = b.act; up.ldc = F; up.epi = EPI_SWIGLU; up.act = L.act; up.c_bf16 = bf;
+  down.A = b.act; down.lda = F; down.W = L.w_down; down.ldw = F; down.w_stride = (long long)D * F; down.N = D; down.K = F; down.tag = "gemm_expert_down";
+  down.C = b.ey; down.ldc = D; down.c_bf16 = bf;
+  up.M = down.M = M;
+  const bool tc = bf && m->use_tc && D % 8 == 0 && tc_detail::encode_fn() != nullptr;
+  if (tc && M <= 256) {
+    VN_LAUNCH_PDL_LEVEL(ctx, 1, "mod_dispatch_kernel", mod_dispatch_kernel<T>, M * S, 128, 0, (const T*)m->h, b.slot_expert, hm.exp_count, hm.exp_off, hm.exp_cur,
+                        b.slot_pos, (T*)b.hs, n, S, D);
+    up.seg_off = down.seg_off = hm.exp_off; up.seg_cnt = down.seg_cnt = hm.exp_count; up.nseg = down.nseg = L.n_exp;
+    const int active = std::min(L.n_exp, M * S);          // segments with rows, at most
+    int sp = 1;
+    TRY(tc_partial(m, up, (long long)M * S, (long long)M * S, &sp, active));
+    const long long pairs = (long long)M * S * F;
+    VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp, (long long)M * S * 2 * F, (T*)b.act, 2 * F,
+                      pairs, L.act);
+    TRY(tc_partial(m, down, (long long)M * S, (long long)M * S, &sp, active));
+    few.y.p = m->partial; few.y.splits = sp; few.y.pstride = (long long)M * S * D;
+    return close_rows<T>(m, few, M, nullptr, next);
+  }
+  VN_LAUNCH(ctx, mod_offsets_kernel, 1, 32, 0, hm.exp_count, hm.exp_off, hm.exp_cur, n);
+  VN_LAUNCH(ctx, mod_scatter_kernel, ceil_div(M * S, 256), 256, 0, b.slot_expert, hm.exp_off, hm.exp_cur, b.sorted_row, b.slot_pos, M * S, S);
+  if (tc) {
+    int *off = b.sub_seg, *cnt = off + b.sub_cap, *w = cnt + b.sub_cap;
+    VN_LAUNCH(ctx, mod_subseg_kernel, 1, 32, 0, (const int*)hm.exp_count, (const int*)hm.exp_off, L.n_exp, off, cnt, w, b.sub_cap);
+    VN_LAUNCH(ctx, gather_sorted_kernel<T>, M * S, 128, 0, (const T*)m->h, (const int*)b.sorted_row, (T*)b.hs, D);
+    TRY(ensure_partial(m, 1024));
+    for (GemmArgs* g : {&up, &down}) {
+      g->M = 256; g->seg_off = off; g->seg_cnt = cnt; g->seg_w = w; g->n_w = L.n_exp; g->nseg = b.sub_cap;
+      TcPlan plan;
+      plan.error_flag = m->tc_error;
+      TRY(launch_gemm_tc(ctx, *g, (long long)M * S, plan));
+    }
+  } else {                                                // the kernels of any shape gather the rows themselves
+    up.A = m->h; up.a_rows = b.sorted_row;
+    for (GemmArgs* g : {&up, &down}) {
+      g->seg_off = hm.exp_off; g->seg_cnt = hm.exp_count; g->nseg = L.n_exp;
+      TRY(linear(m, *g));
+    }
+  }
+  if constexpr (std::is_same<T, __nv_bfloat16>::value) {
+    AddExperts<T, Mat<T>> y;
+    y.y.p = (const T*)b.ey; y.y.ld = D;
+    y.h = few.h; y.slot_pos = few.slot_pos; y.slot_expert = few.slot_expert; y.slot_w = few.slot_w; y.top = S; y.n_real = few.n_real; y.D = D;
+    y.count = few.count; y.cursor = few.cursor; y.n_count = n;
+    return close_rows<T>(m, y, M, nullptr, next);
+  } else {
+    few.y.p = (const float*)b.ey;
+    return close_rows<T>(m, few, M, nullptr, next);
+  }
+}
+
+// x += norm(W_proj (gelu(W_gate x) * e)): e is the layer's part of the tokens' side embeddings, m->h holds x
+template <typename T>
+int32_t side_input(vn_model* m, const int64_t* tokens, const HLayer& L, int layer, int M, const Buffers& b, const Next& next) {
+  vn_ctx* ctx = m->ctx;
+  const Model& hm = *m->hyb;
+  const int D = hm.D;
+  Src gate;
+  TRY(project(m, gemm_args(m->h, D, L.w_sgate, up4(hm.side), D, M, "gemm_side_gate"), b.proj, &gate));
+  const long long total = (long long)M * hm.sidep;
+  VN_LAUNCH_PDL_LEVEL(ctx, 1, "side_act_kernel", side_act_kernel<T>, (unsigned)ceil_div(total, 256ll), 256, 0, gate, (const long long*)tokens, hm.vocab,
+                      (const T*)hm.side_embed, (long long)hm.layers.size() * hm.side, layer * hm.side, hm.side, (T*)b.side_act, hm.sidep, total);
+  const GemmArgs g = gemm_args(b.side_act, hm.sidep, L.w_sproj, D, hm.sidep, M, "gemm_side_proj");
+  if constexpr (std::is_same<T, __nv_bfloat16>::value)
+    if (M > 256) {
+      AddRows<Mat<T>> y;
+      TRY(project(m, g, b.proj, &y.y));
+      return close_rows<T>(m, y, M, L.s_norm, next);
+    }
+  AddRows<Src> y;
+  TRY(project(m, g, b.proj, &y.y));
+  return close_rows<T>(m, y, M, L.s_norm, next);
 }
 
 // act = relu(h W_up^T)^2, and the raw gate of the result beside it when the model has one
@@ -1035,6 +1374,15 @@ int32_t forward_arranged(vn_model* m, vn_kv* kv, const int64_t* tokens, const Ro
   return out_logits ? head(m, pick.n, out_logits) : VN_OK;
 }
 
+// mixers that read a projection of many rows in 16 bits
+template <typename T>
+int32_t dense_projection_mixer(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+  if constexpr (std::is_same<T, __nv_bfloat16>::value)
+    if (rows.M > 256)
+      return L.kind == MAMBA2 ? mamba2<T, Mat<T>>(m, in_rows, kv, hc, L, run, rows, b) : attention<T, Mat<T>>(m, in_rows, kv, hc, L, run, rows, b);
+  return L.kind == MAMBA2 ? mamba2<T, Src>(m, in_rows, kv, hc, L, run, rows, b) : attention<T, Src>(m, in_rows, kv, hc, L, run, rows, b);
+}
+
 template <typename T>
 int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows, const Pick& pick, float* out_hidden,
                 float* out_logits) {
@@ -1067,17 +1415,21 @@ int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows,
     } else if (i == 0) {
       VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, L.norm1, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
     }
-    const float* next_norm = i + 1 < n_runs && !enters_pass(i + 1) ? hm.layers[hm.runs[i + 1].layer].norm1 : nullptr;
+    const Next next_layer{i + 1 < n_runs && !enters_pass(i + 1) ? hm.layers[hm.runs[i + 1].layer].norm1 : nullptr, false};
+    const Next after_ff = hm.side ? Next{nullptr, true} : next_layer, after_mix = L.ff ? Next{L.norm2, false} : after_ff;
     if (L.kind == LATENT) TRY(latent_attention<T>(m, m->h, kv, hc, L, i, rows, b));
     else if (L.kind == MAMBA1) TRY(mamba1<T>(m, m->h, kv, hc, L, i, rows, b));
     else if (L.kind == DELTA) TRY(channel_delta<T>(m, m->h, kv, hc, L, i, rows, b));
-    else TRY((attention<T, Src>(m, m->h, kv, hc, L, i, rows, b)));
+    else TRY((dense_projection_mixer<T>(m, m->h, kv, hc, L, i, rows, b)));
     const int width = L.kind == MAMBA1 ? L.inner : L.H * L.vd;
-    TRY(close_block<T>(m, gemm_args(b.mix, width, L.w_o, D, width, M, "gemm_mix_out"), L.ff ? L.norm2 : next_norm));
-    if (L.ff) {
+    TRY(close_block<T>(m, gemm_args(b.mix, width, L.w_o, D, width, M, "gemm_mix_out"), L.o_b, after_mix));
+    if (L.n_exp) {
+      TRY(mixture<T>(m, L, M, b, after_ff));
+    } else if (L.ff) {
       TRY(gated_up<T>(m, L, M, b));
-      TRY(close_block<T>(m, gemm_args(b.act, L.ffp, L.w_down, D, L.ffp, M, "gemm_ff_down"), next_norm));
+      TRY(close_block<T>(m, gemm_args(b.act, L.ffp, L.w_down, D, L.ffp, M, "gemm_ff_down"), nullptr, after_ff));
     }
+    if (hm.side) TRY(side_input<T>(m, tokens, L, hm.runs[i].layer, M, b, next_layer));
     if (hm.probe)
       VN_CUDA(ctx, cudaMemcpyAsync(hm.probe + (size_t)i * M * D, m->x, (size_t)M * D * 4, cudaMemcpyDeviceToDevice, ctx->stream));
   }

@@ -396,7 +396,7 @@ int32_t linear(vn_model* m, GemmArgs g) {
     // row segments, every segment with the same weight matrix (stride 0).  A weight tile is then fetched once per
     // segment, from L2 after the first.  VN_PREFILL_TC=0 (read per call) keeps the mma.sync kernel.
     const char* pe = getenv("VN_PREFILL_TC");
-    if (m->use_tc && !(pe && pe[0] == '0') && g.M > 256 && !g.seg_cnt && !g.a_rows && g.nseg == 1 && !g.bias &&
+    if (m->use_tc && !(pe && pe[0] == '0') && g.M > 256 && !g.seg_cnt && !g.a_rows && g.nseg == 1 && (!g.bias || g.epi != EPI_SWIGLU) && !g.mul &&
         g.K % tc_detail::BK == 0 && g.N >= tc_detail::BF && g.ldw_k == 1 && tc_detail::encode_fn() != nullptr &&
         (g.epi == EPI_STORE || g.epi == EPI_ADD || g.epi == EPI_SWIGLU) && (!g.post || g.c_bf16)) {
       const int nseg = ceil_div(g.M, 256);
@@ -695,9 +695,10 @@ int32_t tc_launch(vn_ctx* ctx, const GemmArgs& g, long long a_rows, TcPlan& plan
 }
 
 // launches the GEMM into the split-K workspace; returns the number of partial slices through *splits_out
-int32_t tc_partial(vn_model* m, GemmArgs g, long long a_rows, long long c_rows, int* splits_out) {
+// (`active`: how many of the segments have rows, when that is known to be fewer)
+int32_t tc_partial(vn_model* m, GemmArgs g, long long a_rows, long long c_rows, int* splits_out, int active = 0) {
   vn_ctx* ctx = m->ctx;
-  const int splits = tc_splits(ctx, g.N, g.K, g.nseg);
+  const int splits = tc_splits(ctx, g.N, g.K, active > 0 ? active : g.nseg);
   TRY(ensure_partial(m, (size_t)splits * c_rows * g.N * 4));
   TcPlan plan;
   plan.splits = splits; plan.force_partial = true;

@@ -1,0 +1,94 @@
+// Mixture of experts: which experts a row goes to.  Scores are the soft-max over all router outputs; the choice may see a
+// correction per expert and be limited to the best groups of neighbouring experts; the weights are the plain scores.  The last
+// outputs may be identity experts, whose result is their input.  Rows are then laid out expert by expert by the kernels that
+// serve the other mixtures (mod_dispatch_kernel, or mod_offsets / mod_scatter / gather_sorted).
+#pragma once
+#include "rows.cuh"
+#include <math_constants.h>
+
+constexpr int ROUTE_WARPS = 4, MAX_CHOSEN = 32;
+
+struct RouteIn {
+  Src z;                               // [M, E] router outputs
+  const float* correction = nullptr;   // [E] or null
+  int M = 0, E = 0, top = 1, groups = 1, keep = 1;
+  int* slot_expert = nullptr;          // [M, top]
+  float* slot_w = nullptr;             // [M, top]
+  int* count = nullptr;                // [E], zero before the launch
+};
+
+// the largest value over a warp's lanes and its index (the lowest one among equals)
+__device__ __forceinline__ void warp_argmax(float& v, int& i) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+    if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
+  }
+}
+
+// one warp per row; shared memory: ROUTE_WARPS x (2 E + groups) floats.  grid ceil(M / ROUTE_WARPS)
+__global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(RouteIn r) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float s_route[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x * ROUTE_WARPS + warp, E = r.E;
+  if (row >= r.M) return;
+  float* score = s_route + warp * (2 * E + r.groups);
+  float* choice = score + E;
+  float* best = choice + E;
+  float top = -CUDART_INF_F;
+  for (int e = lane; e < E; e += 32) {
+    const float z = r.z.get(row, e);
+    score[e] = z;
+    top = fmaxf(top, z);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+  float sum = 0.f;
+  for (int e = lane; e < E; e += 32) { const float x = expf(score[e] - top); score[e] = x; sum += x; }
+  sum = warp_sum(sum);
+  for (int e = lane; e < E; e += 32) {
+    const float s = score[e] / sum;
+    score[e] = s;
+    choice[e] = r.correction ? s + r.correction[e] : s;
+  }
+  __syncwarp();
+  const int per = E / r.groups;
+  if (r.keep < r.groups) {
+    for (int g = lane; g < r.groups; g += 32) {
+      float m = choice[g * per];
+      for (int i = 1; i < per; ++i) m = fmaxf(m, choice[g * per + i]);
+      best[g] = m;
+    }
+    __syncwarp();
+    // the groups that are not kept: all but `keep` times the largest
+    for (int k = 0; k < r.keep; ++k) {
+      float v = -CUDART_INF_F;
+      int at = r.groups;
+      for (int g = lane; g < r.groups; g += 32)
+        if (best[g] != CUDART_INF_F && (best[g] > v || at == r.groups)) { v = best[g]; at = g; }
+      warp_argmax(v, at);
+      if (lane == 0 && at < r.groups) best[at] = CUDART_INF_F;          // marks a kept group
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (best[e / per] != CUDART_INF_F) choice[e] = -CUDART_INF_F;
+    __syncwarp();
+  }
+  for (int k = 0; k < r.top; ++k) {
+    float v = -CUDART_INF_F;
+    int at = E;
+    for (int e = lane; e < E; e += 32)
+      if (choice[e] > v) { v = choice[e]; at = e; }
+    warp_argmax(v, at);
+    if (lane == 0) {
+      at = at < E ? at : 0;                                             // not finite scores: any expert
+      r.slot_expert[(long long)row * r.top + k] = at;
+      r.slot_w[(long long)row * r.top + k] = score[at];
+      atomicAdd(r.count + at, 1);
+      choice[at] = -CUDART_INF_F;
+    }
+    __syncwarp();
+  }
+}

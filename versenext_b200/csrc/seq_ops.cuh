@@ -69,6 +69,164 @@ __global__ void __launch_bounds__(256) rowsum_norm_kernel(Src src, const float* 
   for (int d = threadIdx.x; d < D; d += 256) y[row * D + d] = from_f<T>(x[row * D + d] / r * norm_w[d]);
 }
 
+// ---- the end of a sublayer in one pass over a row: what it adds, the residual, and what the next product reads -------------
+// Y gives the addend: quad(row, d) of four columns, one(row, d) of one; begin(row) is called by all 256 threads first.
+
+// a projection's result with a bias
+template <typename S>
+struct AddRows {
+  S y;
+  const float* bias = nullptr;
+  __device__ __forceinline__ void begin(int) {}
+  __device__ __forceinline__ float4 quad(int row, int d) const {
+    float4 v = get4(y, row, d);
+    if (bias) { const float4 b = load4(bias + d); v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w; }
+    return v;
+  }
+  __device__ __forceinline__ float one(int row, int d) const { return y.get(row, d) + (bias ? bias[d] : 0.f); }
+};
+
+// the weighted results of a row's experts: rows slot_pos[] of y; experts from n_real on are the input h itself
+template <typename T, typename S>
+struct AddExperts {
+  S y;
+  const T* h = nullptr;
+  const int *slot_pos = nullptr, *slot_expert = nullptr;
+  const float* slot_w = nullptr;
+  int top = 1, n_real = 0, D = 0;
+  int *count = nullptr, *cursor = nullptr;       // left at zero for the next mixture
+  int n_count = 0;
+  int* pos;                                      // of the chosen experts with results; shared memory
+  float* w;
+  int n;
+  float w_self;
+  __device__ __forceinline__ void begin(int row) {
+    __shared__ int s_pos[32];
+    __shared__ float s_w[32];
+    pos = s_pos; w = s_w;
+    const int lane = threadIdx.x & 31;           // every warp finds out for itself; they write the same values
+    const bool has = lane < top;
+    const int e = has ? slot_expert[(long long)row * top + lane] : n_real;
+    const float v = has ? slot_w[(long long)row * top + lane] : 0.f;
+    const unsigned real = __ballot_sync(0xffffffffu, has && e < n_real);
+    if (has && e < n_real) {
+      const int at = __popc(real & ((1u << lane) - 1));
+      s_pos[at] = slot_pos[(long long)row * top + lane];
+      s_w[at] = v;
+    }
+    n = __popc(real);
+    w_self = warp_sum(has && e >= n_real ? v : 0.f);
+    if (blockIdx.x == 0)
+      for (int i = threadIdx.x; i < n_count; i += 256) { count[i] = 0; cursor[i] = 0; }
+    __syncthreads();
+  }
+  __device__ __forceinline__ float4 quad(int row, int d) const {
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (w_self != 0.f) { const float4 t = load4(h + (long long)row * D + d); a = make_float4(t.x * w_self, t.y * w_self, t.z * w_self, t.w * w_self); }
+#pragma unroll 4
+    for (int j = 0; j < n; ++j) {
+      const float4 t = get4(y, pos[j], d);
+      const float f = w[j];
+      a.x = fmaf(t.x, f, a.x); a.y = fmaf(t.y, f, a.y); a.z = fmaf(t.z, f, a.z); a.w = fmaf(t.w, f, a.w);
+    }
+    return a;
+  }
+  __device__ __forceinline__ float one(int row, int d) const {
+    float a = w_self != 0.f ? w_self * to_f<T>(h[(long long)row * D + d]) : 0.f;
+    for (int j = 0; j < n; ++j) a = fmaf(y.get(pos[j], d), w[j], a);
+    return a;
+  }
+};
+
+// x += y, or y over its root mean square times own_norm; then h = RMSNorm(x) * next_norm, or x itself (cast), or nothing.
+// NV > 0: four columns per thread, NV times, held in registers (D % 4 == 0, D <= 1024 NV); 0: any D.  grid M
+template <typename T, typename Y, int NV>
+__global__ void __launch_bounds__(256) residual_kernel(Y y, float* __restrict__ x, const float* __restrict__ own_norm,
+                                                       const float* __restrict__ next_norm, int cast, T* __restrict__ h, int D, float eps) {
+  __shared__ float sm[2][8];
+  pdl_trigger();
+  pdl_wait();
+  const int row = blockIdx.x;
+  float* xr = x + (long long)row * D;
+  T* hr = h + (long long)row * D;
+  y.begin(row);
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+    float4 v[NV], xv[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (threadIdx.x + 256 * i) * 4;
+      v[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (d < D) { xv[i] = load4(xr + d); v[i] = y.quad(row, d); }
+    }
+    if (own_norm) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+      const float r = 1.f / sqrtf(block_sum256(ss, sm[0]) / (float)D + eps);
+      ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int d = (threadIdx.x + 256 * i) * 4;
+        if (d >= D) break;
+        const float4 w = load4(own_norm + d);
+        v[i] = make_float4(v[i].x * r * w.x, v[i].y * r * w.y, v[i].z * r * w.z, v[i].w * r * w.w);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (threadIdx.x + 256 * i) * 4;
+      if (d >= D) break;
+      xv[i] = make_float4(xv[i].x + v[i].x, xv[i].y + v[i].y, xv[i].z + v[i].z, xv[i].w + v[i].w);
+      store4(xr + d, xv[i]);
+      if (cast) store4(hr + d, xv[i]);
+      ss += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+    }
+    if (!next_norm) return;
+    const float r = 1.f / sqrtf(block_sum256(ss, sm[1]) / (float)D + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int d = (threadIdx.x + 256 * i) * 4;
+      if (d >= D) break;
+      const float4 w = load4(next_norm + d);
+      store4(hr + d, make_float4(xv[i].x * r * w.x, xv[i].y * r * w.y, xv[i].z * r * w.z, xv[i].w * r * w.w));
+    }
+  } else {
+    float f = 1.f;
+    if (own_norm) {
+      for (int d = threadIdx.x; d < D; d += 256) { const float v = y.one(row, d); ss += v * v; }
+      f = 1.f / sqrtf(block_sum256(ss, sm[0]) / (float)D + eps);
+      ss = 0.f;
+    }
+    for (int d = threadIdx.x; d < D; d += 256) {
+      float v = y.one(row, d);
+      if (own_norm) v *= f * own_norm[d];
+      v += xr[d];
+      xr[d] = v;
+      if (cast) hr[d] = from_f<T>(v);
+      ss += v * v;
+    }
+    if (!next_norm) return;
+    const float r = 1.f / sqrtf(block_sum256(ss, sm[1]) / (float)D + eps);
+    for (int d = threadIdx.x; d < D; d += 256) hr[d] = from_f<T>(xr[d] * r * next_norm[d]);
+  }
+}
+
+// A layer's own input for a token: act = gelu(gate) * the layer's part of the token's side embedding, n columns padded to ld.
+// table [V, pitch]; grid ceil(M ld / 256)
+template <typename T>
+__global__ void __launch_bounds__(256) side_act_kernel(Src gate, const long long* __restrict__ tokens, int V, const T* __restrict__ table,
+                                                       long long pitch, int col0, int n, T* __restrict__ act, int ld, long long total) {
+  pdl_trigger();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= total) return;
+  const long long row = i / ld;
+  const int j = (int)(i % ld);
+  long long tok = tokens[row];
+  tok = tok < 0 ? 0 : tok >= V ? V - 1 : tok;            // the embedding has raised the flag
+  act[i] = from_f<T>(j < n ? gelu_tanh(gate.get(row, j)) * to_f<T>(table[tok * pitch + col0 + j]) : 0.f);
+}
+
 // y = RMSNorm(x[row_of(i)]) * w: rows picked by a list, by (i * mul + add), or the entries' last rows
 template <typename T>
 __global__ void __launch_bounds__(256) rmsnorm_pick_kernel(const float* __restrict__ x, const float* __restrict__ w,
