@@ -27,6 +27,7 @@ from .speculative import SpeculativeDecoder, Tensor, no_grad
 from .model import VerseNexLM, CometSparkNexLM, KVCache, build_verse_delta_pattern
 from .engine import SpecEngine
 from .composed import ComposedLM
+from .bozasun import BozasunLM
 from .fuzudra import FuzudraLM
 from .musutar import MusutarLM
 from .serving import BatchEngine, StepRunner
@@ -39,6 +40,6 @@ from . import sampling
 from . import quant
 
 __all__ = ["Context", "DeviceArray", "as_device", "DeviceBackend", "B200Backend", "get_backend",
-           "clear_backend_cache", "SpeculativeDecoder", "Tensor", "no_grad", "sampling", "quant", "VerseNexLM", "CometSparkNexLM", "KVCache", "ComposedLM", "FuzudraLM", "MusutarLM",
+           "clear_backend_cache", "SpeculativeDecoder", "Tensor", "no_grad", "sampling", "quant", "VerseNexLM", "CometSparkNexLM", "KVCache", "ComposedLM", "BozasunLM", "FuzudraLM", "MusutarLM",
            "load_model", "BatchEngine", "StepRunner", "build_verse_delta_pattern", "SpecEngine", "TreeSpecEngine",
            "ShardedSpecEngine", "Comm", "rank_seed", "VNFileReader", "load_vn"]

@@ -4,17 +4,20 @@
 optional feed-forward; an optional looped block; the norm and its eps; the kind of positions; the arrangement of the
 residual) and offers what every model of the package offers: weight loading, caches, uniform and ragged steps, generation,
 speculative decoding as target or draft.  A named design is a subclass of `DesignLM` that translates its own config.json
-(see fuzudra.py, musutar.py).
+(see bozasun.py, fuzudra.py, musutar.py).
 
-Mixers: "latent_attention" (heads, dim, vdim, kv_rank, scale, window), "attention" (heads, kv_heads, dim, vdim, scale,
-window, conv, rope {dims, base, scaling {factor, original, fast, slow}}, output_gate, kv_from), "mamba1" (inner, state,
-dt_rank, conv), "channel_delta" (heads, kv_heads, dim, vdim, conv, decay_rank, gate_rank), "lightning" (heads, dim, vdim,
-decay).
+Mixers: "latent_attention" (heads, dim, vdim, kv_rank, scale, window, rot_dim with rope, sink, output_gate "head", "element" or
+"none"), "attention" (heads, kv_heads, dim, vdim, scale, window, chunk, softcap, conv, rope, bias, qk_norm, output_gate, kv_from),
+"mamba1" (inner, state, dt_rank, conv), "mamba2" (heads, vdim, state, groups, norm_groups, conv), "channel_delta" (heads,
+kv_heads, dim, vdim, conv, decay_rank, gate_rank), "lightning" (heads, dim, vdim, decay).  rope: {dims, base, interleaved,
+scaling: YaRN {factor, original, fast, slow} or {kind: "linear", factor}}.
 
-Feed-forwards: mlp_hidden with mlp_act "silu" or "gelu_tanh" (gated) or "relu2" (plain).
+Feed-forwards: mlp_hidden with mlp_act "silu" or "gelu_tanh" (gated) or "relu2" (plain); with experts {count, identity, top,
+groups, keep, correction} a mixture of gated ones.
 
-Model-wide: norm "rms" (weights stored around zero) or "layer" (plain weights); streams (residual streams, hyper-connections);
-input_conv (taps of the convolution that a mixer's input gets); residual_gate (sigmoid gate on every sublayer's result).
+Model-wide: norm "rms" (weights stored around zero, or plain: norm_weight "plain") or "layer" (plain weights); streams (residual
+streams, hyper-connections); input_conv (taps of the convolution that a mixer's input gets); residual_gate (sigmoid gate on every
+sublayer's result); token_side (width of the input that every layer has for each token).
 """
 
 from __future__ import annotations

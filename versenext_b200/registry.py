@@ -5,6 +5,7 @@ from __future__ import annotations
 import json
 import os
 
+from .bozasun import BozasunLM
 from .fuzudra import FuzudraLM
 from .model import DeviceLM, VerseNexLM
 from .musutar import MusutarLM
@@ -39,6 +40,7 @@ def load_model(path: str, dtype: str = "bf16", device: str = "cuda", **kw) -> De
     return VerseNexLM.from_pretrained(path, dtype=dtype, device=device, **kw)
 
 
+register(BozasunLM.ARCHITECTURE, BozasunLM)
 register(FuzudraLM.ARCHITECTURE, FuzudraLM)
 register(MusutarLM.ARCHITECTURE, MusutarLM)
 register("VerseNexLM", VerseNexLM)
