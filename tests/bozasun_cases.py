@@ -179,9 +179,10 @@ def prompt(cfg, n, seed=1, sd=None):
             close = close_calls(sd, cfg, toks)
             if not close.any():
                 return toks
-            first = np.argmax(close)                         # what comes before it stays as it is
-            redo = close & (np.arange(n) < first + 40)
-            toks[redo] = rng.integers(0, cfg["vocab"], redo.sum())
+            new = rng.integers(0, cfg["vocab"], n)
+            if n > 9:                                        # half of them from those that are clear in this prompt
+                new = np.where(rng.random(n) < 0.5, rng.choice(toks[~close], n), new)
+            toks = np.where(close, new, toks)
         raise AssertionError("no prompt without close calls")
     return toks
 

@@ -206,6 +206,67 @@ def musutar_shapes(cfg: dict) -> dict:
     return s
 
 
+def bozasun_config(width: int, vocab: int = 32000, n_layer: int = 4) -> dict:
+    """config.json contents: chunked attention with a dense feed-forward, Mamba-2 and latent attention with mixtures, Mamba-2
+    with a dense feed-forward in turn; heads of 128 (64 below width 2048), four query heads per key head, chunks of 1024, a
+    state of 128 per channel, feed-forwards as wide as VerseNexLM's, mixtures of experts a quarter as wide of which a token
+    uses about as many."""
+    hd = 128 if width >= 2048 else 64
+    heads, ff = width // hd, int((4 * width * 2 / 3 + 63) // 64) * 64
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": (ff // 4 + 63) // 64 * 64},
+           "router": {"experts": 24, "identity": 8, "top": 6, "groups": {"count": 4, "keep": 3}}}
+    rot = {"base": 10000.0, "dims": hd, "scaling": {"factor": 2.0}}
+    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0, "mask": {"size": 1024}, "rot": rot}
+    latent = {"heads": heads, "dim": hd, "rot_dim": hd // 2, "vdim": hd, "kv_rank": width // 4, "scale": (1.5 * hd) ** -0.5,
+              "rot": {"base": 10000.0, "dims": hd // 2}}
+    mamba = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "norm_groups": 1, "conv": 4}
+    kinds = [{"type": "attention", "mixer": attention, "mlp": dense}, {"type": "mamba2", "mixer": mamba, "mlp": moe},
+             {"type": "latent_attention", "mixer": latent, "mlp": moe}, {"type": "mamba2", "mixer": mamba, "mlp": dense}]
+    return {"architecture": "Bozasun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "token_side": {"dim": width // 16},
+            "layers": [kinds[i % 4] for i in range(n_layer)]}
+
+
+def bozasun_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape."""
+    D, V, n = cfg["width"], cfg["vocab"], cfg["token_side"]["dim"]
+    s = {"embed": (V, D), "side.embed": (V, n * len(cfg["layers"])), "head": (V, D), "final.norm": (D,)}
+    for i, L in enumerate(cfg["layers"]):
+        m, mlp = L["mixer"], L.get("mlp")
+        t = {"norm1": (D,), "side.gate": (n, D), "side.proj": (D, n), "side.norm": (D,)}
+        H, v = m["heads"], m["vdim"]
+        if L["type"] == "attention":
+            G, d = m["kv_heads"], m["dim"]
+            for part, w in (("q", H * d), ("k", G * d), ("v", G * v)):
+                t.update({f"mix.{part}": (w, D), f"mix.{part}.b": (w,)})
+            t.update({"mix.q.norm": (d,), "mix.k.norm": (d,), "mix.o": (D, H * v), "mix.o.b": (D,)})
+        elif L["type"] == "latent_attention":
+            d, r, R = m["dim"], m["rot_dim"], m["kv_rank"]
+            t.update({"mix.q": (H * (d + r), D), "mix.dkv": (R + r, D), "mix.dkv.norm": (R,), "mix.uk": (H * d, R), "mix.uv": (H * v, R),
+                      "mix.g": (H * v, D), "mix.o": (D, H * v)})
+        else:
+            C = H * v + 2 * m["groups"] * m["state"]
+            t.update({"mix.in": (H * v + C + H, D), "mix.conv": (C, m["conv"]), "mix.conv.b": (C,), "mix.dt_bias": (H,), "mix.A_log": (H,),
+                      "mix.D": (H,), "mix.norm": (H * v,), "mix.o": (D, H * v)})
+        parts = [("mlp.", mlp["ff"])] if mlp and mlp["kind"] == "dense" else []
+        if mlp:
+            t["norm2"] = (D,)
+            if mlp["kind"] == "moe":
+                r = mlp["router"]
+                t.update({"mlp.router": (r["experts"] + r["identity"], D), "mlp.correction": (r["experts"] + r["identity"],)})
+                parts = [(f"mlp.e{e}.", mlp["expert"]["ff"]) for e in range(r["experts"])]
+        for p, f in parts:
+            t.update({p + "gate": (f, D), p + "up": (f, D), p + "down": (D, f)})
+        s.update({f"l{i}.{k}": x for k, x in t.items()})
+    return s
+
+
+def random_bozasun(cfg: dict, seed: int = 0, **kw):
+    """A BozasunLM with seeded random weights, tensor by tensor."""
+    from .bozasun import BozasunLM
+    return _random_design(BozasunLM, cfg, bozasun_shapes(cfg), seed, **kw)
+
+
 def random_fuzudra(cfg: dict, seed: int = 0, **kw):
     """A FuzudraLM with seeded random weights, tensor by tensor."""
     from .fuzudra import FuzudraLM
@@ -221,7 +282,7 @@ def random_musutar(cfg: dict, seed: int = 0, **kw):
 # (name's end, standard deviation, mean) of the tensors that are not plain linear weights or norms around zero
 _SPECIAL = (("mix.A_log", 1.0, -1.0), ("mix.dt_bias", 1.0, -2.0), ("mix.dt.b", 1.0, -3.0), ("mix.D", 0.1, 1.0), ("mix.sink", 1.0, 0.0),
             (".conv", 0.4, 0.0), ("canon1", 0.3, 0.0), ("mix.norm", 0.1, 1.0), ("dkv.norm", 0.1, 1.0), ("hc1.in", 0.1, 0.25), ("hc2.in", 0.1, 0.25),
-            ("hc1.out", 0.1, 1.0), ("hc2.out", 0.1, 1.0))
+            ("hc1.out", 0.1, 1.0), ("hc2.out", 0.1, 1.0), ("mlp.correction", 0.005, 0.0))
 
 
 def _random_design(cls, cfg: dict, shapes: dict, seed: int, **kw):
@@ -232,8 +293,8 @@ def _random_design(cls, cfg: dict, shapes: dict, seed: int, **kw):
         for end, s, m in _SPECIAL:
             if name.endswith(end):
                 std, mean = s, m
-        if cfg["architecture"] == "Musutar" and name.split(".")[-1] in ("norm", "norm1", "norm2"):
-            mean = 1.0                                     # layer norms: plain weights
+        if cfg["architecture"] in ("Bozasun", "Musutar") and name.split(".")[-1] in ("norm", "norm1", "norm2"):
+            mean = 1.0                                     # plain weights
         w = mean + std * rng.standard_normal(shape, dtype=np.float32)
         model.load_tensor(name, w + np.eye(shape[0], dtype=np.float32) if name.endswith(".mix") else w)
     model.finalize()
