@@ -18,6 +18,7 @@ struct GemmArgs {
   // segmented (grouped) mode: blockIdx.z selects a segment of rows and its own weight matrix
   const int* seg_off = nullptr;   // [nseg] first row of the segment (device)
   const int* seg_cnt = nullptr;   // [nseg] rows in the segment (device)
+  int seg_rows = 0;               // tcgen05 kernel: segments of this many rows each (a multiple of 32), all with the same weights
   const int* seg_w = nullptr;     // [nseg] which of the n_w weight matrices a segment uses (device), or null: segment z uses matrix z
   int n_w = 0;                    // number of weight matrices when seg_w is given
   const int* a_rows = nullptr;    // optional gather: A row = a_rows[row]

@@ -69,6 +69,7 @@ struct TcArgs {
   int post, post_n;        // 16-bit TC_STORE only: GemmArgs::post
   int epi, c_bf16;
   int act;                 // TC_SWIGLU: activation of the gate (GemmArgs::act)
+  int seg_rows, rows_all;  // segments of equal length (the last one may be shorter) over rows_all rows with one weight matrix, or 0
   const int* seg_off;      // segmented mode (blockIdx.z = segment)
   const int* seg_cnt;
   long long w_rows_per_seg;  // rows of W between consecutive weight matrices
@@ -370,12 +371,57 @@ __device__ __forceinline__ void tc_epilogue_chunk(const TcArgs& g, const unsigne
         }
       }
     } else if (MODE == TC_ADD) {
-      if (n < g.N) {
-        float* dst = reinterpret_cast<float*>(g.C) + (long long)(row0 + m0) * g.ldc + n;
-        const float bias = g.bias ? g.bias[n] : 0.f;
+      // staged like the stores, so that a warp reads and writes 512 contiguous bytes of a row, all its loads ahead of its stores
+      float* dst = reinterpret_cast<float*>(g.C) + (long long)(row0 + m0) * g.ldc + n0;
+      const float bias = g.bias && n < g.N ? g.bias[n] : 0.f;
+      if (vec_ok) {
+        float* tile = reinterpret_cast<float*>(base) + buf * (32 * BF);
+#pragma unroll
+        for (int i = 0; i < 32; ++i) tile[i * BF + f] = __uint_as_float(r[i]) + bias;
+        asm volatile("bar.sync %0, 128;" ::"r"(bar_id) : "memory");
+        const int c4 = lane * 4;
+        if (n0 + c4 < g.N) {
+          float4 x[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j)
+            if (q * 8 + j < mrem) x[j] = *reinterpret_cast<const float4*>(dst + (long long)(q * 8 + j) * g.ldc + c4);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            const int row = q * 8 + j;
+            if (row >= mrem) continue;
+            const float4 v = *reinterpret_cast<const float4*>(tile + row * BF + c4);
+            *reinterpret_cast<float4*>(dst + (long long)row * g.ldc + c4) = make_float4(x[j].x + v.x, x[j].y + v.y, x[j].z + v.z, x[j].w + v.w);
+          }
+        }
+      } else if (n < g.N) {
+        float x[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) x[i] = i < mrem ? dst[(long long)i * g.ldc + f] : 0.f;
 #pragma unroll
         for (int i = 0; i < 32; ++i)
-          if (i < mrem) dst[(long long)i * g.ldc] += __uint_as_float(r[i]) + bias;
+          if (i < mrem) dst[(long long)i * g.ldc + f] = x[i] + __uint_as_float(r[i]) + bias;
+      }
+    } else if (MODE == TC_STORE && g.c_bf16 && vec_ok) {
+      // 16-bit rows, staged as well: 256 contiguous bytes of a row per warp
+      float* tile = reinterpret_cast<float*>(base) + buf * (32 * BF);
+      const float bias = g.bias && n < g.N ? g.bias[n] : 0.f;
+      const int post = n < g.post_n ? g.post : 0;
+#pragma unroll
+      for (int i = 0; i < 32; ++i) tile[i * BF + f] = post_act(__uint_as_float(r[i]) + bias, post, true);
+      asm volatile("bar.sync %0, 128;" ::"r"(bar_id) : "memory");
+      const int c4 = lane * 4;
+      if (n0 + c4 < g.N) {
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(g.C) + (long long)(row0 + m0) * g.ldc + n0 + c4;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const int row = q * 8 + j;
+          if (row >= mrem) break;
+          const float4 v = *reinterpret_cast<const float4*>(tile + row * BF + c4);
+          uint2 u;
+          *reinterpret_cast<__nv_bfloat162*>(&u.x) = __floats2bfloat162_rn(v.x, v.y);
+          *reinterpret_cast<__nv_bfloat162*>(&u.y) = __floats2bfloat162_rn(v.z, v.w);
+          *reinterpret_cast<uint2*>(dst + (long long)row * g.ldc) = u;
+        }
       }
     } else {
       if (n < g.N) {
@@ -424,6 +470,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   // segment sizes are written by the routing kernels that precede this one; a dense block only waits
   // once its first weight tiles are on their way (weights never change)
   if (g.seg_cnt) { pdl_wait(); row0 = g.seg_off[z]; cnt = g.seg_cnt[z]; }
+  if (g.seg_rows) { row0 = z * g.seg_rows; cnt = min(g.seg_rows, g.rows_all - row0); }
   if (cnt > g.ntok) cnt = g.ntok;
   const int cnt16 = (cnt + 15) & ~15;      // UMMA N and token rows loaded by this CTA
   const int n0 = blockIdx.x * BF;
@@ -787,6 +834,7 @@ gemm_tc_persist_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_co
     n0 = (rem - y * tiles_x) * BF;
     row0 = 0; cnt = g.M;
     if (g.seg_cnt) { row0 = g.seg_off[z]; cnt = g.seg_cnt[z]; }
+    if (g.seg_rows) { row0 = z * g.seg_rows; cnt = min(g.seg_rows, g.rows_all - row0); }
     if (cnt > g.ntok) cnt = g.ntok;
     kb0 = y * g.kb_per_split;
     nkb = nkb_total - kb0;
@@ -1009,7 +1057,7 @@ inline int persist_level_env() { const char* e = getenv("VN_TC_PERSIST"); return
 inline bool gemm_tc_supported(const GemmArgs& g) {
   return g.M >= 1 && g.M <= 256 && g.a_rows == nullptr && g.ldw_k == 1 && g.K % 8 == 0 && g.lda % 8 == 0 &&
          g.ldw % 8 == 0 && ((uintptr_t)g.A & 15) == 0 && ((uintptr_t)g.W & 15) == 0 &&
-         (g.seg_cnt != nullptr || g.nseg == 1) && tc_detail::encode_fn() != nullptr;
+         (g.seg_cnt != nullptr || g.seg_rows > 0 || g.nseg == 1) && tc_detail::encode_fn() != nullptr;
 }
 
 // a_rows_total: number of valid rows behind g.A (rows beyond are zero-filled by TMA)
@@ -1019,11 +1067,14 @@ inline int32_t launch_gemm_tc(vn_ctx* ctx, const GemmArgs& g, long long a_rows_t
   const int ntok = (g.M + 15) & ~15;
   CUtensorMap tm_w, tm_x;
   const long long w_rows = g.seg_cnt ? (long long)((g.seg_w ? g.n_w : g.nseg) - 1) * (g.w_stride / g.ldw) + g.N : g.N;
-  if (!make_map(&tm_w, g.W, w_rows, g.K, g.ldw, BF) || !make_map(&tm_x, g.A, a_rows_total, g.K, g.lda, g.seg_cnt ? 16 : ntok))
+  // one box per stage, unless segments differ in length
+  const int x_box = g.seg_cnt || (g.seg_rows && a_rows_total % g.seg_rows) ? 16 : ntok;
+  if (!make_map(&tm_w, g.W, w_rows, g.K, g.ldw, BF) || !make_map(&tm_x, g.A, a_rows_total, g.K, g.lda, x_box))
     return vn_fail(ctx, VN_ERR_CUDA, "cuTensorMapEncodeTiled failed");
   TcArgs a = {};
   a.C = g.C; a.bias = g.bias; a.ldc = g.ldc; a.M = g.M; a.N = g.N; a.K = g.K; a.ntok = ntok;
-  a.x_box = g.seg_cnt ? 16 : ntok;
+  a.x_box = x_box;
+  a.seg_rows = g.seg_rows; a.rows_all = g.seg_rows ? (int)a_rows_total : 0;
   const size_t stage_bytes = (size_t)BF * BK * 2 + (size_t)ntok * BK * 2;
   const int nkb = (g.K + BK - 1) / BK;
   const int splits = std::max(1, std::min(plan.splits, nkb));
@@ -1055,7 +1106,7 @@ inline int32_t launch_gemm_tc(vn_ctx* ctx, const GemmArgs& g, long long a_rows_t
   a.run_if = plan.run_if;
   if (plan.filter) a.cand = *plan.filter;
   if (plan.cluster_mode) {
-    if (gy > 8 || g.seg_cnt) return vn_fail(ctx, VN_ERR_INVALID, "cluster split-K: at most 8 K ranges, dense rows only");
+    if (gy > 8 || g.seg_cnt || g.seg_rows) return vn_fail(ctx, VN_ERR_INVALID, "cluster split-K: at most 8 K ranges, dense rows only");
     a.partial = nullptr;
     budget = std::max(budget, (size_t)((g.M + 31) / 32) * 32 * BF * 4);   // the whole partial tile is staged
     a.smem_budget = (unsigned)budget;
@@ -1073,8 +1124,8 @@ inline int32_t launch_gemm_tc(vn_ctx* ctx, const GemmArgs& g, long long a_rows_t
     const bool part = mode == TC_PARTIAL;
     const float* optr = part ? a.partial : reinterpret_cast<const float*>(g.C);
     const long long old_ = part ? g.N : g.ldc;
-    const long long slice = part ? a.partial_stride : (long long)g.M * old_;
-    const long long rows = part ? plan.rows_total : g.M;
+    const long long rows = part ? plan.rows_total : g.seg_rows ? a_rows_total : g.M;
+    const long long slice = part ? a.partial_stride : rows * old_;
     if (((uintptr_t)optr & 15) == 0 && old_ % 4 == 0 && slice % 4 == 0 &&
         make_out_map(&tm_out, optr, g.N, rows, part ? gy : 1, old_, slice)) {
       const int per_group = (((g.M + 31) / 32) + 1) / 2;               // chunks the busier epilogue group drains

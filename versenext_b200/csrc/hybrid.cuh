@@ -769,14 +769,12 @@ int32_t ensure(vn_model* m, int M) {
   Model& hm = *m->hyb;
   VN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
   m->cap_rows = 0;
-  void** bufs[] = {(void**)&m->x, &m->h, (void**)&m->row_seg, (void**)&hm.x0, &hm.cat, (void**)&hm.ws, &hm.hc, (void**)&hm.gate, (void**)&hm.y};
+  void** bufs[] = {(void**)&m->x, &m->h, (void**)&hm.x0, &hm.cat, (void**)&hm.ws, &hm.hc, (void**)&hm.gate, (void**)&hm.y};
   for (void** b : bufs) { if (*b) cudaFree(*b); *b = nullptr; }
   const size_t R = (size_t)M + (M >> 2) + 32, D = hm.D, e = m->esz;
   TRY(dev_alloc(ctx, (void**)&m->x, R * D * 4 * std::max(1, hm.streams)));
   TRY(dev_alloc(ctx, &m->h, R * D * e));
-  m->row_seg_cap = (int)(R / 256 + 2);
-  TRY(dev_alloc(ctx, (void**)&m->row_seg, (size_t)2 * m->row_seg_cap * sizeof(int)));
-  TRY(dev_alloc(ctx, (void**)&hm.x0, R * D * 4));
+  if (hm.arranged || hm.loop_times) TRY(dev_alloc(ctx, (void**)&hm.x0, R * D * 4));
   if (hm.arranged) {
     TRY(dev_alloc(ctx, &hm.hc, R * D * e));
     TRY(dev_alloc(ctx, (void**)&hm.gate, R * D * 4));
@@ -874,7 +872,7 @@ int32_t close_block(vn_model* m, GemmArgs g, const float* bias, const Next& next
   TRY(linear(m, g));
   if (next.cast) {
     const long long n = (long long)M * D;
-    VN_LAUNCH(ctx, cast_rows_kernel<T>, (unsigned)ceil_div(n, 256ll), 256, 0, m->x, (T*)m->h, n);
+    VN_LAUNCH(ctx, cast_rows_kernel<T>, (unsigned)ceil_div(n, 1024ll), 256, 0, m->x, (T*)m->h, n);
   }
   if (next_norm)
     VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, next_norm, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
@@ -888,17 +886,18 @@ int32_t batched(vn_model* m, const GemmArgs& g) {
 }
 
 // ---- mixers: normalised rows -> the input of the output projection -----------------------------------------------------------
-template <typename T>
+// S: Src, or the 16-bit matrix of a forward of many rows
+template <typename T, typename S>
 int32_t latent_attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
   vn_ctx* ctx = m->ctx;
   const int M = rows.M, D = m->hyb->D, H = L.H;
-  Src s;
+  S s;
   TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_latent_in"), b.proj, &s));
   LatentIn in;
   in.H = H; in.d = L.d; in.dp = L.dp; in.rr = L.rr; in.R = L.R; in.Rp = L.Rp; in.rope = L.rope >= 0 ? m->hyb->ropes[L.rope].table : nullptr;
   in.norm_w = L.f_a; in.eps = m->hyb->eps; in.n_gate = L.n_gate(); in.gate = b.gate; in.gate_t = b.gate_t;
   in.q = b.q; in.qc = b.qc; in.plane = kv->k[run]; in.table = hc.table_dev; in.max_pages = hc.max_pages;
-  VN_LAUNCH(ctx, latent_append_kernel<T>, M, 256, (size_t)L.R * 4, s, in, rows);
+  VN_LAUNCH_NAMED(ctx, "latent_append_kernel", (latent_append_kernel<T, S>), M, 256, (size_t)L.R * 4, s, in, rows);
   GemmArgs g = gemm_args(b.q, H * L.dp, L.w_uk, L.rr ? L.R : L.Rp, L.dp, M, "gemm_latent_uk");
   g.C = b.qc; g.ldc = (long long)H * L.Rp; g.c_bf16 = m->cfg.bf16;
   g.nseg = H; g.a_stride = L.dp; g.w_stride = (long long)L.Rp * L.dp; g.c_stride = L.Rp;
@@ -987,7 +986,7 @@ int32_t mamba2(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLa
   a.state = (float*)kv->v[run]; a.R = hc.ring_len; a.pending = hc.pending; a.u = b.u; a.rows = rows;
   bool step = false;
   if constexpr (std::is_same<S, Src>::value) {
-    step = rows.max_n == 1;
+    step = rows.max_n == 1 && M < SSD_STEP_ROWS;      // few rows: one kernel; many: each row's inputs are convolved only once
     if (step) TRY(vn_ssd_step<T>(ctx, cv, a));
   }
   if (!step) {
@@ -1169,8 +1168,9 @@ int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Nex
   TRY(project(m, gemm_args(m->h, D, L.w_router, n, D, M, "gemm_router"), b.logits, &r.z));
   r.correction = L.correction; r.M = M; r.E = n; r.top = S; r.groups = L.exp_groups; r.keep = L.keep;
   r.slot_expert = b.slot_expert; r.slot_w = b.slot_w; r.count = hm.exp_count;
-  VN_LAUNCH_PDL_LEVEL(ctx, 1, "route_kernel", route_kernel, ceil_div(M, ROUTE_WARPS), 32 * ROUTE_WARPS, (size_t)ROUTE_WARPS * (2 * n + L.exp_groups) * 4, r);
-  AddExperts<T, Src> few;
+  r.rows = route_rows(M);
+  VN_LAUNCH_PDL_LEVEL(ctx, 1, "route_kernel", route_kernel, ceil_div(M, ROUTE_WARPS * r.rows), 32 * ROUTE_WARPS, route_smem(n, L.exp_groups), r);
+  AddExperts<T, Src> few;          // results in split-K slices
   few.h = (const T*)m->h; few.slot_pos = b.slot_pos; few.slot_expert = b.slot_expert; few.slot_w = b.slot_w; few.top = S; few.n_real = L.n_exp; few.D = D;
   few.count = hm.exp_count; few.cursor = hm.exp_cur; few.n_count = n;
   few.y.ld = D;
@@ -1345,7 +1345,7 @@ int32_t forward_arranged(vn_model* m, vn_kv* kv, const int64_t* tokens, const Ro
             VN_LAUNCH(ctx, (conv_tail_kernel<T, Mat<T>, false>), dim3(ceil_div(D, 256), rows.n_ent), 256, 0, cv, rows, hc.pending);
         }
       }
-      if (L.kind == LATENT) TRY(latent_attention<T>(m, in_rows, kv, hc, L, i, rows, b));
+      if (L.kind == LATENT) TRY((latent_attention<T, Src>(m, in_rows, kv, hc, L, i, rows, b)));
       else if (L.kind == MAMBA1) TRY(mamba1<T>(m, in_rows, kv, hc, L, i, rows, b));
       else if (L.kind == DELTA) TRY(channel_delta<T>(m, in_rows, kv, hc, L, i, rows, b));
       else if (L.kind == ATTENTION) TRY((attention<T, S>(m, in_rows, kv, hc, L, i, rows, b)));
@@ -1374,13 +1374,18 @@ int32_t forward_arranged(vn_model* m, vn_kv* kv, const int64_t* tokens, const Ro
   return out_logits ? head(m, pick.n, out_logits) : VN_OK;
 }
 
-// mixers that read a projection of many rows in 16 bits
+// mixers that read the projection of many rows in 16 bits
 template <typename T>
 int32_t dense_projection_mixer(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLayer& L, int run, const Rows& rows, const Buffers& b) {
+  auto run_as = [&](auto tag) -> int32_t {
+    using S = decltype(tag);
+    if (L.kind == LATENT) return latent_attention<T, S>(m, in_rows, kv, hc, L, run, rows, b);
+    if (L.kind == MAMBA2) return mamba2<T, S>(m, in_rows, kv, hc, L, run, rows, b);
+    return attention<T, S>(m, in_rows, kv, hc, L, run, rows, b);
+  };
   if constexpr (std::is_same<T, __nv_bfloat16>::value)
-    if (rows.M > 256)
-      return L.kind == MAMBA2 ? mamba2<T, Mat<T>>(m, in_rows, kv, hc, L, run, rows, b) : attention<T, Mat<T>>(m, in_rows, kv, hc, L, run, rows, b);
-  return L.kind == MAMBA2 ? mamba2<T, Src>(m, in_rows, kv, hc, L, run, rows, b) : attention<T, Src>(m, in_rows, kv, hc, L, run, rows, b);
+    if (rows.M > 256) return run_as(Mat<T>());
+  return run_as(Src());
 }
 
 template <typename T>
@@ -1417,8 +1422,7 @@ int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows,
     }
     const Next next_layer{i + 1 < n_runs && !enters_pass(i + 1) ? hm.layers[hm.runs[i + 1].layer].norm1 : nullptr, false};
     const Next after_ff = hm.side ? Next{nullptr, true} : next_layer, after_mix = L.ff ? Next{L.norm2, false} : after_ff;
-    if (L.kind == LATENT) TRY(latent_attention<T>(m, m->h, kv, hc, L, i, rows, b));
-    else if (L.kind == MAMBA1) TRY(mamba1<T>(m, m->h, kv, hc, L, i, rows, b));
+    if (L.kind == MAMBA1) TRY(mamba1<T>(m, m->h, kv, hc, L, i, rows, b));
     else if (L.kind == DELTA) TRY(channel_delta<T>(m, m->h, kv, hc, L, i, rows, b));
     else TRY((dense_projection_mixer<T>(m, m->h, kv, hc, L, i, rows, b)));
     const int width = L.kind == MAMBA1 ? L.inner : L.H * L.vd;

@@ -47,8 +47,8 @@ struct LatentIn {
 
 // latent of the row: RMS norm with a plain weight, appended to its page with the rotated key; queries to the storage dtype
 // (head pitch dp), their rotated parts to their places behind the carried queries; sigmoid of the gates.  grid M
-template <typename T>
-__global__ void __launch_bounds__(256) latent_append_kernel(Src src, LatentIn a, Rows rows) {
+template <typename T, typename S>
+__global__ void __launch_bounds__(256) latent_append_kernel(S src, LatentIn a, Rows rows) {
   __shared__ float sm[8];
   const int H = a.H, d = a.d, dp = a.dp, rr = a.rr, R = a.R, Rp = a.Rp, max_pages = a.max_pages, qd = d + rr, np = rr / 2;
   extern __shared__ float s_c[];

@@ -176,8 +176,6 @@ struct vn_model {
   int* tc_error = nullptr;       // device word raised by a bounded wait that ran out
   int* sub_seg = nullptr;        // [3][sub_cap] offsets, counts and experts of the experts' 256-row pieces (prompt forwards)
   int sub_cap = 0;
-  int* row_seg = nullptr;        // [2][row_seg_n] offsets and counts of the 256-row segments a prompt's GEMMs use
-  int row_seg_cap = 0;
   unsigned* stack_bar = nullptr; // two device words: arrivals and generation of the fused layer stack's grid barrier
   std::vector<int> pair0;        // per layer: its first K / V plane pair in a cache (a vda layer owns three pairs)
   int n_pairs = 0;
@@ -354,11 +352,8 @@ int32_t ensure_rows(vn_model* m, int M) {
   }
   // segment tables of a prompt's GEMMs (rows in blocks of 256; the experts' pieces), sized for the row capacity so
   // that a forward never allocates them: filled by kernels on the stream
-  if (m->row_seg) cudaFree(m->row_seg);
   if (m->sub_seg) cudaFree(m->sub_seg);
-  m->row_seg = m->sub_seg = nullptr;
-  m->row_seg_cap = (int)(R / 256 + 2);
-  TRY(dev_alloc(ctx, (void**)&m->row_seg, (size_t)2 * m->row_seg_cap * sizeof(int)));
+  m->sub_seg = nullptr;
   m->sub_cap = (int)(c.P * c.E + R * S / 256 + 2);
   TRY(dev_alloc(ctx, (void**)&m->sub_seg, (size_t)3 * m->sub_cap * sizeof(int)));
   if (has_mod) {
@@ -392,24 +387,22 @@ int32_t linear(vn_model* m, GemmArgs g) {
     return launch_gemm_mma_q(ctx, g);
   }
   if (m->cfg.bf16) {
-    // Many rows (a prompt): the tcgen05 kernel takes the rows as segments of 256 -- the same code path as the experts'
-    // row segments, every segment with the same weight matrix (stride 0).  A weight tile is then fetched once per
-    // segment, from L2 after the first.  VN_PREFILL_TC=0 (read per call) keeps the mma.sync kernel.
+    // Many rows (a prompt): the tcgen05 kernel takes the rows as segments of at most 256, every segment with the same
+    // weight matrix.  A weight tile is then fetched once per segment, from L2 after the first.  Shorter segments where
+    // there would be fewer tiles than SMs.  VN_PREFILL_TC=0 (read per call) keeps the mma.sync kernel.
     const char* pe = getenv("VN_PREFILL_TC");
     if (m->use_tc && !(pe && pe[0] == '0') && g.M > 256 && !g.seg_cnt && !g.a_rows && g.nseg == 1 && (!g.bias || g.epi != EPI_SWIGLU) && !g.mul &&
-        g.K % tc_detail::BK == 0 && g.N >= tc_detail::BF && g.ldw_k == 1 && tc_detail::encode_fn() != nullptr &&
+        g.K % tc_detail::BK == 0 && g.N >= 16 && g.ldw_k == 1 && tc_detail::encode_fn() != nullptr &&
         (g.epi == EPI_STORE || g.epi == EPI_ADD || g.epi == EPI_SWIGLU) && (!g.post || g.c_bf16)) {
-      const int nseg = ceil_div(g.M, 256);
-      if (nseg <= m->row_seg_cap) {
-      VN_LAUNCH(ctx, row_segments_kernel, ceil_div(nseg, 128), 128, 0, m->row_seg, m->row_seg + m->row_seg_cap, nseg, g.M);
       TRY(ensure_partial(m, 1024));                               // the error word
+      int rows = 256;
+      while (rows > 32 && ceil_div(g.M, rows) * ceil_div(g.N, tc_detail::BF) < ctx->sm_count) rows >>= 1;
       GemmArgs g2 = g;
-      g2.M = 256; g2.seg_off = m->row_seg; g2.seg_cnt = m->row_seg + m->row_seg_cap; g2.nseg = nseg; g2.w_stride = 0;
-      if (gemm_tc_supported(g2)) {
+      g2.M = rows; g2.seg_rows = rows; g2.nseg = ceil_div(g.M, rows); g2.w_stride = 0;
+      if (g2.nseg <= 65535 && gemm_tc_supported(g2)) {
         TcPlan plan;
         plan.error_flag = m->tc_error;
         return launch_gemm_tc(ctx, g2, g.M, plan);
-      }
       }
     }
     if (gemm_mma_supported(g)) return launch_gemm_mma(ctx, g);
@@ -1346,7 +1339,7 @@ int32_t vn_model_destroy(vn_model* m) {
   }
   F(m->x); F(m->h); F(m->h32); F(m->qkv); F(m->attn); F(m->act); F(m->y); F(m->slot_expert); F(m->slot_w); F(m->part_w);
   F(m->expert_count); F(m->expert_off); F(m->expert_cur); F(m->sorted_row); F(m->slot_pos); F(m->depth_dev);
-  F(m->anc_dev); F(m->rows_dev); F(m->stage); F(m->hs); F(m->partial); F(m->tc_error); F(m->stack_bar); F(m->row_seg); F(m->sub_seg); F(m->head_q); F(m->head_qs);
+  F(m->anc_dev); F(m->rows_dev); F(m->stage); F(m->hs); F(m->partial); F(m->tc_error); F(m->stack_bar); F(m->sub_seg); F(m->head_q); F(m->head_qs);
   for (auto& L : m->layers) for (int i = 0; i < 6; ++i) { F(L.q[i]); F(L.qs[i]); }
   for (auto& L : m->layers)
     for (auto& S : L.sub) { F(S.wqkv); F(S.w_up); F(S.sink); F(S.sink_k); F(S.sink_v); F(S.head_gate); F(S.head_w); F(S.w_abs); F(S.q[0]); F(S.q[1]); F(S.qs[0]); F(S.qs[1]); }
@@ -1803,7 +1796,7 @@ int32_t vn_model_head(vn_model* m, const float* hidden_dev, int32_t rows, int32_
     g.tag = "gemm_head_shard";
     const long long n = (long long)nr * D;
     if (c.bf16) {
-      VN_LAUNCH(ctx, cast_rows_kernel<__nv_bfloat16>, (unsigned)ceil_div(n, 256ll), 256, 0, hidden_dev + (long long)r0 * D,
+      VN_LAUNCH(ctx, cast_rows_kernel<__nv_bfloat16>, (unsigned)ceil_div(n, 1024ll), 256, 0, hidden_dev + (long long)r0 * D,
                 (__nv_bfloat16*)m->h, n);
       g.A = m->h;
       if (m->qmode) {     // the quantised head copy: rows v_lo .. of the bytes (or nibbles) and of the scales

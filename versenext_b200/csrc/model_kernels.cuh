@@ -17,11 +17,15 @@ __global__ void convert_rows_kernel(const float* __restrict__ src, T* __restrict
   dst[(r * row_mul + row_off) * dst_ld + c] = from_f<T>(src[i]);
 }
 
-// fp32 rows -> storage dtype (the GEMM's activation format)
+// fp32 rows -> storage dtype (the GEMM's activation format), four values per thread
 template <typename T>
 __global__ void cast_rows_kernel(const float* __restrict__ src, T* __restrict__ dst, long long n) {
-  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < n) dst[i] = from_f<T>(src[i]);
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i + 3 < n && ((uintptr_t)src & 15) == 0 && ((uintptr_t)dst & (4 * sizeof(T) - 1)) == 0) {
+    store4(dst + i, load4(src + i));
+  } else {
+    for (long long j = i; j < min(i + 4, n); ++j) dst[j] = from_f<T>(src[j]);
+  }
 }
 
 // ---- embedding gather (verse_torch/vnnn.py:453-460) + optional sqrt(dim) scale (base_model.py:201-203)
@@ -466,12 +470,6 @@ __global__ void mod_offsets_kernel(const int* __restrict__ count, int* __restric
     int acc = 0;
     for (int e = 0; e < n_expert; ++e) { offset[e] = acc; acc += count[e]; cursor[e] = 0; }
   }
-}
-
-// rows 0 .. M-1 in blocks of 256: off[i] = 256 i, cnt[i] = rows in block i
-__global__ void row_segments_kernel(int* __restrict__ off, int* __restrict__ cnt, int nseg, int M) {
-  const int i = blockIdx.x * blockDim.x + threadIdx.x;
-  if (i < nseg) { off[i] = 256 * i; cnt[i] = min(256, M - 256 * i); }
 }
 
 // The experts' row segments cut into pieces of at most 256 rows (what one CTA of the tensor-core GEMM takes as its

@@ -346,7 +346,7 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
   }
   const int w_lo = start + min(f0 + 16 * warp, nf - 1) / hg, w_hi = start + min(f0 + 16 * warp + 15, nf - 1) / hg;
   const int k_lo = a.first_key(w_lo), k_hi = a.first_key(w_hi);
-  const float sc = a.scale * 1.4426950408889634f;
+  const float sc = a.softcap > 0.f ? 1.f : a.scale * 1.4426950408889634f;
   fetch(pg0, 0);
   for (int pg = pg0, buf = 0; pg < pg1; ++pg, buf ^= 1) {
     if (pg + 1 < pg1) { fetch(pg + 1, buf ^ 1); cp_async_wait<1>(); } else cp_async_wait<0>();
@@ -380,12 +380,17 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
       }
       const bool whole = pg * KV_PAGE + KV_PAGE - 1 <= w_lo && pg * KV_PAGE >= k_hi;
       float mx[2] = {m_run[0], m_run[1]};
+      if (a.softcap > 0.f)
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) s[j][x] = softcap_log2(s[j][x] * a.scale, a.softcap);
 #pragma unroll
       for (int j = 0; j < 8; ++j)
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
           const int e = x >> 1;
-          float v = a.softcap > 0.f ? softcap_log2(s[j][x] * a.scale, a.softcap) : s[j][x] * sc;
+          float v = s[j][x] * sc;
           if (!whole) {
             const int key = pg * KV_PAGE + 8 * j + (lane & 3) * 2 + (x & 1);
             if (key > rp[e] || key < rk[e]) v = -CUDART_INF_F;

@@ -7,11 +7,13 @@
 #include <math_constants.h>
 
 constexpr int ROUTE_WARPS = 4, MAX_CHOSEN = 32;
+inline int route_rows(int M) { return M >= 2048 ? 8 : 1; }      // rows per warp: a block's counts are added up before they leave it
+inline size_t route_smem(int E, int groups) { return ((size_t)ROUTE_WARPS * (2 * E + groups) + E) * 4; }
 
 struct RouteIn {
   Src z;                               // [M, E] router outputs
   const float* correction = nullptr;   // [E] or null
-  int M = 0, E = 0, top = 1, groups = 1, keep = 1;
+  int M = 0, E = 0, top = 1, groups = 1, keep = 1, rows = 1;      // rows: per warp
   int* slot_expert = nullptr;          // [M, top]
   float* slot_w = nullptr;             // [M, top]
   int* count = nullptr;                // [E], zero before the launch
@@ -27,68 +29,77 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
   }
 }
 
-// one warp per row; shared memory: ROUTE_WARPS x (2 E + groups) floats.  grid ceil(M / ROUTE_WARPS)
+// one warp per `rows` rows.  grid ceil(M / (ROUTE_WARPS rows)), shared memory route_smem
 __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(RouteIn r) {
   pdl_trigger();
   pdl_wait();
   extern __shared__ float s_route[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x * ROUTE_WARPS + warp, E = r.E;
-  if (row >= r.M) return;
-  float* score = s_route + warp * (2 * E + r.groups);
-  float* choice = score + E;
-  float* best = choice + E;
-  float top = -CUDART_INF_F;
-  for (int e = lane; e < E; e += 32) {
-    const float z = r.z.get(row, e);
-    score[e] = z;
-    top = fmaxf(top, z);
-  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, E = r.E;
+  int* s_count = reinterpret_cast<int*>(s_route + ROUTE_WARPS * (2 * E + r.groups));
+  for (int e = threadIdx.x; e < E; e += 32 * ROUTE_WARPS) s_count[e] = 0;
+  __syncthreads();
+  const int first = (blockIdx.x * ROUTE_WARPS + warp) * r.rows;
+#pragma unroll 1
+  for (int row = first; row < min(r.M, first + r.rows); ++row) {
+    float* score = s_route + warp * (2 * E + r.groups);
+    float* choice = score + E;
+    float* best = choice + E;
+    float top = -CUDART_INF_F;
+    for (int e = lane; e < E; e += 32) {
+      const float z = r.z.get(row, e);
+      score[e] = z;
+      top = fmaxf(top, z);
+    }
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) { const float x = expf(score[e] - top); score[e] = x; sum += x; }
-  sum = warp_sum(sum);
-  for (int e = lane; e < E; e += 32) {
-    const float s = score[e] / sum;
-    score[e] = s;
-    choice[e] = r.correction ? s + r.correction[e] : s;
-  }
-  __syncwarp();
-  const int per = E / r.groups;
-  if (r.keep < r.groups) {
-    for (int g = lane; g < r.groups; g += 32) {
-      float m = choice[g * per];
-      for (int i = 1; i < per; ++i) m = fmaxf(m, choice[g * per + i]);
-      best[g] = m;
+    for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) { const float x = expf(score[e] - top); score[e] = x; sum += x; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      const float s = score[e] / sum;
+      score[e] = s;
+      choice[e] = r.correction ? s + r.correction[e] : s;
     }
     __syncwarp();
-    // the groups that are not kept: all but `keep` times the largest
-    for (int k = 0; k < r.keep; ++k) {
-      float v = -CUDART_INF_F;
-      int at = r.groups;
-      for (int g = lane; g < r.groups; g += 32)
-        if (best[g] != CUDART_INF_F && (best[g] > v || at == r.groups)) { v = best[g]; at = g; }
-      warp_argmax(v, at);
-      if (lane == 0 && at < r.groups) best[at] = CUDART_INF_F;          // marks a kept group
+    const int per = E / r.groups;
+    if (r.keep < r.groups) {
+      for (int g = lane; g < r.groups; g += 32) {
+        float m = choice[g * per];
+        for (int i = 1; i < per; ++i) m = fmaxf(m, choice[g * per + i]);
+        best[g] = m;
+      }
+      __syncwarp();
+      // the groups that are not kept: all but `keep` times the largest
+      for (int k = 0; k < r.keep; ++k) {
+        float v = -CUDART_INF_F;
+        int at = r.groups;
+        for (int g = lane; g < r.groups; g += 32)
+          if (best[g] != CUDART_INF_F && (best[g] > v || at == r.groups)) { v = best[g]; at = g; }
+        warp_argmax(v, at);
+        if (lane == 0 && at < r.groups) best[at] = CUDART_INF_F;          // marks a kept group
+        __syncwarp();
+      }
+      for (int e = lane; e < E; e += 32)
+        if (best[e / per] != CUDART_INF_F) choice[e] = -CUDART_INF_F;
       __syncwarp();
     }
-    for (int e = lane; e < E; e += 32)
-      if (best[e / per] != CUDART_INF_F) choice[e] = -CUDART_INF_F;
-    __syncwarp();
-  }
-  for (int k = 0; k < r.top; ++k) {
-    float v = -CUDART_INF_F;
-    int at = E;
-    for (int e = lane; e < E; e += 32)
-      if (choice[e] > v) { v = choice[e]; at = e; }
-    warp_argmax(v, at);
-    if (lane == 0) {
-      at = at < E ? at : 0;                                             // not finite scores: any expert
-      r.slot_expert[(long long)row * r.top + k] = at;
-      r.slot_w[(long long)row * r.top + k] = score[at];
-      atomicAdd(r.count + at, 1);
-      choice[at] = -CUDART_INF_F;
+    for (int k = 0; k < r.top; ++k) {
+      float v = -CUDART_INF_F;
+      int at = E;
+      for (int e = lane; e < E; e += 32)
+        if (choice[e] > v) { v = choice[e]; at = e; }
+      warp_argmax(v, at);
+      if (lane == 0) {
+        at = at < E ? at : 0;                                             // not finite scores: any expert
+        r.slot_expert[(long long)row * r.top + k] = at;
+        r.slot_w[(long long)row * r.top + k] = score[at];
+        atomicAdd(s_count + at, 1);
+        choice[at] = -CUDART_INF_F;
+      }
+      __syncwarp();
     }
-    __syncwarp();
   }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += 32 * ROUTE_WARPS)
+    if (s_count[e]) atomicAdd(r.count + e, s_count[e]);
 }

@@ -3,7 +3,7 @@
 #pragma once
 #include "model_kernels.cuh"
 
-// ---- token embedding + sinusoidal position vector: entry 2i sin, 2i+1 cos of pos * freq[i]; x and a copy x0.
+// ---- token embedding + sinusoidal position vector: entry 2i sin, 2i+1 cos of pos * freq[i]; x and a copy x0 (or null).
 // The angle is reduced to one turn in double before the float sine, so far positions lose nothing.
 template <typename T>
 __global__ void __launch_bounds__(256) embed_pos_kernel(const long long* __restrict__ tokens, const T* __restrict__ emb,
@@ -30,10 +30,12 @@ __global__ void __launch_bounds__(256) embed_pos_kernel(const long long* __restr
     }
     const long long o = (long long)row * D + 2 * i;
     const float v0 = to_f<T>(e[2 * i]) + sn;
-    x[o] = v0; x0[o] = v0;
+    x[o] = v0;
+    if (x0) x0[o] = v0;
     if (2 * i + 1 < D) {
       const float v1 = to_f<T>(e[2 * i + 1]) + cs;
-      x[o + 1] = v1; x0[o + 1] = v1;
+      x[o + 1] = v1;
+      if (x0) x0[o + 1] = v1;
     }
   }
 }

@@ -185,6 +185,77 @@ __global__ void __launch_bounds__(SCAN_TH) ssd_scan_kernel(ConvIn<T, S> in, SsdA
   }
 }
 
+// One row per entry, inputs convolved: bound by the state's bytes, so no barrier and nothing in shared memory; every thread
+// reads its rows of B and C itself.  Columns as above.  grid (H * ceil(P / (32 NP)), n_ent)
+template <typename T, typename S, int DK, int NP>
+__global__ void __launch_bounds__(SCAN_TH) ssd_token_kernel(SsdArgs a, S proj) {
+  constexpr int COLS = SCAN_COLS * NP;
+  const int tid = threadIdx.x, nb = (a.P + COLS - 1) / COLS, h = blockIdx.x / nb, cb = (blockIdx.x % nb) * COLS;
+  const int N = a.N, P = a.P, cl = tid >> 3, li = tid & 7, inner = a.inner(), g = h / (a.H / a.G);
+  int slot, row, n, start;
+  a.rows.entry(blockIdx.y, &slot, &row, &n, &start);
+  if (n <= 0) return;
+  const long long one = (long long)P * N;
+  const float* st_in = a.state + (((long long)slot * a.R + start % a.R) * a.H + h) * one;
+  float* st_out = a.state + (((long long)slot * a.R + (start + 1) % a.R) * a.H + h) * one;
+  float St[NP][DK];
+#pragma unroll
+  for (int p = 0; p < NP; ++p) {
+    const int c = cb + cl + SCAN_COLS * p;
+    delta_col_load<DK>(st_in + (long long)c * N, N, li, start > 0 && c < P, St[p]);
+  }
+  const T* in = reinterpret_cast<const T*>(a.xbc) + (long long)row * a.ld;
+  const float dt = a.dt[(long long)row * a.H + h], D = a.D[h], dec = exp2f(a.A[h] * LOG2E * dt);
+  float x[NP], z = 0.f;
+#pragma unroll
+  for (int p = 0; p < NP; ++p) {
+    const int c = cb + cl + SCAN_COLS * p;
+    x[p] = c < P ? to_f<T>(in[h * P + c]) : 0.f;
+    if (li == p && c < P) z = proj.get(row, h * P + c);
+  }
+  const T *B = in + inner + g * N, *C = B + a.G * N;
+  const bool quads = N % 4 == 0 && (inner & 3) == 0 && (a.ld & 3) == 0;
+  float o[NP];
+#pragma unroll
+  for (int p = 0; p < NP; ++p) o[p] = 0.f;
+#pragma unroll
+  for (int i = 0; i < DK / 4; ++i) {
+    const int r = 32 * i + 4 * li;
+    float b[4] = {0.f, 0.f, 0.f, 0.f}, cc[4] = {0.f, 0.f, 0.f, 0.f};
+    if (quads && r < N) {
+      const float4 b4 = load4(B + r), c4 = load4(C + r);
+      b[0] = b4.x; b[1] = b4.y; b[2] = b4.z; b[3] = b4.w;
+      cc[0] = c4.x; cc[1] = c4.y; cc[2] = c4.z; cc[3] = c4.w;
+    } else {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (r + e < N) { b[e] = to_f<T>(B[r + e]); cc[e] = to_f<T>(C[r + e]); }
+    }
+#pragma unroll
+    for (int p = 0; p < NP; ++p) {
+      const float v = dt * x[p];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float& s = St[p][4 * i + e];
+        s = fmaf(dec, s, b[e] * v);
+        o[p] = fmaf(s, cc[e], o[p]);
+      }
+    }
+  }
+  float mine = 0.f, xm = 0.f;
+#pragma unroll
+  for (int p = 0; p < NP; ++p) {
+    const int c = cb + cl + SCAN_COLS * p;
+    if (c < P) delta_col_store<DK>(st_out + (long long)c * N, N, li, St[p]);
+    o[p] += __shfl_xor_sync(0xffffffffu, o[p], 1);
+    o[p] += __shfl_xor_sync(0xffffffffu, o[p], 2);
+    o[p] += __shfl_xor_sync(0xffffffffu, o[p], 4);
+    if (li == p) { mine = o[p]; xm = x[p]; }
+  }
+  const int c = cb + cl + SCAN_COLS * li;
+  if (li < NP && c < P) reinterpret_cast<T*>(a.u)[(long long)row * inner + h * P + c] = from_f<T>((mine + D * xm) * silu_as<T>(z));
+}
+
 // columns per group: more fetch B and C fewer times, fewer make more CTAs
 int scan_np(const vn_ctx* ctx, int H, int P, int N, int n_ent) {
   if (N > 128) return 1;
@@ -608,7 +679,7 @@ int32_t vn_ssd_inputs(vn_ctx* ctx, const ConvIn<T, S>& conv, const SsdArgs& a) {
     }
   }
   const int gx = ceil_div(conv.C, 32) + ceil_div(a.H, 32);
-  if (M >= 64)
+  if (M >= 64 && a.rows.max_n > 4)
     VN_LAUNCH_NAMED(ctx, "ssd_inputs_kernel", (ssd_inputs_kernel<T, S, 8>), dim3(gx, ceil_div(M, 64)), dim3(32, 8), 0, conv, a);
   else
     VN_LAUNCH_NAMED(ctx, "ssd_inputs_kernel", (ssd_inputs_kernel<T, S, 1>), dim3(gx, ceil_div(M, 8)), dim3(32, 8), 0, conv, a);
@@ -620,6 +691,16 @@ template int32_t vn_ssd_inputs(vn_ctx*, const ConvIn<bf16, Mat<bf16>>&, const Ss
 
 template <typename T, typename S>
 int32_t vn_ssd_scan(vn_ctx* ctx, const S& proj, const SsdArgs& a) {
+  if (a.rows.max_n == 1 && a.N <= 256) {
+    const int np = a.N <= 128 && a.P > SCAN_COLS ? 2 : 1;
+    const dim3 grid(a.H * ceil_div(a.P, SCAN_COLS * np), a.rows.n_ent);
+#define TOKEN(DK, NP) VN_LAUNCH_NAMED(ctx, "ssd_token_kernel", (ssd_token_kernel<T, S, DK, NP>), grid, SCAN_TH, 0, a, proj)
+#define TOKENS(DK) do { if (np == 2) TOKEN(DK, 2); else TOKEN(DK, 1); } while (0)
+    if (a.N <= 32) TOKENS(4); else if (a.N <= 64) TOKENS(8); else if (a.N <= 128) TOKENS(16); else TOKEN(32, 1);
+#undef TOKENS
+#undef TOKEN
+    return VN_OK;
+  }
   ConvIn<T, S> in;
   in.src = proj;
   return launch_scan<T, S, false>(ctx, in, a);

@@ -40,11 +40,12 @@ SsdPlan vn_ssd_plan(const vn_ctx* ctx, bool bf16, int H, int N, int P, const Row
 
 // convolution of x, B and C, step sizes (everything but the one-token kernel needs them)
 template <typename T, typename S> int32_t vn_ssd_inputs(vn_ctx* ctx, const ConvIn<T, S>& conv, const SsdArgs& a);
-// token after token: any dtype, any count; the states behind all tokens are kept when there are fewer than R
+// token after token (all entries of one row: a kernel of its own): any dtype, any count; the states behind all tokens are kept when there are fewer than R
 template <typename T, typename S> int32_t vn_ssd_scan(vn_ctx* ctx, const S& proj, const SsdArgs& a);
 // chunks of 64 tokens on the tensor cores (N <= 128)
 template <typename S> int32_t vn_ssd_chunks(vn_ctx* ctx, const S& proj, const SsdArgs& a);
-// one new row per sequence: convolution, step size, recurrence and gate
+constexpr int SSD_STEP_ROWS = 16;
+// one new row per sequence, few of them: convolution, step size, recurrence and gate
 template <typename T> int32_t vn_ssd_step(vn_ctx* ctx, const ConvIn<T>& conv, const SsdArgs& a);
 // out = u over the root mean square of its part (`parts` equal ones) times w
 template <typename T> int32_t vn_ssd_norm(vn_ctx* ctx, const T* u, const float* w, T* out, int M, int n, int parts, float eps);
