@@ -13,7 +13,8 @@ constexpr int WARPS = 4;
 template <int P> constexpr int stages() { return P > 128 ? 2 : 3; }
 template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2; }
 
-template <int P>
+// HEADS: biases, norms, interleaved pairs, capped scores (an instance of its own: the code is fetched anew at every step)
+template <int P, bool HEADS>
 __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(ConvIn<bf16, Src, false> in, PagedAttnArgs a) {
   using namespace mma_detail;
   constexpr int LD = P + 8, ST = stages<P>(), TH = 32 * WARPS, CH = P / 8, TILE = 16 * LD;
@@ -91,7 +92,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
             acc.x = fmaf(x[j].x, w[-j], acc.x); acc.y = fmaf(x[j].y, w[taps - j], acc.y);
             acc.z = fmaf(x[j].z, w[2 * taps - j], acc.z); acc.w = fmaf(x[j].w, w[3 * taps - j], acc.w);
           }
-        if (in.bias) { const float4 b = load4(in.bias + c); acc.x += b.x; acc.y += b.y; acc.z += b.z; acc.w += b.w; }
+        if (HEADS && in.bias) { const float4 b = load4(in.bias + c); acc.x += b.x; acc.y += b.y; acc.z += b.z; acc.w += b.w; }
         store4(dst, acc);
       }
     } else {
@@ -104,7 +105,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
       }
     }
     __syncthreads();
-    if (a.qn) {                                                       // factors of the heads' norms
+    if (HEADS && a.qn) {                                              // factors of the heads' norms
 #pragma unroll 1
       for (int head = warp; head < nq + (fresh ? 1 : 0); head += WARPS) {
         const float* src = sConv(head < nq ? head : 16);
@@ -123,16 +124,22 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
       const int head = i / half, x = i - head * half;
       const float* src = sConv(head < nq ? head : 16);
       bf16* to = head < nq ? sQ + head * LD : sNew;
-      const int cu = x >= np ? np + x : a.interleaved ? 2 * x : x, cv = x >= np ? cu : a.interleaved ? 2 * x + 1 : np + x;
-      float u = src[cu], v = src[cv];
-      if (a.qn) {
+      const bool pair = x < np, next = HEADS && a.interleaved;
+      const int cu = !pair ? np + x : next ? 2 * x : x, cv = !pair ? cu : next ? 2 * x + 1 : np + x;
+      float fu = 1.f, fv = 1.f;
+      if (HEADS && a.qn) {
         const float* nw = head < nq ? a.qn : a.kn;
-        u *= s_norm[head] * nw[cu];
-        v *= s_norm[head] * nw[cv];
+        fu = s_norm[head] * nw[cu];
+        fv = s_norm[head] * nw[cv];
       }
-      const float2 cs = x < np ? rope[x] : make_float2(1.f, 0.f);
-      to[cu] = __float2bfloat16_rn(u * cs.x - v * cs.y);
-      if (x < np) to[cv] = __float2bfloat16_rn(v * cs.x + u * cs.y);
+      if (pair) {
+        const float2 cs = rope[x];
+        const float u = src[cu] * fu, v = src[cv] * fv;
+        to[cu] = __float2bfloat16_rn(u * cs.x - v * cs.y);
+        to[cv] = __float2bfloat16_rn(v * cs.x + u * cs.y);
+      } else {
+        to[cu] = __float2bfloat16_rn(src[cu] * fu);
+      }
     }
     if (fresh)
       for (int x = tid; x < vd; x += TH) sNew[P + x] = __float2bfloat16_rn(sConv(17)[x]);
@@ -160,7 +167,8 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
   float m_run[2] = {-CUDART_INF_F, -CUDART_INF_F}, l_run[2] = {0.f, 0.f};
-  const float sc = a.scale * 1.4426950408889634f;
+  const bool capped = HEADS && a.softcap > 0.f;
+  const float sc = capped ? 1.f : a.scale * 1.4426950408889634f;
   const bf16* q_at = sQ + (lane & 15) * LD + ((lane >> 4) << 3);
   int st = 0;
   for (int c = c0 + warp; c < c1; c += WARPS) {
@@ -185,14 +193,18 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
       mma_bf16(s[0], af, b0);
       mma_bf16(s[1], af, b1);
     }
+    if (capped)
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) s[j][x] = softcap_log2(s[j][x] * a.scale, a.softcap);
     float mx[2] = {m_run[0], m_run[1]};
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int x = 0; x < 4; ++x) {
         const int key = 16 * c + 8 * j + (lane & 3) * 2 + (x & 1);
-        const float v = a.softcap > 0.f ? softcap_log2(s[j][x] * a.scale, a.softcap) : s[j][x] * sc;
-        s[j][x] = key >= lo && key <= pos ? v : -CUDART_INF_F;
+        s[j][x] = key >= lo && key <= pos ? s[j][x] * sc : -CUDART_INF_F;
         mx[x >> 1] = fmaxf(mx[x >> 1], s[j][x]);
       }
     float f[2];
@@ -343,13 +355,15 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
 int32_t vn_attn_step(vn_ctx* ctx, const ConvIn<bf16, Src, false>& conv, const PagedAttnArgs& a) {
   const dim3 grid(a.splits, a.KH * ceil_div(a.H / a.KH, 16), a.rows.M);
   VN_REQUIRE(ctx, a.splits >= 1 && a.splits <= 32 && (a.splits == 1 || (long long)grid.y * grid.z <= VN_TICKETS), "key ranges of the one-token kernel");
-#define STEP(P) do { \
+  const bool heads = conv.bias || a.qn || a.interleaved || a.softcap > 0.f;
+#define STEP1(P, HEADS) do { \
     static unsigned long long done = 0; \
     if (!((done >> (ctx->device & 63)) & 1ull)) { \
-      VN_CUDA(ctx, cudaFuncSetAttribute(attn_step_kernel<P>, cudaFuncAttributeMaxDynamicSharedMemorySize, step_smem<P>())); \
+      VN_CUDA(ctx, cudaFuncSetAttribute((attn_step_kernel<P, HEADS>), cudaFuncAttributeMaxDynamicSharedMemorySize, step_smem<P>())); \
       done |= 1ull << (ctx->device & 63); \
     } \
-    VN_LAUNCH_NAMED(ctx, "attn_step_kernel", attn_step_kernel<P>, grid, 32 * WARPS, step_smem<P>(), conv, a); } while (0)
+    VN_LAUNCH_NAMED(ctx, "attn_step_kernel", (attn_step_kernel<P, HEADS>), grid, 32 * WARPS, step_smem<P>(), conv, a); } while (0)
+#define STEP(P) do { if (heads) STEP1(P, true); else STEP1(P, false); } while (0)
   switch (a.P) {
     case 32: STEP(32); break;
     case 64: STEP(64); break;
@@ -360,5 +374,6 @@ int32_t vn_attn_step(vn_ctx* ctx, const ConvIn<bf16, Src, false>& conv, const Pa
     default: return vn_fail(ctx, VN_ERR_UNSUPPORTED, "key pitch %d", a.P);
   }
 #undef STEP
+#undef STEP1
   return VN_OK;
 }

@@ -141,10 +141,6 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
         float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
         if (n < g.post_n) v0 = post_act(v0, g.post, g.c_bf16);       // no bias goes with it
         if (n + 1 < g.post_n) v1 = post_act(v1, g.post, g.c_bf16);
-        if (g.mul) {                                                 // nor with this
-          if (n < g.N) v0 *= mul_at(g, crow + n);
-          if (n + 1 < g.N) v1 *= mul_at(g, crow + n + 1);
-        }
         if (g.epi == EPI_SWIGLU) {
           if (n + 1 < g.N) store_out<float>(g.C, crow + (n >> 1), glu_act(v0, g.act) * v1, g.c_bf16);
         } else if (g.epi == EPI_ADD) {
@@ -152,8 +148,16 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
           if (n < g.N) c[0] += v0 + (g.bias ? g.bias[n] : 0.f);
           if (n + 1 < g.N) c[1] += v1 + (g.bias ? g.bias[n + 1] : 0.f);
         } else if (g.c_bf16 && !g.bias && n + 1 < g.N && ((crow + n) & 1) == 0) {
+          if (g.mul) {
+            const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(reinterpret_cast<const __nv_bfloat16*>(g.mul) + crow + n));
+            v0 *= f.x; v1 *= f.y;
+          }
           *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(g.C) + crow + n) = __floats2bfloat162_rn(v0, v1);
         } else {
+          if (g.mul) {
+            if (n < g.N) v0 *= mul_at(g, crow + n);
+            if (n + 1 < g.N) v1 *= mul_at(g, crow + n + 1);
+          }
           if (n < g.N) store_out<float>(g.C, crow + n, v0 + (g.bias ? g.bias[n] : 0.f), g.c_bf16);
           if (n + 1 < g.N) store_out<float>(g.C, crow + n + 1, v1 + (g.bias ? g.bias[n + 1] : 0.f), g.c_bf16);
         }

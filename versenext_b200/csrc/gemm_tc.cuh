@@ -485,7 +485,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
   unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   // a stage holds the weight tile and the token rows this CTA really has, so a short segment gets more
   // stages out of the same shared memory
-  const unsigned w_bytes = BF * BK * 2, x_bytes = (unsigned)cnt16 * BK * 2;
+  const int x_rows = g.x_box < g.ntok ? cnt16 : g.ntok;      // one whole box, or as many boxes as the segment needs
+  const unsigned w_bytes = BF * BK * 2, x_bytes = (unsigned)x_rows * BK * 2;
   const unsigned stage_bytes = w_bytes + x_bytes;
   int S = (int)(g.smem_budget / stage_bytes);
   S = S > 8 ? 8 : S;
@@ -524,8 +525,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         }
         pdl_wait();
         for (int kb = 0; kb < npre; ++kb) {
-          mbar_expect_tx(&bar_full[kb], (unsigned)cnt16 * BK * 2);
-          for (int r16 = 0; r16 < cnt16; r16 += g.x_box)
+          mbar_expect_tx(&bar_full[kb], x_bytes);
+          for (int r16 = 0; r16 < x_rows; r16 += g.x_box)
             tma_load_2d(base + (size_t)kb * stage_bytes + w_bytes + (size_t)r16 * BK * 2, &tm_x, &bar_full[kb],
                         (kb0 + kb) * BK, row0 + r16);
         }
@@ -535,11 +536,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         const int s = kb % S;
         if (!mbar_wait(&bar_empty[s], ((kb / S) & 1) ^ 1)) { s_error = 1; break; }
         unsigned char* st = base + (size_t)s * stage_bytes;
-        mbar_expect_tx(&bar_full[s], w_bytes + (unsigned)cnt16 * BK * 2);
+        mbar_expect_tx(&bar_full[s], stage_bytes);
         const int kx = (kb0 + kb) * BK;
         tma_load_2d(st, &tm_w, &bar_full[s], kx, w_row);
-        // tokens in boxes of 16 rows (two swizzle atoms each): only the rows this segment has
-        for (int r16 = 0; r16 < cnt16; r16 += g.x_box)
+        // tokens in boxes of 16 rows (two swizzle atoms each): only the rows this segment has; or all rows in one box, of
+        // which those beyond the segment (another's, or zeros beyond the matrix) are not used
+        for (int r16 = 0; r16 < x_rows; r16 += g.x_box)
           tma_load_2d(st + w_bytes + (size_t)r16 * BK * 2, &tm_x, &bar_full[s], kx, row0 + r16);
       }
     }
@@ -795,7 +797,7 @@ gemm_tc_persist_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_co
   }
   if (maxcnt > g.ntok) maxcnt = g.ntok;
   if (maxcnt <= 0 || (int)blockIdx.x >= tiles_total) return;     // uniform: nothing allocated yet
-  const int max16 = (maxcnt + 15) & ~15;
+  const int max16 = g.x_box < g.ntok ? (maxcnt + 15) & ~15 : g.ntok;
 
   unsigned char* base = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   unsigned char* stages = base + PERSIST_STAGING;
@@ -856,10 +858,11 @@ gemm_tc_persist_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_co
           const int s = it % S;
           if (!mbar_wait(&bar_empty[s], ((it / S) & 1) ^ 1)) { s_error = 1; ok = false; break; }
           unsigned char* st = stages + (size_t)s * stage_bytes;
-          mbar_expect_tx(&bar_full[s], w_bytes + (unsigned)cnt16 * BK * 2);
+          const int x_rows = g.x_box < g.ntok ? cnt16 : g.ntok;
+          mbar_expect_tx(&bar_full[s], w_bytes + (unsigned)x_rows * BK * 2);
           const int kx = (kb0 + kb) * BK;
           tma_load_2d(st, &tm_w, &bar_full[s], kx, w_row);
-          for (int r16 = 0; r16 < cnt16; r16 += g.x_box)
+          for (int r16 = 0; r16 < x_rows; r16 += g.x_box)
             tma_load_2d(st + w_bytes + (size_t)r16 * BK * 2, &tm_x, &bar_full[s], kx, row0 + r16);
         }
       }
@@ -1067,8 +1070,8 @@ inline int32_t launch_gemm_tc(vn_ctx* ctx, const GemmArgs& g, long long a_rows_t
   const int ntok = (g.M + 15) & ~15;
   CUtensorMap tm_w, tm_x;
   const long long w_rows = g.seg_cnt ? (long long)((g.seg_w ? g.n_w : g.nseg) - 1) * (g.w_stride / g.ldw) + g.N : g.N;
-  // one box per stage, unless segments differ in length
-  const int x_box = g.seg_cnt || (g.seg_rows && a_rows_total % g.seg_rows) ? 16 : ntok;
+  // one box per stage; segments that may be short (a row block of few tokens) take boxes of 16 rows
+  const int x_box = g.seg_cnt && !g.seg_w ? 16 : ntok;
   if (!make_map(&tm_w, g.W, w_rows, g.K, g.ldw, BF) || !make_map(&tm_x, g.A, a_rows_total, g.K, g.lda, x_box))
     return vn_fail(ctx, VN_ERR_CUDA, "cuTensorMapEncodeTiled failed");
   TcArgs a = {};
@@ -1161,7 +1164,7 @@ inline int32_t launch_gemm_tc(vn_ctx* ctx, const GemmArgs& g, long long a_rows_t
   // Unset (-1): only where a tile's K range is at most four blocks and there are more than two tiles per SM (the
   // draft model's LM head: 1,940 tiles of four k blocks), where the per-tile set-up is what the tile loop saves;
   // measured -15 us per round there, +24 us on the target's GEMMs when forced everywhere.
-  const bool persist_auto = persist_level < 0 && a.kb_per_split <= 4 && tiles_total > 2ll * ctx->sm_count;
+  const bool persist_auto = persist_level < 0 && !g.seg_rows && a.kb_per_split <= 4 && tiles_total > 2ll * ctx->sm_count;
   if ((persist_level > 0 || persist_auto || plan.force_persist) && (mode == TC_STORE || mode == TC_SWIGLU || mode == TC_PARTIAL || mode == TC_FILTER) &&
       (persist_level >= 2 || plan.force_persist || tiles_total > 2ll * ctx->sm_count) && tiles_total < (1ll << 30)) {
     const size_t stages_max = (216 * 1024 - PERSIST_STAGING) / stage_bytes;

@@ -897,7 +897,8 @@ int32_t latent_attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc,
   in.H = H; in.d = L.d; in.dp = L.dp; in.rr = L.rr; in.R = L.R; in.Rp = L.Rp; in.rope = L.rope >= 0 ? m->hyb->ropes[L.rope].table : nullptr;
   in.norm_w = L.f_a; in.eps = m->hyb->eps; in.n_gate = L.n_gate(); in.gate = b.gate; in.gate_t = b.gate_t;
   in.q = b.q; in.qc = b.qc; in.plane = kv->k[run]; in.table = hc.table_dev; in.max_pages = hc.max_pages;
-  VN_LAUNCH_NAMED(ctx, "latent_append_kernel", (latent_append_kernel<T, S>), M, 256, (size_t)L.R * 4, s, in, rows);
+  const int parts = M > 256 ? 1 : std::min(16, ceil_div(L.n_in, 512));
+  VN_LAUNCH_NAMED(ctx, "latent_append_kernel", (latent_append_kernel<T, S>), dim3(M, parts), 256, (size_t)L.R * 4, s, in, rows);
   GemmArgs g = gemm_args(b.q, H * L.dp, L.w_uk, L.rr ? L.R : L.Rp, L.dp, M, "gemm_latent_uk");
   g.C = b.qc; g.ldc = (long long)H * L.Rp; g.c_bf16 = m->cfg.bf16;
   g.nseg = H; g.a_stride = L.dp; g.w_stride = (long long)L.Rp * L.dp; g.c_stride = L.Rp;

@@ -46,7 +46,8 @@ struct LatentIn {
 };
 
 // latent of the row: RMS norm with a plain weight, appended to its page with the rotated key; queries to the storage dtype
-// (head pitch dp), their rotated parts to their places behind the carried queries; sigmoid of the gates.  grid M
+// (head pitch dp), their rotated parts to their places behind the carried queries; sigmoid of the gates.  grid (M, parts): the
+// queries and gates are shared out, the first part has the latent
 template <typename T, typename S>
 __global__ void __launch_bounds__(256) latent_append_kernel(S src, LatentIn a, Rows rows) {
   __shared__ float sm[8];
@@ -56,12 +57,7 @@ __global__ void __launch_bounds__(256) latent_append_kernel(S src, LatentIn a, R
   int slot, r0, n, start;
   rows.entry(rows.entry_of(row), &slot, &r0, &n, &start);
   const int pos = start + row - r0;
-  float ss = 0.f;
-  for (int j = threadIdx.x; j < R; j += 256) {
-    const float v = src.get(row, H * qd + j);
-    s_c[j] = v;
-    ss += v * v;
-  }
+  const int t0 = blockIdx.y * 256 + threadIdx.x, stride = gridDim.y * 256;
   const float2* rope = a.rope + (long long)pos * np;
   // pair i of the rr values from column c on, rotated by the row's position
   auto rotated = [&](int c, int i) {
@@ -69,35 +65,43 @@ __global__ void __launch_bounds__(256) latent_append_kernel(S src, LatentIn a, R
     const float2 cs = rope[i];
     return make_float2(u * cs.x - v * cs.y, v * cs.x + u * cs.y);
   };
-  const float r = sqrtf(block_sum256(ss, sm) / (float)R + a.eps);
-  const int pg = pos / KV_PAGE;
-  if (pg < max_pages) {
-    T* dst = reinterpret_cast<T*>(a.plane) + ((long long)a.table[(long long)slot * max_pages + pg] * KV_PAGE + pos % KV_PAGE) * Rp;
-    for (int j = threadIdx.x; j < Rp; j += 256)
-      if (j < R || j >= R + rr) dst[j] = from_f<T>(j < R ? s_c[j] / r * a.norm_w[j] : 0.f);
-    for (int i = threadIdx.x; i < np; i += 256) {
-      const float2 v = rotated(H * qd + R, i);
-      dst[R + 2 * i] = from_f<T>(v.x);
-      dst[R + 2 * i + 1] = from_f<T>(v.y);
+  if (blockIdx.y == 0) {
+    float ss = 0.f;
+    for (int j = threadIdx.x; j < R; j += 256) {
+      const float v = src.get(row, H * qd + j);
+      s_c[j] = v;
+      ss += v * v;
+    }
+    const float r = sqrtf(block_sum256(ss, sm) / (float)R + a.eps);
+    const int pg = pos / KV_PAGE;
+    if (pg < max_pages) {
+      T* dst = reinterpret_cast<T*>(a.plane) + ((long long)a.table[(long long)slot * max_pages + pg] * KV_PAGE + pos % KV_PAGE) * Rp;
+      for (int j = threadIdx.x; j < Rp; j += 256)
+        if (j < R || j >= R + rr) dst[j] = from_f<T>(j < R ? s_c[j] / r * a.norm_w[j] : 0.f);
+      for (int i = threadIdx.x; i < np; i += 256) {
+        const float2 v = rotated(H * qd + R, i);
+        dst[R + 2 * i] = from_f<T>(v.x);
+        dst[R + 2 * i + 1] = from_f<T>(v.y);
+      }
     }
   }
   T* q = reinterpret_cast<T*>(a.q) + (long long)row * H * dp;
-  for (int i = threadIdx.x; i < H * dp; i += 256) {
+  for (int i = t0; i < H * dp; i += stride) {
     const int h = i / dp, j = i % dp;
     q[i] = from_f<T>(j < d ? src.get(row, h * qd + j) : 0.f);
   }
   if (rr) {
     T* qc = reinterpret_cast<T*>(a.qc) + (long long)row * H * Rp;
-    for (int i = threadIdx.x; i < H * np; i += 256) {
+    for (int i = t0; i < H * np; i += stride) {
       const int h = i / np, j = i % np;
       const float2 v = rotated(h * qd + d, j);
       qc[h * Rp + R + 2 * j] = from_f<T>(v.x);
       qc[h * Rp + R + 2 * j + 1] = from_f<T>(v.y);
     }
     const int pad = Rp - R - rr;
-    for (int i = threadIdx.x; i < H * pad; i += 256) qc[(i / pad) * Rp + R + rr + i % pad] = from_f<T>(0.f);
+    for (int i = t0; i < H * pad; i += stride) qc[(i / pad) * Rp + R + rr + i % pad] = from_f<T>(0.f);
   }
-  for (int i = threadIdx.x; i < a.n_gate; i += 256) {
+  for (int i = t0; i < a.n_gate; i += stride) {
     const float v = sigmoid_f(src.get(row, H * qd + R + rr + i));
     if (a.gate) a.gate[(long long)row * a.n_gate + i] = v;
     if (a.gate_t) reinterpret_cast<T*>(a.gate_t)[(long long)row * a.n_gate + i] = from_f<T>(v);

@@ -6,8 +6,8 @@
 #include "rows.cuh"
 #include <math_constants.h>
 
-constexpr int ROUTE_WARPS = 4, MAX_CHOSEN = 32;
-inline int route_rows(int M) { return M >= 2048 ? 8 : 1; }      // rows per warp: a block's counts are added up before they leave it
+constexpr int ROUTE_WARPS = 8, MAX_CHOSEN = 32;
+inline int route_rows(int M) { return M >= 2048 ? 2 : 1; }      // rows per warp: a block's counts are added up before they leave it
 inline size_t route_smem(int E, int groups) { return ((size_t)ROUTE_WARPS * (2 * E + groups) + E) * 4; }
 
 struct RouteIn {
@@ -19,14 +19,11 @@ struct RouteIn {
   int* count = nullptr;                // [E], zero before the launch
 };
 
-// the largest value over a warp's lanes and its index (the lowest one among equals)
-__device__ __forceinline__ void warp_argmax(float& v, int& i) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
-    if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
-  }
+// index of the largest value over a warp's lanes (the lowest one among equals), by way of integers in the same order
+__device__ __forceinline__ int warp_argmax(float v, int i) {
+  const unsigned bits = __float_as_uint(v), key = bits ^ ((bits >> 31) ? 0xffffffffu : 0x80000000u);
+  const unsigned top = __reduce_max_sync(0xffffffffu, key);
+  return (int)__reduce_min_sync(0xffffffffu, key == top ? (unsigned)i : 0xffffffffu);
 }
 
 // one warp per `rows` rows.  grid ceil(M / (ROUTE_WARPS rows)), shared memory route_smem
@@ -75,7 +72,7 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(RouteIn r) {
         int at = r.groups;
         for (int g = lane; g < r.groups; g += 32)
           if (best[g] != CUDART_INF_F && (best[g] > v || at == r.groups)) { v = best[g]; at = g; }
-        warp_argmax(v, at);
+        at = warp_argmax(v, at);
         if (lane == 0 && at < r.groups) best[at] = CUDART_INF_F;          // marks a kept group
         __syncwarp();
       }
@@ -88,7 +85,7 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(RouteIn r) {
       int at = E;
       for (int e = lane; e < E; e += 32)
         if (choice[e] > v) { v = choice[e]; at = e; }
-      warp_argmax(v, at);
+      at = warp_argmax(v, at);
       if (lane == 0) {
         at = at < E ? at : 0;                                             // not finite scores: any expert
         r.slot_expert[(long long)row * r.top + k] = at;

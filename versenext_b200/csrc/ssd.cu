@@ -692,7 +692,8 @@ template int32_t vn_ssd_inputs(vn_ctx*, const ConvIn<bf16, Mat<bf16>>&, const Ss
 template <typename T, typename S>
 int32_t vn_ssd_scan(vn_ctx* ctx, const S& proj, const SsdArgs& a) {
   if (a.rows.max_n == 1 && a.N <= 256) {
-    const int np = a.N <= 128 && a.P > SCAN_COLS ? 2 : 1;
+    static const int np_env = getenv("VN_SSD_NP") ? atoi(getenv("VN_SSD_NP")) : 2;
+    const int np = a.N <= 128 && a.P > SCAN_COLS ? np_env : 1;
     const dim3 grid(a.H * ceil_div(a.P, SCAN_COLS * np), a.rows.n_ent);
 #define TOKEN(DK, NP) VN_LAUNCH_NAMED(ctx, "ssd_token_kernel", (ssd_token_kernel<T, S, DK, NP>), grid, SCAN_TH, 0, a, proj)
 #define TOKENS(DK) do { if (np == 2) TOKEN(DK, 2); else TOKEN(DK, 1); } while (0)
