@@ -202,6 +202,7 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
     A.take(&b.xbc, M * up8(L.conv_ch()) * e);
     A.take(&b.dt, M * L.H * 4);
     A.take(&b.u, M * L.inner * e);
+    A.take(&b.z, M * L.inner * e);
   } else if (L.kind == ATTENTION) {
     A.take(&b.q, M * L.H * L.P * e);
     if (M <= SPLIT_ROWS) {
@@ -989,6 +990,7 @@ int32_t mamba2(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const HLa
   if constexpr (std::is_same<S, Src>::value) {
     step = rows.max_n == 1 && M < SSD_STEP_ROWS;      // few rows: one kernel; many: each row's inputs are convolved only once
     if (step) TRY(vn_ssd_step<T>(ctx, cv, a));
+    else if (rows.max_n == 1) a.z = b.z;
   }
   if (!step) {
     TRY((vn_ssd_inputs<T, S>(ctx, cv, a)));

@@ -13,15 +13,20 @@ constexpr float LOG2E = 1.4426950408889634f;
 constexpr int SCAN_TH = 256, SCAN_COLS = SCAN_TH / 8;
 
 // ---- inputs --------------------------------------------------------------------------------------------------------------
-// grid (ceil(C / 32) + ceil(H / 32), ceil(M / (8 RB))), block (32, 8): a thread takes one channel, or one head's step size,
-// of RB rows
+// grid (ceil(C / 32) + ceil(H / 32) [+ ceil(H P / 32): z], ceil(M / (8 RB))), block (32, 8): a thread takes one channel, one
+// head's step size or one gate of RB rows
 template <typename T, typename S, int RB>
 __global__ void __launch_bounds__(256) ssd_inputs_kernel(ConvIn<T, S> in, SsdArgs a) {
   const int blocks = (in.C + 31) / 32;
   int row = (blockIdx.y * 8 + threadIdx.y) * RB;
   const int last = min(row + RB, a.rows.M);
   if ((int)blockIdx.x >= blocks) {
-    const int h = ((int)blockIdx.x - blocks) * 32 + threadIdx.x;
+    const int h = ((int)blockIdx.x - blocks) * 32 + threadIdx.x, hp = (a.H + 31) / 32 * 32;
+    if (h >= hp) {
+      const int c = h - hp, n = a.inner();
+      for (; c < n && row < last; ++row) reinterpret_cast<T*>(a.z)[(long long)row * n + c] = from_f<T>(in.src.get(row, c));
+      return;
+    }
     if (h >= a.H) return;
     const float bias = a.dt_bias[h];
     for (; row < last; ++row) a.dt[(long long)row * a.H + h] = softplus_f(in.src.get_rare(row, a.col_dt() + h) + bias);
@@ -40,11 +45,12 @@ __global__ void __launch_bounds__(256) ssd_inputs_kernel(ConvIn<T, S> in, SsdArg
     } else {
 #pragma unroll
       for (int r = 0; r < RB; ++r) {
-        float cur;
+        float cur = 0.f;
         v[r] = first + r < end ? in.at(first + r, r0, start, slot, c, &cur) : 0.f;
+        if (RB == 1 && n <= a.pending && in.taps > 1) in.keep(slot, start + first - r0, c, cur);
       }
     }
-    if (n <= a.pending && in.taps > 1)
+    if (RB > 1 && n <= a.pending && in.taps > 1)
       for (int r = first; r < end; ++r) in.keep(slot, start + r - r0, c, in.src.get_rare(r, in.col0 + c));
 #pragma unroll
     for (int r = 0; r < RB; ++r) {
@@ -185,75 +191,74 @@ __global__ void __launch_bounds__(SCAN_TH) ssd_scan_kernel(ConvIn<T, S> in, SsdA
   }
 }
 
-// One row per entry, inputs convolved: bound by the state's bytes, so no barrier and nothing in shared memory; every thread
-// reads its rows of B and C itself.  Columns as above.  grid (H * ceil(P / (32 NP)), n_ent)
-template <typename T, typename S, int DK, int NP>
-__global__ void __launch_bounds__(SCAN_TH) ssd_token_kernel(SsdArgs a, S proj) {
+// One row per entry, inputs convolved: bound by the state's bytes, so no barrier and nothing in shared memory.  A CTA takes
+// `heads` heads in turn, the next one's state on its way while this one's is updated; B and C stay in registers within a group.
+// N, H P and the pitch multiples of 4.  grid (ceil(H / heads) * ceil(P / (32 NP)), n_ent)
+template <typename T, int DK, int NP>
+__global__ void __launch_bounds__(SCAN_TH, 2) ssd_token_kernel(SsdArgs a, Mat<T> z, int heads) {
   constexpr int COLS = SCAN_COLS * NP;
-  const int tid = threadIdx.x, nb = (a.P + COLS - 1) / COLS, h = blockIdx.x / nb, cb = (blockIdx.x % nb) * COLS;
-  const int N = a.N, P = a.P, cl = tid >> 3, li = tid & 7, inner = a.inner(), g = h / (a.H / a.G);
+  const int tid = threadIdx.x, nb = (a.P + COLS - 1) / COLS, h0 = (blockIdx.x / nb) * heads, h1 = min(a.H, h0 + heads);
+  const int N = a.N, P = a.P, li = tid & 7, c0 = (blockIdx.x % nb) * COLS + (tid >> 3), inner = a.inner(), per = a.H / a.G;
   int slot, row, n, start;
   a.rows.entry(blockIdx.y, &slot, &row, &n, &start);
   if (n <= 0) return;
   const long long one = (long long)P * N;
-  const float* st_in = a.state + (((long long)slot * a.R + start % a.R) * a.H + h) * one;
-  float* st_out = a.state + (((long long)slot * a.R + (start + 1) % a.R) * a.H + h) * one;
-  float St[NP][DK];
-#pragma unroll
-  for (int p = 0; p < NP; ++p) {
-    const int c = cb + cl + SCAN_COLS * p;
-    delta_col_load<DK>(st_in + (long long)c * N, N, li, start > 0 && c < P, St[p]);
-  }
+  const float* st_in = a.state + ((long long)slot * a.R + start % a.R) * a.H * one + (long long)c0 * N + 4 * li;
+  float* st_out = a.state + ((long long)slot * a.R + (start + 1) % a.R) * a.H * one + (long long)c0 * N + 4 * li;
   const T* in = reinterpret_cast<const T*>(a.xbc) + (long long)row * a.ld;
-  const float dt = a.dt[(long long)row * a.H + h], D = a.D[h], dec = exp2f(a.A[h] * LOG2E * dt);
-  float x[NP], z = 0.f;
-#pragma unroll
-  for (int p = 0; p < NP; ++p) {
-    const int c = cb + cl + SCAN_COLS * p;
-    x[p] = c < P ? to_f<T>(in[h * P + c]) : 0.f;
-    if (li == p && c < P) z = proj.get(row, h * P + c);
-  }
-  const T *B = in + inner + g * N, *C = B + a.G * N;
-  const bool quads = N % 4 == 0 && (inner & 3) == 0 && (a.ld & 3) == 0;
-  float o[NP];
-#pragma unroll
-  for (int p = 0; p < NP; ++p) o[p] = 0.f;
-#pragma unroll
-  for (int i = 0; i < DK / 4; ++i) {
-    const int r = 32 * i + 4 * li;
-    float b[4] = {0.f, 0.f, 0.f, 0.f}, cc[4] = {0.f, 0.f, 0.f, 0.f};
-    if (quads && r < N) {
-      const float4 b4 = load4(B + r), c4 = load4(C + r);
-      b[0] = b4.x; b[1] = b4.y; b[2] = b4.z; b[3] = b4.w;
-      cc[0] = c4.x; cc[1] = c4.y; cc[2] = c4.z; cc[3] = c4.w;
-    } else {
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (r + e < N) { b[e] = to_f<T>(B[r + e]); cc[e] = to_f<T>(C[r + e]); }
-    }
+  struct Head { float4 st[NP][DK / 4]; float x[NP], z, dt; };
+  auto fetch = [&](int h, Head& f) {
 #pragma unroll
     for (int p = 0; p < NP; ++p) {
-      const float v = dt * x[p];
+      const int c = c0 + SCAN_COLS * p;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        float& s = St[p][4 * i + e];
-        s = fmaf(dec, s, b[e] * v);
-        o[p] = fmaf(s, cc[e], o[p]);
+      for (int i = 0; i < DK / 4; ++i)
+        f.st[p][i] = start > 0 && c < P && 32 * i + 4 * li < N ? load4(st_in + h * one + (long long)SCAN_COLS * p * N + 32 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      f.x[p] = c < P ? to_f<T>(in[h * P + c]) : 0.f;
+    }
+    f.dt = a.dt[(long long)row * a.H + h];
+    const int c = c0 + SCAN_COLS * li;
+    f.z = li < NP && c < P ? z.get(row, h * P + c) : 0.f;
+  };
+  Head cur, next;
+  fetch(h0, cur);
+  float4 B[DK / 4], C[DK / 4];
+  int group = -1;
+#pragma unroll 1
+  for (int h = h0; h < h1; ++h) {
+    if (h + 1 < h1) fetch(h + 1, next);
+    if (h / per != group) {
+      group = h / per;
+      const T* b = in + inner + group * N + 4 * li;
+#pragma unroll
+      for (int i = 0; i < DK / 4; ++i) {
+        const bool ok = 32 * i + 4 * li < N;
+        B[i] = ok ? load4(b + 32 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        C[i] = ok ? load4(b + a.G * N + 32 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
     }
-  }
-  float mine = 0.f, xm = 0.f;
+    const float dec = exp2f(a.A[h] * LOG2E * cur.dt), D = a.D[h];
+    float mine = 0.f, xm = 0.f;
 #pragma unroll
-  for (int p = 0; p < NP; ++p) {
-    const int c = cb + cl + SCAN_COLS * p;
-    if (c < P) delta_col_store<DK>(st_out + (long long)c * N, N, li, St[p]);
-    o[p] += __shfl_xor_sync(0xffffffffu, o[p], 1);
-    o[p] += __shfl_xor_sync(0xffffffffu, o[p], 2);
-    o[p] += __shfl_xor_sync(0xffffffffu, o[p], 4);
-    if (li == p) { mine = o[p]; xm = x[p]; }
+    for (int p = 0; p < NP; ++p) {
+      const float v = cur.dt * cur.x[p];
+      float o = 0.f;
+#pragma unroll
+      for (int i = 0; i < DK / 4; ++i) {
+        float4& s = cur.st[p][i];
+        s = make_float4(fmaf(dec, s.x, B[i].x * v), fmaf(dec, s.y, B[i].y * v), fmaf(dec, s.z, B[i].z * v), fmaf(dec, s.w, B[i].w * v));
+        o = fmaf(s.x, C[i].x, fmaf(s.y, C[i].y, fmaf(s.z, C[i].z, fmaf(s.w, C[i].w, o))));
+        if (c0 + SCAN_COLS * p < P && 32 * i + 4 * li < N) store4(st_out + h * one + (long long)SCAN_COLS * p * N + 32 * i, s);
+      }
+      o += __shfl_xor_sync(0xffffffffu, o, 1);
+      o += __shfl_xor_sync(0xffffffffu, o, 2);
+      o += __shfl_xor_sync(0xffffffffu, o, 4);
+      if (li == p) { mine = o; xm = cur.x[p]; }
+    }
+    const int c = c0 + SCAN_COLS * li;
+    if (li < NP && c < P) reinterpret_cast<T*>(a.u)[(long long)row * inner + h * P + c] = from_f<T>((mine + D * xm) * silu_as<T>(cur.z));
+    cur = next;
   }
-  const int c = cb + cl + SCAN_COLS * li;
-  if (li < NP && c < P) reinterpret_cast<T*>(a.u)[(long long)row * inner + h * P + c] = from_f<T>((mine + D * xm) * silu_as<T>(z));
 }
 
 // columns per group: more fetch B and C fewer times, fewer make more CTAs
@@ -678,7 +683,7 @@ int32_t vn_ssd_inputs(vn_ctx* ctx, const ConvIn<T, S>& conv, const SsdArgs& a) {
       return VN_OK;
     }
   }
-  const int gx = ceil_div(conv.C, 32) + ceil_div(a.H, 32);
+  const int gx = ceil_div(conv.C, 32) + ceil_div(a.H, 32) + (a.z ? ceil_div(a.inner(), 32) : 0);
   if (M >= 64 && a.rows.max_n > 4)
     VN_LAUNCH_NAMED(ctx, "ssd_inputs_kernel", (ssd_inputs_kernel<T, S, 8>), dim3(gx, ceil_div(M, 64)), dim3(32, 8), 0, conv, a);
   else
@@ -691,13 +696,17 @@ template int32_t vn_ssd_inputs(vn_ctx*, const ConvIn<bf16, Mat<bf16>>&, const Ss
 
 template <typename T, typename S>
 int32_t vn_ssd_scan(vn_ctx* ctx, const S& proj, const SsdArgs& a) {
-  if (a.rows.max_n == 1 && a.N <= 256) {
-    static const int np_env = getenv("VN_SSD_NP") ? atoi(getenv("VN_SSD_NP")) : 2;
-    const int np = a.N <= 128 && a.P > SCAN_COLS ? np_env : 1;
-    const dim3 grid(a.H * ceil_div(a.P, SCAN_COLS * np), a.rows.n_ent);
-#define TOKEN(DK, NP) VN_LAUNCH_NAMED(ctx, "ssd_token_kernel", (ssd_token_kernel<T, S, DK, NP>), grid, SCAN_TH, 0, a, proj)
+  if (a.rows.max_n == 1 && (a.z || std::is_same<S, Mat<T>>::value) && a.N <= 128 && a.N % 4 == 0 && a.inner() % 4 == 0 && a.ld % 4 == 0) {
+    const int np = a.P > SCAN_COLS ? 2 : 1, nb = ceil_div(a.P, SCAN_COLS * np);
+    int heads = 8;                                       // as many as leave enough CTAs
+    while (heads > 1 && (long long)ceil_div(a.H, heads) * nb * a.rows.n_ent < 3 * ctx->sm_count) heads /= 2;
+    const dim3 grid(ceil_div(a.H, heads) * nb, a.rows.n_ent);
+    Mat<T> z;
+    z.p = (const T*)a.z; z.ld = a.inner();
+    if constexpr (std::is_same<S, Mat<T>>::value) z = proj;
+#define TOKEN(DK, NP) VN_LAUNCH_NAMED(ctx, "ssd_token_kernel", (ssd_token_kernel<T, DK, NP>), grid, SCAN_TH, 0, a, z, heads)
 #define TOKENS(DK) do { if (np == 2) TOKEN(DK, 2); else TOKEN(DK, 1); } while (0)
-    if (a.N <= 32) TOKENS(4); else if (a.N <= 64) TOKENS(8); else if (a.N <= 128) TOKENS(16); else TOKEN(32, 1);
+    if (a.N <= 32) TOKENS(4); else if (a.N <= 64) TOKENS(8); else TOKENS(16);
 #undef TOKENS
 #undef TOKEN
     return VN_OK;

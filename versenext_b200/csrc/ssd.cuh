@@ -16,6 +16,7 @@ struct SsdArgs {
   void* xbc = nullptr;             // [M, ld] convolved and activated x | B | C, storage dtype
   int ld = 0;
   float* dt = nullptr;             // [M, H] step sizes
+  void* z = nullptr;               // [M, H P] the gates in the storage dtype, or null: read off the projection (see vn_ssd_scan)
   const float* dt_bias = nullptr;  // [H]
   const float* A = nullptr;        // [H] -exp(A_log)
   const float* D = nullptr;        // [H]
@@ -40,7 +41,7 @@ SsdPlan vn_ssd_plan(const vn_ctx* ctx, bool bf16, int H, int N, int P, const Row
 
 // convolution of x, B and C, step sizes (everything but the one-token kernel needs them)
 template <typename T, typename S> int32_t vn_ssd_inputs(vn_ctx* ctx, const ConvIn<T, S>& conv, const SsdArgs& a);
-// token after token (all entries of one row: a kernel of its own): any dtype, any count; the states behind all tokens are kept when there are fewer than R
+// token after token (all entries of one row: a kernel of its own, which reads z when the projection is Src): any dtype, any count; the states behind all tokens are kept when there are fewer than R
 template <typename T, typename S> int32_t vn_ssd_scan(vn_ctx* ctx, const S& proj, const SsdArgs& a);
 // chunks of 64 tokens on the tensor cores (N <= 128)
 template <typename S> int32_t vn_ssd_chunks(vn_ctx* ctx, const S& proj, const SsdArgs& a);
