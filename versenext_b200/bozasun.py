@@ -63,7 +63,7 @@ def composed_config(config: dict, shapes: Dict[str, Tuple[int, ...]]) -> dict:
             out.update(_mlp(entry["mlp"], i))
         layers.append(out)
     return {"vocab_size": int(config["vocab"]), "dim": int(config["width"]), "norm_eps": float(config["norm"]["eps"]),
-            "norm_weight": "plain", "token_side": int(config["token_side"]["dim"]), "layers": layers}
+            "norm_weight": "plain", "token_side": int((config.get("token_side") or {}).get("dim") or 0), "layers": layers}
 
 
 class BozasunLM(DesignLM):

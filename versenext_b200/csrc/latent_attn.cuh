@@ -86,6 +86,31 @@ __global__ void __launch_bounds__(256) latent_append_kernel(S src, LatentIn a, R
     }
   }
   T* q = reinterpret_cast<T*>(a.q) + (long long)row * H * dp;
+  if (d % 4 == 0 && dp == d && rr % 4 == 0 && R % 4 == 0 && a.n_gate % 4 == 0 && src.ld % 4 == 0) {      // four columns at a time
+    for (int i = t0; i < H * d / 4; i += stride) {
+      const int h = 4 * i / d, j = 4 * i % d;
+      store4(q + 4 * i, get4(src, row, h * qd + j));
+    }
+    T* qc = reinterpret_cast<T*>(a.qc) + (long long)row * H * Rp + R;
+    const int tail = Rp - R;
+    if (rr)
+      for (int i = t0; i < H * tail / 4; i += stride) {
+        const int h = 4 * i / tail, j = 4 * i % tail;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < rr) {
+          const float4 u = get4(src, row, h * qd + d + j), cs = load4(reinterpret_cast<const float*>(rope + j / 2));
+          v = make_float4(u.x * cs.x - u.y * cs.y, u.y * cs.x + u.x * cs.y, u.z * cs.z - u.w * cs.w, u.w * cs.z + u.z * cs.w);
+        }
+        store4(qc + h * Rp + j, v);
+      }
+    for (int i = 4 * t0; i < a.n_gate; i += 4 * stride) {
+      float4 v = get4(src, row, H * qd + R + rr + i);
+      v = make_float4(sigmoid_f(v.x), sigmoid_f(v.y), sigmoid_f(v.z), sigmoid_f(v.w));
+      if (a.gate) store4(a.gate + (long long)row * a.n_gate + i, v);
+      if (a.gate_t) store4(reinterpret_cast<T*>(a.gate_t) + (long long)row * a.n_gate + i, v);
+    }
+    return;
+  }
   for (int i = t0; i < H * dp; i += stride) {
     const int h = i / dp, j = i % dp;
     q[i] = from_f<T>(j < d ? src.get(row, h * qd + j) : 0.f);

@@ -678,8 +678,8 @@ int32_t vn_ssd_inputs(vn_ctx* ctx, const ConvIn<T, S>& conv, const SsdArgs& a) {
   const int M = a.rows.M;
   if constexpr (std::is_same<S, Mat<T>>::value) {
     if (conv.taps <= 4 && conv.C % 4 == 0 && conv.col0 % 4 == 0 && conv.src.ld % 4 == 0 && a.ld % 4 == 0) {
-      const int rep = M >= 4096 ? 4 : 1;
-      VN_LAUNCH_NAMED(ctx, "ssd_inputs_kernel", (ssd_inputs4_kernel<T, 8>), dim3(ceil_div(conv.C / 4 + a.H, 256), ceil_div(M, 8 * rep)), 256, 0, conv, a, rep);
+      const int rep = M >= 4096 ? 8 : 2;
+      VN_LAUNCH_NAMED(ctx, "ssd_inputs_kernel", (ssd_inputs4_kernel<T, 4>), dim3(ceil_div(conv.C / 4 + a.H, 256), ceil_div(M, 4 * rep)), 256, 0, conv, a, rep);
       return VN_OK;
     }
   }
