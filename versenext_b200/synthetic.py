@@ -208,7 +208,7 @@ def musutar_shapes(cfg: dict) -> dict:
 
 def bozasun_config(width: int, vocab: int = 32000, n_layer: int = 4) -> dict:
     """config.json contents: chunked attention with a dense feed-forward, Mamba-2 and latent attention with mixtures, Mamba-2
-    with a dense feed-forward in turn; heads of 128 (64 below width 2048), four query heads per key head, chunks of 1024, a
+    with a dense feed-forward in turn; heads of 128 (64 below width 2048), four query heads per key head, chunks of 2048, a
     state of 128 per channel, feed-forwards as wide as VerseNexLM's, mixtures of experts a quarter as wide of which a token
     uses about as many."""
     hd = 128 if width >= 2048 else 64
@@ -217,7 +217,7 @@ def bozasun_config(width: int, vocab: int = 32000, n_layer: int = 4) -> dict:
     moe = {"kind": "moe", "expert": {"ff": (ff // 4 + 63) // 64 * 64},
            "router": {"experts": 24, "identity": 8, "top": 6, "groups": {"count": 4, "keep": 3}}}
     rot = {"base": 10000.0, "dims": hd, "scaling": {"factor": 2.0}}
-    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0, "mask": {"size": 1024}, "rot": rot}
+    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0, "mask": {"size": 2048}, "rot": rot}
     latent = {"heads": heads, "dim": hd, "rot_dim": hd // 2, "vdim": hd, "kv_rank": width // 4, "scale": (1.5 * hd) ** -0.5,
               "rot": {"base": 10000.0, "dims": hd // 2}}
     mamba = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "norm_groups": 1, "conv": 4}
