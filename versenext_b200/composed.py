@@ -4,20 +4,23 @@
 optional feed-forward; an optional looped block; the norm and its eps; the kind of positions; the arrangement of the
 residual) and offers what every model of the package offers: weight loading, caches, uniform and ragged steps, generation,
 speculative decoding as target or draft.  A named design is a subclass of `DesignLM` that translates its own config.json
-(see bozasun.py, fuzudra.py, musutar.py).
+(see bozasun.py, fuzudra.py, givozen.py, musutar.py).
 
 Mixers: "latent_attention" (heads, dim, vdim, kv_rank, scale, window, rot_dim with rope, sink, output_gate "head", "element" or
-"none"), "attention" (heads, kv_heads, dim, vdim, scale, window, chunk, softcap, conv, rope, bias, qk_norm, output_gate, kv_from),
+"none"), "attention" (heads, kv_heads, dim, vdim, scale, window, chunk, softcap, conv, rope, bias, out_bias, qk_norm,
+temperature, output_gate "head", "element" or "none", kv_from),
 "mamba1" (inner, state, dt_rank, conv), "mamba2" (heads, vdim, state, groups, norm_groups, conv), "channel_delta" (heads,
 kv_heads, dim, vdim, conv, decay_rank, gate_rank), "lightning" (heads, dim, vdim, decay).  rope: {dims, base, interleaved,
-scaling: YaRN {factor, original, fast, slow} or {kind: "linear", factor}}.
+scaling: YaRN {factor, original, fast, slow}, {kind: "linear", factor} or {kind: "wavelength", factor, low, high, original}}.
 
-Feed-forwards: mlp_hidden with mlp_act "silu" or "gelu_tanh" (gated) or "relu2" (plain); with experts {count, identity, top,
-groups, keep, correction} a mixture of gated ones.
+Feed-forwards: mlp_hidden with mlp_act "silu", "gelu_tanh" or "clamped" (gated; the last one with mlp_limit) or "relu2" or
+"poly_norm" (plain); with experts {count, identity, top, groups, keep, correction, score "softmax" or "sigmoid", weight of the
+"result" or the "input", shared {hidden, limit}} a mixture of gated ones.
 
 Model-wide: norm "rms" (weights stored around zero, or plain: norm_weight "plain") or "layer" (plain weights); streams (residual
 streams, hyper-connections); input_conv (taps of the convolution that a mixer's input gets); residual_gate (sigmoid gate on every
-sublayer's result); token_side (width of the input that every layer has for each token).
+sublayer's result); post_norm (an RMS norm of every sublayer's result); token_side (width of the input that every layer has for
+each token); tie_weights; loop {start, stop, times, entry "project" or "add"}.
 """
 
 from __future__ import annotations

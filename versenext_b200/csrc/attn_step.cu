@@ -13,7 +13,7 @@ constexpr int WARPS = 4;
 template <int P> constexpr int stages() { return P > 128 ? 2 : 3; }
 template <int P> constexpr int step_smem() { return WARPS * stages<P>() * 2 * 16 * (P + 8) * 2 + 16 * (P + 8) * 2 + 2 * P * 2; }
 
-// HEADS: biases, norms, interleaved pairs, capped scores (an instance of its own: the code is fetched anew at every step)
+// HEADS: biases, norms, interleaved pairs, factors of and caps on the scores, gates per head (an instance of its own: the code is fetched anew at every step)
 template <int P, bool HEADS>
 __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(ConvIn<bf16, Src, false> in, PagedAttnArgs a) {
   using namespace mma_detail;
@@ -25,7 +25,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
   // convolved channels: query heads 0 .. 15, key (16), value (17); they lie in ring stages that no prefetch has reached yet
   auto sConv = [&](int r) { return reinterpret_cast<float*>(ring + ((r < 16 ? 0 : ST * 2) + (ST - 1) * 2) * TILE) + (r < 16 ? r : r - 16) * P; };
   __shared__ int s_last;
-  __shared__ float s_ml[WARPS][16][2], s_f[WARPS][16], s_norm[17];
+  __shared__ float s_ml[WARPS][16][2], s_f[WARPS][16], s_norm[17], s_gate[16];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = blockIdx.z;
   const int hg = a.H / a.KH, tiles = (hg + 15) / 16, g = blockIdx.y / tiles, q0 = (blockIdx.y % tiles) * 16, nq = min(16, hg - q0);
   int slot, r0, n, pos;
@@ -119,6 +119,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
     // rotation of the queries and the key
     const int np = a.rd / 2, half = np + d - a.rd;
     const float2* rope = a.rope + (long long)pos * np;
+    if (HEADS && a.gate_head && tid < nq) s_gate[tid] = in.src.get_rare(row, a.col_g + g * hg + q0 + tid);
 #pragma unroll 1
     for (int i = tid; i < (nq + (fresh ? 1 : 0)) * half; i += TH) {
       const int head = i / half, x = i - head * half;
@@ -131,6 +132,11 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
         const float* nw = head < nq ? a.qn : a.kn;
         fu = s_norm[head] * nw[cu];
         fv = s_norm[head] * nw[cv];
+      }
+      if (HEADS && a.temp && head < nq) {
+        const float t = a.temp[g * hg + q0 + head];
+        fu *= t;
+        fv *= t;
       }
       if (pair) {
         const float2 cs = rope[x];
@@ -270,10 +276,11 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
   }
   __syncthreads();
   // four columns of a head: divided by the sum, gated, stored
-  const bool vec = a.vd % 4 == 0 && a.col_g % 4 == 0 && in.src.ld % 4 == 0;
+  const bool vec = a.vd % 4 == 0 && (a.gate_head || (a.col_g % 4 == 0 && in.src.ld % 4 == 0));
   auto gates = [&](int r, int c) {
     const int col = a.col_g + (g * hg + q0 + r) * a.vd + c;
     if (a.col_g < 0 || c >= a.vd) return make_float4(0.f, 0.f, 0.f, 0.f);
+    if (HEADS && a.gate_head) return make_float4(s_gate[r], s_gate[r], s_gate[r], s_gate[r]);
     if (vec) return get4(in.src, row, col);
     const int last = a.vd - 1 - c;
     return make_float4(in.src.get_rare(row, col), in.src.get_rare(row, col + min(1, last)), in.src.get_rare(row, col + min(2, last)),
@@ -355,7 +362,7 @@ __global__ void __launch_bounds__(32 * WARPS, P > 128 ? 1 : 2) attn_step_kernel(
 int32_t vn_attn_step(vn_ctx* ctx, const ConvIn<bf16, Src, false>& conv, const PagedAttnArgs& a) {
   const dim3 grid(a.splits, a.KH * ceil_div(a.H / a.KH, 16), a.rows.M);
   VN_REQUIRE(ctx, a.splits >= 1 && a.splits <= 32 && (a.splits == 1 || (long long)grid.y * grid.z <= VN_TICKETS), "key ranges of the one-token kernel");
-  const bool heads = conv.bias || a.qn || a.interleaved || a.softcap > 0.f;
+  const bool heads = conv.bias || a.qn || a.interleaved || a.temp || a.gate_head || a.softcap > 0.f;
 #define STEP1(P, HEADS) do { \
     static unsigned long long done = 0; \
     if (!((done >> (ctx->device & 63)) & 1ull)) { \

@@ -5,8 +5,10 @@
 enum GemmEpilogue {
   EPI_STORE = 0,    // C = acc (+ bias)
   EPI_ADD = 1,      // C += acc              (residual stream, fp32)
-  EPI_SWIGLU = 2    // out[m, n/2] = act(acc[m, n]) * acc[m, n+1], n even (gate / up rows interleaved in W), act: GemmArgs::act
+  EPI_SWIGLU = 2    // out[m, n/2] = glu(acc[m, n], acc[m, n+1]), n even (gate / up rows interleaved in W), see GemmArgs::act
 };
+
+enum GluAct { GLU_SILU = 0, GLU_GELU = 1, GLU_CLAMP = 2 };
 
 struct GemmArgs {
   const void* A = nullptr;    // [rows, K]
@@ -28,7 +30,8 @@ struct GemmArgs {
   int nseg = 1;
   int epi = EPI_STORE;
   int c_bf16 = 0;
-  int act = 0;                    // gate activation of EPI_SWIGLU: 0 silu, 1 gelu (tanh form)
+  int act = GLU_SILU;             // function of EPI_SWIGLU's pairs
+  float act_limit = 0.f;          // of GLU_CLAMP
   int post = 0;                   // EPI_STORE: function of columns [0, post_n): 0 none, POST_SILU, POST_RELU2
   int post_n = 0;
   const void* mul = nullptr;      // EPI_STORE, plain and batched modes: factors of the results, laid out and typed as C
@@ -57,7 +60,16 @@ __device__ __forceinline__ float silu_ref(float x) { return x * (0.5f * (1.0f + 
 __device__ __forceinline__ float gelu_tanh(float x) {
   return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
 }
-__device__ __forceinline__ float glu_act(float x, int act) { return act ? gelu_tanh(x) : silu_ref(x); }
+// a gated feed-forward's function of gate g and up u (GluAct).  GLU_CLAMP: g capped from above, u from both sides, g sigmoid(1.702 g) (u + 1);
+// `fast`: the result is kept in 16 bits
+__device__ __forceinline__ float glu(float g, float u, int act, float limit, bool fast) {
+  if (act == GLU_CLAMP) {
+    g = fminf(g, limit);
+    const float b = fminf(fmaxf(u, -limit), limit) + 1.f;
+    return (fast ? __fdividef(g, 1.0f + __expf(-1.702f * g)) : g / (1.0f + expf(-1.702f * g))) * b;
+  }
+  return (act == GLU_GELU ? gelu_tanh(g) : silu_ref(g)) * u;
+}
 
 __device__ __forceinline__ float mul_at(const GemmArgs& g, long long idx) {
   return g.c_bf16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(g.mul)[idx]) : reinterpret_cast<const float*>(g.mul)[idx];
@@ -129,7 +141,7 @@ __global__ void __launch_bounds__(256) gemm_nt_simt_kernel(GemmArgs g) {
       for (int j = 0; j < 4; j += 2) {
         const int n = n0 + tx * 4 + j;
         if (n + 1 < g.N) {
-          const float v = glu_act(acc[i][j], g.act) * acc[i][j + 1];
+          const float v = glu(acc[i][j], acc[i][j + 1], g.act, g.act_limit, g.c_bf16);
           store_out<float>(g.C, c_base + crow * g.ldc + (n >> 1), v, g.c_bf16);
         }
       }

@@ -142,7 +142,7 @@ __global__ void __launch_bounds__(BM * 2) gemm_mma_kernel(GemmArgs g) {
         if (n < g.post_n) v0 = post_act(v0, g.post, g.c_bf16);       // no bias goes with it
         if (n + 1 < g.post_n) v1 = post_act(v1, g.post, g.c_bf16);
         if (g.epi == EPI_SWIGLU) {
-          if (n + 1 < g.N) store_out<float>(g.C, crow + (n >> 1), glu_act(v0, g.act) * v1, g.c_bf16);
+          if (n + 1 < g.N) store_out<float>(g.C, crow + (n >> 1), glu(v0, v1, g.act, g.act_limit, g.c_bf16), g.c_bf16);
         } else if (g.epi == EPI_ADD) {
           float* c = reinterpret_cast<float*>(g.C) + crow + n;
           if (n < g.N) c[0] += v0 + (g.bias ? g.bias[n] : 0.f);

@@ -68,7 +68,8 @@ struct TcArgs {
   int kb_per_split;        // k blocks (of 64) per blockIdx.y
   int post, post_n;        // 16-bit TC_STORE only: GemmArgs::post
   int epi, c_bf16;
-  int act;                 // TC_SWIGLU: activation of the gate (GemmArgs::act)
+  int act;                 // TC_SWIGLU: GemmArgs::act, act_limit
+  float act_limit;
   int seg_rows, rows_all;  // segments of equal length (the last one may be shorter) over rows_all rows with one weight matrix, or 0
   const int* seg_off;      // segmented mode (blockIdx.z = segment)
   const int* seg_cnt;
@@ -351,7 +352,7 @@ __device__ __forceinline__ void tc_epilogue_chunk(const TcArgs& g, const unsigne
             const int row = q * 8 + j;
             if (row < mrem) {
               const float4 v = *reinterpret_cast<const float4*>(tile + row * BF + c4);
-              const float o0 = glu_act(v.x, g.act) * v.y, o1 = glu_act(v.z, g.act) * v.w;
+              const float o0 = glu(v.x, v.y, g.act, g.act_limit, g.c_bf16), o1 = glu(v.z, v.w, g.act, g.act_limit, g.c_bf16);
               const long long at = (long long)(row0 + m0 + row) * g.ldc + ((n0 + c4) >> 1);
               if (g.c_bf16)
                 *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(g.C) + at) =
@@ -367,7 +368,7 @@ __device__ __forceinline__ void tc_epilogue_chunk(const TcArgs& g, const unsigne
           const float v = __uint_as_float(r[i]);
           const float other = __shfl_xor_sync(0xffffffffu, v, 1);
           if (i < mrem && !(lane & 1) && n + 1 < g.N)
-            store_out<float>(g.C, (long long)(row0 + m0 + i) * g.ldc + (n >> 1), glu_act(v, g.act) * other, g.c_bf16);
+            store_out<float>(g.C, (long long)(row0 + m0 + i) * g.ldc + (n >> 1), glu(v, other, g.act, g.act_limit, g.c_bf16), g.c_bf16);
         }
       }
     } else if (MODE == TC_ADD) {
@@ -1094,7 +1095,7 @@ inline int32_t launch_gemm_tc(vn_ctx* ctx, const GemmArgs& g, long long a_rows_t
   budget = std::max(budget, 2 * stage_bytes);
   budget = std::max<size_t>(budget, 64 * 1024);       // the epilogue stages four 16 KB tiles in the freed stage memory
   a.smem_budget = (unsigned)budget;
-  a.epi = g.epi; a.c_bf16 = g.c_bf16; a.act = g.act; a.post = g.post; a.post_n = g.post_n;
+  a.epi = g.epi; a.c_bf16 = g.c_bf16; a.act = g.act; a.act_limit = g.act_limit; a.post = g.post; a.post_n = g.post_n;
   a.seg_off = g.seg_off; a.seg_cnt = g.seg_cnt;
   a.w_rows_per_seg = g.seg_cnt ? g.w_stride / g.ldw : 0;
   a.seg_w = g.seg_w;

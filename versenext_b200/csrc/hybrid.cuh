@@ -25,7 +25,7 @@
 namespace hybrid {
 
 enum Kind { LATENT = 0, MAMBA1 = 1, DELTA = 2, ATTENTION = 3, LIGHTNING = 4, MAMBA2 = 5 };
-enum Gate { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };
+enum Gate { GATE_NONE = 0, GATE_HEAD = 1, GATE_ELEMENT = 2 };       // output gates of attention layers
 
 struct HLayer {
   int kind = 0;
@@ -34,19 +34,25 @@ struct HLayer {
   float scale = 1.f;
   // attention: H, KH, d, vd, taps, window, scale and the line below (conv_named: the convolutions are in the checkpoint).
   // lightning: H, d, vd, decay
-  int kv_from = -1, gated = 0, P = 0, rd = 0, rope = -1, conv_named = 0;
-  int chunk = 0, qk_norm = 0, bias = 0, interleaved = 0;
+  int kv_from = -1, gated = GATE_NONE, P = 0, rd = 0, rope = -1, conv_named = 0;
+  int chunk = 0, qk_norm = 0, bias = 0, out_bias = 0, temps = 0, interleaved = 0;
   float softcap = 0.f;
   // latent, besides: rotated dimensions rr, what the output gate multiplies, sink.  mamba2: H, vd, nstate, taps, groups, norm_groups
   int rr = 0, gate = GATE_HEAD, sinks = 1, groups = 1, norm_groups = 1;
   std::vector<double> decay;
-  int ff = 0, act = 0;             // feed-forward width (0: none), activation of its gate: 0 silu, 1 gelu
+  int ff = 0, act = GLU_SILU;      // feed-forward width (0: none), function of its gate and up
+  float limit = 0.f;               // of GLU_CLAMP
   // mixture: n_exp experts of width ff and n_id identity experts (0: a dense feed-forward), of which a row uses `top`, out of
   // the `keep` best of exp_groups groups
   int n_exp = 0, n_id = 0, top = 0, exp_groups = 1, keep = 1, corrected = 0;
+  int sigmoid = 0, weigh_input = 0;    // scores by sigmoid; a weight multiplies the expert's input instead of its result
+  int sff = 0, sffp = 0;           // width of the gated expert that serves every row (0: none)
+  float s_limit = 0.f;
   int ff_plain = 0;                // no gate: squared relu
+  int poly = 0;                    // no gate: PolyNorm
   int dp = 0, Rp = 0, dtp = 0, rap = 0, rgp = 0, n_in = 0, n_x = 0, ffp = 0;    // padded sizes
   float* norm1 = nullptr; float* norm2 = nullptr;                               // 1 + stored weight
+  float* post[2] = {nullptr, nullptr};                                          // norms of the sublayers' results
   void* w_in = nullptr;            // first projection, all its parts stacked [n_in, D]
   void* w_o = nullptr;
   void* w_uk = nullptr;            // latent: per head W_uk^T [H][Rp][dp];  delta: a2 [H d, rap];  mamba: dt [inner, dtp]
@@ -63,9 +69,15 @@ struct HLayer {
   void* w_gu = nullptr; void* w_down = nullptr;                                 // of a mixture: per expert
   float* f_d = nullptr;                   // mamba2: -exp(A_log) [H]
   float* o_b = nullptr;                   // bias of the output projection
-  void* w_router = nullptr; float* correction = nullptr;                        // [n_exp + n_id, D], [n_exp + n_id]
+  float* temp = nullptr;                  // attention: factors of the heads' scores [H]
+  float* coef = nullptr;                  // PolyNorm's four numbers
+  void *w_sgu = nullptr, *w_sdown = nullptr;                                    // of the expert that serves every row
+  void* w_router = nullptr; float* correction = nullptr;                        // [n_router, D], [n_out]
   void *w_sgate = nullptr, *w_sproj = nullptr; float* s_norm = nullptr;         // the token's own input
   int n_out() const { return n_exp + n_id; }
+  int n_router() const { return sff ? (n_out() + 4) & ~3 : n_out(); }          // the shared expert's gate is row n_out
+  int single_up() const { return ff_plain || poly; }                            // one matrix in front of the activation
+  int attn_gates() const { return gated == GATE_HEAD ? H : gated ? H * vd : 0; }
   int n_gate() const { return gate == GATE_HEAD ? H : gate == GATE_ELEMENT ? H * vd : 0; }      // latent
   int conv_ch() const {
     if (kind == MAMBA1) return inner;
@@ -90,6 +102,9 @@ struct Model {
   float eps = 1e-6f;
   std::vector<HLayer> layers;
   int loop_start = 0, loop_stop = 0, loop_times = 0;
+  bool loop_add = false;           // a pass begins with x + x0 (but the first) + step vector, else with W [x | x0] + step vector
+  bool post_norm = false;          // norms of the sublayers' results
+  bool tied = false;               // the head is the embedding table
   std::vector<Run> runs;
   void* w_loop = nullptr;          // [D, 2 D]
   float* loop_step = nullptr;      // [times, D]
@@ -156,7 +171,8 @@ struct Buffers {
   void* gate_t = nullptr;                        // latent: output gates in the storage dtype
   void *xbc = nullptr, *u = nullptr;             // mamba2
   // mixture of experts
-  float *logits = nullptr, *slot_w = nullptr;
+  float *logits = nullptr, *slot_w = nullptr, *sorted_w = nullptr, *sgate = nullptr, *sy = nullptr;
+  void* sact = nullptr;
   int *slot_expert = nullptr, *slot_pos = nullptr, *sorted_row = nullptr, *sub_seg = nullptr;
   void *hs = nullptr, *ey = nullptr;
   int sub_cap = 0;
@@ -166,16 +182,22 @@ constexpr int SPLIT_ROWS = 64, MAX_SPLITS = 16;   // key splits of the latent at
 
 inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& A, Buffers& b) {
   A.off = 0;
-  A.take(&b.proj, M * std::max(std::max(L.n_in, hm.D), L.ff_plain ? L.ffp + hm.D : 0) * 4);
+  A.take(&b.proj, M * std::max(std::max(L.n_in, hm.D), L.single_up() ? L.ffp + hm.D : 0) * 4);
   A.take(&b.mix, M * (size_t)(L.kind == MAMBA1 ? L.inner : L.H * L.vd) * e);
   if (L.ff) A.take(&b.act, M * std::max(1, L.top) * L.ffp * e);
   if (L.n_exp) {
     const size_t slots = M * L.top;
-    A.take(&b.logits, M * L.n_out() * 4);
+    A.take(&b.logits, M * L.n_router() * 4);
     A.take(&b.slot_w, slots * 4);
     A.take(&b.slot_expert, slots * 4);
     A.take(&b.slot_pos, slots * 4);
     A.take(&b.sorted_row, slots * 4);
+    A.take(&b.sorted_w, slots * 4);
+    if (L.sff) {
+      A.take(&b.sgate, M * 4);
+      A.take(&b.sact, M * L.sffp * e);
+      A.take(&b.sy, M * hm.D * 4);
+    }
     A.take(&b.hs, slots * hm.D * e);
     A.take(&b.ey, slots * hm.D * e);
     b.sub_cap = (int)(L.n_exp + slots / 256 + 1);
@@ -225,8 +247,9 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
   }
 }
 
-// Rotary frequencies f_i = base^(-2 i / dims).  Linear scaling divides them all by `factor`; YaRN divides those of pairs that
-// turn slowly over the original context, keeps those that turn fast, with a linear ramp between the two.
+// Rotary frequencies f_i = base^(-2 i / dims).  Linear scaling divides them all by `factor`; scaling by wavelength divides those
+// with fewer than `low` turns over the original context, keeps those with more than `high`, and blends linearly in the number of
+// turns between the two (Llama 3.1); YaRN does it with a ramp over the pairs.
 inline Rope make_rope(const JsonValue& r) {
   Rope out;
   const int dims = (int)r.number("dims", 0);
@@ -237,6 +260,16 @@ inline Rope make_rope(const JsonValue& r) {
   const double factor = s->number("factor", 1), original = s->number("original", 1);
   if (s->text("kind") == "linear") {
     for (double& f : out.freq) f /= factor;
+    return out;
+  }
+  if (s->text("kind") == "wavelength") {
+    const double low = s->number("low", 1), high = s->number("high", 4);
+    for (double& f : out.freq) {
+      const double wave = 2 * M_PI / f;
+      if (wave < original / high) continue;
+      const double share = wave > original / low ? 0.0 : (original / wave - low) / (high - low);
+      f = (1 - share) * f / factor + share * f;
+    }
     return out;
   }
   auto dim_of = [&](double turns) { return dims * log(original / (2 * M_PI * turns)) / (2 * log(base)); };
@@ -257,7 +290,7 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
   const std::string dt = j.text("dtype");
   VN_REQUIRE(ctx, dt.empty() || dt == "f32" || dt == "bf16", "dtype must be \"f32\" or \"bf16\", got %s", dt.c_str());
   c->bf16 = dt == "bf16";
-  c->tie = 0;
+  c->tie = hm->tied = j.number("tie_weights", 0) != 0;
   c->max_seq_len = (int)j.number("max_seq_len", 2048);
   hm->D = c->dim; hm->vocab = c->vocab;
   hm->eps = (float)j.number("norm_eps", 1e-6);
@@ -273,6 +306,7 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
   const std::string nw = j.text("norm_weight");
   VN_REQUIRE(ctx, nw.empty() || nw == "plain" || nw == "around_zero", "norm_weight %s unknown (plain | around_zero)", nw.c_str());
   hm->plain_norm = hm->layer_norm || nw == "plain";
+  hm->post_norm = j.number("post_norm", 0) != 0;
   hm->side = (int)j.number("token_side", 0);
   hm->sidep = up8(hm->side);
   VN_REQUIRE(ctx, hm->side >= 0, "token_side out of range");
@@ -301,16 +335,32 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
     };
     L.ff = I("mlp_hidden");
     const std::string act = l.text("mlp_act");
-    VN_REQUIRE(ctx, !L.ff || act == "gelu_tanh" || act == "silu" || act == "relu2", "layer %zu: activation %s unknown (gelu_tanh | silu | relu2)", i, act.c_str());
-    L.act = act == "gelu_tanh";
+    VN_REQUIRE(ctx, !L.ff || act == "gelu_tanh" || act == "silu" || act == "clamped" || act == "relu2" || act == "poly_norm",
+               "layer %zu: activation %s unknown (gelu_tanh | silu | clamped | relu2 | poly_norm)", i, act.c_str());
+    L.act = act == "gelu_tanh" ? GLU_GELU : act == "clamped" ? GLU_CLAMP : GLU_SILU;
+    L.limit = (float)l.number("mlp_limit", 0);
     L.ff_plain = act == "relu2";
+    L.poly = act == "poly_norm";
     if (const JsonValue* x = l.find("experts"))
       if (x->kind == JsonValue::OBJ) {
         L.n_exp = (int)x->number("count", 0); L.n_id = (int)x->number("identity", 0); L.top = (int)x->number("top", 0);
         L.exp_groups = (int)x->number("groups", 1); L.keep = (int)x->number("keep", L.exp_groups);
         L.corrected = x->number("correction", 0) != 0;
+        const std::string score = x->text("score"), weight = x->text("weight");
+        VN_REQUIRE(ctx, (score.empty() || score == "softmax" || score == "sigmoid") && (weight.empty() || weight == "result" || weight == "input"),
+                   "layer %zu: experts' score %s (softmax | sigmoid) or weight %s (result | input) unknown", i, score.c_str(), weight.c_str());
+        L.sigmoid = score == "sigmoid";
+        L.weigh_input = weight == "input";
+        if (const JsonValue* sh = x->find("shared"))
+          if (sh->kind == JsonValue::OBJ) {
+            L.sff = (int)sh->number("hidden", 0);
+            L.s_limit = (float)sh->number("limit", L.limit);
+            L.sffp = up8(L.sff);
+            VN_REQUIRE(ctx, L.sff > 0, "layer %zu: shared expert of width %d", i, L.sff);
+          }
+        VN_REQUIRE(ctx, !(L.weigh_input && L.n_id), "layer %zu: identity experts take their weights on the result", i);
         const int n = L.n_out();
-        VN_REQUIRE(ctx, L.ff > 0 && !L.ff_plain && L.n_exp > 0 && L.n_id >= 0 && n <= 1024 && L.exp_groups >= 1 && n % L.exp_groups == 0 &&
+        VN_REQUIRE(ctx, L.ff > 0 && !L.single_up() && L.n_exp > 0 && L.n_id >= 0 && n <= 1024 && L.exp_groups >= 1 && n % L.exp_groups == 0 &&
                    L.keep >= 1 && L.keep <= L.exp_groups && L.top >= 1 && L.top <= MAX_CHOSEN && L.top <= L.keep * (n / L.exp_groups),
                    "layer %zu: mixture of %d experts and %d identities in %d groups, %d kept, %d chosen", i, L.n_exp, L.n_id, L.exp_groups, L.keep, L.top);
         hm->max_out = std::max(hm->max_out, n);
@@ -343,7 +393,11 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
     } else if (L.kind == ATTENTION) {
       L.KH = I("kv_heads"); L.window = I("window"); L.scale = (float)l.number("scale", 0); L.kv_from = I("kv_from", -1);
       L.chunk = I("chunk"); L.softcap = (float)l.number("softcap", 0); L.qk_norm = l.number("qk_norm", 0) != 0; L.bias = l.number("bias", 0) != 0;
-      L.gated = l.number("output_gate", 0) != 0;
+      const std::string gate = l.text("output_gate");
+      VN_REQUIRE(ctx, gate.empty() || gate == "head" || gate == "element" || gate == "none", "layer %zu: output gate %s unknown (head | element | none)", i, gate.c_str());
+      L.gated = gate == "head" ? GATE_HEAD : gate == "element" || (gate.empty() && l.number("output_gate", 0) != 0) ? GATE_ELEMENT : GATE_NONE;
+      L.out_bias = l.number("out_bias", L.bias) != 0;
+      L.temps = l.number("temperature", 0) != 0;
       L.conv_named = l.find("conv") && l.find("conv")->kind == JsonValue::NUM;
       TRY(rope(L.d));
       VN_REQUIRE(ctx, !(L.conv_named && (L.qk_norm || L.bias)) && !(L.kv_from >= 0 && L.qk_norm), "layer %zu: norms and biases of the heads together with "
@@ -357,7 +411,7 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
                    "layer %zu: keys and values of layer %d have other sizes, or are not its own", i, L.kv_from);
       }
       L.P = attn_pitch(std::max(L.d, L.vd));
-      L.n_in = up8(L.conv_ch() + (L.gated ? L.H * L.vd : 0));
+      L.n_in = up8(L.conv_ch() + L.attn_gates());
     } else if (L.kind == LIGHTNING) {
       const JsonValue* dec = l.find("decay");
       VN_REQUIRE(ctx, L.H > 0 && L.d > 0 && L.d <= 512 && L.vd > 0 && dec && dec->kind == JsonValue::ARR && (int)dec->arr.size() == L.H,
@@ -381,6 +435,9 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
       hm->loop_times = (int)lp->number("times", 0);
       VN_REQUIRE(ctx, hm->loop_start >= 0 && hm->loop_start < hm->loop_stop && hm->loop_stop <= n && hm->loop_times >= 1,
                  "loop over layers %d .. %d, %d times, of %d layers", hm->loop_start, hm->loop_stop, hm->loop_times, n);
+      const std::string entry = lp->text("entry");
+      VN_REQUIRE(ctx, entry.empty() || entry == "project" || entry == "add", "entry of a looped block %s unknown (project | add)", entry.c_str());
+      hm->loop_add = entry == "add";
     }
   }
   const int a = hm->loop_times ? hm->loop_start : n, b = hm->loop_times ? hm->loop_stop : n;
@@ -398,7 +455,8 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
   VN_REQUIRE(ctx, !hm->side || !hm->loop_times, "tokens' own inputs do not go with a looped block");
   if (hm->arranged)
     for (const HLayer& L : hm->layers)
-      VN_REQUIRE(ctx, !L.n_exp && !hm->side && L.kind != MAMBA2 && !L.bias, "mixtures, state-space layers, biases and tokens' own inputs need the plain residual");
+      VN_REQUIRE(ctx, !L.n_exp && !hm->side && L.kind != MAMBA2 && !L.bias && !L.out_bias && !L.poly && !hm->post_norm,
+                 "mixtures, state-space layers, biases, PolyNorm, norms of results and tokens' own inputs need the plain residual");
   return VN_OK;
 }
 
@@ -415,15 +473,19 @@ int32_t alloc(vn_model* m) {
   auto W = [&](void** p, size_t n) { return zalloc(m, p, n * e); };
   auto F = [&](float** p, size_t n) { return zalloc(m, (void**)p, n * 4); };
   TRY(W(&m->emb, hm.vocab * D));
-  TRY(W(&m->head, hm.vocab * D));
+  if (hm.tied) m->head = m->emb; else TRY(W(&m->head, hm.vocab * D));
   TRY(F(&m->norm_f, D));
   TRY(dev_alloc(m->ctx, (void**)&m->status, 4));
   VN_CUDA(m->ctx, cudaMemsetAsync(m->status, 0, 4, m->ctx->stream));
-  hm.want = {"embed", "head", "final.norm"};
+  hm.want = {"embed", "final.norm"};
+  if (!hm.tied) hm.want.insert("head");
   if (hm.loop_times) {
-    TRY(W(&hm.w_loop, D * 2 * D));
     TRY(F(&hm.loop_step, hm.loop_times * D));
-    hm.want.insert("loop.in"); hm.want.insert("loop.step");
+    hm.want.insert("loop.step");
+    if (!hm.loop_add) {
+      TRY(W(&hm.w_loop, D * 2 * D));
+      hm.want.insert("loop.in");
+    }
   }
   if (hm.side) {
     TRY(W(&hm.side_embed, (size_t)hm.vocab * hm.layers.size() * hm.side));
@@ -474,10 +536,11 @@ int32_t alloc(vn_model* m) {
       }
       if (L.bias) {
         TRY(F(&L.f_c, L.conv_ch()));
-        TRY(F(&L.o_b, D));
-        need({"mix.q.b", "mix.o.b"});
+        need({"mix.q.b"});
         if (L.kv_from < 0) need({"mix.k.b", "mix.v.b"});
       }
+      if (L.out_bias) { TRY(F(&L.o_b, D)); need({"mix.o.b"}); }
+      if (L.temps) { TRY(F(&L.temp, L.H)); need({"mix.temp"}); }
       if (L.conv_named) need({"mix.q.conv"});
       if (L.conv_named && L.kv_from < 0) need({"mix.k.conv", "mix.v.conv"});
     } else if (L.kind == LIGHTNING) {
@@ -528,18 +591,24 @@ int32_t alloc(vn_model* m) {
       const bool stacked = L.ff_plain && hm.res_gate;          // up | gate of the result: both read the same rows
       const size_t n = std::max(1, L.n_exp);
       TRY(F(&L.norm2, D));
-      TRY(W(&L.w_gu, n * (L.ff_plain ? L.ffp + (stacked ? D : 0) : 2 * L.ffp) * D));
+      TRY(W(&L.w_gu, n * (L.single_up() ? L.ffp + (stacked ? D : 0) : 2 * L.ffp) * D));
       TRY(W(&L.w_down, n * D * L.ffp));
       need({"norm2"});
       if (L.n_exp) {
-        TRY(W(&L.w_router, (size_t)L.n_out() * D));
+        TRY(W(&L.w_router, (size_t)L.n_router() * D));
         need({"mlp.router"});
+        if (L.sff) {
+          TRY(W(&L.w_sgu, (size_t)2 * L.sffp * D));
+          TRY(W(&L.w_sdown, D * L.sffp));
+          need({"mlp.shared.gate", "mlp.shared.up", "mlp.shared.down", "mlp.shared.sg"});
+        }
         if (L.corrected) { TRY(F(&L.correction, L.n_out())); need({"mlp.correction"}); }
         for (int x = 0; x < L.n_exp; ++x)
           for (const char* part : {".gate", ".up", ".down"}) hm.want.insert(p + "mlp.e" + std::to_string(x) + part);
       } else {
         need({"mlp.up", "mlp.down"});
-        if (!L.ff_plain) need({"mlp.gate"});
+        if (!L.single_up()) need({"mlp.gate"});
+        if (L.poly) { TRY(F(&L.coef, 4)); need({"mlp.act"}); }
       }
       if (stacked) L.w_rg[1] = (char*)L.w_gu + (size_t)L.ffp * D * e;
     }
@@ -551,6 +620,10 @@ int32_t alloc(vn_model* m) {
     }
     for (int q = 0; q < (L.ff ? 2 : 1); ++q) {
       const std::string k = std::to_string(q + 1);
+      if (hm.post_norm) {
+        TRY(F(&L.post[q], D));
+        hm.want.insert(p + "norm" + k + "b");
+      }
       if (hm.streams) {
         TRY(F(&L.hc_in[q], hm.streams));
         TRY(F(&L.hc_out[q], hm.streams));
@@ -581,7 +654,8 @@ void destroy(vn_model* m) {
     if (!(L.ff_plain && hm.res_gate)) F(L.w_rg[1]);            // else part of w_gu
     F(L.w_gu); F(L.w_down); F(L.w_rg[0]); F(L.in_conv);
     F(L.f_d); F(L.o_b); F(L.w_router); F(L.correction); F(L.w_sgate); F(L.w_sproj); F(L.s_norm);
-    for (int q = 0; q < 2; ++q) { F(L.hc_in[q]); F(L.hc_out[q]); F(L.hc_mix[q]); F(L.rg_b[q]); }
+    F(L.temp); F(L.coef); F(L.w_sgu); F(L.w_sdown);
+    for (int q = 0; q < 2; ++q) { F(L.post[q]); F(L.hc_in[q]); F(L.hc_out[q]); F(L.hc_mix[q]); F(L.rg_b[q]); }
   }
   for (Rope& r : hm.ropes) F(r.table);
   for (void* t : hm.retired) F(t);
@@ -623,7 +697,7 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
     const int i = n[0] == 'l' && at != std::string::npos ? atoi(n.substr(1, at - 1).c_str()) : -1;
     const std::string part = at != std::string::npos ? n.substr(at + 1) : "";
     if (i >= 0 && i < (int)hm.layers.size() && !hm.layers[i].ff && n.substr(0, at) == "l" + std::to_string(i) &&
-        (part == "norm2" || part.compare(0, 4, "hc2.") == 0 || part == "rg2" || part == "rg2.b"))
+        (part == "norm2" || part == "norm2b" || part.compare(0, 4, "hc2.") == 0 || part == "rg2" || part == "rg2.b"))
       return VN_OK;
     return vn_fail(ctx, VN_ERR_INVALID, "unexpected tensor %s", n.c_str());
   }
@@ -642,11 +716,18 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
   const std::string s = n.substr(dot + 1);
   if (s == "norm1") PUT(D, 1, weight(L.norm1, D));
   if (s == "norm2") PUT(D, 1, weight(L.norm2, D));
+  if (s == "norm1b") PUT(D, 1, weight(L.post[0], D));
+  if (s == "norm2b") PUT(D, 1, weight(L.post[1], D));
+  if (s == "mlp.act") PUT(4, 1, f32(data, L.coef, 4));
   if (s == "mlp.gate") PUT(L.ff, D, rows(L.w_gu, D, 0, 2));
-  if (s == "mlp.up" && L.ff_plain) PUT(L.ff, D, rows(L.w_gu, D));
+  if (s == "mlp.up" && L.single_up()) PUT(L.ff, D, rows(L.w_gu, D));
   if (s == "mlp.up") PUT(L.ff, D, rows(L.w_gu, D, 1, 2));
   if (s == "mlp.down") PUT(D, L.ff, rows(L.w_down, L.ffp));
   if (s == "mlp.router") PUT(L.n_out(), D, rows(L.w_router, D));
+  if (s == "mlp.shared.sg") PUT(1, D, rows(L.w_router, D, L.n_out()));
+  if (s == "mlp.shared.gate") PUT(L.sff, D, rows(L.w_sgu, D, 0, 2));
+  if (s == "mlp.shared.up") PUT(L.sff, D, rows(L.w_sgu, D, 1, 2));
+  if (s == "mlp.shared.down") PUT(D, L.sff, rows(L.w_sdown, L.sffp));
   if (s == "mlp.correction") PUT(L.n_out(), 1, f32(data, L.correction, r));
   if (s.compare(0, 5, "mlp.e") == 0) {
     const size_t end = s.find('.', 4);
@@ -674,7 +755,8 @@ int32_t load(vn_model* m, const std::string& n, const float* data, long long r, 
     if (s == "mix.q") PUT(qd, D, rows(L.w_in, D));
     if (s == "mix.k") PUT(kd, D, rows(L.w_in, D, qd));
     if (s == "mix.v") PUT(vd, D, rows(L.w_in, D, qd + kd));
-    if (s == "mix.g") PUT(hv, D, rows(L.w_in, D, L.conv_ch()));
+    if (s == "mix.g") PUT(L.attn_gates(), D, rows(L.w_in, D, L.conv_ch()));
+    if (s == "mix.temp") PUT(L.H, 1, f32(data, L.temp, r));
     if (s == "mix.q.norm") PUT(L.d, 1, f32(data, L.f_a, r));
     if (s == "mix.k.norm") PUT(L.d, 1, f32(data, L.f_b, r));
     if (s == "mix.q.b") PUT(qd, 1, f32(data, L.f_c, r));
@@ -781,7 +863,7 @@ int32_t ensure(vn_model* m, int M) {
     TRY(dev_alloc(ctx, (void**)&hm.gate, R * D * 4));
     TRY(dev_alloc(ctx, (void**)&hm.y, R * D * 4));
   }
-  if (hm.loop_times) TRY(dev_alloc(ctx, &hm.cat, R * 2 * D * e));
+  if (hm.loop_times && !hm.loop_add) TRY(dev_alloc(ctx, &hm.cat, R * 2 * D * e));
   size_t need = 0;
   for (auto& L : hm.layers)
     for (size_t rows : {R, std::min(R, (size_t)SPLIT_ROWS)}) {
@@ -829,8 +911,8 @@ int32_t project(vn_model* m, GemmArgs g, float* direct, Mat<__nv_bfloat16>* out,
   out->p = (const __nv_bfloat16*)direct; out->ld = g.N;
   return linear(m, g);
 }
-// what m->h holds behind a sublayer: RMSNorm(x) * norm_w, x itself, or nothing
-struct Next { const float* norm_w = nullptr; bool cast = false; };
+// what follows a sublayer: the entry of a looped block's pass, and in m->h RMSNorm(x) * norm_w, x itself, or nothing
+struct Next { const float* norm_w = nullptr; bool cast = false; PassEntry pass; };
 
 // x += y (or y over its root mean square times own_norm), and what the next product reads, in one pass over the rows
 template <typename T, typename Y>
@@ -838,13 +920,29 @@ int32_t close_rows(vn_model* m, const Y& y, int M, const float* own_norm, const 
   vn_ctx* ctx = m->ctx;
   const int D = m->hyb->D;
   const float eps = m->hyb->eps;
-#define RESIDUAL(NV) VN_LAUNCH_PDL_LEVEL(ctx, 1, "residual_kernel", (residual_kernel<T, Y, NV>), M, 256, 0, y, m->x, own_norm, next.norm_w, (int)next.cast, (T*)m->h, D, eps)
+#define RESIDUAL(NV) VN_LAUNCH_PDL_LEVEL(ctx, 1, "residual_kernel", (residual_kernel<T, Y, NV>), M, 256, 0, y, m->x, own_norm, next.pass, next.norm_w, (int)next.cast, (T*)m->h, D, eps)
   if (D % 4 || D > 8192) RESIDUAL(0); else if (D <= 1024) RESIDUAL(1); else if (D <= 2048) RESIDUAL(2); else if (D <= 4096) RESIDUAL(4); else RESIDUAL(8);
 #undef RESIDUAL
   return VN_OK;
 }
 
-// x += A W^T (+ bias); then m->h as `next` says
+// x += A W^T over its root mean square times own_norm; then as `next` says.  direct: [M, D] fp32 scratch
+template <typename T>
+int32_t close_normed(vn_model* m, const GemmArgs& g, const float* bias, float* direct, const float* own_norm, const Next& next) {
+  if constexpr (std::is_same<T, __nv_bfloat16>::value)
+    if (g.M > 256) {
+      AddRows<Mat<T>> y;
+      y.bias = bias;
+      TRY(project(m, g, direct, &y.y));
+      return close_rows<T>(m, y, g.M, own_norm, next);
+    }
+  AddRows<Src> y;
+  y.bias = bias;
+  TRY(project(m, g, direct, &y.y));
+  return close_rows<T>(m, y, g.M, own_norm, next);
+}
+
+// x += A W^T (+ bias); then as `next` says
 template <typename T>
 int32_t close_block(vn_model* m, GemmArgs g, const float* bias, const Next& next) {
   vn_ctx* ctx = m->ctx;
@@ -854,7 +952,7 @@ int32_t close_block(vn_model* m, GemmArgs g, const float* bias, const Next& next
   if (tc_rows(m, g)) {
     int sp = 1;
     TRY(tc_partial(m, g, M, M, &sp));
-    if (bias || next.cast) {
+    if (bias || next.cast || next.pass.step) {
       AddRows<Src> y;
       y.y.p = m->partial; y.y.splits = sp; y.y.pstride = (long long)M * D; y.y.ld = D; y.bias = bias;
       return close_rows<T>(m, y, M, nullptr, next);
@@ -875,7 +973,9 @@ int32_t close_block(vn_model* m, GemmArgs g, const float* bias, const Next& next
     const long long n = (long long)M * D;
     VN_LAUNCH(ctx, cast_rows_kernel<T>, (unsigned)ceil_div(n, 1024ll), 256, 0, m->x, (T*)m->h, n);
   }
-  if (next_norm)
+  if (next.pass.step)
+    VN_LAUNCH(ctx, enter_pass_kernel<T>, M, 256, 0, next.pass, m->x, next_norm, (T*)m->h, D, hm.eps);
+  else if (next_norm)
     VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, next_norm, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
   return VN_OK;
 }
@@ -1067,6 +1167,8 @@ int32_t attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const 
   a.own_kv = from == run;
   a.kplane = kv->k[from]; a.vplane = kv->v[from]; a.table = hc.table_dev; a.max_pages = hc.max_pages;
   a.col_g = L.gated ? L.conv_ch() : -1;
+  a.gate_head = L.gated == GATE_HEAD;
+  a.temp = L.temp;
   a.q = b.q; a.out = b.mix; a.pending = hc.pending; a.rows = rows;
   const bool mma = m->cfg.bf16 && attn_mma_ok(L.P) && !m->force_simt_attn;
   if constexpr (std::is_same<T, __nv_bfloat16>::value && std::is_same<S, Src>::value) {
@@ -1141,26 +1243,58 @@ int32_t head(vn_model* m, int n_rows, float* out_logits) {
   return linear(m, g);
 }
 
-// act = f(h W_gate^T) * (h W_up^T) of a gated feed-forward
+// out = glu(h W_gate^T, h W_up^T) of a gated feed-forward of padded width n, w: both matrices, rows in turn
 template <typename T>
-int32_t gated_up(vn_model* m, const HLayer& L, int M, const Buffers& b) {
+int32_t gated_up(vn_model* m, const void* w, int n, int act, float limit, int M, void* out, const char* tag) {
   vn_ctx* ctx = m->ctx;
   const int D = m->hyb->D;
-  GemmArgs g = gemm_args(m->h, D, L.w_gu, 2 * L.ffp, D, M, "gemm_ff_gateup");
+  GemmArgs g = gemm_args(m->h, D, w, 2 * n, D, M, tag);
   if (tc_rows(m, g)) {
     int sp = 1;
     TRY(tc_partial(m, g, M, M, &sp));
-    const long long pairs = (long long)M * L.ffp;
+    const long long pairs = (long long)M * n;
     VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp,
-                      (long long)M * 2 * L.ffp, (T*)b.act, 2 * L.ffp, pairs, L.act);
+                      (long long)M * 2 * n, (T*)out, 2 * n, pairs, act, limit);
     return VN_OK;
   }
-  g.C = b.act; g.ldc = L.ffp; g.epi = EPI_SWIGLU; g.act = L.act; g.c_bf16 = m->cfg.bf16;
+  g.C = out; g.ldc = n; g.epi = EPI_SWIGLU; g.act = act; g.act_limit = limit; g.c_bf16 = m->cfg.bf16;
   return linear(m, g);
 }
+template <typename T>
+int32_t gated_up(vn_model* m, const HLayer& L, int M, const Buffers& b) {
+  return gated_up<T>(m, L.w_gu, L.ffp, L.act, L.limit, M, b.act, "gemm_ff_gateup");
+}
 
-// Mixture of experts: x += the weighted results of each row's experts, m->h as `next` says.  The rows are copied into expert
-// order; few rows go as one segment per expert through split-K GEMMs, many as pieces of 256 rows.
+// act = PolyNorm(h W_up^T)
+template <typename T, typename S>
+int32_t poly_up(vn_model* m, const HLayer& L, int M, const Buffers& b) {
+  vn_ctx* ctx = m->ctx;
+  S z;
+  TRY(project(m, gemm_args(m->h, m->hyb->D, L.w_gu, L.ffp, m->hyb->D, M, "gemm_ff_up"), b.proj, &z));
+  const int n = L.ffp;
+#define POLY(NV) VN_LAUNCH_PDL_LEVEL(ctx, 1, "poly_norm_kernel", (poly_norm_kernel<T, S, NV>), M, 256, 0, z, L.coef, (T*)b.act, L.ff, n, m->hyb->eps)
+  if (n > 8192) POLY(0); else if (n <= 1024) POLY(1); else if (n <= 2048) POLY(2); else if (n <= 4096) POLY(4); else POLY(8);
+#undef POLY
+  return VN_OK;
+}
+template <typename T>
+int32_t poly_up(vn_model* m, const HLayer& L, int M, const Buffers& b) {
+  if constexpr (std::is_same<T, __nv_bfloat16>::value)
+    if (M > 256) return poly_up<T, Mat<T>>(m, L, M, b);
+  return poly_up<T, Src>(m, L, M, b);
+}
+
+// result of the expert that serves every row
+template <typename T, typename S>
+int32_t shared_expert(vn_model* m, const HLayer& L, int M, const Buffers& b, S* out) {
+  TRY(gated_up<T>(m, L.w_sgu, L.sffp, L.act, L.s_limit, M, b.sact, "gemm_shared_gateup"));
+  return project(m, gemm_args(b.sact, L.sffp, L.w_sdown, m->hyb->D, L.sffp, M, "gemm_shared_down"), b.sy, out, true);
+}
+
+// Mixture of experts: x += the weighted results of each row's experts and the gated one of the expert that serves every row (or
+// their sum over its root mean square times the sublayer's norm); then as `next` says.  The rows are copied into expert order, times
+// their weights where those belong to the input; few rows go as one segment per expert through split-K GEMMs, many as pieces of
+// 256 rows.
 template <typename T>
 int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Next& next) {
   vn_ctx* ctx = m->ctx;
@@ -1168,42 +1302,47 @@ int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Nex
   const int D = hm.D, n = L.n_out(), S = L.top, F = L.ffp;
   const bool bf = m->cfg.bf16;
   RouteIn r;
-  TRY(project(m, gemm_args(m->h, D, L.w_router, n, D, M, "gemm_router"), b.logits, &r.z));
+  TRY(project(m, gemm_args(m->h, D, L.w_router, L.n_router(), D, M, "gemm_router"), b.logits, &r.z));
+  r.sigmoid = L.sigmoid; r.shared_gate = L.sff ? b.sgate : nullptr;
   r.correction = L.correction; r.M = M; r.E = n; r.top = S; r.groups = L.exp_groups; r.keep = L.keep;
   r.slot_expert = b.slot_expert; r.slot_w = b.slot_w; r.count = hm.exp_count;
   r.rows = route_rows(M);
   VN_LAUNCH_PDL_LEVEL(ctx, 1, "route_kernel", route_kernel, ceil_div(M, ROUTE_WARPS * r.rows), 32 * ROUTE_WARPS, route_smem(n, L.exp_groups), r);
   AddExperts<T, Src> few;          // results in split-K slices
-  few.h = (const T*)m->h; few.slot_pos = b.slot_pos; few.slot_expert = b.slot_expert; few.slot_w = b.slot_w; few.top = S; few.n_real = L.n_exp; few.D = D;
+  few.h = (const T*)m->h; few.slot_pos = b.slot_pos; few.slot_expert = b.slot_expert; few.slot_w = L.weigh_input ? nullptr : b.slot_w; few.top = S; few.n_real = L.n_exp; few.D = D;
   few.count = hm.exp_count; few.cursor = hm.exp_cur; few.n_count = n;
   few.y.ld = D;
+  few.shared_gate = r.shared_gate;
+  const float* scale = L.weigh_input ? b.slot_w : nullptr;
   GemmArgs up, down;
   up.A = b.hs; up.lda = D; up.W = L.w_gu; up.ldw = D; up.w_stride = (long long)2 * F * D; up.N = 2 * F; up.K = D; up.tag = "gemm_expert_gateup";
-  up.C = b.act; up.ldc = F; up.epi = EPI_SWIGLU; up.act = L.act; up.c_bf16 = bf;
+  up.C = b.act; up.ldc = F; up.epi = EPI_SWIGLU; up.act = L.act; up.act_limit = L.limit; up.c_bf16 = bf;
   down.A = b.act; down.lda = F; down.W = L.w_down; down.ldw = F; down.w_stride = (long long)D * F; down.N = D; down.K = F; down.tag = "gemm_expert_down";
   down.C = b.ey; down.ldc = D; down.c_bf16 = bf;
   up.M = down.M = M;
   const bool tc = bf && m->use_tc && D % 8 == 0 && tc_detail::encode_fn() != nullptr;
   if (tc && M <= 256) {
+    if (L.sff) TRY((shared_expert<T, Src>(m, L, M, b, &few.shared)));
     VN_LAUNCH_PDL_LEVEL(ctx, 1, "mod_dispatch_kernel", mod_dispatch_kernel<T>, M * S, 128, 0, (const T*)m->h, b.slot_expert, hm.exp_count, hm.exp_off, hm.exp_cur,
-                        b.slot_pos, (T*)b.hs, n, S, D);
+                        b.slot_pos, (T*)b.hs, n, S, D, scale);
     up.seg_off = down.seg_off = hm.exp_off; up.seg_cnt = down.seg_cnt = hm.exp_count; up.nseg = down.nseg = L.n_exp;
     const int active = std::min(L.n_exp, M * S);          // segments with rows, at most
     int sp = 1;
     TRY(tc_partial(m, up, (long long)M * S, (long long)M * S, &sp, active));
     const long long pairs = (long long)M * S * F;
     VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp, (long long)M * S * 2 * F, (T*)b.act, 2 * F,
-                      pairs, L.act);
+                      pairs, L.act, L.limit);
     TRY(tc_partial(m, down, (long long)M * S, (long long)M * S, &sp, active));
     few.y.p = m->partial; few.y.splits = sp; few.y.pstride = (long long)M * S * D;
-    return close_rows<T>(m, few, M, nullptr, next);
+    return close_rows<T>(m, few, M, L.post[1], next);
   }
   VN_LAUNCH(ctx, mod_offsets_kernel, 1, 32, 0, hm.exp_count, hm.exp_off, hm.exp_cur, n);
-  VN_LAUNCH(ctx, mod_scatter_kernel, ceil_div(M * S, 256), 256, 0, b.slot_expert, hm.exp_off, hm.exp_cur, b.sorted_row, b.slot_pos, M * S, S);
+  VN_LAUNCH(ctx, mod_scatter_kernel, ceil_div(M * S, 256), 256, 0, b.slot_expert, hm.exp_off, hm.exp_cur, b.sorted_row, b.slot_pos, M * S, S, scale, scale ? b.sorted_w : (float*)nullptr);
+  const float* sorted_w = scale ? b.sorted_w : nullptr;
   if (tc) {
     int *off = b.sub_seg, *cnt = off + b.sub_cap, *w = cnt + b.sub_cap;
     VN_LAUNCH(ctx, mod_subseg_kernel, 1, 32, 0, (const int*)hm.exp_count, (const int*)hm.exp_off, L.n_exp, off, cnt, w, b.sub_cap);
-    VN_LAUNCH(ctx, gather_sorted_kernel<T>, M * S, 128, 0, (const T*)m->h, (const int*)b.sorted_row, (T*)b.hs, D);
+    VN_LAUNCH(ctx, gather_sorted_kernel<T>, M * S, 128, 0, (const T*)m->h, (const int*)b.sorted_row, (T*)b.hs, D, sorted_w);
     TRY(ensure_partial(m, 1024));
     for (GemmArgs* g : {&up, &down}) {
       g->M = 256; g->seg_off = off; g->seg_cnt = cnt; g->seg_w = w; g->n_w = L.n_exp; g->nseg = b.sub_cap;
@@ -1211,8 +1350,12 @@ int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Nex
       plan.error_flag = m->tc_error;
       TRY(launch_gemm_tc(ctx, *g, (long long)M * S, plan));
     }
-  } else {                                                // the kernels of any shape gather the rows themselves
-    up.A = m->h; up.a_rows = b.sorted_row;
+  } else {                                                // the kernels of any shape gather rows themselves, as they are
+    if (scale) {
+      VN_LAUNCH(ctx, gather_sorted_kernel<T>, M * S, 128, 0, (const T*)m->h, (const int*)b.sorted_row, (T*)b.hs, D, sorted_w);
+    } else {
+      up.A = m->h; up.a_rows = b.sorted_row;
+    }
     for (GemmArgs* g : {&up, &down}) {
       g->seg_off = hm.exp_off; g->seg_cnt = hm.exp_count; g->nseg = L.n_exp;
       TRY(linear(m, *g));
@@ -1221,12 +1364,14 @@ int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Nex
   if constexpr (std::is_same<T, __nv_bfloat16>::value) {
     AddExperts<T, Mat<T>> y;
     y.y.p = (const T*)b.ey; y.y.ld = D;
-    y.h = few.h; y.slot_pos = few.slot_pos; y.slot_expert = few.slot_expert; y.slot_w = few.slot_w; y.top = S; y.n_real = few.n_real; y.D = D;
+    y.h = few.h; y.slot_pos = few.slot_pos; y.slot_expert = few.slot_expert; y.slot_w = few.slot_w; y.shared_gate = few.shared_gate; y.top = S; y.n_real = few.n_real; y.D = D;
     y.count = few.count; y.cursor = few.cursor; y.n_count = n;
-    return close_rows<T>(m, y, M, nullptr, next);
+    if (L.sff) TRY((shared_expert<T, Mat<T>>(m, L, M, b, &y.shared)));
+    return close_rows<T>(m, y, M, L.post[1], next);
   } else {
     few.y.p = (const float*)b.ey;
-    return close_rows<T>(m, few, M, nullptr, next);
+    if (L.sff) TRY((shared_expert<T, Src>(m, L, M, b, &few.shared)));
+    return close_rows<T>(m, few, M, L.post[1], next);
   }
 }
 
@@ -1241,16 +1386,7 @@ int32_t side_input(vn_model* m, const int64_t* tokens, const HLayer& L, int laye
   const long long total = (long long)M * hm.sidep;
   VN_LAUNCH_PDL_LEVEL(ctx, 1, "side_act_kernel", side_act_kernel<T>, (unsigned)ceil_div(total, 256ll), 256, 0, gate, (const long long*)tokens, hm.vocab,
                       (const T*)hm.side_embed, (long long)hm.layers.size() * hm.side, layer * hm.side, hm.side, (T*)b.side_act, hm.sidep, total);
-  const GemmArgs g = gemm_args(b.side_act, hm.sidep, L.w_sproj, D, hm.sidep, M, "gemm_side_proj");
-  if constexpr (std::is_same<T, __nv_bfloat16>::value)
-    if (M > 256) {
-      AddRows<Mat<T>> y;
-      TRY(project(m, g, b.proj, &y.y));
-      return close_rows<T>(m, y, M, L.s_norm, next);
-    }
-  AddRows<Src> y;
-  TRY(project(m, g, b.proj, &y.y));
-  return close_rows<T>(m, y, M, L.s_norm, next);
+  return close_normed<T>(m, gemm_args(b.side_act, hm.sidep, L.w_sproj, D, hm.sidep, M, "gemm_side_proj"), nullptr, b.proj, L.s_norm, next);
 }
 
 // act = relu(h W_up^T)^2, and the raw gate of the result beside it when the model has one
@@ -1407,34 +1543,46 @@ int32_t forward(vn_model* m, vn_kv* kv, const int64_t* tokens, const Rows& rows,
   VN_LAUNCH(ctx, embed_pos_kernel<T>, M, 256, 0, (const long long*)tokens, (const T*)m->emb, hm.freq, m->x, hm.x0, rows, D,
             hm.vocab, m->status);
   auto enters_pass = [&](int i) { return i < n_runs && hm.runs[i].pass >= 0 && hm.runs[i].layer == hm.loop_start; };
+  auto pass_entry = [&](int i) {
+    PassEntry p;
+    if (enters_pass(i) && hm.loop_add) { p.step = hm.loop_step + (long long)hm.runs[i].pass * D; p.x0 = hm.runs[i].pass > 0 ? hm.x0 : nullptr; }
+    return p;
+  };
   for (int i = 0; i < n_runs; ++i) {
     const HLayer& L = hm.layers[hm.runs[i].layer];
     Arena A;
     Buffers b;
     A.base = hm.ws;
     layout(hm, L, M, m->esz, A, b);
-    if (enters_pass(i)) {
+    if (enters_pass(i) && !hm.loop_add) {
       // x = W [x | x0] + step vector of the pass, and the first layer's norm
       VN_LAUNCH(ctx, concat_cast_kernel<T>, M, 256, 0, m->x, hm.x0, (T*)hm.cat, D);
       Src s;
       TRY(project(m, gemm_args(hm.cat, 2 * D, hm.w_loop, D, 2 * D, M, "gemm_loop_in"), b.proj, &s));
       VN_LAUNCH(ctx, rowsum_norm_kernel<T>, M, 256, 0, s, hm.loop_step + (long long)hm.runs[i].pass * D, 0, m->x, L.norm1,
                 (T*)m->h, D, hm.eps);
+    } else if (enters_pass(i) && (i == 0 || hm.probe)) {
+      VN_LAUNCH(ctx, enter_pass_kernel<T>, M, 256, 0, pass_entry(i), m->x, L.norm1, (T*)m->h, D, hm.eps);
     } else if (i == 0) {
       VN_LAUNCH(ctx, rmsnorm_kernel<T>, M, 256, 0, m->x, L.norm1, (T*)m->h, (float*)nullptr, 1, 0, D, hm.eps);
     }
-    const Next next_layer{i + 1 < n_runs && !enters_pass(i + 1) ? hm.layers[hm.runs[i + 1].layer].norm1 : nullptr, false};
-    const Next after_ff = hm.side ? Next{nullptr, true} : next_layer, after_mix = L.ff ? Next{L.norm2, false} : after_ff;
+    Next next_layer;                                      // an entry that adds is part of the sublayer's end before it
+    if (i + 1 < n_runs && (!enters_pass(i + 1) || (hm.loop_add && !hm.probe)))
+      next_layer = {hm.layers[hm.runs[i + 1].layer].norm1, false, pass_entry(i + 1)};
+    const Next after_ff = hm.side ? Next{nullptr, true, {}} : next_layer, after_mix = L.ff ? Next{L.norm2, false, {}} : after_ff;
+    auto close = [&](const GemmArgs& g, const float* bias, const float* own_norm, const Next& next) {
+      return own_norm ? close_normed<T>(m, g, bias, b.proj, own_norm, next) : close_block<T>(m, g, bias, next);
+    };
     if (L.kind == MAMBA1) TRY(mamba1<T>(m, m->h, kv, hc, L, i, rows, b));
     else if (L.kind == DELTA) TRY(channel_delta<T>(m, m->h, kv, hc, L, i, rows, b));
     else TRY((dense_projection_mixer<T>(m, m->h, kv, hc, L, i, rows, b)));
     const int width = L.kind == MAMBA1 ? L.inner : L.H * L.vd;
-    TRY(close_block<T>(m, gemm_args(b.mix, width, L.w_o, D, width, M, "gemm_mix_out"), L.o_b, after_mix));
+    TRY(close(gemm_args(b.mix, width, L.w_o, D, width, M, "gemm_mix_out"), L.o_b, L.post[0], after_mix));
     if (L.n_exp) {
       TRY(mixture<T>(m, L, M, b, after_ff));
     } else if (L.ff) {
-      TRY(gated_up<T>(m, L, M, b));
-      TRY(close_block<T>(m, gemm_args(b.act, L.ffp, L.w_down, D, L.ffp, M, "gemm_ff_down"), nullptr, after_ff));
+      if (L.poly) TRY(poly_up<T>(m, L, M, b)); else TRY(gated_up<T>(m, L, M, b));
+      TRY(close(gemm_args(b.act, L.ffp, L.w_down, D, L.ffp, M, "gemm_ff_down"), nullptr, L.post[1], after_ff));
     }
     if (hm.side) TRY(side_input<T>(m, tokens, L, hm.runs[i].layer, M, b, next_layer));
     if (hm.probe)

@@ -585,7 +585,7 @@ int32_t forward_t(vn_model* m, vn_kv* kv, const int64_t* tokens, int B, int Tn, 
       VN_LAUNCH(ctx, mod_route_kernel, M, 128, 0, r);
       VN_LAUNCH(ctx, mod_offsets_kernel, 1, 32, 0, m->expert_count, m->expert_off, m->expert_cur, ne);
       VN_LAUNCH(ctx, mod_scatter_kernel, ceil_div(M * S, 256), 256, 0, m->slot_expert, m->expert_off, m->expert_cur,
-                m->sorted_row, m->slot_pos, M * S, S);
+                m->sorted_row, m->slot_pos, M * S, S, (const float*)nullptr, (float*)nullptr);
       // Many routed rows on a bf16 model: the experts' segments are cut into pieces of at most 256 rows and run on
       // the tcgen05 kernel (rows copied into expert order first, so that TMA loads them; a piece names its expert's
       // weights through seg_w).  Otherwise the mma.sync kernels gather the rows themselves.
@@ -598,7 +598,7 @@ int32_t forward_t(vn_model* m, vn_kv* kv, const int64_t* tokens, int B, int Tn, 
         int* sub_off = m->sub_seg; int* sub_cnt = m->sub_seg + m->sub_cap; int* sub_w = m->sub_seg + 2 * m->sub_cap;
         VN_LAUNCH(ctx, mod_subseg_kernel, 1, 32, 0, (const int*)m->expert_count, (const int*)m->expert_off, ne, sub_off,
                   sub_cnt, sub_w, n_sub);
-        VN_LAUNCH(ctx, gather_sorted_kernel<T>, M * S, 128, 0, (const T*)m->h, (const int*)m->sorted_row, (T*)m->hs, D);
+        VN_LAUNCH(ctx, gather_sorted_kernel<T>, M * S, 128, 0, (const T*)m->h, (const int*)m->sorted_row, (T*)m->hs, D, (const float*)nullptr);
         TRY(ensure_partial(m, 1024));
         TcPlan plan;
         plan.error_flag = m->tc_error;
@@ -992,7 +992,7 @@ int32_t forward_tc(vn_model* m, vn_kv* kv, const int64_t* tokens, int B, int Tn,
         TRY(tc_partial(m, g, cap, M, &sp));
         const long long pairs = (long long)M * c.mlp_hidden;
         VN_LAUNCH_PDL_BIT(ctx, 8, splitk_swiglu_kernel<T>, (unsigned)ceil_div(pairs, 512ll), 256, 0, m->partial, sp,
-                  (long long)M * 2 * c.mlp_hidden, (T*)m->act, 2 * c.mlp_hidden, pairs, 0);
+                  (long long)M * 2 * c.mlp_hidden, (T*)m->act, 2 * c.mlp_hidden, pairs, (int)GLU_SILU, 0.f);
       }
       g = GemmArgs();
       g.A = m->act; g.lda = c.mlp_hidden; g.W = L.w_down; g.ldw = c.mlp_hidden; g.M = M; g.N = D; g.K = c.mlp_hidden;
@@ -1009,7 +1009,7 @@ int32_t forward_tc(vn_model* m, vn_kv* kv, const int64_t* tokens, int B, int Tn,
       r.expert_count = m->expert_count; r.M = M; r.D = D; r.P = c.P; r.E = c.E; r.top_k = c.top_k;
       VN_LAUNCH_PDL_BIT(ctx, 16, mod_route_kernel, M, 512, 0, r);
       VN_LAUNCH_PDL_BIT(ctx, 16, mod_dispatch_kernel<T>, M * S, 128, 0, (const T*)m->h, m->slot_expert, m->expert_count,
-                    m->expert_off, m->expert_cur, m->slot_pos, (T*)m->hs, ne, S, D);
+                    m->expert_off, m->expert_cur, m->slot_pos, (T*)m->hs, ne, S, D, (const float*)nullptr);
       g = GemmArgs();
       g.A = m->hs; g.lda = D; g.W = L.e_gateup; g.ldw = D; g.w_stride = (long long)2 * eh * D;
       g.C = m->act; g.ldc = eh; g.M = M; g.N = 2 * eh; g.K = D; g.epi = EPI_SWIGLU; g.c_bf16 = 1;

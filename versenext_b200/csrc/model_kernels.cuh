@@ -488,10 +488,11 @@ __global__ void mod_subseg_kernel(const int* __restrict__ count, const int* __re
   }
 }
 
-// place every (token, slot) in its expert's segment; sorted_row[pos] = token row, slot_pos[token, slot] = pos
+// place every (token, slot) in its expert's segment; sorted_row[pos] = token row, slot_pos[token, slot] = pos and, where asked
+// for, sorted_w[pos] = the slot's weight
 __global__ void mod_scatter_kernel(const int* __restrict__ slot_expert, const int* __restrict__ offset,
                                    int* __restrict__ cursor, int* __restrict__ sorted_row, int* __restrict__ slot_pos,
-                                   int n_slots_total, int S) {
+                                   int n_slots_total, int S, const float* __restrict__ slot_w, float* __restrict__ sorted_w) {
   pdl_trigger();
   pdl_wait();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
@@ -500,6 +501,7 @@ __global__ void mod_scatter_kernel(const int* __restrict__ slot_expert, const in
   const int pos = offset[e] + atomicAdd(&cursor[e], 1);
   sorted_row[pos] = i / S;
   slot_pos[i] = pos;
+  if (sorted_w) sorted_w[pos] = slot_w[i];
 }
 
 // x[row] += sum_p part_w[p] * (sum_j slot_w[p, j] * y[slot_pos[p, j]])   (mod.py:196-211, :604-605, :779-781)
@@ -644,10 +646,11 @@ __global__ void splitk_store_kernel(const float* __restrict__ partial, int split
   out[row * ld + n] = acc;
 }
 
-// act[row, j] = f(sum_s partial[.., 2j]) * sum_s partial[.., 2j+1]
+// act[row, j] = glu(sum_s partial[.., 2j], sum_s partial[.., 2j+1])
 template <typename T>
 __global__ void splitk_swiglu_kernel(const float* __restrict__ partial, int splits, long long pstride,
-                                     T* __restrict__ act, int N, long long total_pairs, int fn) {
+                                     T* __restrict__ act, int N, long long total_pairs, int fn, float limit) {
+  constexpr bool fast = sizeof(T) == 2;
   pdl_trigger();
   pdl_wait();
   const int half = N / 2;
@@ -664,8 +667,8 @@ __global__ void splitk_swiglu_kernel(const float* __restrict__ partial, int spli
       const float4 t = *reinterpret_cast<const float4*>(p + (long long)s * pstride);
       acc.x += t.x; acc.y += t.y; acc.z += t.z; acc.w += t.w;
     }
-    act[row * half + j] = from_f<T>(glu_act(acc.x, fn) * acc.y);
-    act[row * half + j + 1] = from_f<T>(glu_act(acc.z, fn) * acc.w);
+    act[row * half + j] = from_f<T>(glu(acc.x, acc.y, fn, limit, fast));
+    act[row * half + j + 1] = from_f<T>(glu(acc.z, acc.w, fn, limit, fast));
     return;
   }
   for (long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 2, e = 0; e < 2 && i < total_pairs; ++e, ++i) {
@@ -676,18 +679,35 @@ __global__ void splitk_swiglu_kernel(const float* __restrict__ partial, int spli
       const float2 p = *reinterpret_cast<const float2*>(partial + (long long)s * pstride + row * N + 2 * j);
       g += p.x; u += p.y;
     }
-    act[row * half + j] = from_f<T>(glu_act(g, fn) * u);
+    act[row * half + j] = from_f<T>(glu(g, u, fn, limit, fast));
   }
+}
+
+// sixteen bytes of a row times a factor
+template <typename T> __device__ __forceinline__ uint4 scaled16(uint4 p, float f);
+template <> __device__ __forceinline__ uint4 scaled16<float>(uint4 p, float f) {
+  return make_uint4(__float_as_uint(__uint_as_float(p.x) * f), __float_as_uint(__uint_as_float(p.y) * f),
+                    __float_as_uint(__uint_as_float(p.z) * f), __float_as_uint(__uint_as_float(p.w) * f));
+}
+template <> __device__ __forceinline__ uint4 scaled16<__nv_bfloat16>(uint4 p, float f) {
+  auto two = [f](unsigned u) {
+    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u));
+    const __nv_bfloat162 r = __floats2bfloat162_rn(v.x * f, v.y * f);
+    return *reinterpret_cast<const unsigned*>(&r);
+  };
+  return make_uint4(two(p.x), two(p.y), two(p.z), two(p.w));
 }
 
 // copy the routed tokens' normalised activations into expert order: dst[pos] = src[sorted_row[pos]]
 // ---- MoD dispatch in one launch: segment offsets, a place for every routed (token, slot) pair inside its
 // expert's segment, and the copy of the token's normalised row to that place (the expert GEMMs load their rows
 // contiguously with TMA).  One CTA per pair.  `cursor` must be zero on entry (the combine kernel leaves it so).
+// scale: a factor per pair, or null.
 template <typename T>
 __global__ void mod_dispatch_kernel(const T* __restrict__ src, const int* __restrict__ slot_expert,
                                     const int* __restrict__ count, int* __restrict__ offset, int* __restrict__ cursor,
-                                    int* __restrict__ slot_pos, T* __restrict__ dst, int n_expert, int S, int D) {
+                                    int* __restrict__ slot_pos, T* __restrict__ dst, int n_expert, int S, int D,
+                                    const float* __restrict__ scale) {
   pdl_trigger();
   pdl_wait();
   __shared__ int s_pos;
@@ -701,6 +721,7 @@ __global__ void mod_dispatch_kernel(const T* __restrict__ src, const int* __rest
     const int j = threadIdx.x + u * blockDim.x;
     piece[u] = j < n16 ? a[j] : make_uint4(0u, 0u, 0u, 0u);
   }
+  const float f = scale ? scale[i] : 1.f;
   if (threadIdx.x < 32) {
     // exclusive prefix of the expert counts by the lanes of one warp: all counts are requested at once (a loop of
     // one thread waited for every count before it could ask for the next)
@@ -732,21 +753,30 @@ __global__ void mod_dispatch_kernel(const T* __restrict__ src, const int* __rest
 #pragma unroll
   for (int u = 0; u < 2; ++u) {
     const int j = threadIdx.x + u * blockDim.x;
-    if (j < n16) b[j] = piece[u];
+    if (j < n16) b[j] = scale ? scaled16<T>(piece[u], f) : piece[u];
   }
-  for (int j = threadIdx.x + 2 * blockDim.x; j < n16; j += blockDim.x) b[j] = a[j];
+  for (int j = threadIdx.x + 2 * blockDim.x; j < n16; j += blockDim.x) b[j] = scale ? scaled16<T>(a[j], f) : a[j];
 }
 
+// sorted_w: a factor per copied row, or null.  Rows that are not whole 16-byte pieces go element by element.
 template <typename T>
 __global__ void gather_sorted_kernel(const T* __restrict__ src, const int* __restrict__ sorted_row, T* __restrict__ dst,
-                                     int D) {
+                                     int D, const float* __restrict__ sorted_w) {
   pdl_trigger();
   pdl_wait();
   const long long s = sorted_row[blockIdx.x];
+  const float f = sorted_w ? sorted_w[blockIdx.x] : 1.f;
+  if (D * sizeof(T) % 16) {
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+      const T v = src[s * D + i];
+      dst[(long long)blockIdx.x * D + i] = sorted_w ? from_f<T>(to_f<T>(v) * f) : v;
+    }
+    return;
+  }
   const uint4* a = reinterpret_cast<const uint4*>(src + s * D);
   uint4* b = reinterpret_cast<uint4*>(dst + (long long)blockIdx.x * D);
   const int n16 = D * (int)sizeof(T) / 16;
-  for (int i = threadIdx.x; i < n16; i += blockDim.x) b[i] = a[i];
+  for (int i = threadIdx.x; i < n16; i += blockDim.x) b[i] = sorted_w ? scaled16<T>(a[i], f) : a[i];
 }
 
 // combine with split-K partials of the expert outputs: y = sum_s ypart[s]; x[row] += the weighted sum; then, if

@@ -30,6 +30,7 @@ __global__ void __launch_bounds__(256) attn_inputs_kernel(ConvIn<T, S, false> in
   const int w = is_v ? a.vd : a.d;
   const int c0 = is_v ? (a.H + a.KH) * a.d + head * a.vd : unit * a.d;
   const int np = is_v ? 0 : a.rd / 2, items = w - np;       // pairs first, then single channels
+  const float tf = is_q && a.temp ? a.temp[head] : 1.f;
   while (row < last) {                                      // stretches of one entry
     int slot, r0, n, start;
     a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
@@ -62,10 +63,10 @@ __global__ void __launch_bounds__(256) attn_inputs_kernel(ConvIn<T, S, false> in
         T* dst = dest(first + r);
         if (pair) {
           const float2 cs = a.rope[(long long)(start + first + r - r0) * np + i];
-          dst[cu] = from_f<T>(u[r] * cs.x - v[r] * cs.y);
-          dst[cv] = from_f<T>(v[r] * cs.x + u[r] * cs.y);
+          dst[cu] = from_f<T>((u[r] * cs.x - v[r] * cs.y) * tf);
+          dst[cv] = from_f<T>((v[r] * cs.x + u[r] * cs.y) * tf);
         } else {
-          dst[cu] = from_f<T>(u[r]);
+          dst[cu] = from_f<T>(u[r] * tf);
         }
       }
     }
@@ -90,6 +91,7 @@ __global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, fal
   else if (it < qk_heads * (nr + nu)) { const int i = it - qk_heads * nr; head = i / nu; c = a.rd + i % nu * 4; }
   else { const int i = it - qk_heads * (nr + nu); is_v = true; head = i / nv; c = i % nv * 4; }
   const int col = is_v ? (a.H + a.KH) * a.d + head * a.vd + c : head * a.d + c;
+  const float tf = !is_v && head < a.H && a.temp ? a.temp[head] : 1.f;
   int row = blockIdx.y * rep * RB;
   const int last = min(row + rep * RB, a.rows.M);
   float wu[4][4], wv[4][4];
@@ -117,11 +119,11 @@ __global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, fal
       }
       if (pair) {
         const float4* cs = reinterpret_cast<const float4*>(a.rope + (long long)pos * np + c);   // two pairs each
-        const float4 p0 = cs[0], p1 = cs[1], x = u[r], y = v[r];
+        const float4 p0 = cs[0], p1 = cs[1], x = scaled(u[r], tf), y = scaled(v[r], tf);
         store4(dst, make_float4(x.x * p0.x - y.x * p0.y, x.y * p0.z - y.y * p0.w, x.z * p1.x - y.z * p1.y, x.w * p1.z - y.w * p1.w));
         store4(dst + np, make_float4(y.x * p0.x + x.x * p0.y, y.y * p0.z + x.y * p0.w, y.z * p1.x + x.z * p1.y, y.w * p1.z + x.w * p1.w));
       } else {
-        store4(dst, u[r]);
+        store4(dst, scaled(u[r], tf));
       }
       const int w = is_v ? a.vd : a.d;
       if (c + 4 == w || (pair && np + c + 4 == w))         // the last quad of a head also pads it
@@ -136,7 +138,7 @@ __global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, fal
   }
 }
 
-// Heads with a norm (or interleaved pairs), without convolutions: bias, norm, rotation.  One warp per (row, unit) with the
+// Heads with a norm (or with interleaved pairs and biases), without convolutions: bias, norm, rotation.  One warp per (row, unit) with the
 // head staged in shared memory; units as above.  grid (units, ceil(M / 8)), block (32, 8), 8 max(d, vd) floats
 template <typename T, typename S>
 __global__ void __launch_bounds__(256) attn_heads_kernel(ConvIn<T, S, false> in, PagedAttnArgs a) {
@@ -162,7 +164,8 @@ __global__ void __launch_bounds__(256) attn_heads_kernel(ConvIn<T, S, false> in,
   T* dst = is_q ? reinterpret_cast<T*>(a.q) + ((long long)row * a.H + head) * a.P
                 : reinterpret_cast<T*>(is_v ? a.vplane : a.kplane) +
                       (((long long)a.table[(long long)slot * a.max_pages + pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.KH + head) * a.P;
-  auto value = [&](int c) { return nw ? s[c] * r * nw[c] : s[c]; };
+  const float tf = is_q && a.temp ? a.temp[head] : 1.f;
+  auto value = [&](int c) { return nw ? s[c] * r * nw[c] * tf : s[c] * tf; };
   for (int i = lane; i < w - np; i += 32) {
     if (i < np) {
       const int cu = a.interleaved ? 2 * i : i, cv = a.interleaved ? 2 * i + 1 : np + i;
@@ -194,6 +197,7 @@ __global__ void __launch_bounds__(256) attn_heads4_kernel(ConvIn<T, S, false> in
     x[r] = mine ? get4(in.src, min(row0 + r, a.rows.M - 1), in.col0 + c0) : make_float4(0.f, 0.f, 0.f, 0.f);
   if (mine && in.bias) b = load4(in.bias + c0);
   if (mine && nw) wt = load4(nw + c);
+  const float tf = live && is_q && a.temp ? a.temp[head] : 1.f;
   float ss[RB];
 #pragma unroll
   for (int r = 0; r < RB; ++r) {
@@ -223,7 +227,7 @@ __global__ void __launch_bounds__(256) attn_heads4_kernel(ConvIn<T, S, false> in
       const float4 cs = *reinterpret_cast<const float4*>(a.rope + (long long)pos * np + 2 * l);
       v = make_float4(v.x * cs.x - v.y * cs.y, v.y * cs.x + v.x * cs.y, v.z * cs.z - v.w * cs.w, v.w * cs.z + v.z * cs.w);
     }
-    store4(dst + c, v);                                    // pads too: their quads are zero
+    store4(dst + c, scaled(v, tf));                        // pads too: their quads are zero
   }
 }
 
@@ -266,10 +270,12 @@ __global__ void __launch_bounds__(256) paged_attn_kernel(PagedAttnArgs a, S proj
     m = m2;
   }
   T* o = reinterpret_cast<T*>(a.out) + ((long long)row * a.H + h) * a.vd;
+  const bool each = a.col_g >= 0 && !a.gate_head;
+  if (a.gate_head) l /= sigmoid_f(proj.get_rare(row, a.col_g + h));
 #pragma unroll
   for (int i = 0; i < NR; ++i) {
     const int j = lane + 32 * i;
-    if (j < a.vd) o[j] = from_f<T>(acc[i] / l * (a.col_g >= 0 ? sigmoid_f(proj.get_rare(row, a.col_g + h * a.vd + j)) : 1.f));
+    if (j < a.vd) o[j] = from_f<T>(acc[i] / l * (each ? sigmoid_f(proj.get_rare(row, a.col_g + h * a.vd + j)) : 1.f));
   }
 }
 
@@ -435,19 +441,22 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
   }
   // through shared memory, so that rows are gated and stored in whole lines
   float* sO = reinterpret_cast<float*>(raw) + 16 * warp * P;
+  const int fw = f0 + 16 * warp;
+  const bool each = a.col_g >= 0 && !a.gate_head;         // a gate per element, else per head or none
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
     float l = l_run[e];
     l += __shfl_xor_sync(0xffffffffu, l, 1);
     l += __shfl_xor_sync(0xffffffffu, l, 2);
-    const float inv = 1.f / l;
+    float inv = 1.f / l;
+    const int f = fw + (lane >> 2) + 8 * e;
+    if (a.gate_head && f < nf) inv *= sigmoid_f(proj.get_rare(r0 + f / hg, a.col_g + g * hg + f % hg));
 #pragma unroll
     for (int j = 0; j < P / 8; ++j)
       *reinterpret_cast<float2*>(sO + ((lane >> 2) + 8 * e) * P + 8 * j + (lane & 3) * 2) = make_float2(acc[j][2 * e] * inv, acc[j][2 * e + 1] * inv);
   }
   __syncwarp();
-  const int fw = f0 + 16 * warp;
-  if (a.vd % 4 == 0 && (a.col_g < 0 || (a.col_g % 4 == 0 && proj.ld % 4 == 0))) {
+  if (a.vd % 4 == 0 && (!each || (a.col_g % 4 == 0 && proj.ld % 4 == 0))) {
     // four columns per lane, eight rows' gates requested at a time
 #pragma unroll 1
     for (int c = lane * 4; c < a.vd; c += 128)
@@ -457,14 +466,14 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
 #pragma unroll
         for (int y = 0; y < 8; ++y) {
           const int f = min(fw + r + y, nf - 1);
-          if (a.col_g >= 0) gt[y] = get4(proj, r0 + f / hg, a.col_g + (g * hg + f % hg) * a.vd + c);
+          if (each) gt[y] = get4(proj, r0 + f / hg, a.col_g + (g * hg + f % hg) * a.vd + c);
         }
 #pragma unroll
         for (int y = 0; y < 8; ++y) {
           const int f = fw + r + y;
           if (f >= nf) break;
           float4 v = load4(sO + (r + y) * P + c);
-          if (a.col_g >= 0) { v.x *= sigmoid_f(gt[y].x); v.y *= sigmoid_f(gt[y].y); v.z *= sigmoid_f(gt[y].z); v.w *= sigmoid_f(gt[y].w); }
+          if (each) { v.x *= sigmoid_f(gt[y].x); v.y *= sigmoid_f(gt[y].y); v.z *= sigmoid_f(gt[y].z); v.w *= sigmoid_f(gt[y].w); }
           store4(reinterpret_cast<bf16*>(a.out) + ((long long)(r0 + f / hg) * a.H + g * hg + f % hg) * a.vd + c, v);
         }
       }
@@ -477,7 +486,7 @@ __global__ void __launch_bounds__(32 * W) paged_attn_mma_kernel(PagedAttnArgs a,
     const int h = g * hg + f % hg;
     bf16* o = reinterpret_cast<bf16*>(a.out) + (row * a.H + h) * a.vd;
     for (int c = lane; c < a.vd; c += 32)
-      o[c] = __float2bfloat16_rn(sO[r * P + c] * (a.col_g >= 0 ? sigmoid_f(proj.get_rare(row, a.col_g + h * a.vd + c)) : 1.f));
+      o[c] = __float2bfloat16_rn(sO[r * P + c] * (each ? sigmoid_f(proj.get_rare(row, a.col_g + h * a.vd + c)) : 1.f));
   }
 }
 
@@ -533,7 +542,7 @@ template <typename T, typename S>
 int32_t vn_attn_inputs(vn_ctx* ctx, const ConvIn<T, S, false>& conv, const PagedAttnArgs& a) {
   const int units = a.H + (a.own_kv ? 2 * a.KH : 0);
   const dim3 block(32, 8);
-  if (a.qn || conv.bias) {
+  if (a.qn || (conv.bias && a.interleaved)) {
     VN_REQUIRE(ctx, conv.taps == 1, "norms and biases of the heads stand without convolutions");
     const int w = std::max(a.d, a.vd);
     if (a.d % 4 == 0 && a.vd % 4 == 0 && a.rd % 4 == 0 && conv.src.ld % 4 == 0 && w <= 128 && (a.interleaved || !a.rd)) {

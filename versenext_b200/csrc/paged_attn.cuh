@@ -1,8 +1,8 @@
 // Grouped-query attention over paged keys and values: query head h reads key/value head h / (H / KH).  Optional sliding
 // window or chunks, rotary positions on the first rd dimensions of a head (half-split or interleaved pairs; frequencies and
 // amplitude come as a table), biases, an RMS norm of every query and key head, short causal convolutions on q, k and v, a
-// soft cap of the scores, a sigmoid gate on every output element; scores and soft-max in fp32.  A layer may read another
-// layer's planes instead of owning some.
+// factor of every query head's scores, a soft cap of the scores, a sigmoid gate on every output element or every head; scores
+// and soft-max in fp32.  A layer may read another layer's planes instead of owning some.
 //
 // Cache: plane[page * KV_PAGE + pos % KV_PAGE][KH][P], P = padded width of a key or value; table[slot * max_pages + pos / KV_PAGE].
 #pragma once
@@ -18,6 +18,7 @@ struct PagedAttnArgs {
   const float* qn = nullptr;       // [d] weights of the query heads' and key heads' norms, or null
   const float* kn = nullptr;
   float eps = 0.f;
+  const float* temp = nullptr;     // [H] factors of the scores (the queries are stored times them), or null
   int rd = 0;                      // rotated dimensions (even)
   int interleaved = 0;             // dimension 2 i is rotated with 2 i + 1, else i with i + rd / 2
   const float2* rope = nullptr;    // [positions][rd / 2] cos, sin
@@ -26,6 +27,7 @@ struct PagedAttnArgs {
   const int* table = nullptr;
   int max_pages = 0;
   int col_g = -1;                  // first gate column of the projection, or -1
+  int gate_head = 0;               // gates: one per head, else one per output element
   void* q = nullptr;               // [M, H, P] storage dtype
   void* out = nullptr;             // [M, H vd] storage dtype
   // one-token kernel: key ranges of a sequence, merged by the CTA that finishes last

@@ -1,6 +1,7 @@
-// Mixture of experts: which experts a row goes to.  Scores are the soft-max over all router outputs; the choice may see a
-// correction per expert and be limited to the best groups of neighbouring experts; the weights are the plain scores.  The last
-// outputs may be identity experts, whose result is their input.  Rows are then laid out expert by expert by the kernels that
+// Mixture of experts: which experts a row goes to.  Scores are the soft-max over all router outputs, or the sigmoid of each;
+// the choice may see a correction per expert and be limited to the best groups of neighbouring experts; the weights are the
+// plain scores.  The last outputs may be identity experts, whose result is their input.  A further column of the router's
+// product may hold the raw gate of an expert that serves every row.  Rows are then laid out expert by expert by the kernels that
 // serve the other mixtures (mod_dispatch_kernel, or mod_offsets / mod_scatter / gather_sorted).
 #pragma once
 #include "rows.cuh"
@@ -11,12 +12,14 @@ inline int route_rows(int M) { return M >= 2048 ? 2 : 1; }      // rows per warp
 inline size_t route_smem(int E, int groups) { return ((size_t)ROUTE_WARPS * (2 * E + groups) + E) * 4; }
 
 struct RouteIn {
-  Src z;                               // [M, E] router outputs
+  Src z;                               // [M, E or more] router outputs
+  int sigmoid = 0;                     // scores: sigmoid of each output, else soft-max over all
   const float* correction = nullptr;   // [E] or null
   int M = 0, E = 0, top = 1, groups = 1, keep = 1, rows = 1;      // rows: per warp
   int* slot_expert = nullptr;          // [M, top]
   float* slot_w = nullptr;             // [M, top]
   int* count = nullptr;                // [E], zero before the launch
+  float* shared_gate = nullptr;        // [M] sigmoid of column E, or null
 };
 
 // index of the largest value over a warp's lanes (the lowest one among equals), by way of integers in the same order
@@ -50,10 +53,12 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) route_kernel(RouteIn r) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
     float sum = 0.f;
-    for (int e = lane; e < E; e += 32) { const float x = expf(score[e] - top); score[e] = x; sum += x; }
+    if (!r.sigmoid)
+      for (int e = lane; e < E; e += 32) { const float x = expf(score[e] - top); score[e] = x; sum += x; }
     sum = warp_sum(sum);
+    if (r.shared_gate && lane == 0) r.shared_gate[row] = sigmoid_f(r.z.get(row, E));
     for (int e = lane; e < E; e += 32) {
-      const float s = score[e] / sum;
+      const float s = r.sigmoid ? sigmoid_f(score[e]) : score[e] / sum;
       score[e] = s;
       choice[e] = r.correction ? s + r.correction[e] : s;
     }

@@ -96,6 +96,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<__nv_bfloat162*>(&u.y) = __floats2bfloat162_rn(v.z, v.w);
   *reinterpret_cast<uint2*>(p) = u;
 }
+__device__ __forceinline__ float4 scaled(float4 v, float f) { return make_float4(v.x * f, v.y * f, v.z * f, v.w * f); }
 __device__ __forceinline__ float4 get4(const Src& s, long long row, int col) {
   const float* q = s.p + row * s.ld + col;
   float4 a = load4(q);
@@ -242,7 +243,10 @@ struct ConvIn {
     const auto* p = src.p + (long long)row * src.ld + col0 + c;
 #pragma unroll
     for (int i = 0; i < RB; ++i) x[3 + i] = load4(p + (long long)(min(row + i, row_end - 1) - row) * src.ld);
-    if (row - r0 >= 3) {
+    if (taps == 1) {
+#pragma unroll
+      for (int i = 0; i < 3; ++i) x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    } else if (row - r0 >= 3) {
 #pragma unroll
       for (int i = 0; i < 3; ++i) x[i] = load4(p + (long long)(i - 3) * src.ld);
     } else {

@@ -1,5 +1,6 @@
 // Kernels shared by the layer kinds of composed models (hybrid.cuh): embedding with position vectors, the entry of a
-// looped block, row sums with a norm, picked rows, and the tail of the convolution inputs.
+// looped block, row sums with a norm, the end of a sublayer, activations of feed-forwards, picked rows, and the tail of the
+// convolution inputs.
 #pragma once
 #include "model_kernels.cuh"
 
@@ -71,6 +72,27 @@ __global__ void __launch_bounds__(256) rowsum_norm_kernel(Src src, const float* 
   for (int d = threadIdx.x; d < D; d += 256) y[row * D + d] = from_f<T>(x[row * D + d] / r * norm_w[d]);
 }
 
+// Entry of a looped block that adds instead of projecting: x += x0 (from the second pass on) + step vector of the pass.
+struct PassEntry { const float* x0 = nullptr; const float* step = nullptr; };
+
+// the same by itself, with the norm of the pass's first layer behind it.  Any D, grid M
+template <typename T>
+__global__ void __launch_bounds__(256) enter_pass_kernel(PassEntry pass, float* __restrict__ x, const float* __restrict__ norm_w,
+                                                         T* __restrict__ y, int D, float eps) {
+  __shared__ float sm[8];
+  const long long row = blockIdx.x;
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < D; d += 256) {
+    float v = x[row * D + d];
+    if (pass.x0) v += pass.x0[row * D + d];
+    v += pass.step[d];
+    x[row * D + d] = v;
+    ss += v * v;
+  }
+  const float r = sqrtf(block_sum256(ss, sm) / (float)D + eps);
+  for (int d = threadIdx.x; d < D; d += 256) y[row * D + d] = from_f<T>(x[row * D + d] / r * norm_w[d]);
+}
+
 // ---- the end of a sublayer in one pass over a row: what it adds, the residual, and what the next product reads -------------
 // Y gives the addend: quad(row, d) of four columns, one(row, d) of one; begin(row) is called by all 256 threads first.
 
@@ -88,13 +110,16 @@ struct AddRows {
   __device__ __forceinline__ float one(int row, int d) const { return y.get(row, d) + (bias ? bias[d] : 0.f); }
 };
 
-// the weighted results of a row's experts: rows slot_pos[] of y; experts from n_real on are the input h itself
+// the results of a row's experts: rows slot_pos[] of y, weighted unless the weights are null; experts from n_real on are the
+// input h itself; and the gated result of the expert that serves every row
 template <typename T, typename S>
 struct AddExperts {
   S y;
   const T* h = nullptr;
   const int *slot_pos = nullptr, *slot_expert = nullptr;
   const float* slot_w = nullptr;
+  S shared;                                      // [M, D], times shared_gate [M] (null: none)
+  const float* shared_gate = nullptr;
   int top = 1, n_real = 0, D = 0;
   int *count = nullptr, *cursor = nullptr;       // left at zero for the next mixture
   int n_count = 0;
@@ -109,7 +134,7 @@ struct AddExperts {
     const int lane = threadIdx.x & 31;           // every warp finds out for itself; they write the same values
     const bool has = lane < top;
     const int e = has ? slot_expert[(long long)row * top + lane] : n_real;
-    const float v = has ? slot_w[(long long)row * top + lane] : 0.f;
+    const float v = !has ? 0.f : slot_w ? slot_w[(long long)row * top + lane] : 1.f;
     const unsigned real = __ballot_sync(0xffffffffu, has && e < n_real);
     if (has && e < n_real) {
       const int at = __popc(real & ((1u << lane) - 1));
@@ -124,7 +149,8 @@ struct AddExperts {
   }
   __device__ __forceinline__ float4 quad(int row, int d) const {
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (w_self != 0.f) { const float4 t = load4(h + (long long)row * D + d); a = make_float4(t.x * w_self, t.y * w_self, t.z * w_self, t.w * w_self); }
+    if (shared_gate) a = scaled(get4(shared, row, d), shared_gate[row]);
+    if (w_self != 0.f) { const float4 t = load4(h + (long long)row * D + d); a = make_float4(fmaf(t.x, w_self, a.x), fmaf(t.y, w_self, a.y), fmaf(t.z, w_self, a.z), fmaf(t.w, w_self, a.w)); }
 #pragma unroll 4
     for (int j = 0; j < n; ++j) {
       const float4 t = get4(y, pos[j], d);
@@ -135,16 +161,17 @@ struct AddExperts {
   }
   __device__ __forceinline__ float one(int row, int d) const {
     float a = w_self != 0.f ? w_self * to_f<T>(h[(long long)row * D + d]) : 0.f;
+    if (shared_gate) a = fmaf(shared.get(row, d), shared_gate[row], a);
     for (int j = 0; j < n; ++j) a = fmaf(y.get(pos[j], d), w[j], a);
     return a;
   }
 };
 
-// x += y, or y over its root mean square times own_norm; then h = RMSNorm(x) * next_norm, or x itself (cast), or nothing.
+// x += y, or y over its root mean square times own_norm, and what a pass of a looped block begins with; then h = RMSNorm(x) * next_norm, or x itself (cast), or nothing.
 // NV > 0: four columns per thread, NV times, held in registers (D % 4 == 0, D <= 1024 NV); 0: any D.  grid M
 template <typename T, typename Y, int NV>
 __global__ void __launch_bounds__(256) residual_kernel(Y y, float* __restrict__ x, const float* __restrict__ own_norm,
-                                                       const float* __restrict__ next_norm, int cast, T* __restrict__ h, int D, float eps) {
+                                                       PassEntry pass, const float* __restrict__ next_norm, int cast, T* __restrict__ h, int D, float eps) {
   __shared__ float sm[2][8];
   pdl_trigger();
   pdl_wait();
@@ -179,6 +206,11 @@ __global__ void __launch_bounds__(256) residual_kernel(Y y, float* __restrict__ 
       const int d = (threadIdx.x + 256 * i) * 4;
       if (d >= D) break;
       xv[i] = make_float4(xv[i].x + v[i].x, xv[i].y + v[i].y, xv[i].z + v[i].z, xv[i].w + v[i].w);
+      if (pass.step) {
+        if (pass.x0) { const float4 t = load4(pass.x0 + (long long)row * D + d); xv[i] = make_float4(xv[i].x + t.x, xv[i].y + t.y, xv[i].z + t.z, xv[i].w + t.w); }
+        const float4 t = load4(pass.step + d);
+        xv[i] = make_float4(xv[i].x + t.x, xv[i].y + t.y, xv[i].z + t.z, xv[i].w + t.w);
+      }
       store4(xr + d, xv[i]);
       if (cast) store4(hr + d, xv[i]);
       ss += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
@@ -203,6 +235,8 @@ __global__ void __launch_bounds__(256) residual_kernel(Y y, float* __restrict__ 
       float v = y.one(row, d);
       if (own_norm) v *= f * own_norm[d];
       v += xr[d];
+      if (pass.x0) v += pass.x0[(long long)row * D + d];
+      if (pass.step) v += pass.step[d];
       xr[d] = v;
       if (cast) hr[d] = from_f<T>(v);
       ss += v * v;
@@ -227,6 +261,54 @@ __global__ void __launch_bounds__(256) side_act_kernel(Src gate, const long long
   long long tok = tokens[row];
   tok = tok < 0 ? 0 : tok >= V ? V - 1 : tok;            // the embedding has raised the flag
   act[i] = from_f<T>(j < n ? gelu_tanh(gate.get(row, j)) * to_f<T>(table[tok * pitch + col0 + j]) : 0.f);
+}
+
+// PolyNorm: act = a N(z) + b N(z^2) + c N(z^3) + e over a row of n columns, N: over the root mean square; coef = {a, b, c, e}.
+// Columns n .. ld - 1 of z are zero (and meet zero weights behind).  NV > 0: four columns per thread, NV times, held in
+// registers (ld % 4 == 0, ld <= 1024 NV); 0: any ld, z is read twice.  grid M
+template <typename T, typename S, int NV>
+__global__ void __launch_bounds__(256) poly_norm_kernel(S z, const float* __restrict__ coef, T* __restrict__ act, int n, int ld, float eps) {
+  __shared__ float sm[3][8];
+  pdl_trigger();
+  pdl_wait();
+  const int row = blockIdx.x;
+  T* out = act + (long long)row * ld;
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto count = [&](float v) { const float q = v * v; s2 += q; s4 = fmaf(q, q, s4); s6 = fmaf(q * q, q, s6); };
+  float4 v[NV > 0 ? NV : 1];
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + 256 * i) * 4;
+      v[i] = c < ld ? get4(z, row, c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { count(v[i].x); count(v[i].y); count(v[i].z); count(v[i].w); }
+  } else {
+    for (int c = threadIdx.x; c < n; c += 256) count(z.get(row, c));
+  }
+  s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
+  if ((threadIdx.x & 31) == 0) { const int w = threadIdx.x >> 5; sm[0][w] = s2; sm[1][w] = s4; sm[2][w] = s6; }
+  __syncthreads();
+  float f[3];
+#pragma unroll
+  for (int k = 0; k < 3; ++k) {
+    float t = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) t += sm[k][w];
+    f[k] = coef[k] / sqrtf(t / (float)n + eps);
+  }
+  const float e = coef[3];
+  auto value = [&](float x) { return fmaf(x, fmaf(x, fmaf(x, f[2], f[1]), f[0]), e); };
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + 256 * i) * 4;
+      if (c < ld) store4(out + c, make_float4(value(v[i].x), value(v[i].y), value(v[i].z), value(v[i].w)));
+    }
+  } else {
+    for (int c = threadIdx.x; c < ld; c += 256) out[c] = from_f<T>(value(c < n ? z.get(row, c) : 0.f));
+  }
 }
 
 // y = RMSNorm(x[row_of(i)]) * w: rows picked by a list, by (i * mul + add), or the entries' last rows
