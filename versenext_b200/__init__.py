@@ -4,7 +4,8 @@ Public surface (names follow the reference):
   SpeculativeDecoder                      verse_nex/speculative.py:55
   VerseNexLM (= CometSparkNexLM), KVCache verse_nex/cometspark.py:294, kv_cache_parallel.py:42
   build_verse_delta_pattern               verse_nex/delta_attention.py:1218 (layer kinds vda / dsa / kda / gmla)
-  ComposedLM, FuzudraLM, MusutarLM        models composed of attention, latent attention, scan, delta rule, lightning layers
+  ComposedLM, BozasunLM, FuzudraLM, GivozenLM, MusutarLM
+                                          models composed of attention, latent attention, scan, delta rule, lightning layers
   load_model                              a model by the architecture its config.json names
   BatchEngine, StepRunner                 ragged batches: portions of prompts beside single tokens, slots and pages reused
   SpecEngine                              batched draft -> verify -> accept -> commit loop
@@ -29,6 +30,7 @@ from .engine import SpecEngine
 from .composed import ComposedLM
 from .bozasun import BozasunLM
 from .fuzudra import FuzudraLM
+from .givozen import GivozenLM
 from .musutar import MusutarLM
 from .serving import BatchEngine, StepRunner
 from .registry import load_model
@@ -40,6 +42,6 @@ from . import sampling
 from . import quant
 
 __all__ = ["Context", "DeviceArray", "as_device", "DeviceBackend", "B200Backend", "get_backend",
-           "clear_backend_cache", "SpeculativeDecoder", "Tensor", "no_grad", "sampling", "quant", "VerseNexLM", "CometSparkNexLM", "KVCache", "ComposedLM", "BozasunLM", "FuzudraLM", "MusutarLM",
+           "clear_backend_cache", "SpeculativeDecoder", "Tensor", "no_grad", "sampling", "quant", "VerseNexLM", "CometSparkNexLM", "KVCache", "ComposedLM", "BozasunLM", "FuzudraLM", "GivozenLM", "MusutarLM",
            "load_model", "BatchEngine", "StepRunner", "build_verse_delta_pattern", "SpecEngine", "TreeSpecEngine",
            "ShardedSpecEngine", "Comm", "rank_seed", "VNFileReader", "load_vn"]

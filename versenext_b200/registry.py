@@ -7,6 +7,7 @@ import os
 
 from .bozasun import BozasunLM
 from .fuzudra import FuzudraLM
+from .givozen import GivozenLM
 from .model import DeviceLM, VerseNexLM
 from .musutar import MusutarLM
 
@@ -42,6 +43,7 @@ def load_model(path: str, dtype: str = "bf16", device: str = "cuda", **kw) -> De
 
 register(BozasunLM.ARCHITECTURE, BozasunLM)
 register(FuzudraLM.ARCHITECTURE, FuzudraLM)
+register(GivozenLM.ARCHITECTURE, GivozenLM)
 register(MusutarLM.ARCHITECTURE, MusutarLM)
 register("VerseNexLM", VerseNexLM)
 register("CometSparkNexLM", VerseNexLM)
