@@ -1122,7 +1122,7 @@ def _prefill_ms(m, ctx, B, T, V, steps, profile=False):
 def run_composed(args):
     """Prefill and decode of a composed design (random weights, 4 layers) beside VerseNexLM models of the same width, depth,
     feed-forward weights, window and vocabulary: all TriSparse, and all GMLA (a latent behind K and V); with Musutar also
-    Fuzudra, with Bozasun both: the other composed designs."""
+    Fuzudra, with Bozasun both, with Givozen Bozasun and Musutar: the other composed designs."""
     import versenext_b200 as vn
     from versenext_b200 import synthetic as S
     design = args.workload
@@ -1143,7 +1143,7 @@ def run_composed(args):
             m = vn.VerseNexLM(dtype="bf16", device=f"cuda:{local}", **kw)
             S.load_random(m, kw, seed=3)
             return m
-        for name in {"bozasun": ["bozasun", "fuzudra", "musutar"], "musutar": ["musutar", "fuzudra"], "fuzudra": ["fuzudra"]}[design] + ["trisparse", "gmla"]:
+        for name in {"givozen": ["givozen", "bozasun", "musutar"], "bozasun": ["bozasun", "fuzudra", "musutar"], "musutar": ["musutar", "fuzudra"], "fuzudra": ["fuzudra"]}[design] + ["trisparse", "gmla"]:
             if args.only and name not in args.only.split(","):
                 continue
             m = verse(name) if name in ("trisparse", "gmla") else composed(name)
@@ -1168,7 +1168,7 @@ def run_composed(args):
         line = {"metric": "composed-model decode throughput", "value": head["decode_B32_tok_s"], "unit": "tokens/s",
                 "n_gpus": world, "steps": steps, "warmup": 3, "ms_per_step": head["decode_B32_ms"], "higher_is_better": True,
                 "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-                "config": {"workload": f"{design}: 4 layers, widths {COMPOSED_WIDTHS}, V={V}, context {COMPOSED_CTX}, L2 flushed "
+                "config": {"workload": f"{design}: 4 layer runs, widths {COMPOSED_WIDTHS}, V={V}, context {COMPOSED_CTX}, L2 flushed "
                                        "between steps, decode replayed from a CUDA graph"},
                 "rows": rows, "clocks": clk, "gpu_launches": ctx.launch_count() - l0}
         if profs:
@@ -1392,7 +1392,7 @@ def main():
     ap.add_argument("--steps", type=int, default=32)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--workload", default="spec", choices=["spec", "accept", "sharded", "tree", "small", "layer", "delta", "fuzudra", "musutar", "bozasun"])
+    ap.add_argument("--workload", default="spec", choices=["spec", "accept", "sharded", "tree", "small", "layer", "delta", "fuzudra", "musutar", "bozasun", "givozen"])
     ap.add_argument("--weak", action="store_true",
                     help="spec workload: 32 requests on every rank (default: the configuration's 32 split over the ranks)")
     ap.add_argument("--no-weak", action="store_true", help="N > 1: skip the extra 32-per-GPU measurement")
@@ -1401,8 +1401,8 @@ def main():
                     help="spec workload: quantise the target's linear weights (not the default benchmark line)")
     ap.add_argument("--pattern", default="mod,trisparse", help="layer workload: comma-separated layer kinds")
     ap.add_argument("--context", type=int, default=1100, help="layer workload: cached positions (a multiple of 220)")
-    ap.add_argument("--kernels", action="store_true", help="fuzudra / musutar / bozasun workloads: per-kernel times of every case")
-    ap.add_argument("--only", default=None, help="fuzudra / musutar / bozasun workloads: these models only (comma-separated)")
+    ap.add_argument("--kernels", action="store_true", help="fuzudra / musutar / bozasun / givozen workloads: per-kernel times of every case")
+    ap.add_argument("--only", default=None, help="fuzudra / musutar / bozasun / givozen workloads: these models only (comma-separated)")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU-baseline leg")
     ap.add_argument("--no-sampler", action="store_true", help="spec workload: skip the sampler GB/s measurement")
     args = ap.parse_args()
@@ -1410,7 +1410,7 @@ def main():
         {"accept": run_reference, "small": run_reference_small}.get(args.workload, run_reference_spec)(args)
     else:
         {"spec": run_spec, "accept": run_accept, "sharded": run_sharded, "tree": run_tree,
-         "small": run_small, "layer": run_layer, "delta": run_delta, "fuzudra": run_composed, "musutar": run_composed, "bozasun": run_composed}[args.workload](args)
+         "small": run_small, "layer": run_layer, "delta": run_delta, "fuzudra": run_composed, "musutar": run_composed, "bozasun": run_composed, "givozen": run_composed}[args.workload](args)
 
 
 if __name__ == "__main__":

@@ -261,6 +261,54 @@ def bozasun_shapes(cfg: dict) -> dict:
     return s
 
 
+def givozen_config(width: int, vocab: int = 32000, n_run: int = 4) -> dict:
+    """config.json contents: `n_run` layer runs out of n_run - 1 layers, PolyNorm feed-forwards and mixtures, the mixture in the
+    middle run twice; heads of 128 (64 below width 2048), four query heads per key head; feed-forwards with as many weights as
+    VerseNexLM's gated ones, experts and the one that serves every token a quarter as wide, of which a token uses three."""
+    hd = 128 if width >= 2048 else 64
+    heads, ff = width // hd, int((4 * width * 2 / 3 + 63) // 64) * 64
+    part = {"ff": (ff // 4 + 63) // 64 * 64, "limit": 7.0}
+    dense, moe = {"kind": "dense", "ff": 4 * width}, {"kind": "moe", "expert": part, "shared": part, "router": {"experts": 24, "top": 3}}
+    rot = {"base": 500000.0, "dims": hd, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}
+    mixer = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": hd, "vdim": hd, "scale": hd ** -0.5, "rot": rot}
+    return {"architecture": "Givozen", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "loop": {"start": 1, "stop": 2, "times": 2},
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": moe if i % 2 else dense} for i in range(n_run - 1)]}
+
+
+def givozen_shapes(cfg: dict) -> dict:
+    """Tensor name -> shape."""
+    D, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, D), "final.norm": (D,)}
+    if cfg.get("loop"):
+        s["loop.step"] = (cfg["loop"]["times"], D)
+    for i, L in enumerate(cfg["layers"]):
+        m, mlp = L["mixer"], L.get("mlp")
+        H, G, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        t = {"norm1": (D,), "norm1b": (D,), "mix.temp": (H,), "mix.g": (H, D), "mix.o": (D, H * v)}
+        for part, w in (("q", H * d), ("k", G * d), ("v", G * v)):
+            t.update({f"mix.{part}": (w, D), f"mix.{part}.b": (w,)})
+        if mlp:
+            t.update({"norm2": (D,), "norm2b": (D,)})
+        if mlp and mlp["kind"] == "dense":
+            t.update({"mlp.up": (mlp["ff"], D), "mlp.down": (D, mlp["ff"]), "mlp.act": (4,)})
+        elif mlp:
+            parts = [(f"mlp.e{e}.", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])]
+            t["mlp.router"] = (mlp["router"]["experts"], D)
+            if mlp.get("shared"):
+                parts.append(("mlp.shared.", mlp["shared"]["ff"]))
+                t["mlp.shared.sg"] = (1, D)
+            for p, f in parts:
+                t.update({p + "gate": (f, D), p + "up": (f, D), p + "down": (D, f)})
+        s.update({f"l{i}.{k}": x for k, x in t.items()})
+    return s
+
+
+def random_givozen(cfg: dict, seed: int = 0, **kw):
+    """A GivozenLM with seeded random weights, tensor by tensor."""
+    from .givozen import GivozenLM
+    return _random_design(GivozenLM, cfg, givozen_shapes(cfg), seed, **kw)
+
+
 def random_bozasun(cfg: dict, seed: int = 0, **kw):
     """A BozasunLM with seeded random weights, tensor by tensor."""
     from .bozasun import BozasunLM
@@ -282,7 +330,7 @@ def random_musutar(cfg: dict, seed: int = 0, **kw):
 # (name's end, standard deviation, mean) of the tensors that are not plain linear weights or norms around zero
 _SPECIAL = (("mix.A_log", 1.0, -1.0), ("mix.dt_bias", 1.0, -2.0), ("mix.dt.b", 1.0, -3.0), ("mix.D", 0.1, 1.0), ("mix.sink", 1.0, 0.0),
             (".conv", 0.4, 0.0), ("canon1", 0.3, 0.0), ("mix.norm", 0.1, 1.0), ("dkv.norm", 0.1, 1.0), ("hc1.in", 0.1, 0.25), ("hc2.in", 0.1, 0.25),
-            ("hc1.out", 0.1, 1.0), ("hc2.out", 0.1, 1.0), ("mlp.correction", 0.005, 0.0))
+            ("hc1.out", 0.1, 1.0), ("hc2.out", 0.1, 1.0), ("mlp.correction", 0.005, 0.0), ("mix.temp", 0.1, 1.0), ("mlp.act", 0.1, 0.5))
 
 
 def _random_design(cls, cfg: dict, shapes: dict, seed: int, **kw):
