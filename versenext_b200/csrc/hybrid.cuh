@@ -75,7 +75,11 @@ struct HLayer {
   void* w_router = nullptr; float* correction = nullptr;                        // [n_router, D], [n_out]
   void *w_sgate = nullptr, *w_sproj = nullptr; float* s_norm = nullptr;         // the token's own input
   int n_out() const { return n_exp + n_id; }
-  int n_router() const { return sff ? (n_out() + 4) & ~3 : n_out(); }          // the shared expert's gate is row n_out
+  int n_router() const { return sff ? (n_out() + 8) & ~7 : n_out(); }          // the shared expert's gate is row n_out
+  // the shared expert is stored, and run, as one more of the others where it has their shape
+  int joined() const { return sff == ff && sff && s_limit == limit && !n_id && top < MAX_CHOSEN; }
+  int n_mats() const { return n_exp + joined(); }
+  int slots() const { return top + joined(); }
   int single_up() const { return ff_plain || poly; }                            // one matrix in front of the activation
   int attn_gates() const { return gated == GATE_HEAD ? H : gated ? H * vd : 0; }
   int n_gate() const { return gate == GATE_HEAD ? H : gate == GATE_ELEMENT ? H * vd : 0; }      // latent
@@ -184,23 +188,23 @@ inline void layout(const Model& hm, const HLayer& L, size_t M, size_t e, Arena& 
   A.off = 0;
   A.take(&b.proj, M * std::max(std::max(L.n_in, hm.D), L.single_up() ? L.ffp + hm.D : 0) * 4);
   A.take(&b.mix, M * (size_t)(L.kind == MAMBA1 ? L.inner : L.H * L.vd) * e);
-  if (L.ff) A.take(&b.act, M * std::max(1, L.top) * L.ffp * e);
+  if (L.ff) A.take(&b.act, M * std::max(1, L.slots()) * L.ffp * e);
   if (L.n_exp) {
-    const size_t slots = M * L.top;
+    const size_t slots = M * L.slots();
     A.take(&b.logits, M * L.n_router() * 4);
     A.take(&b.slot_w, slots * 4);
     A.take(&b.slot_expert, slots * 4);
     A.take(&b.slot_pos, slots * 4);
     A.take(&b.sorted_row, slots * 4);
     A.take(&b.sorted_w, slots * 4);
-    if (L.sff) {
-      A.take(&b.sgate, M * 4);
+    if (L.sff) A.take(&b.sgate, M * 4);
+    if (L.sff && !L.joined()) {
       A.take(&b.sact, M * L.sffp * e);
       A.take(&b.sy, M * hm.D * 4);
     }
     A.take(&b.hs, slots * hm.D * e);
     A.take(&b.ey, slots * hm.D * e);
-    b.sub_cap = (int)(L.n_exp + slots / 256 + 1);
+    b.sub_cap = (int)(L.n_mats() + slots / 256 + 1);
     A.take(&b.sub_seg, (size_t)3 * b.sub_cap * 4);
   }
   if (hm.side) A.take(&b.side_act, M * hm.sidep * e);
@@ -363,7 +367,7 @@ int32_t parse(vn_ctx* ctx, const JsonValue& j, Model* hm, Config* c) {
         VN_REQUIRE(ctx, L.ff > 0 && !L.single_up() && L.n_exp > 0 && L.n_id >= 0 && n <= 1024 && L.exp_groups >= 1 && n % L.exp_groups == 0 &&
                    L.keep >= 1 && L.keep <= L.exp_groups && L.top >= 1 && L.top <= MAX_CHOSEN && L.top <= L.keep * (n / L.exp_groups),
                    "layer %zu: mixture of %d experts and %d identities in %d groups, %d kept, %d chosen", i, L.n_exp, L.n_id, L.exp_groups, L.keep, L.top);
-        hm->max_out = std::max(hm->max_out, n);
+        hm->max_out = std::max(hm->max_out, n + L.joined());
       }
     if (L.ff_plain || L.kind == LIGHTNING) hm->arranged = true;
     L.ffp = up8(L.ff);
@@ -589,7 +593,7 @@ int32_t alloc(vn_model* m) {
     }
     if (L.ff) {
       const bool stacked = L.ff_plain && hm.res_gate;          // up | gate of the result: both read the same rows
-      const size_t n = std::max(1, L.n_exp);
+      const size_t n = std::max(1, L.n_mats());
       TRY(F(&L.norm2, D));
       TRY(W(&L.w_gu, n * (L.single_up() ? L.ffp + (stacked ? D : 0) : 2 * L.ffp) * D));
       TRY(W(&L.w_down, n * D * L.ffp));
@@ -598,8 +602,13 @@ int32_t alloc(vn_model* m) {
         TRY(W(&L.w_router, (size_t)L.n_router() * D));
         need({"mlp.router"});
         if (L.sff) {
-          TRY(W(&L.w_sgu, (size_t)2 * L.sffp * D));
-          TRY(W(&L.w_sdown, D * L.sffp));
+          if (L.joined()) {
+            L.w_sgu = (char*)L.w_gu + (size_t)L.n_exp * 2 * L.ffp * D * e;
+            L.w_sdown = (char*)L.w_down + (size_t)L.n_exp * D * L.ffp * e;
+          } else {
+            TRY(W(&L.w_sgu, (size_t)2 * L.sffp * D));
+            TRY(W(&L.w_sdown, D * L.sffp));
+          }
           need({"mlp.shared.gate", "mlp.shared.up", "mlp.shared.down", "mlp.shared.sg"});
         }
         if (L.corrected) { TRY(F(&L.correction, L.n_out())); need({"mlp.correction"}); }
@@ -654,7 +663,8 @@ void destroy(vn_model* m) {
     if (!(L.ff_plain && hm.res_gate)) F(L.w_rg[1]);            // else part of w_gu
     F(L.w_gu); F(L.w_down); F(L.w_rg[0]); F(L.in_conv);
     F(L.f_d); F(L.o_b); F(L.w_router); F(L.correction); F(L.w_sgate); F(L.w_sproj); F(L.s_norm);
-    F(L.temp); F(L.coef); F(L.w_sgu); F(L.w_sdown);
+    F(L.temp); F(L.coef);
+    if (!L.joined()) { F(L.w_sgu); F(L.w_sdown); }             // else part of w_gu, w_down
     for (int q = 0; q < 2; ++q) { F(L.post[q]); F(L.hc_in[q]); F(L.hc_out[q]); F(L.hc_mix[q]); F(L.rg_b[q]); }
   }
   for (Rope& r : hm.ropes) F(r.table);
@@ -1158,7 +1168,7 @@ int32_t attention(vn_model* m, const void* in_rows, vn_kv* kv, Cache& hc, const 
   const int M = rows.M, D = hm.D, from = hm.runs[run].kv_run;
   ConvIn<T, S, false> cv;
   TRY(project(m, gemm_args(in_rows, D, L.w_in, L.n_in, D, M, "gemm_attn_in"), b.proj, &cv.src));
-  cv.ring = (T*)hc.ring[run]; cv.RC = L.taps - 1 + hc.pending; cv.C = L.conv_ch(); cv.taps = L.taps; cv.w = L.conv;
+  cv.ring = (T*)hc.ring[run]; cv.RC = L.taps - 1 + hc.pending; cv.C = L.conv_ch(); cv.taps = L.taps; cv.w = L.conv; cv.named = L.conv_named;
   PagedAttnArgs a;
   a.H = L.H; a.KH = L.KH; a.d = L.d; a.vd = L.vd; a.P = L.P; a.window = L.window; a.chunk = L.chunk; a.scale = L.scale; a.softcap = L.softcap; a.rd = L.rd;
   a.interleaved = L.interleaved; a.qn = L.f_a; a.kn = L.f_b; a.eps = hm.eps;
@@ -1299,20 +1309,21 @@ template <typename T>
 int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Next& next) {
   vn_ctx* ctx = m->ctx;
   Model& hm = *m->hyb;
-  const int D = hm.D, n = L.n_out(), S = L.top, F = L.ffp;
+  const int D = hm.D, n = L.n_out() + L.joined(), S = L.slots(), F = L.ffp, mats = L.n_mats();
+  const bool apart = L.sff && !L.joined();
   const bool bf = m->cfg.bf16;
   RouteIn r;
   TRY(project(m, gemm_args(m->h, D, L.w_router, L.n_router(), D, M, "gemm_router"), b.logits, &r.z));
-  r.sigmoid = L.sigmoid; r.shared_gate = L.sff ? b.sgate : nullptr;
-  r.correction = L.correction; r.M = M; r.E = n; r.top = S; r.groups = L.exp_groups; r.keep = L.keep;
+  r.sigmoid = L.sigmoid; r.shared_gate = L.sff ? b.sgate : nullptr; r.shared_slot = L.joined();
+  r.correction = L.correction; r.M = M; r.E = L.n_out(); r.top = L.top; r.groups = L.exp_groups; r.keep = L.keep;
   r.slot_expert = b.slot_expert; r.slot_w = b.slot_w; r.count = hm.exp_count;
   r.rows = route_rows(M);
-  VN_LAUNCH_PDL_LEVEL(ctx, 1, "route_kernel", route_kernel, ceil_div(M, ROUTE_WARPS * r.rows), 32 * ROUTE_WARPS, route_smem(n, L.exp_groups), r);
+  VN_LAUNCH_PDL_LEVEL(ctx, 1, "route_kernel", route_kernel, ceil_div(M, ROUTE_WARPS * r.rows), 32 * ROUTE_WARPS, route_smem(r.E, L.exp_groups), r);
   AddExperts<T, Src> few;          // results in split-K slices
-  few.h = (const T*)m->h; few.slot_pos = b.slot_pos; few.slot_expert = b.slot_expert; few.slot_w = L.weigh_input ? nullptr : b.slot_w; few.top = S; few.n_real = L.n_exp; few.D = D;
+  few.h = (const T*)m->h; few.slot_pos = b.slot_pos; few.slot_expert = b.slot_expert; few.slot_w = L.weigh_input ? nullptr : b.slot_w; few.top = S; few.n_real = mats; few.D = D;
   few.count = hm.exp_count; few.cursor = hm.exp_cur; few.n_count = n;
   few.y.ld = D;
-  few.shared_gate = r.shared_gate;
+  if (apart) few.shared_gate = r.shared_gate; else few.slot_gate = r.shared_gate;
   const float* scale = L.weigh_input ? b.slot_w : nullptr;
   GemmArgs up, down;
   up.A = b.hs; up.lda = D; up.W = L.w_gu; up.ldw = D; up.w_stride = (long long)2 * F * D; up.N = 2 * F; up.K = D; up.tag = "gemm_expert_gateup";
@@ -1322,11 +1333,11 @@ int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Nex
   up.M = down.M = M;
   const bool tc = bf && m->use_tc && D % 8 == 0 && tc_detail::encode_fn() != nullptr;
   if (tc && M <= 256) {
-    if (L.sff) TRY((shared_expert<T, Src>(m, L, M, b, &few.shared)));
+    if (apart) TRY((shared_expert<T, Src>(m, L, M, b, &few.shared)));
     VN_LAUNCH_PDL_LEVEL(ctx, 1, "mod_dispatch_kernel", mod_dispatch_kernel<T>, M * S, 128, 0, (const T*)m->h, b.slot_expert, hm.exp_count, hm.exp_off, hm.exp_cur,
                         b.slot_pos, (T*)b.hs, n, S, D, scale);
-    up.seg_off = down.seg_off = hm.exp_off; up.seg_cnt = down.seg_cnt = hm.exp_count; up.nseg = down.nseg = L.n_exp;
-    const int active = std::min(L.n_exp, M * S);          // segments with rows, at most
+    up.seg_off = down.seg_off = hm.exp_off; up.seg_cnt = down.seg_cnt = hm.exp_count; up.nseg = down.nseg = mats;
+    const int active = std::min(mats, M * S);          // segments with rows, at most
     int sp = 1;
     TRY(tc_partial(m, up, (long long)M * S, (long long)M * S, &sp, active));
     const long long pairs = (long long)M * S * F;
@@ -1341,11 +1352,11 @@ int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Nex
   const float* sorted_w = scale ? b.sorted_w : nullptr;
   if (tc) {
     int *off = b.sub_seg, *cnt = off + b.sub_cap, *w = cnt + b.sub_cap;
-    VN_LAUNCH(ctx, mod_subseg_kernel, 1, 32, 0, (const int*)hm.exp_count, (const int*)hm.exp_off, L.n_exp, off, cnt, w, b.sub_cap);
+    VN_LAUNCH(ctx, mod_subseg_kernel, 1, 32, 0, (const int*)hm.exp_count, (const int*)hm.exp_off, mats, off, cnt, w, b.sub_cap);
     VN_LAUNCH(ctx, gather_sorted_kernel<T>, M * S, 128, 0, (const T*)m->h, (const int*)b.sorted_row, (T*)b.hs, D, sorted_w);
     TRY(ensure_partial(m, 1024));
     for (GemmArgs* g : {&up, &down}) {
-      g->M = 256; g->seg_off = off; g->seg_cnt = cnt; g->seg_w = w; g->n_w = L.n_exp; g->nseg = b.sub_cap;
+      g->M = 256; g->seg_off = off; g->seg_cnt = cnt; g->seg_w = w; g->n_w = mats; g->nseg = b.sub_cap;
       TcPlan plan;
       plan.error_flag = m->tc_error;
       TRY(launch_gemm_tc(ctx, *g, (long long)M * S, plan));
@@ -1357,20 +1368,20 @@ int32_t mixture(vn_model* m, const HLayer& L, int M, const Buffers& b, const Nex
       up.A = m->h; up.a_rows = b.sorted_row;
     }
     for (GemmArgs* g : {&up, &down}) {
-      g->seg_off = hm.exp_off; g->seg_cnt = hm.exp_count; g->nseg = L.n_exp;
+      g->seg_off = hm.exp_off; g->seg_cnt = hm.exp_count; g->nseg = mats;
       TRY(linear(m, *g));
     }
   }
   if constexpr (std::is_same<T, __nv_bfloat16>::value) {
     AddExperts<T, Mat<T>> y;
     y.y.p = (const T*)b.ey; y.y.ld = D;
-    y.h = few.h; y.slot_pos = few.slot_pos; y.slot_expert = few.slot_expert; y.slot_w = few.slot_w; y.shared_gate = few.shared_gate; y.top = S; y.n_real = few.n_real; y.D = D;
+    y.h = few.h; y.slot_pos = few.slot_pos; y.slot_expert = few.slot_expert; y.slot_w = few.slot_w; y.shared_gate = few.shared_gate; y.slot_gate = few.slot_gate; y.top = S; y.n_real = few.n_real; y.D = D;
     y.count = few.count; y.cursor = few.cursor; y.n_count = n;
-    if (L.sff) TRY((shared_expert<T, Mat<T>>(m, L, M, b, &y.shared)));
+    if (apart) TRY((shared_expert<T, Mat<T>>(m, L, M, b, &y.shared)));
     return close_rows<T>(m, y, M, L.post[1], next);
   } else {
     few.y.p = (const float*)b.ey;
-    if (L.sff) TRY((shared_expert<T, Src>(m, L, M, b, &few.shared)));
+    if (apart) TRY((shared_expert<T, Src>(m, L, M, b, &few.shared)));
     return close_rows<T>(m, few, M, L.post[1], next);
   }
 }

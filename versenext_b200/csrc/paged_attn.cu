@@ -138,6 +138,67 @@ __global__ void __launch_bounds__(256) attn_inputs4_kernel(ConvIn<T, Mat<T>, fal
   }
 }
 
+// The same without convolutions: a thread takes four channels of one row (with the four they are rotated with) in up to `per`
+// heads, four at a time.  d, vd, rd / 2 and the source's pitch multiples of 4; bias [channels] or null.
+// grid (ceil(M max(quads of a head) / 256), slices of the query and key heads, and one of the values)
+template <typename T, typename S>
+__global__ void __launch_bounds__(256) attn_rows4_kernel(S src, const float* __restrict__ bias, PagedAttnArgs a, int qk_heads, int per) {
+  const int np = a.rd / 2, nr = np / 4;
+  const bool is_v = a.own_kv && blockIdx.y == gridDim.y - 1;
+  const int w = is_v ? a.vd : a.d, quads = is_v ? a.vd / 4 : nr + (a.d - a.rd) / 4;
+  const long long t = (long long)blockIdx.x * 256 + threadIdx.x;
+  const int row = (int)(t / quads), i = (int)(t % quads);
+  if (row >= a.rows.M) return;
+  const bool pair = !is_v && i < nr;
+  const int c = is_v || pair ? 4 * i : a.rd + 4 * (i - nr), col0 = is_v ? (a.H + a.KH) * a.d : 0;
+  const int last = is_v ? a.KH : min(qk_heads, ((int)blockIdx.y + 1) * per);
+  int slot, r0, n, start;
+  a.rows.entry(a.rows.entry_of(row), &slot, &r0, &n, &start);
+  const int pos = start + row - r0;
+  const long long page = ((long long)a.table[(long long)slot * a.max_pages + pos / KV_PAGE] * KV_PAGE + pos % KV_PAGE) * a.KH;
+  float4 p0 = make_float4(1.f, 0.f, 1.f, 0.f), p1 = p0;
+  if (pair) {
+    const float4* cs = reinterpret_cast<const float4*>(a.rope + (long long)pos * np + c);          // two pairs each
+    p0 = cs[0]; p1 = cs[1];
+  }
+  const bool pads = a.P > w && (c + 4 == w || (pair && np + c + 4 == w));       // the last quad of a head also pads it
+#pragma unroll 1
+  for (int head = is_v ? 0 : blockIdx.y * per; head < last; head += 4) {
+    float4 x[4], y[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int col = col0 + min(head + k, last - 1) * w + c;
+      x[k] = get4(src, row, col);
+      if (pair) y[k] = get4(src, row, col + np);
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int h = head + k;
+      if (h >= last) break;
+      const int col = col0 + h * w + c;
+      const bool is_q = !is_v && h < a.H;
+      const float tf = is_q && a.temp ? a.temp[h] : 1.f;
+      T* dst = is_q ? reinterpret_cast<T*>(a.q) + ((long long)row * a.H + h) * a.P + c
+                    : reinterpret_cast<T*>(is_v ? a.vplane : a.kplane) + (page + (is_v ? h : h - a.H)) * a.P + c;
+      auto value = [&](float4 v, int at) {
+        v = make_float4(round_to<T>(v.x), round_to<T>(v.y), round_to<T>(v.z), round_to<T>(v.w));
+        if (bias) { const float4 b = load4(bias + at); v = make_float4(v.x + b.x, v.y + b.y, v.z + b.z, v.w + b.w); }
+        return scaled(v, tf);
+      };
+      const float4 u = value(x[k], col);
+      if (pair) {
+        const float4 v = value(y[k], col + np);
+        store4(dst, make_float4(u.x * p0.x - v.x * p0.y, u.y * p0.z - v.y * p0.w, u.z * p1.x - v.z * p1.y, u.w * p1.z - v.w * p1.w));
+        store4(dst + np, make_float4(v.x * p0.x + u.x * p0.y, v.y * p0.z + u.y * p0.w, v.z * p1.x + u.z * p1.y, v.w * p1.z + u.w * p1.w));
+      } else {
+        store4(dst, u);
+      }
+      if (pads)
+        for (int j = w - c; j < a.P - c; j += 4) store4(dst + j, make_float4(0.f, 0.f, 0.f, 0.f));
+    }
+  }
+}
+
 // Heads with a norm (or with interleaved pairs and biases), without convolutions: bias, norm, rotation.  One warp per (row, unit) with the
 // head staged in shared memory; units as above.  grid (units, ceil(M / 8)), block (32, 8), 8 max(d, vd) floats
 template <typename T, typename S>
@@ -556,6 +617,14 @@ int32_t vn_attn_inputs(vn_ctx* ctx, const ConvIn<T, S, false>& conv, const Paged
       return VN_OK;
     }
     VN_LAUNCH_NAMED(ctx, "attn_heads_kernel", (attn_heads_kernel<T, S>), dim3(units, ceil_div(a.rows.M, 8)), block, (size_t)8 * w * 4, conv, a);
+    return VN_OK;
+  }
+  if (!conv.named && conv.taps == 1 && a.d % 4 == 0 && a.vd % 4 == 0 && a.rd % 8 == 0 && conv.src.ld % 4 == 0 && !a.interleaved) {
+    const int qk = a.H + (a.own_kv ? a.KH : 0), quads = std::max((a.d - a.rd / 2) / 4, a.own_kv ? a.vd / 4 : 0);
+    const long long blocks = ceil_div((long long)a.rows.M * quads, 256ll);
+    int per = 4;                                           // more heads per thread where there are threads enough
+    while (per < qk && blocks * ceil_div(qk, 2 * per) >= 8ll * ctx->sm_count) per *= 2;
+    VN_LAUNCH_NAMED(ctx, "attn_inputs_kernel", (attn_rows4_kernel<T, S>), dim3((unsigned)blocks, ceil_div(qk, per) + (a.own_kv ? 1 : 0)), 256, 0, conv.src, conv.bias, a, qk, per);
     return VN_OK;
   }
   if constexpr (std::is_same<S, Mat<T>>::value) {

@@ -148,6 +148,7 @@ struct ConvIn {
   int RC = 1, C = 0, taps = 1;
   const float* w = nullptr;      // [C, taps]
   const float* bias = nullptr;   // [C] or null
+  bool named = true;             // false: one tap of weight 1, the inputs themselves
 
   template <bool RARE = false>
   __device__ __forceinline__ float input(int row, int r0, int start, int slot, int pos, int c) const {

@@ -111,7 +111,7 @@ struct AddRows {
 };
 
 // the results of a row's experts: rows slot_pos[] of y, weighted unless the weights are null; experts from n_real on are the
-// input h itself; and the gated result of the expert that serves every row
+// input h itself; and the gated result of the expert that serves every row, a matrix of its own or that of a row's last slot
 template <typename T, typename S>
 struct AddExperts {
   S y;
@@ -120,6 +120,7 @@ struct AddExperts {
   const float* slot_w = nullptr;
   S shared;                                      // [M, D], times shared_gate [M] (null: none)
   const float* shared_gate = nullptr;
+  const float* slot_gate = nullptr;              // [M] factor of slot top - 1, or null
   int top = 1, n_real = 0, D = 0;
   int *count = nullptr, *cursor = nullptr;       // left at zero for the next mixture
   int n_count = 0;
@@ -134,7 +135,7 @@ struct AddExperts {
     const int lane = threadIdx.x & 31;           // every warp finds out for itself; they write the same values
     const bool has = lane < top;
     const int e = has ? slot_expert[(long long)row * top + lane] : n_real;
-    const float v = !has ? 0.f : slot_w ? slot_w[(long long)row * top + lane] : 1.f;
+    const float v = !has ? 0.f : slot_gate && lane == top - 1 ? slot_gate[row] : slot_w ? slot_w[(long long)row * top + lane] : 1.f;
     const unsigned real = __ballot_sync(0xffffffffu, has && e < n_real);
     if (has && e < n_real) {
       const int at = __popc(real & ((1u << lane) - 1));
