@@ -101,7 +101,7 @@ MODELS = {
                         width=50, vocab=77, eps=1e-2, loop=(1, 2, 2)),
     "ones": config([A(heads=1, kv_heads=1, dim=16, vdim=16, rot=rot(16), mlp=E(experts=1, top=1, ff=8, shared_ff=8)),
                     A(heads=1, kv_heads=1, dim=2, vdim=1, rot=None, mlp=E(experts=4, top=4, ff=1, shared_ff=None)), A(mlp=dense(1))], width=40, loop=(0, 3, 1)),
-    "no_loop": config([A(rot=rot(24, 1e6, 4.0, 1.0, 4.0, 1024), mlp=E(top=2)), A(mlp=dense())]),
+    "no_loop": config([A(rot=rot(24, 2e5, 6.0, 1.5, 5.0, 700), mlp=E(top=2)), A(mlp=dense())]),
 }
 
 
